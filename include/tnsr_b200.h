@@ -56,7 +56,8 @@ typedef enum tnsr_b200_status {
 typedef enum tnsr_b200_activation {
     TNSR_B200_ACT_RELU = 0,
     TNSR_B200_ACT_GELU = 1,
-    TNSR_B200_ACT_SWIGLU = 2
+    TNSR_B200_ACT_SWIGLU = 2,
+    TNSR_B200_ACT_GELU_TANH = 3   /* 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))): operator calls and described models */
 } tnsr_b200_activation;
 
 typedef enum tnsr_b200_dtype {
@@ -140,6 +141,62 @@ typedef struct tnsr_b200_config {
 
 typedef struct tnsr_b200_decoder tnsr_b200_decoder;
 
+/* Models described layer by layer (no reference counterpart: tnsr has one GPT
+ * block).  A described model is an embedding table, a list of layers and an
+ * output head; every layer is one pre-norm block whose mixer and feed-forward
+ * read the same normalised rows and are added to the residual together:
+ *     h = rms(x) * (norm_offset + w);   x <- x + mixer(h) + feed_forward(h)
+ * (feed_forward(h) = W_down gelu_tanh(W_up h), left out when feed_forward is 0).
+ *
+ * MIXER_ATTENTION: projections with bias, a causal per-channel convolution of
+ * conv_taps taps on q, k and v, per-head RMS norm of q and k, interleaved rotary
+ * positions on the first rotary_dims dimensions (frequencies scaled by
+ * wavelength when rotary_factor > 0), grouped-query causal softmax attention on
+ * softcap * tanh(q.k * score_scale / softcap) (softcap 0: none), and one sigmoid
+ * output gate per head.
+ * MIXER_MAMBA2: the state-space-duality layer: causal convolution + silu on
+ * x|B|C, dt = softplus(dt + bias), a [state, vdim] f32 state per head with scalar
+ * decay exp(-exp(A_log) dt), skip D x, gate silu(z), RMS norm in norm_groups
+ * parts.
+ *
+ * weights_of >= 0: the layer has no tensors of its own and uses those of that
+ * layer (same sizes), with a cache or state of its own. */
+typedef enum tnsr_b200_mixer {
+    TNSR_B200_MIXER_ATTENTION = 0,
+    TNSR_B200_MIXER_MAMBA2 = 1
+} tnsr_b200_mixer;
+
+typedef struct tnsr_b200_layer {
+    uint32_t mixer;         /* tnsr_b200_mixer */
+    int32_t weights_of;     /* -1: tensors of its own */
+    uint32_t heads;
+    uint32_t vdim;          /* value width per head */
+    uint32_t conv_taps;     /* 1..16 */
+    uint32_t feed_forward;  /* 0: no feed-forward */
+    /* attention */
+    uint32_t kv_heads;      /* divides heads */
+    uint32_t dim;           /* query / key width per head, <= 256 */
+    uint32_t rotary_dims;   /* even, <= dim */
+    uint32_t pad0;
+    double rotary_base;
+    double rotary_factor;   /* 0: frequencies as they are */
+    double rotary_low, rotary_high, rotary_original;
+    double score_scale;
+    double score_softcap;   /* 0: no cap */
+    /* mamba2 */
+    uint32_t state;         /* <= 256 */
+    uint32_t groups;        /* divides heads */
+    uint32_t norm_groups;   /* divides heads * vdim */
+    uint32_t pad1;
+} tnsr_b200_layer;
+
+typedef struct tnsr_b200_stack {
+    double embedding_scale;
+    double norm_offset;     /* added to the weights of the layers' and the final norm (1: stored around zero) */
+    const tnsr_b200_layer* layers;
+    uint32_t num_layers;
+} tnsr_b200_stack;
+
 /* ---- library ------------------------------------------------------------ */
 
 TNSR_B200_API const char* tnsr_b200_version(void);
@@ -183,6 +240,20 @@ TNSR_B200_API int tnsr_b200_test_lose_gemm_stage(uint32_t k_block);
  * the 2*num_layers cache tensors (src/nn/kv_cache.rs:188-195) and zeroed
  * parameters.  Size arithmetic is overflow-checked like src/nn/kv_cache.rs:173-187. */
 TNSR_B200_API int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder** out);
+/* The same handle for a model described layer by layer.  Of `config`, vocab_size,
+ * embed_dim, layer_norm_epsilon (the epsilon of every norm), weight_dtype,
+ * kv_dtype (must equal weight_dtype), batch, capacity, max_sequence_length,
+ * device, logits_mode, and the paging fields apply; num_layers must equal the
+ * stack's.  Every call below works on such a handle.  Parameter order: embedding
+ * [vocab, d], head [vocab, d], final norm [d], then for every layer with tensors
+ * of its own: norm [d]; attention: q, q bias, k, k bias, v, v bias, q norm, k
+ * norm, q conv, k conv, v conv, gate, output; mamba2: in, conv, conv bias, dt
+ * bias, A_log, D, norm, output; then up, down if it has a feed-forward.  Matrices
+ * are [out, in] here, convolutions [channels, taps].  The attention caches are
+ * [batch, capacity, kv_heads * width]; paging applies to them only.  Sessions at
+ * position 0 start from empty states whatever their slot held before. */
+TNSR_B200_API int tnsr_b200_decoder_create_stack(const tnsr_b200_config* config, const tnsr_b200_stack* stack,
+                                                 tnsr_b200_decoder** out);
 /* Drop (src/nn/kv_cache/cuda.rs:56-62): waits for queued work, then frees. */
 TNSR_B200_API void tnsr_b200_decoder_destroy(tnsr_b200_decoder* dec);
 
@@ -260,6 +331,12 @@ TNSR_B200_API int tnsr_b200_decoder_synchronize(tnsr_b200_decoder* dec);
 /* The session's private stream as a cudaStream_t (for event timing). */
 TNSR_B200_API void* tnsr_b200_decoder_stream(tnsr_b200_decoder* dec);
 
+/* Number of cache and state tensors of the handle, and the elements of one: a GPT
+ * handle has keys and values of every layer; a described model has, per layer in
+ * order, keys, values and convolution inputs (attention) or convolution inputs
+ * and recurrent state (mamba2). */
+TNSR_B200_API uint32_t tnsr_b200_decoder_cache_count(const tnsr_b200_decoder* dec);
+TNSR_B200_API uint64_t tnsr_b200_decoder_cache_elems(const tnsr_b200_decoder* dec, uint32_t index);
 /* Cache tensor `index` (2*layer = keys, 2*layer+1 = values) as f32
  * [batch, capacity, embed_dim]; the counterpart of reading the reference's
  * `cache: Vec<Parameter<f32>>` (src/nn/kv_cache.rs:76).  `write` exists so

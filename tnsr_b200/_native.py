@@ -17,7 +17,8 @@ STATUS = {
     0: "OK", -1: "ERR_INVALID_ARGUMENT", -2: "ERR_CUDA", -3: "ERR_OUT_OF_MEMORY", -4: "ERR_CAPACITY",
     -5: "ERR_TOKEN_RANGE", -6: "ERR_FAILED_STATE", -7: "ERR_TIMEOUT", -8: "ERR_UNSUPPORTED", -9: "ERR_NO_DEVICE",
 }
-ACT = {"relu": 0, "gelu": 1, "swiglu": 2}
+ACT = {"relu": 0, "gelu": 1, "swiglu": 2, "gelu_tanh": 3}
+MIXER = {"attention": 0, "mamba2": 1}
 DTYPE = {"f32": 0, "bf16": 1}
 LOGITS = {"all": 0, "last": 1, "none": 2}
 PREFILL = {"auto": 0, "scalar": 1}
@@ -34,6 +35,21 @@ class Config(C.Structure):
     ]
 
 
+class LayerDesc(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_uint32), ("weights_of", C.c_int32), ("heads", C.c_uint32), ("vdim", C.c_uint32), ("conv_taps", C.c_uint32),
+        ("feed_forward", C.c_uint32), ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("rotary_dims", C.c_uint32), ("pad0", C.c_uint32),
+        ("rotary_base", C.c_double), ("rotary_factor", C.c_double), ("rotary_low", C.c_double), ("rotary_high", C.c_double),
+        ("rotary_original", C.c_double), ("score_scale", C.c_double), ("score_softcap", C.c_double), ("state", C.c_uint32),
+        ("groups", C.c_uint32), ("norm_groups", C.c_uint32), ("pad1", C.c_uint32),
+    ]
+
+
+class StackDesc(C.Structure):
+    _fields_ = [("embedding_scale", C.c_double), ("norm_offset", C.c_double), ("layers", C.POINTER(LayerDesc)),
+                ("num_layers", C.c_uint32)]
+
+
 _vp, _u32, _u64, _i, _f = C.c_void_p, C.c_uint32, C.c_uint64, C.c_int, C.c_float
 _fp, _u32p = C.POINTER(C.c_float), C.POINTER(C.c_uint32)
 
@@ -47,6 +63,7 @@ SIGNATURES = {
     "tnsr_b200_set_wait_limit_ns": (_i, [_u64]),
     "tnsr_b200_test_lose_gemm_stage": (_i, [_u32]),
     "tnsr_b200_decoder_create": (_i, [C.POINTER(Config), C.POINTER(_vp)]),
+    "tnsr_b200_decoder_create_stack": (_i, [C.POINTER(Config), C.POINTER(StackDesc), C.POINTER(_vp)]),
     "tnsr_b200_decoder_destroy": (None, [_vp]),
     "tnsr_b200_decoder_param_count": (_u32, [_vp]),
     "tnsr_b200_decoder_param_elems": (_u64, [_vp, _u32]),
@@ -59,6 +76,8 @@ SIGNATURES = {
     "tnsr_b200_decoder_stream": (_vp, [_vp]),
     "tnsr_b200_decoder_profile_attention": (_i, [_vp, _i]),
     "tnsr_b200_decoder_attention_profile": (_i, [_vp, C.POINTER(C.c_double), C.POINTER(C.c_uint64)]),
+    "tnsr_b200_decoder_cache_count": (_u32, [_vp]),
+    "tnsr_b200_decoder_cache_elems": (_u64, [_vp, _u32]),
     "tnsr_b200_decoder_read_cache": (_i, [_vp, _u32, _fp]),
     "tnsr_b200_decoder_write_cache": (_i, [_vp, _u32, _fp]),
     "tnsr_b200_embedding": (_i, [_vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _u32, _i, _vp, _vp]),

@@ -84,7 +84,7 @@ inline uint32_t ceil_div(uint32_t a, uint32_t b) { return (a + b - 1) / b; }
 inline uint64_t ceil_div64(uint64_t a, uint64_t b) { return (a + b - 1) / b; }
 
 // FFN / epilogue activation codes shared by host and device.
-enum : int { ACT_NONE = -1, ACT_RELU = 0, ACT_GELU = 1 };
+enum : int { ACT_NONE = -1, ACT_RELU = 0, ACT_GELU = 1, ACT_GELU_TANH = 3 };   // values of tnsr_b200_activation
 
 // Device-side status word: kernels never trap; they record the first problem
 // here and carry on with harmless values.
@@ -142,7 +142,20 @@ enum GemmMode : int {
     GEMM_PLAIN = 0,   // out[m, n] (f32 or bf16) = act(acc + bias) (+ residual)
     GEMM_QKV = 1,     // n = 3*d: columns [0,d) -> q (bf16), [d,2d) -> K cache rows, [2d,3d) -> V cache rows
     GEMM_SWIGLU = 2,  // n = 2*f packed in blocks of 16: out[m, f] bf16 = silu(gate) * up
-    GEMM_ARGMAX = 3   // no matrix leaves the kernel: per (row, column tile) the greedy candidate (key, index)
+    GEMM_ARGMAX = 3,  // no matrix leaves the kernel: per (row, column tile) the greedy candidate (key, index)
+    GEMM_SEGMENTS = 4 // column ranges with destinations of their own (GemmSegments): one product for all projections of a layer
+};
+// Destinations of the column ranges of one product: range i covers accumulator columns [col0, col0 of i + 1) and lands in
+// `out` (row pitch ld, local column = column - col0), bf16 or f32, with an activation of its own.  Range boundaries and n
+// are multiples of 32, so that a 32-column block belongs to one range.
+struct GemmSegment {
+    void* out = nullptr;
+    uint32_t col0 = 0, ld = 0;
+    int out_dtype = TNSR_B200_BF16, activation = ACT_NONE;
+};
+struct GemmSegments {
+    GemmSegment s[3];
+    uint32_t count = 0;
 };
 // Paged K/V: a cache tensor is a pool [pages, page_rows, d] shared by all sessions; logical row r of session s lives
 // in page table[s * pages_per_session + r / page_rows] at row r % page_rows.  table == nullptr: the contiguous
@@ -172,6 +185,9 @@ struct GemmQkvTargets {
 int launch_gemm_bf16(const bf16* a, const bf16* bt, void* out, uint32_t ldc, uint32_t m, uint32_t n,
                      uint32_t k, GemmMode mode, const GemmEpilogue& ep, const GemmQkvTargets* qkv,
                      int* d_status, cudaStream_t stream);
+// a[m, k] . bt[n, k]^T (+ bias), every column range to its own destination.
+int launch_gemm_segments(const bf16* a, const bf16* bt, uint32_t m, uint32_t n, uint32_t k, const float* bias,
+                         const GemmSegments& segments, int* d_status, cudaStream_t stream);
 extern int g_gemm_engine;  // 0 auto, 1 CUDA-core only, 2 tcgen05 only, 3 auto + the tcgen05 few-row engine for every eligible shape, 4 auto + the streaming engine for every eligible shape
 // Few rows (m <= 64): weights on the M side of the MMA, optional split-K (gemm_skinny.cu).
 uint64_t gemm_skinny_workspace_bytes();
@@ -190,9 +206,13 @@ int launch_lm_head_argmax(const bf16* a, const bf16* bt, uint32_t m, uint32_t n,
 
 int launch_embedding(const void* tok, const void* pos, const uint32_t* ids, float* out, uint32_t rows,
                      uint32_t chunk, uint32_t position0, const uint32_t* d_position, uint32_t vocab,
-                     uint32_t width, int dtype, int* d_status, cudaStream_t stream, uint32_t position_stride = 0);
+                     uint32_t width, int dtype, int* d_status, cudaStream_t stream, uint32_t position_stride = 0,
+                     float scale = 1.0f);   // pos == nullptr: token row * scale, no position table
 int launch_layernorm(const float* x, const float* w, const float* b, void* out, uint32_t rows,
                      uint32_t width, float eps, int out_dtype, bool strict, cudaStream_t stream);
+// x / sqrt(mean(x^2) + eps) * (w_add + w), statistics in f32.
+int launch_rmsnorm(const float* x, const float* w, float w_add, void* out, uint32_t rows, uint32_t width, float eps,
+                   int out_dtype, cudaStream_t stream);
 // Gathers row (s * chunk + chunk - 1) of x for every session s into out[s, :] (f32).
 int launch_gather_last_rows(const float* x, float* out, uint32_t sessions, uint32_t chunk, uint32_t width,
                             cudaStream_t stream);
@@ -216,6 +236,11 @@ int launch_transpose_f32_to_bf16_mapped(const float* in, bf16* out, uint32_t k, 
 bool layernorm_fold_supported(uint32_t width);
 int launch_layernorm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, const float* b,
                           void* out, uint32_t rows, uint32_t width, float eps, cudaStream_t stream);
+int launch_rmsnorm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, float w_add,
+                        void* out, uint32_t rows, uint32_t width, float eps, cudaStream_t stream);
+// out[(row0 + r) * ld + col0 + c] = in[r, c] (f32 or bf16 out): one stored weight into its place in a packed operand.
+int launch_pack_rows(const float* in, void* out, int dtype, uint32_t rows, uint32_t cols, uint32_t row0, uint32_t col0,
+                     uint32_t ld, cudaStream_t stream);
 int launch_layernorm_strict(const float* x, const float* w, const float* b, float* out, uint32_t rows,
                             uint32_t width, float eps, cudaStream_t stream);
 int launch_swiglu_strict(const float* gate, const float* up, float* out, size_t n, cudaStream_t stream);
@@ -314,6 +339,14 @@ __device__ __forceinline__ float bf16_bits_to_f32(uint32_t hi16) { return __uint
 __device__ __forceinline__ float2 bf16x2_to_f32(uint32_t v) {
     return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
 }
+template <typename T>
+__device__ __forceinline__ T from_f32(float x);
+template <>
+__device__ __forceinline__ float from_f32<float>(float x) { return x; }
+template <>
+__device__ __forceinline__ bf16 from_f32<bf16>(float x) { return __float2bfloat16_rn(x); }
+__device__ __forceinline__ float to_f32(float x) { return x; }
+__device__ __forceinline__ float to_f32(bf16 x) { return __bfloat162float(x); }
 // Round to nearest even to bf16 and widen again; NaN stays a quiet NaN.
 __device__ __forceinline__ float round_to_bf16(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
@@ -337,9 +370,14 @@ __device__ __forceinline__ float fast_gelu(float x) {
     float cdf = (x < 0.0f) ? tail : 1.0f - tail;
     return x * cdf;
 }
+// tanh form of gelu: 0.5 x (1 + tanh(u)) = x * sigmoid(2u), u = sqrt(2/pi) (x + 0.044715 x^3)
+__device__ __forceinline__ float fast_gelu_tanh(float x) {
+    return x * fast_sigmoid(1.5957691216057308f * (x + 0.044715f * x * x * x));
+}
 __device__ __forceinline__ float apply_activation(float x, int act) {
     if (act == ACT_RELU) return fmaxf(x, 0.0f);
     if (act == ACT_GELU) return fast_gelu(x);
+    if (act == ACT_GELU_TANH) return fast_gelu_tanh(x);
     return x;
 }
 

@@ -10,7 +10,7 @@
 #include <unordered_set>
 #include <vector>
 
-#include "common.cuh"
+#include "decoder.cuh"
 
 namespace tb {
 std::atomic<uint64_t> g_launches{0};
@@ -41,188 +41,6 @@ bool debug_sync_enabled() {
 using namespace tb;
 
 namespace {
-
-constexpr uint32_t kNoPage = 0xffffffffu;
-
-struct Buffer {
-    void* ptr = nullptr;
-    size_t bytes = 0;
-};
-
-enum ParamKind { P_TOK, P_POS, P_VEC, P_QKV_W, P_QKV_B, P_O_W, P_FF_IN_W, P_FF_IN_B, P_FF_OUT_W, P_GATE_W, P_GATE_B, P_UP_W, P_UP_B };
-
-struct ParamInfo {
-    ParamKind kind;
-    uint64_t elems;
-    uint32_t rows, cols;  // [rows, cols] as the reference stores it ([in, out] for matrices)
-    uint32_t layer;
-    uint32_t slot;        // 0/1/2 = q/k/v for QKV params
-    void* dev = nullptr;  // where the values live (f32 path: as given; bf16 path: see upload)
-};
-
-struct Layer {
-    // f32 path: the reference layout, f32.  bf16 path: matrices are [out, in] bf16.
-    void *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr;
-    float *bq = nullptr, *bk = nullptr, *bv = nullptr, *bo = nullptr;
-    float *ln1w = nullptr, *ln1b = nullptr, *ln2w = nullptr, *ln2b = nullptr;
-    void *w_in = nullptr, *w_out = nullptr, *w_gate = nullptr, *w_up = nullptr;
-    float *b_in = nullptr, *b_out = nullptr, *b_gate = nullptr, *b_up = nullptr;
-    // bf16 path fused forms
-    bf16* wqkv = nullptr;  // [3d, d]
-    float* bqkv = nullptr; // [3d]
-    bf16* wgu = nullptr;   // packed [2f, d] when f % 16 == 0
-    float* bgu = nullptr;  // packed [2f]
-    void *kcache = nullptr, *vcache = nullptr;
-};
-
-}  // namespace
-
-struct tnsr_b200_decoder {
-    tnsr_b200_config cfg;
-    cudaStream_t stream = nullptr;
-    bool bf16_path = false, kv_bf16 = false, swiglu = false, fused_gu = false;
-    bool failed = false;
-    std::string error;
-    std::vector<ParamInfo> params;
-    std::vector<Layer> layers;
-    void *tok = nullptr, *pos = nullptr;
-    float *fnw = nullptr, *fnb = nullptr;
-    std::vector<void*> allocations;
-    // activations (grow with the chunk)
-    uint32_t rows_cap = 0, logit_rows_cap = 0;
-    float* h = nullptr;      // residual stream [rows, d] f32
-    void* n = nullptr;       // normalised rows: f32 (strict) or bf16
-    void* q = nullptr;       // queries: f32 (strict) or bf16
-    void* att = nullptr;     // attention output: f32 (strict) or bf16
-    void* ff = nullptr;      // FFN hidden [rows, f]
-    void* ff2 = nullptr;     // second FFN buffer (up projection) when gate/up are not fused
-    float* hl = nullptr;     // last rows [batch, d] f32
-    float* logits = nullptr; // [logit_rows, vocab]
-    uint32_t* d_tokens = nullptr;
-    uint32_t tokens_cap = 0;
-    uint32_t* d_argmax = nullptr;
-    int* d_status = nullptr;
-    void* attn_ws = nullptr;
-    // a single-token step may be divided into up to kMaxParts session ranges on as many streams (see step_bf16):
-    // range 0 runs on `stream` with `attn_ws`, range i > 0 on side_stream[i - 1] with side_ws[i - 1]
-    void* side_ws[3] = {nullptr, nullptr, nullptr};
-    // partial sums of the split-K projections of an undivided single-token step: [4][split_rows][d] f32
-    float* split_ws = nullptr;
-    uint32_t split_rows = 0;
-    uint32_t split_pending = 0;   // partial sums of the last layer's down projection, for the final LayerNorm to add
-    uint64_t attn_ws_bytes = 0;
-    cudaStream_t side_stream[3] = {nullptr, nullptr, nullptr};   // forked from and joined to `stream` by events
-    cudaEvent_t ev_fork = nullptr, ev_join[3] = {nullptr, nullptr, nullptr};
-    uint32_t parts = 1;
-    // small batches: one persistent kernel per layer between the attention scans (decode_tail.cu); its barrier words
-    void* tail_ws = nullptr;
-    bool use_tail = true;
-    // paged K/V: every cache tensor is a pool [pool_pages, page_rows, d]; h_table[s * pps + i] is the pool page of
-    // session s's i-th page, kNoPage while unassigned (the device copy is refreshed before the step that needs it)
-    bool paged = false;
-    uint32_t page_rows = 0, pool_pages = 0, pps = 0;
-    std::vector<uint32_t> h_table_shadow;   // the table as the host knows it
-    std::vector<uint32_t> free_pages;       // stack of unassigned pool pages
-    uint32_t* h_table = nullptr;            // pinned copy used for the upload
-    uint32_t* d_table = nullptr;
-    bool table_dirty = false;
-    // next-token sampling instead of the greedy pick (temperature <= 0: greedy)
-    float sample_temperature = 0.0f;
-    uint32_t sample_top_k = 0;
-    uint64_t sample_seed = 0;
-    uint32_t* d_positions = nullptr;   // [batch] per-session positions of a ragged step
-    uint32_t* h_positions = nullptr;   // pinned staging for them
-    // pinned staging
-    uint32_t* h_tokens = nullptr;
-    uint32_t* h_argmax = nullptr;
-    int* h_status = nullptr;
-    float* h_stage = nullptr;  // upload staging (pinned)
-    size_t h_stage_bytes = 0;
-    float* d_stage = nullptr;  // upload staging (device, f32)
-    size_t d_stage_bytes = 0;
-    std::vector<float> host_bqkv, host_bgu;
-    bool profile_attention = false;
-    KernelTimer attention_timer;
-    void* lm_candidates = nullptr;  // per (session, vocabulary tile) greedy candidates of the fused LM head
-    // single-token steps are replayed from a captured CUDA graph; the position lives in d_pos
-    uint32_t* d_pos = nullptr;
-    struct StepGraph {
-        const uint32_t* tokens;
-        uint32_t* argmax;
-        cudaGraphExec_t exec;
-        uint64_t kernels;
-    };
-    std::vector<StepGraph> graphs;
-    bool use_graphs = true;
-    bool use_pdl = true;
-    bool stepped_once = false;  // a plain (uncaptured) single-token step has run: buffers and attributes are set
-};
-
-namespace {
-
-int fail(tnsr_b200_decoder* dec, int code, const std::string& msg) {
-    if (dec) dec->error = msg;
-    set_thread_error(msg);
-    return code;
-}
-
-int cuda_fail(tnsr_b200_decoder* dec, cudaError_t e, const char* what) {
-    std::string msg = std::string(what) + ": " + cudaGetErrorString(e);
-    int code = (e == cudaErrorMemoryAllocation) ? TNSR_B200_ERR_OUT_OF_MEMORY : TNSR_B200_ERR_CUDA;
-    if (dec && code == TNSR_B200_ERR_CUDA) dec->failed = true;
-    cudaGetLastError();
-    return fail(dec, code, msg);
-}
-
-#define CU(dec, call)                                                   \
-    do {                                                                \
-        cudaError_t e__ = (call);                                       \
-        if (e__ != cudaSuccess) return cuda_fail(dec, e__, #call);      \
-    } while (0)
-
-#define RUN(dec, call)                                                  \
-    do {                                                                \
-        int rc__ = (call);                                              \
-        if (rc__ != TNSR_B200_OK) {                                     \
-            (dec)->error = thread_error();                              \
-            if (rc__ == TNSR_B200_ERR_CUDA) (dec)->failed = true;       \
-            return rc__;                                                \
-        }                                                               \
-    } while (0)
-
-void drop_graphs(tnsr_b200_decoder* dec) {
-    for (auto& g : dec->graphs) cudaGraphExecDestroy(g.exec);
-    dec->graphs.clear();
-}
-
-int dev_alloc(tnsr_b200_decoder* dec, void** out, size_t bytes, bool zero) {
-    if (bytes == 0) bytes = 16;
-    void* p = nullptr;
-    cudaError_t e = cudaMalloc(&p, bytes);
-    if (e != cudaSuccess) return cuda_fail(dec, e, "cudaMalloc");
-    dec->allocations.push_back(p);
-    if (zero) {
-        e = cudaMemsetAsync(p, 0, bytes, dec->stream);
-        if (e != cudaSuccess) return cuda_fail(dec, e, "cudaMemsetAsync");
-    }
-    *out = p;
-    return TNSR_B200_OK;
-}
-
-void dev_free(tnsr_b200_decoder* dec, void* p) {
-    if (!p) return;
-    for (size_t i = 0; i < dec->allocations.size(); ++i)
-        if (dec->allocations[i] == p) {
-            dec->allocations.erase(dec->allocations.begin() + i);
-            break;
-        }
-    cudaFree(p);
-}
-
-size_t elt(const tnsr_b200_decoder* dec) { return dec->bf16_path ? 2 : 4; }
-size_t kv_elt(const tnsr_b200_decoder* dec) { return dec->kv_bf16 ? 2 : 4; }
-
-bool mul_overflow(uint64_t a, uint64_t b, uint64_t* out) { return __builtin_mul_overflow(a, b, out); }
 
 // model_parameters order (src/nn/kv_cache.rs:392-421) + the SwiGLU extension.
 void describe_params(tnsr_b200_decoder* dec) {
@@ -324,11 +142,15 @@ int ensure_rows(tnsr_b200_decoder* dec, uint32_t rows, uint32_t logit_rows) {
         dec->rows_cap = 0;
         if ((rc = dev_alloc(dec, (void**)&dec->h, rows * d * 4, false))) return rc;
         if ((rc = dev_alloc(dec, &dec->n, rows * d * a, false))) return rc;
-        if ((rc = dev_alloc(dec, &dec->q, rows * d * a, false))) return rc;
-        if ((rc = dev_alloc(dec, &dec->att, rows * d * a, false))) return rc;
-        if ((rc = dev_alloc(dec, &dec->ff, rows * f * a, false))) return rc;
-        if (dec->swiglu && !dec->fused_gu)
-            if ((rc = dev_alloc(dec, &dec->ff2, rows * f * a, false))) return rc;
+        if (dec->stack) {   // projections and mixer outputs are the stack's own
+            if ((rc = stack_alloc_rows(dec, rows))) return rc;
+        } else {
+            if ((rc = dev_alloc(dec, &dec->q, rows * d * a, false))) return rc;
+            if ((rc = dev_alloc(dec, &dec->att, rows * d * a, false))) return rc;
+            if ((rc = dev_alloc(dec, &dec->ff, rows * f * a, false))) return rc;
+            if (dec->swiglu && !dec->fused_gu)
+                if ((rc = dev_alloc(dec, &dec->ff2, rows * f * a, false))) return rc;
+        }
         dec->rows_cap = rows;
     }
     if (logit_rows > dec->logit_rows_cap) {
@@ -691,7 +513,8 @@ int run_step_direct(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t c
     t_attention_timer = dec->profile_attention ? &dec->attention_timer : nullptr;
     t_pdl = dec->use_pdl && dec->bf16_path && chunk == 1;
     t_single_token_step = chunk == 1;
-    int rc = dec->bf16_path ? step_bf16(dec, d_tokens, chunk, position, d_position, logit_rows, fuse_ids ? d_argmax_out : nullptr)
+    int rc = dec->stack ? stack_step(dec, d_tokens, chunk, position, d_position, false, logit_rows, fuse_ids ? d_argmax_out : nullptr)
+           : dec->bf16_path ? step_bf16(dec, d_tokens, chunk, position, d_position, logit_rows, fuse_ids ? d_argmax_out : nullptr)
                             : step_strict(dec, d_tokens, chunk, position, d_position, logit_rows);
     t_attention_timer = nullptr;
     if (rc) { t_pdl = t_single_token_step = false; return rc; }
@@ -844,11 +667,12 @@ int tnsr_b200_set_gemm_engine(int engine) {
     return TNSR_B200_OK;
 }
 
-int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder** out) {
+// `stack`: the model is described layer by layer; nullptr: the GPT of the configuration.
+static int create_decoder(const tnsr_b200_config* config, const tnsr_b200_stack* stack, tnsr_b200_decoder** out) {
     if (!out) return fail(nullptr, TNSR_B200_ERR_INVALID_ARGUMENT, "null output handle");
     *out = nullptr;
     std::string why;
-    int rc = validate_config(config, why);
+    int rc = stack ? stack_check(config, stack, why) : validate_config(config, why);
     if (rc) return fail(nullptr, rc, why);
     int count = 0;
     if (cudaGetDeviceCount(&count) != cudaSuccess || count == 0) {
@@ -867,7 +691,7 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
     dec->cfg = *config;
     dec->bf16_path = config->weight_dtype == TNSR_B200_BF16;
     dec->kv_bf16 = config->kv_dtype == TNSR_B200_BF16;
-    dec->swiglu = config->activation == TNSR_B200_ACT_SWIGLU;
+    dec->swiglu = !stack && config->activation == TNSR_B200_ACT_SWIGLU;
     dec->fused_gu = dec->bf16_path && dec->swiglu && config->feed_forward_dim % 16 == 0;
     auto bail = [&](int code) {
         std::string msg = dec->error;
@@ -878,7 +702,7 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
     if (cudaSetDevice(config->device) != cudaSuccess) return bail(cuda_fail(dec, cudaGetLastError(), "cudaSetDevice"));
     cudaError_t e = cudaStreamCreateWithFlags(&dec->stream, cudaStreamNonBlocking);
     if (e != cudaSuccess) return bail(cuda_fail(dec, e, "cudaStreamCreate"));
-    describe_params(dec);
+    if (!stack) describe_params(dec);
     if (config->kv_page_rows) {
         dec->paged = true;
         dec->page_rows = config->kv_page_rows;
@@ -892,7 +716,7 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
         if (cudaMallocHost((void**)&dec->h_table, dec->h_table_shadow.size() * 4) != cudaSuccess)
             return bail(cuda_fail(dec, cudaGetLastError(), "cudaMallocHost"));
     }
-    if ((rc = allocate_weights(dec))) return bail(rc);
+    if ((rc = stack ? stack_create(dec, stack) : allocate_weights(dec))) return bail(rc);
     const uint64_t d = config->embed_dim;
     if ((rc = dev_alloc(dec, (void**)&dec->hl, (size_t)config->batch * d * 4, false))) return bail(rc);
     if ((rc = dev_alloc(dec, (void**)&dec->d_argmax, (size_t)config->batch * 4, true))) return bail(rc);
@@ -912,7 +736,7 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
         cudaMallocHost((void**)&dec->h_status, 16) != cudaSuccess)
         return bail(cuda_fail(dec, cudaGetLastError(), "cudaMallocHost"));
     *dec->h_status = 0;
-    if (dec->bf16_path && decode_attention_supported(config->num_heads, config->embed_dim / config->num_heads)) {
+    if (!stack && dec->bf16_path && decode_attention_supported(config->num_heads, config->embed_dim / config->num_heads)) {
         dec->attn_ws_bytes = decode_attention_workspace_bytes(config->batch, config->capacity, config->num_heads,
                                                               config->embed_dim / config->num_heads);
         if ((rc = dev_alloc(dec, &dec->attn_ws, dec->attn_ws_bytes, true))) return bail(rc);
@@ -942,7 +766,7 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
             dec->use_tail = config->small_batch_mode == 0;
         }
     }
-    if (dec->bf16_path) {
+    if (!stack && dec->bf16_path) {
         dec->host_bqkv.assign((size_t)config->num_layers * 3 * d, 0.0f);
         if (dec->fused_gu) dec->host_bgu.assign((size_t)config->num_layers * 2 * config->feed_forward_dim, 0.0f);
     }
@@ -952,10 +776,18 @@ int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder**
     return TNSR_B200_OK;
 }
 
+int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_b200_decoder** out) { return create_decoder(config, nullptr, out); }
+
+int tnsr_b200_decoder_create_stack(const tnsr_b200_config* config, const tnsr_b200_stack* stack, tnsr_b200_decoder** out) {
+    if (!stack) return fail(nullptr, TNSR_B200_ERR_INVALID_ARGUMENT, "null model description");
+    return create_decoder(config, stack, out);
+}
+
 void tnsr_b200_decoder_destroy(tnsr_b200_decoder* dec) {
     if (!dec) return;
     cudaSetDevice(dec->cfg.device);
     if (dec->stream) cudaStreamSynchronize(dec->stream);
+    stack_destroy(dec);
     for (void* p : dec->allocations) cudaFree(p);
     if (dec->h_tokens) cudaFreeHost(dec->h_tokens);
     if (dec->h_argmax) cudaFreeHost(dec->h_argmax);
@@ -975,14 +807,21 @@ void tnsr_b200_decoder_destroy(tnsr_b200_decoder* dec) {
     delete dec;
 }
 
-uint32_t tnsr_b200_decoder_param_count(const tnsr_b200_decoder* dec) { return dec ? (uint32_t)dec->params.size() : 0; }
+uint32_t tnsr_b200_decoder_param_count(const tnsr_b200_decoder* dec) { return dec && dec->stack ? stack_param_count(dec) : dec ? (uint32_t)dec->params.size() : 0; }
 
 uint64_t tnsr_b200_decoder_param_elems(const tnsr_b200_decoder* dec, uint32_t index) {
+    if (dec && dec->stack) return stack_param_elems(dec, index);
     return (dec && index < dec->params.size()) ? dec->params[index].elems : 0;
 }
 
 int tnsr_b200_decoder_upload(tnsr_b200_decoder* dec, uint32_t index, const float* host, uint64_t elems) {
     if (!dec) return fail(nullptr, TNSR_B200_ERR_INVALID_ARGUMENT, "null decoder");
+    if (dec->stack) {
+        if (index >= stack_param_count(dec) || !host) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "parameter index or pointer invalid");
+        if (elems != stack_param_elems(dec, index)) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "parameter length mismatch");
+        CU(dec, cudaSetDevice(dec->cfg.device));
+        return stack_upload(dec, index, host);
+    }
     if (index >= dec->params.size() || !host) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "parameter index or pointer invalid");
     const ParamInfo& p = dec->params[index];
     if (elems != p.elems) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "parameter length mismatch");
@@ -1090,6 +929,10 @@ int tnsr_b200_decoder_reset(tnsr_b200_decoder* dec) {
         std::fill(dec->h_table_shadow.begin(), dec->h_table_shadow.end(), kNoPage);
         dec->table_dirty = true;
     }
+    if (dec->stack) {
+        int rc = stack_reset(dec);
+        if (rc) return rc;
+    }
     for (Layer& L : dec->layers) {
         CU(dec, cudaMemsetAsync(L.kcache, 0, cache_bytes, dec->stream));
         CU(dec, cudaMemsetAsync(L.vcache, 0, cache_bytes, dec->stream));
@@ -1162,7 +1005,7 @@ int tnsr_b200_decoder_decode_ragged(tnsr_b200_decoder* dec, const uint32_t* toke
     if (!dec) return fail(nullptr, TNSR_B200_ERR_INVALID_ARGUMENT, "null decoder");
     if (dec->failed) return fail(dec, TNSR_B200_ERR_FAILED_STATE, "decoder execution failed; reset the cache before reuse");
     const tnsr_b200_config& c = dec->cfg;
-    if (!dec->bf16_path) return fail(dec, TNSR_B200_ERR_UNSUPPORTED, "ragged decode is implemented for bf16 weights only");
+    if (!dec->bf16_path && !dec->stack) return fail(dec, TNSR_B200_ERR_UNSUPPORTED, "ragged decode is implemented for bf16 weights only");
     if (!tokens || !positions) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "null token or position pointer");
     if (c.logits_mode == TNSR_B200_LOGITS_NONE && logits_out)
         return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "logits_out must be NULL when logits_mode is NONE");
@@ -1190,7 +1033,11 @@ int tnsr_b200_decoder_decode_ragged(tnsr_b200_decoder* dec, const uint32_t* toke
     CU(dec, cudaMemcpyAsync(dec->d_positions, dec->h_positions, (size_t)c.batch * 4, cudaMemcpyHostToDevice, dec->stream));
     const bool sampling = dec->sample_temperature > 0.0f;
     const bool fuse_ids = c.logits_mode == TNSR_B200_LOGITS_NONE && argmax_out && dec->lm_candidates && !sampling;
-    if ((rc = step_bf16(dec, dec->d_tokens, 1, 0, dec->d_positions, c.batch, fuse_ids ? dec->d_argmax : nullptr, true))) return rc;
+    t_single_token_step = true;
+    rc = dec->stack ? stack_step(dec, dec->d_tokens, 1, 0, dec->d_positions, true, c.batch, fuse_ids ? dec->d_argmax : nullptr)
+                    : step_bf16(dec, dec->d_tokens, 1, 0, dec->d_positions, c.batch, fuse_ids ? dec->d_argmax : nullptr, true);
+    t_single_token_step = false;
+    if (rc) return rc;
     if (argmax_out && !fuse_ids) {
         // session b's new token will sit at positions[b] + 1
         rc = sampling ? launch_sample_top_k(dec->logits, dec->d_argmax, c.batch, c.vocab_size, c.vocab_size, dec->sample_temperature,
@@ -1299,8 +1146,49 @@ int tnsr_b200_decoder_attention_profile(tnsr_b200_decoder* dec, double* total_ms
 
 void* tnsr_b200_decoder_stream(tnsr_b200_decoder* dec) { return dec ? (void*)dec->stream : nullptr; }
 
+uint32_t tnsr_b200_decoder_cache_count(const tnsr_b200_decoder* dec) {
+    return !dec ? 0 : dec->stack ? stack_cache_count(dec) : 2 * dec->cfg.num_layers;
+}
+
+uint64_t tnsr_b200_decoder_cache_elems(const tnsr_b200_decoder* dec, uint32_t index) {
+    if (!dec || index >= tnsr_b200_decoder_cache_count(dec)) return 0;
+    if (!dec->stack) return (uint64_t)dec->cfg.batch * dec->cfg.capacity * dec->cfg.embed_dim;
+    void* ptr;
+    uint64_t elems = 0;
+    int dtype;
+    stack_cache(dec, index, &ptr, &elems, &dtype);
+    return elems;
+}
+
+// Whole cache or state tensors of a described model (contiguous layout), as f32 on the host side.
+static int copy_stack_cache(tnsr_b200_decoder* dec, uint32_t index, float* host_out, const float* host_in) {
+    void* ptr;
+    uint64_t elems;
+    int dtype;
+    if (!stack_cache(dec, index, &ptr, &elems, &dtype)) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "cache index out of range");
+    if (dec->paged) return fail(dec, TNSR_B200_ERR_UNSUPPORTED, "caches of a paged described model are not read or written as whole tensors");
+    CU(dec, cudaSetDevice(dec->cfg.device));
+    float* tmp = (float*)ptr;
+    int rc = TNSR_B200_OK;
+    if (dtype == TNSR_B200_BF16 && (rc = dev_alloc(dec, (void**)&tmp, elems * 4, false))) return rc;
+    cudaError_t e = cudaSuccess;
+    if (host_out) {
+        if (dtype == TNSR_B200_BF16) rc = launch_bf16_to_f32((const bf16*)ptr, tmp, elems, dec->stream);
+        if (rc == TNSR_B200_OK) e = cudaMemcpyAsync(host_out, tmp, elems * 4, cudaMemcpyDeviceToHost, dec->stream);
+    } else {
+        e = cudaMemcpyAsync(tmp, host_in, elems * 4, cudaMemcpyHostToDevice, dec->stream);
+        if (e == cudaSuccess && dtype == TNSR_B200_BF16) rc = launch_f32_to_bf16(tmp, (bf16*)ptr, elems, dec->stream);
+    }
+    if (rc) dec->error = thread_error();
+    if (e == cudaSuccess) e = cudaStreamSynchronize(dec->stream);
+    if (dtype == TNSR_B200_BF16) dev_free(dec, tmp);
+    if (e != cudaSuccess) return cuda_fail(dec, e, "cache copy");
+    return rc;
+}
+
 int tnsr_b200_decoder_read_cache(tnsr_b200_decoder* dec, uint32_t index, float* host_out) {
     if (!dec || !host_out) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "null argument");
+    if (dec->stack) return copy_stack_cache(dec, index, host_out, nullptr);
     if (index >= 2 * dec->cfg.num_layers) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "cache index out of range");
     CU(dec, cudaSetDevice(dec->cfg.device));
     const uint64_t elems = (uint64_t)dec->cfg.batch * dec->cfg.capacity * dec->cfg.embed_dim;
@@ -1356,6 +1244,7 @@ int tnsr_b200_decoder_read_cache(tnsr_b200_decoder* dec, uint32_t index, float* 
 
 int tnsr_b200_decoder_write_cache(tnsr_b200_decoder* dec, uint32_t index, const float* host_in) {
     if (!dec || !host_in) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "null argument");
+    if (dec->stack) return copy_stack_cache(dec, index, nullptr, host_in);
     if (index >= 2 * dec->cfg.num_layers) return fail(dec, TNSR_B200_ERR_INVALID_ARGUMENT, "cache index out of range");
     CU(dec, cudaSetDevice(dec->cfg.device));
     const uint64_t elems = (uint64_t)dec->cfg.batch * dec->cfg.capacity * dec->cfg.embed_dim;

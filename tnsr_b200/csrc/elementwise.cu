@@ -15,6 +15,7 @@ int launch_layernorm_strict(const float* x, const float* w, const float* b, floa
 // Embedding: out[r, :] = tok[ids[r], :] + pos[position + r % chunk, :]
 // (src/nn/kv_cache/graph.rs:30-41).  The gather is an exact copy and the sum one
 // f32 add per element, so f32 tables reproduce the reference bit for bit.
+// Without a position table (rotary models): out[r, :] = tok[ids[r], :] * scale.
 // One block per row; 4 elements per thread per step.
 // ---------------------------------------------------------------------------
 template <typename T>
@@ -39,7 +40,7 @@ __global__ void __launch_bounds__(128)
 embedding_kernel(const T* __restrict__ tok, const T* __restrict__ pos, const uint32_t* __restrict__ ids,
                  float* __restrict__ out, uint32_t chunk, uint32_t position0,
                  const uint32_t* __restrict__ d_position, uint32_t position_stride, uint32_t vocab, uint32_t width,
-                 int* __restrict__ d_status) {
+                 float scale, int* __restrict__ d_status) {
     pdl_wait();
     pdl_trigger();
     const uint32_t r = blockIdx.x;
@@ -53,6 +54,10 @@ embedding_kernel(const T* __restrict__ tok, const T* __restrict__ pos, const uin
         return;
     }
     const T* tr = tok + (size_t)id * width;
+    if (!pos) {
+        for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) o[c] = load1<T>(tr + c) * scale;
+        return;
+    }
     const T* pr = pos + (size_t)position * width;
     if (width % 4 == 0) {
         for (uint32_t c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
@@ -68,15 +73,15 @@ embedding_kernel(const T* __restrict__ tok, const T* __restrict__ pos, const uin
 
 int launch_embedding(const void* tok, const void* pos, const uint32_t* ids, float* out, uint32_t rows,
                      uint32_t chunk, uint32_t position0, const uint32_t* d_position, uint32_t vocab,
-                     uint32_t width, int dtype, int* d_status, cudaStream_t stream, uint32_t position_stride) {
+                     uint32_t width, int dtype, int* d_status, cudaStream_t stream, uint32_t position_stride, float scale) {
     if (rows == 0) return TNSR_B200_OK;
     if (chunk == 0) return TNSR_B200_ERR_INVALID_ARGUMENT;
     if (dtype == TNSR_B200_BF16)
         launch_kernel(embedding_kernel<bf16>, dim3(rows), dim3(128), 0, stream, (const bf16*)tok, (const bf16*)pos, ids, out,
-                      chunk, position0, d_position, position_stride, vocab, width, d_status);
+                      chunk, position0, d_position, position_stride, vocab, width, scale, d_status);
     else
         launch_kernel(embedding_kernel<float>, dim3(rows), dim3(128), 0, stream, (const float*)tok, (const float*)pos, ids, out,
-                      chunk, position0, d_position, position_stride, vocab, width, d_status);
+                      chunk, position0, d_position, position_stride, vocab, width, scale, d_status);
     count_launch();
     return check_launch("embedding");
 }
@@ -95,10 +100,11 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
-template <bool OUT_BF16>
+// RMS: y = x / sqrt(mean(x^2) + eps) * (w_add + w) -- no mean, no shift; w_add is 1 for weights stored around zero.
+template <bool OUT_BF16, bool RMS>
 __global__ void __launch_bounds__(128)
 layernorm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
-                      void* __restrict__ out, uint32_t rows, uint32_t width, float eps) {
+                      void* __restrict__ out, uint32_t rows, uint32_t width, float eps, float w_add) {
     pdl_wait();
     pdl_trigger();
     const uint32_t lane = threadIdx.x & 31;
@@ -116,13 +122,13 @@ layernorm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w, 
             sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
         }
     }
-    const float mean = warp_sum(sum) / (float)width;
+    const float mean = RMS ? 0.0f : warp_sum(sum) / (float)width;
     float sq = 0.0f;
 #pragma unroll
     for (int i = 0; i < LN_MAX_VEC; ++i) {
         uint32_t c = lane + i * 32;
         if (c < nvec) {
-            v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+            if (!RMS) { v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean; }
             sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
         }
     }
@@ -133,7 +139,8 @@ layernorm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w, 
     for (int i = 0; i < LN_MAX_VEC; ++i) {
         uint32_t c = lane + i * 32;
         if (c < nvec) {
-            float4 ww = wr[c], bb = br[c];
+            float4 ww = wr[c], bb = RMS ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : br[c];
+            if (RMS) { ww.x += w_add; ww.y += w_add; ww.z += w_add; ww.w += w_add; }
             float4 y = make_float4(v[i].x * inv * ww.x + bb.x, v[i].y * inv * ww.y + bb.y,
                                    v[i].z * inv * ww.z + bb.z, v[i].w * inv * ww.w + bb.w);
             if (OUT_BF16) {
@@ -166,10 +173,11 @@ __device__ __forceinline__ float ln_fold_block_sum(float x, float* red) {
     return t;
 }
 
+template <bool RMS>
 __global__ void __launch_bounds__(LN_FOLD_THREADS)
 layernorm_fold_kernel(float* __restrict__ h, const float* __restrict__ partials, uint32_t split_k, uint32_t split_rows,
                       const float* __restrict__ w, const float* __restrict__ b, bf16* __restrict__ out, uint32_t rows,
-                      uint32_t width, float eps) {
+                      uint32_t width, float eps, float w_add) {
     __shared__ float red[LN_FOLD_THREADS / 32];
     pdl_wait();
     pdl_trigger();
@@ -181,7 +189,8 @@ layernorm_fold_kernel(float* __restrict__ h, const float* __restrict__ partials,
     if (live) {
         v = xr[c];
         ww = reinterpret_cast<const float4*>(w)[c];
-        bb = reinterpret_cast<const float4*>(b)[c];
+        if (!RMS) bb = reinterpret_cast<const float4*>(b)[c];
+        else { ww.x += w_add; ww.y += w_add; ww.z += w_add; ww.w += w_add; }
     }
 #pragma unroll
     for (uint32_t s = 0; s < LN_FOLD_MAX; ++s)
@@ -191,8 +200,10 @@ layernorm_fold_kernel(float* __restrict__ h, const float* __restrict__ partials,
         if (s < split_k) { v.x += p[s].x; v.y += p[s].y; v.z += p[s].z; v.w += p[s].w; }
     }
     if (live && split_k) xr[c] = v;
-    const float mean = ln_fold_block_sum(live ? (v.x + v.y) + (v.z + v.w) : 0.0f, red) / (float)width;
-    v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean;
+    if (!RMS) {
+        const float mean = ln_fold_block_sum(live ? (v.x + v.y) + (v.z + v.w) : 0.0f, red) / (float)width;
+        v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean;
+    }
     const float sq = ln_fold_block_sum(live ? (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w) : 0.0f, red);
     const float inv = rsqrtf(sq / (float)width + eps);
     if (live)
@@ -203,10 +214,10 @@ layernorm_fold_kernel(float* __restrict__ h, const float* __restrict__ partials,
 }
 
 // Any width: one block per row, three passes over global memory (L2-resident).
-template <bool OUT_BF16>
+template <bool OUT_BF16, bool RMS>
 __global__ void __launch_bounds__(256)
 layernorm_block_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
-                       void* __restrict__ out, uint32_t width, float eps) {
+                       void* __restrict__ out, uint32_t width, float eps, float w_add) {
     __shared__ float red[8];
     __shared__ float bc;
     pdl_wait();
@@ -224,7 +235,7 @@ layernorm_block_kernel(const float* __restrict__ x, const float* __restrict__ w,
         bc = t / (float)width;
     }
     __syncthreads();
-    const float mean = bc;
+    const float mean = RMS ? 0.0f : bc;
     float sq = 0.0f;
     for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) {
         float d = xr[c] - mean;
@@ -242,10 +253,40 @@ layernorm_block_kernel(const float* __restrict__ x, const float* __restrict__ w,
     __syncthreads();
     const float inv = bc;
     for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) {
-        float y = (xr[c] - mean) * inv * w[c] + b[c];
+        float y = RMS ? xr[c] * inv * (w_add + w[c]) : (xr[c] - mean) * inv * w[c] + b[c];
         if (OUT_BF16) reinterpret_cast<bf16*>(out)[(size_t)blockIdx.x * width + c] = __float2bfloat16_rn(y);
         else reinterpret_cast<float*>(out)[(size_t)blockIdx.x * width + c] = y;
     }
+}
+
+// The fast (non-strict) norms: LayerNorm (RMS = false) and RMS norm share the choice of kernel.
+template <bool RMS>
+static int launch_norm(const float* x, const float* w, const float* b, void* out, uint32_t rows, uint32_t width, float eps,
+                       float w_add, int out_dtype, cudaStream_t stream) {
+    const bool vec_ok = width % 4 == 0 && width <= 32 * 4 * LN_MAX_VEC &&
+                        (reinterpret_cast<uintptr_t>(x) % 16 == 0) && (reinterpret_cast<uintptr_t>(w) % 16 == 0) &&
+                        (reinterpret_cast<uintptr_t>(b) % 16 == 0) && (reinterpret_cast<uintptr_t>(out) % 16 == 0);
+    // Single-token steps (few rows): one block per row with every load of a thread issued at once (layernorm_fold_kernel
+    // with nothing to fold); the row-per-warp kernel fetches scale and shift only after the statistics, a second round
+    // trip that a launch of a few hundred rows has nothing to hide behind.  Many rows (prefill): row per warp, which
+    // runs at 0.94 of the HBM copy rate.
+    if (vec_ok && out_dtype == TNSR_B200_BF16 && t_single_token_step) {
+        launch_kernel(layernorm_fold_kernel<RMS>, dim3(rows), dim3(LN_FOLD_THREADS), 0, stream, const_cast<float*>(x),
+                      static_cast<const float*>(nullptr), 0u, 0u, w, b, reinterpret_cast<bf16*>(out), rows, width, eps, w_add);
+    } else if (vec_ok) {
+        dim3 grid(ceil_div(rows, 4));
+        if (out_dtype == TNSR_B200_BF16)
+            launch_kernel(layernorm_warp_kernel<true, RMS>, grid, dim3(128), 0, stream, x, w, b, out, rows, width, eps, w_add);
+        else
+            launch_kernel(layernorm_warp_kernel<false, RMS>, grid, dim3(128), 0, stream, x, w, b, out, rows, width, eps, w_add);
+    } else {
+        if (out_dtype == TNSR_B200_BF16)
+            launch_kernel(layernorm_block_kernel<true, RMS>, dim3(rows), dim3(256), 0, stream, x, w, b, out, width, eps, w_add);
+        else
+            launch_kernel(layernorm_block_kernel<false, RMS>, dim3(rows), dim3(256), 0, stream, x, w, b, out, width, eps, w_add);
+    }
+    count_launch();
+    return check_launch(RMS ? "rmsnorm" : "layernorm");
 }
 
 int launch_layernorm(const float* x, const float* w, const float* b, void* out, uint32_t rows,
@@ -258,39 +299,20 @@ int launch_layernorm(const float* x, const float* w, const float* b, void* out, 
         }
         return launch_layernorm_strict(x, w, b, (float*)out, rows, width, eps, stream);
     }
-    const bool vec_ok = width % 4 == 0 && width <= 32 * 4 * LN_MAX_VEC &&
-                        (reinterpret_cast<uintptr_t>(x) % 16 == 0) && (reinterpret_cast<uintptr_t>(w) % 16 == 0) &&
-                        (reinterpret_cast<uintptr_t>(b) % 16 == 0) && (reinterpret_cast<uintptr_t>(out) % 16 == 0);
-    // Single-token steps (few rows): one block per row with every load of a thread issued at once (layernorm_fold_kernel
-    // with nothing to fold); the row-per-warp kernel fetches scale and shift only after the statistics, a second round
-    // trip that a launch of a few hundred rows has nothing to hide behind.  Many rows (prefill): row per warp, which
-    // runs at 0.94 of the HBM copy rate.
-    if (vec_ok && out_dtype == TNSR_B200_BF16 && t_single_token_step) {
-        launch_kernel(layernorm_fold_kernel, dim3(rows), dim3(LN_FOLD_THREADS), 0, stream, const_cast<float*>(x),
-                      static_cast<const float*>(nullptr), 0u, 0u, w, b, reinterpret_cast<bf16*>(out), rows, width, eps);
-        count_launch();
-        return check_launch("layernorm");
-    }
-    if (vec_ok) {
-        dim3 grid(ceil_div(rows, 4));
-        if (out_dtype == TNSR_B200_BF16)
-            launch_kernel(layernorm_warp_kernel<true>, grid, dim3(128), 0, stream, x, w, b, out, rows, width, eps);
-        else
-            launch_kernel(layernorm_warp_kernel<false>, grid, dim3(128), 0, stream, x, w, b, out, rows, width, eps);
-    } else {
-        if (out_dtype == TNSR_B200_BF16)
-            launch_kernel(layernorm_block_kernel<true>, dim3(rows), dim3(256), 0, stream, x, w, b, out, width, eps);
-        else
-            launch_kernel(layernorm_block_kernel<false>, dim3(rows), dim3(256), 0, stream, x, w, b, out, width, eps);
-    }
-    count_launch();
-    return check_launch("layernorm");
+    return launch_norm<false>(x, w, b, out, rows, width, eps, 0.0f, out_dtype, stream);
+}
+
+int launch_rmsnorm(const float* x, const float* w, float w_add, void* out, uint32_t rows, uint32_t width, float eps,
+                   int out_dtype, cudaStream_t stream) {
+    if (rows == 0) return TNSR_B200_OK;
+    return launch_norm<true>(x, w, nullptr, out, rows, width, eps, w_add, out_dtype, stream);
 }
 
 bool layernorm_fold_supported(uint32_t width) { return width % 4 == 0 && width <= LN_FOLD_THREADS * 4; }
 
-int launch_layernorm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, const float* b,
-                          void* out, uint32_t rows, uint32_t width, float eps, cudaStream_t stream) {
+template <bool RMS>
+static int launch_norm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, const float* b,
+                            void* out, uint32_t rows, uint32_t width, float eps, float w_add, cudaStream_t stream) {
     if (rows == 0) return TNSR_B200_OK;
     const bool aligned = (reinterpret_cast<uintptr_t>(h) % 16 == 0) && (reinterpret_cast<uintptr_t>(partials) % 16 == 0) &&
                          (reinterpret_cast<uintptr_t>(w) % 16 == 0) && (reinterpret_cast<uintptr_t>(b) % 16 == 0) &&
@@ -299,10 +321,20 @@ int launch_layernorm_fold(float* h, const float* partials, uint32_t split_k, uin
         set_thread_error("layernorm_fold: width, alignment or partial layout outside the kernel");
         return TNSR_B200_ERR_UNSUPPORTED;
     }
-    launch_kernel(layernorm_fold_kernel, dim3(rows), dim3(LN_FOLD_THREADS), 0, stream, h, partials, split_k, split_rows, w, b,
-                  reinterpret_cast<bf16*>(out), rows, width, eps);
+    launch_kernel(layernorm_fold_kernel<RMS>, dim3(rows), dim3(LN_FOLD_THREADS), 0, stream, h, partials, split_k, split_rows, w, b,
+                  reinterpret_cast<bf16*>(out), rows, width, eps, w_add);
     count_launch();
     return check_launch("layernorm_fold");
+}
+
+int launch_layernorm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, const float* b,
+                          void* out, uint32_t rows, uint32_t width, float eps, cudaStream_t stream) {
+    return launch_norm_fold<false>(h, partials, split_k, split_rows, w, b, out, rows, width, eps, 0.0f, stream);
+}
+
+int launch_rmsnorm_fold(float* h, const float* partials, uint32_t split_k, uint32_t split_rows, const float* w, float w_add,
+                        void* out, uint32_t rows, uint32_t width, float eps, cudaStream_t stream) {
+    return launch_norm_fold<true>(h, partials, split_k, split_rows, w, nullptr, out, rows, width, eps, w_add, stream);
 }
 
 // ---------------------------------------------------------------------------
@@ -549,6 +581,28 @@ int launch_pack_gate_up(const bf16* wg, const bf16* wu, const float* bg, const f
     pack_gate_up_kernel<<<flat_grid((uint64_t)2 * f * d), 256, 0, stream>>>(wg, wu, bg, bu, w_out, b_out, d, f);
     count_launch();
     return check_launch("pack_gate_up");
+}
+
+// out[(row0 + r) * ld + col0 + c] = in[r, c] for an [rows, cols] f32 matrix: places one stored [out, in] weight inside a
+// packed operand.
+template <typename T>
+__global__ void pack_rows_kernel(const float* __restrict__ in, T* __restrict__ out, uint32_t rows, uint32_t cols, uint32_t row0,
+                                 uint32_t col0, uint32_t ld) {
+    const uint64_t total = (uint64_t)rows * cols;
+    for (uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (uint64_t)gridDim.x * blockDim.x) {
+        const size_t o = (size_t)(row0 + i / cols) * ld + col0 + i % cols;
+        out[o] = from_f32<T>(in[i]);
+    }
+}
+
+int launch_pack_rows(const float* in, void* out, int dtype, uint32_t rows, uint32_t cols, uint32_t row0, uint32_t col0,
+                     uint32_t ld, cudaStream_t stream) {
+    if (rows == 0 || cols == 0) return TNSR_B200_OK;
+    const unsigned grid = flat_grid((uint64_t)rows * cols);
+    if (dtype == TNSR_B200_BF16) pack_rows_kernel<bf16><<<grid, 256, 0, stream>>>(in, (bf16*)out, rows, cols, row0, col0, ld);
+    else pack_rows_kernel<float><<<grid, 256, 0, stream>>>(in, (float*)out, rows, cols, row0, col0, ld);
+    count_launch();
+    return check_launch("pack_rows");
 }
 
 __global__ void fill_u32_kernel(uint32_t* p, uint32_t value, uint32_t n) {

@@ -28,6 +28,7 @@ thread_local uint32_t t_lose_gemm_stage = 0;
 struct EpiParams {
     GemmEpilogue ep;
     GemmQkvTargets qkv;
+    GemmSegments seg;
     void* out;
     uint32_t ldc;
     uint32_t m, n;  // n = columns of the accumulator (packed width for SWIGLU)
@@ -65,6 +66,22 @@ __device__ __forceinline__ void store_qkv(const EpiParams& P, uint32_t row, uint
         size_t crow = kv_row(P.qkv.paging, session, pos + row % P.qkv.chunk, P.qkv.capacity);
         (which == 1 ? P.qkv.k_cache : P.qkv.v_cache)[crow * d + c] = __float2bfloat16_rn(v);
     }
+}
+
+// Range of column `col` (GEMM_SEGMENTS).
+__device__ __forceinline__ uint32_t segment_of(const EpiParams& P, uint32_t col) {
+    uint32_t i = 0;
+    if (P.seg.count > 1 && col >= P.seg.s[1].col0) i = 1;
+    if (P.seg.count > 2 && col >= P.seg.s[2].col0) i = 2;
+    return i;
+}
+
+__device__ __forceinline__ void store_segment(const EpiParams& P, uint32_t row, uint32_t col, float acc) {
+    const GemmSegment& g = P.seg.s[segment_of(P, col)];
+    const float v = apply_activation(P.ep.bias ? acc + P.ep.bias[col] : acc, g.activation);
+    const size_t o = (size_t)row * g.ld + (col - g.col0);
+    if (g.out_dtype == TNSR_B200_BF16) reinterpret_cast<bf16*>(g.out)[o] = __float2bfloat16_rn(v);
+    else reinterpret_cast<float*>(g.out)[o] = v;
 }
 
 // g, u: accumulators of packed columns pc and pc + 16; output column oc.
@@ -153,6 +170,7 @@ gemm_simple_kernel(const bf16* __restrict__ a, uint32_t lda, const bf16* __restr
             uint32_t r = e / SB, c = e % SB, row = m0 + r, col = n0 + c;
             if (row < P.m && col < P.n) {
                 if (MODE == GEMM_QKV) store_qkv(P, row, col, cs[r][c]);
+                else if (MODE == GEMM_SEGMENTS) store_segment(P, row, col, cs[r][c]);
                 else store_plain(P, row, col, cs[r][c]);
             }
         }
@@ -171,6 +189,7 @@ static int launch_simple(const bf16* a, uint32_t lda, const bf16* bt, const EpiP
         case GEMM_QKV: launch_kernel(gemm_simple_kernel<GEMM_QKV>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
         case GEMM_SWIGLU: launch_kernel(gemm_simple_kernel<GEMM_SWIGLU>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
         case GEMM_ARGMAX: launch_kernel(gemm_simple_kernel<GEMM_ARGMAX>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
+        case GEMM_SEGMENTS: launch_kernel(gemm_simple_kernel<GEMM_SEGMENTS>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
     }
     count_launch();
     return check_launch("gemm_simple");
@@ -403,7 +422,37 @@ __device__ __forceinline__ void epilogue_block(const EpiParams& P, float* stage,
     const uint32_t rows = min(32u, P.m - row0);
     // the vector paths need the whole 32-column block inside the matrix and a 16-byte aligned bias (if any)
     const bool full_cols = col0 + 32 <= P.n && (reinterpret_cast<uintptr_t>(P.ep.bias) & 15) == 0;
-    if (MODE == GEMM_SWIGLU) {
+    if (MODE == GEMM_SEGMENTS) {
+        // the whole block belongs to one column range: bf16, a lane converts 8 columns of one row; f32, 4 columns
+        const uint32_t si = segment_of(P, col0);
+        void* base = P.seg.s[si].out;
+        const uint32_t ld = P.seg.s[si].ld, c0 = col0 - P.seg.s[si].col0;
+        const int act = P.seg.s[si].activation;
+        const bool to_bf16 = P.seg.s[si].out_dtype == TNSR_B200_BF16;
+        if (full_cols && to_bf16 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(base) & 15) == 0) {
+            const uint32_t cg = lane & 3, rsub = lane >> 2, c8 = 8 * cg;
+            bf16* out = reinterpret_cast<bf16*>(base);
+            float4 b0 = make_float4(0.f, 0.f, 0.f, 0.f), b1 = b0;
+            if (P.ep.bias) {
+                b0 = __ldg(reinterpret_cast<const float4*>(P.ep.bias + col0 + c8));
+                b1 = __ldg(reinterpret_cast<const float4*>(P.ep.bias + col0 + c8 + 4));
+            }
+#pragma unroll
+            for (uint32_t it = 0; it < 4; ++it) {
+                const uint32_t rr = it * 8 + rsub;
+                if (rr < rows) {
+                    float4 v0 = stage_load4(stage, rr, c8), v1 = stage_load4(stage, rr, c8 + 4);
+                    v0 = act4(make_float4(v0.x + b0.x, v0.y + b0.y, v0.z + b0.z, v0.w + b0.w), act);
+                    v1 = act4(make_float4(v1.x + b1.x, v1.y + b1.y, v1.z + b1.z, v1.w + b1.w), act);
+                    *reinterpret_cast<uint4*>(out + (size_t)(row0 + rr) * ld + c0 + c8) =
+                        make_uint4(pack_bf16x2(v0.x, v0.y), pack_bf16x2(v0.z, v0.w), pack_bf16x2(v1.x, v1.y), pack_bf16x2(v1.z, v1.w));
+                }
+            }
+        } else {
+            for (uint32_t rr = 0; rr < rows; ++rr)
+                if (col0 + lane < P.n) store_segment(P, row0 + rr, col0 + lane, stage[stage_index(rr, lane)]);
+        }
+    } else if (MODE == GEMM_SWIGLU) {
         // columns [0,16) are gate, [16,32) the matching up columns.  A lane makes 4 outputs of one row:
         // 4 lanes per row, 8 rows per step.
         const uint32_t j = lane & 3, rsub = lane >> 2;
@@ -789,6 +838,7 @@ static int launch_tc_mode(const CUtensorMap& ma, const CUtensorMap& mb, const CU
         case GEMM_QKV: return launch_tc_t<BN, GEMM_QKV>(ma, mb, mo, prm, stream);
         case GEMM_SWIGLU: return launch_tc_t<BN, GEMM_SWIGLU>(ma, mb, mo, prm, stream);
         case GEMM_ARGMAX: return launch_tc_t<BN, GEMM_ARGMAX>(ma, mb, mo, prm, stream);
+        case GEMM_SEGMENTS: return launch_tc_t<BN, GEMM_SEGMENTS>(ma, mb, mo, prm, stream);
     }
     return TNSR_B200_ERR_INVALID_ARGUMENT;
 }
@@ -802,7 +852,7 @@ static bool tc_eligible(const bf16* a, uint32_t lda, const bf16* bt, uint32_t k)
 // tiles the chosen engine used, which GEMM_ARGMAX callers need to read the candidates back.
 static int launch_gemm_impl(const bf16* a, const bf16* bt, void* out, uint32_t ldc, uint32_t m, uint32_t n, uint32_t k,
                             GemmMode mode, const GemmEpilogue& ep, const GemmQkvTargets* qkv, int* d_status,
-                            uint32_t* tiles_n_out, cudaStream_t stream) {
+                            uint32_t* tiles_n_out, cudaStream_t stream, const GemmSegments* segments = nullptr) {
     if (m == 0 || n == 0) return TNSR_B200_OK;
     if (k == 0) return TNSR_B200_ERR_INVALID_ARGUMENT;
     if (mode == GEMM_QKV && (!qkv || qkv->d == 0 || n != 3 * qkv->d || qkv->chunk == 0)) return TNSR_B200_ERR_INVALID_ARGUMENT;
@@ -812,6 +862,17 @@ static int launch_gemm_impl(const bf16* a, const bf16* bt, void* out, uint32_t l
     }
     if (ep.residual && ep.out_dtype != TNSR_B200_F32) return TNSR_B200_ERR_INVALID_ARGUMENT;
     EpiParams P;
+    if (mode == GEMM_SEGMENTS) {
+        bool fits = segments && segments->count >= 1 && segments->count <= 3 && segments->s[0].col0 == 0 && n % 32 == 0;
+        for (uint32_t i = 0; fits && i < segments->count; ++i)
+            fits = segments->s[i].out && segments->s[i].col0 % 32 == 0 && segments->s[i].col0 < n &&
+                   (i == 0 || segments->s[i].col0 > segments->s[i - 1].col0);
+        if (!fits) {
+            set_thread_error("gemm: column ranges must start at multiples of 32, in order, inside the matrix");
+            return TNSR_B200_ERR_INVALID_ARGUMENT;
+        }
+        P.seg = *segments;
+    }
     P.ep = ep;
     if (qkv) P.qkv = *qkv;
     P.out = out;
@@ -988,8 +1049,15 @@ uint32_t gemm_split_k(const bf16* a, const bf16* bt, uint32_t m, uint32_t n, uin
 int launch_gemm_bf16(const bf16* a, const bf16* bt, void* out, uint32_t ldc, uint32_t m, uint32_t n,
                      uint32_t k, GemmMode mode, const GemmEpilogue& ep, const GemmQkvTargets* qkv,
                      int* d_status, cudaStream_t stream) {
-    if (mode == GEMM_ARGMAX) return TNSR_B200_ERR_INVALID_ARGUMENT;  // use launch_lm_head_argmax
+    if (mode == GEMM_ARGMAX || mode == GEMM_SEGMENTS) return TNSR_B200_ERR_INVALID_ARGUMENT;  // launchers of their own below
     return launch_gemm_impl(a, bt, out, ldc, m, n, k, mode, ep, qkv, d_status, nullptr, stream);
+}
+
+int launch_gemm_segments(const bf16* a, const bf16* bt, uint32_t m, uint32_t n, uint32_t k, const float* bias,
+                         const GemmSegments& segments, int* d_status, cudaStream_t stream) {
+    GemmEpilogue ep;
+    ep.bias = bias;
+    return launch_gemm_impl(a, bt, nullptr, n, m, n, k, GEMM_SEGMENTS, ep, nullptr, d_status, nullptr, stream, &segments);
 }
 
 // ---- greedy ids from the LM head without materialising logits --------------------

@@ -1,0 +1,279 @@
+// The attention mixer of models described layer by layer: projections pass a short causal convolution, q and k an RMS
+// norm per head and a rotation, and grouped-query attention runs on capped scores with a sigmoid gate per head.
+//
+//  * attention_prep_kernel     one warp per (head unit, run of tokens): the convolution slides over the run in
+//                              registers, so every projected value is read once; q rows and cache rows come out.
+//  * grouped_attention_rows    one warp per (session, head, query), keys in order: f32 sessions, and every shape the
+//                              tensor-core kernels (grouped_attention.cu) leave out.
+#include <algorithm>
+
+#include "mixers.cuh"
+
+namespace tb {
+
+__device__ __forceinline__ float mx_warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+template <typename T>
+__device__ __forceinline__ float2 load_pair(const T* p, bool vec, bool second);
+template <>
+__device__ __forceinline__ float2 load_pair<float>(const float* p, bool vec, bool second) {
+    if (vec) return *reinterpret_cast<const float2*>(p);
+    return make_float2(p[0], second ? p[1] : 0.0f);
+}
+template <>
+__device__ __forceinline__ float2 load_pair<bf16>(const bf16* p, bool vec, bool second) {
+    if (vec) return bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(p));
+    return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.0f);
+}
+template <typename T>
+__device__ __forceinline__ void store_pair(T* p, float2 v, bool vec, bool second);
+template <>
+__device__ __forceinline__ void store_pair<float>(float* p, float2 v, bool vec, bool second) {
+    if (vec) { *reinterpret_cast<float2*>(p) = v; return; }
+    p[0] = v.x;
+    if (second) p[1] = v.y;
+}
+template <>
+__device__ __forceinline__ void store_pair<bf16>(bf16* p, float2 v, bool vec, bool second) {
+    if (vec) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); return; }
+    p[0] = __float2bfloat16_rn(v.x);
+    if (second) p[1] = __float2bfloat16_rn(v.y);
+}
+
+// NP: channel pairs per lane (a head unit has at most 64 NP channels).  TAPS: compiled window length; shorter filters are
+// padded with zero weights at the old end and never touch the padded rows.
+template <typename T, int NP, int TAPS>
+__global__ void __launch_bounds__(128)
+attention_prep_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t runs, uint32_t total, uint32_t vec) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t lane = threadIdx.x & 31;
+    const uint32_t task = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (task >= total) return;
+    const uint32_t units = a.heads + 2 * a.kv_heads;
+    const uint32_t unit = task % units, r = (task / units) % runs, s = task / (units * runs);
+    const uint32_t nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
+    const uint32_t channels = nq + nk + a.kv_heads * a.vdim;
+    const uint32_t which = unit < a.heads ? 0u : unit < a.heads + a.kv_heads ? 1u : 2u;
+    const uint32_t head = which == 0 ? unit : which == 1 ? unit - a.heads : unit - a.heads - a.kv_heads;
+    const uint32_t width = which == 2 ? a.vdim : a.dim;
+    const uint32_t ch0 = which == 0 ? head * a.dim : which == 1 ? nq + head * a.dim : nq + nk + head * a.vdim;
+    const T* rows = reinterpret_cast<const T*>(a.proj) + (size_t)s * place.chunk * a.ld + ch0;
+    T* ring = reinterpret_cast<T*>(a.ring) + (size_t)s * a.taps * channels + ch0;
+    const uint32_t p0 = place.pos(s);
+    const uint32_t t0 = r * run, t1 = min(place.chunk, t0 + run);
+
+    float2 w[TAPS][NP], nw[NP], win[TAPS][NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const uint32_t c = 2 * (lane + 32 * i);
+        nw[i] = make_float2(1.0f, 1.0f);
+        if (which < 2 && c < width) {
+            const float* g = which == 0 ? a.q_norm : a.k_norm;
+            nw[i] = make_float2(g[c], c + 1 < width ? g[c + 1] : 0.0f);
+        }
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const int src = j - (TAPS - (int)a.taps);
+            const bool ok = src >= 0 && c < width;
+            w[j][i].x = ok ? a.conv_w[(size_t)(ch0 + c) * a.taps + src] : 0.0f;
+            w[j][i].y = ok && c + 1 < width ? a.conv_w[(size_t)(ch0 + c + 1) * a.taps + src] : 0.0f;
+            // the window holds tokens t - TAPS + 1 .. t; before the first token: t0 - TAPS + 1 .. t0 - 1 in slots 1 ..
+            win[j][i] = make_float2(0.0f, 0.0f);
+            const int t = (int)t0 - TAPS + j;      // token that slot j holds before the first shift
+            if (j > 0 && (int)t0 - t < (int)a.taps && c < width) {
+                const long long pos = (long long)p0 + t;
+                if (t >= 0) win[j][i] = load_pair<T>(rows + (size_t)t * a.ld + c, vec, c + 1 < width);
+                else if (pos >= 0) win[j][i] = load_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, vec, c + 1 < width);
+            }
+        }
+    }
+    const uint32_t pairs = a.rotary_dims / 2;
+    for (uint32_t t = t0; t < t1; ++t) {
+        float2 y[NP];
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const uint32_t c = 2 * (lane + 32 * i);
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
+            win[TAPS - 1][i] = c < width ? load_pair<T>(rows + (size_t)t * a.ld + c, vec, c + 1 < width) : make_float2(0.0f, 0.0f);
+            y[i] = make_float2(0.0f, 0.0f);
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                y[i].x = fmaf(w[j][i].x, win[j][i].x, y[i].x);
+                y[i].y = fmaf(w[j][i].y, win[j][i].y, y[i].y);
+            }
+            ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, ss));
+        }
+        const uint32_t pos = p0 + t;
+        if (place.chunk == 1) {
+            // the slot of this position held the oldest row, which no single-token step reads
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                const uint32_t c = 2 * (lane + 32 * i);
+                if (c < width) store_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, win[TAPS - 1][i], vec, c + 1 < width);
+            }
+        }
+        if (which < 2) {
+            const float inv = rsqrtf(mx_warp_sum(ss) / (float)width + a.eps);
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                const uint32_t pi = lane + 32 * i;
+                y[i].x *= inv * nw[i].x;
+                y[i].y *= inv * nw[i].y;
+                if (pi < pairs) {
+                    const float2 cs = a.rotation[(size_t)pos * pairs + pi];
+                    y[i] = make_float2(y[i].x * cs.x - y[i].y * cs.y, y[i].y * cs.x + y[i].x * cs.y);
+                }
+            }
+        }
+        T* dst;
+        if (which == 0) dst = reinterpret_cast<T*>(a.q) + ((size_t)s * place.chunk + t) * nq + head * a.dim;
+        else {
+            const size_t row = kv_row(a.paging, s, pos, a.capacity);
+            dst = which == 1 ? reinterpret_cast<T*>(a.k_cache) + row * nk + head * a.dim
+                             : reinterpret_cast<T*>(a.v_cache) + row * ((size_t)a.kv_heads * a.vdim) + head * a.vdim;
+        }
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const uint32_t c = 2 * (lane + 32 * i);
+            if (c < width) store_pair<T>(dst + c, y[i], vec, c + 1 < width);
+        }
+    }
+}
+
+template <typename T, int NP>
+static void prep_taps(const AttentionPrep& a, const StepPlace& place, uint32_t run, uint32_t runs, uint32_t total, uint32_t vec,
+                      cudaStream_t stream) {
+    const dim3 grid(ceil_div(total, 4)), block(128);
+    if (a.taps <= 4) launch_kernel(attention_prep_kernel<T, NP, 4>, grid, block, 0, stream, a, place, run, runs, total, vec);
+    else launch_kernel(attention_prep_kernel<T, NP, kMaxConvTaps>, grid, block, 0, stream, a, place, run, runs, total, vec);
+}
+
+template <typename T>
+static void prep_width(const AttentionPrep& a, const StepPlace& place, uint32_t run, uint32_t runs, uint32_t total, cudaStream_t stream) {
+    const uint32_t width = std::max(a.dim, a.vdim);
+    // pairs move as one access when every head starts at an even channel of an even row
+    const uint32_t vec = a.dim % 2 == 0 && a.vdim % 2 == 0 && a.ld % 2 == 0;
+    if (width <= 64) prep_taps<T, 1>(a, place, run, runs, total, vec, stream);
+    else if (width <= 128) prep_taps<T, 2>(a, place, run, runs, total, vec, stream);
+    else prep_taps<T, 4>(a, place, run, runs, total, vec, stream);
+}
+
+int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dtype, cudaStream_t stream) {
+    if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
+    if (a.dim > 256 || a.vdim > 256 || a.taps == 0 || a.taps > kMaxConvTaps || a.rotary_dims > a.dim || a.rotary_dims % 2) {
+        set_thread_error("attention: head widths up to 256, 1..16 convolution taps, an even number of rotated dimensions");
+        return TNSR_B200_ERR_UNSUPPORTED;
+    }
+    const uint32_t run = std::min(place.chunk, 16u), runs = ceil_div(place.chunk, run);
+    const uint64_t total = (uint64_t)place.sessions * runs * (a.heads + 2 * a.kv_heads);
+    if (total > 0x7fffffffull) { set_thread_error("attention: too many rows for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
+    if (dtype == TNSR_B200_BF16) prep_width<bf16>(a, place, run, runs, (uint32_t)total, stream);
+    else prep_width<float>(a, place, run, runs, (uint32_t)total, stream);
+    count_launch();
+    return check_launch("attention_prep");
+}
+
+// ---- convolution inputs of a multi-token chunk into the session's ring ---------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_ring_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, T* __restrict__ ring, StepPlace place) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t s = blockIdx.y, keep = min(place.chunk, taps);
+    const uint32_t p0 = place.pos(s);
+    for (uint32_t i = blockIdx.x * blockDim.x + threadIdx.x; i < keep * channels; i += gridDim.x * blockDim.x) {
+        const uint32_t t = place.chunk - keep + i / channels, c = i % channels;
+        ring[((size_t)s * taps + (p0 + t) % taps) * channels + c] = rows[((size_t)s * place.chunk + t) * ld + c];
+    }
+}
+
+int launch_conv_ring(const void* rows, uint32_t ld, uint32_t channels, uint32_t taps, void* ring, const StepPlace& place,
+                     int dtype, cudaStream_t stream) {
+    if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
+    if (place.sessions > 65535u) { set_thread_error("convolution: too many sessions for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
+    const dim3 grid(std::min(ceil_div(std::min(place.chunk, taps) * channels, 256u), 64u), place.sessions);
+    if (dtype == TNSR_B200_BF16)
+        launch_kernel(conv_ring_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)rows, ld, channels, taps, (bf16*)ring, place);
+    else
+        launch_kernel(conv_ring_kernel<float>, grid, dim3(256), 0, stream, (const float*)rows, ld, channels, taps, (float*)ring, place);
+    count_launch();
+    return check_launch("conv_ring");
+}
+
+// ---- one warp per (session, head, query) -----------------------------------------------------
+constexpr int GR_SLOTS = 8;   // widths up to 256: lane owns columns lane, lane + 32, ...
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+grouped_attention_rows_kernel(GroupedAttention a, StepPlace place, uint32_t total) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t lane = threadIdx.x & 31;
+    const uint32_t task = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (task >= total) return;
+    const uint32_t t = task % place.chunk, h = (task / place.chunk) % a.heads, s = task / (place.chunk * a.heads);
+    const uint32_t g = h / (a.heads / a.kv_heads);
+    const size_t row = (size_t)s * place.chunk + t;
+    const T* qr = reinterpret_cast<const T*>(a.q) + row * ((size_t)a.heads * a.dim) + (size_t)h * a.dim;
+    const T* kb = reinterpret_cast<const T*>(a.k_cache) + (size_t)g * a.dim;
+    const T* vb = reinterpret_cast<const T*>(a.v_cache) + (size_t)g * a.vdim;
+    const size_t k_ld = (size_t)a.kv_heads * a.dim, v_ld = (size_t)a.kv_heads * a.vdim;
+    const uint32_t keys = min(place.pos(s) + t + 1, a.capacity);
+    float q[GR_SLOTS], acc[GR_SLOTS];
+#pragma unroll
+    for (int i = 0; i < GR_SLOTS; ++i) {
+        const uint32_t c = lane + 32 * i;
+        q[i] = c < a.dim ? to_f32(qr[c]) : 0.0f;
+        acc[i] = 0.0f;
+    }
+    float m = -INFINITY, l = 0.0f;
+    for (uint32_t j = 0; j < keys; ++j) {
+        const size_t kr = kv_row(a.paging, s, j, a.capacity);
+        float part = 0.0f;
+#pragma unroll
+        for (int i = 0; i < GR_SLOTS; ++i) {
+            const uint32_t c = lane + 32 * i;
+            if (c < a.dim) part = fmaf(q[i], to_f32(kb[kr * k_ld + c]), part);
+        }
+        float sc = mx_warp_sum(part) * a.scale;
+        if (a.softcap > 0.0f) sc = a.softcap * tanhf(sc / a.softcap);
+        const float m_new = fmaxf(m, sc);
+        const float corr = expf(m - m_new), p = expf(sc - m_new);
+        l = l * corr + p;
+#pragma unroll
+        for (int i = 0; i < GR_SLOTS; ++i) {
+            const uint32_t c = lane + 32 * i;
+            if (c < a.vdim) acc[i] = fmaf(acc[i], corr, p * to_f32(vb[kr * v_ld + c]));
+        }
+        m = m_new;
+    }
+    const float gate = a.gate ? 1.0f / (1.0f + expf(-a.gate[row * a.gate_ld + h])) : 1.0f;
+    T* orow = reinterpret_cast<T*>(a.out) + row * a.out_ld;
+#pragma unroll
+    for (int i = 0; i < GR_SLOTS; ++i) {
+        const uint32_t c = lane + 32 * i;
+        if (c < a.vdim) orow[(size_t)h * a.vdim + c] = from_f32<T>(acc[i] / l * gate);
+    }
+    if (h + 1 == a.heads)
+        for (uint32_t c = a.heads * a.vdim + lane; c < a.out_cols; c += 32) orow[c] = from_f32<T>(0.0f);
+}
+
+int launch_grouped_attention_rows(const GroupedAttention& a, const StepPlace& place, int dtype, cudaStream_t stream) {
+    const uint64_t total = (uint64_t)place.sessions * place.chunk * a.heads;
+    if (total > 0x7fffffffull) { set_thread_error("attention: too many rows for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
+    if (dtype == TNSR_B200_BF16)
+        launch_kernel(grouped_attention_rows_kernel<bf16>, dim3((unsigned)ceil_div64(total, 4)), dim3(128), 0, stream, a, place, (uint32_t)total);
+    else
+        launch_kernel(grouped_attention_rows_kernel<float>, dim3((unsigned)ceil_div64(total, 4)), dim3(128), 0, stream, a, place, (uint32_t)total);
+    count_launch();
+    return check_launch("grouped_attention_rows");
+}
+
+}  // namespace tb

@@ -1,0 +1,234 @@
+// The mamba2 (state-space duality) mixer of models described layer by layer.  Per head an f32 state S [state, vdim]:
+//     S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t
+// with x, B, C behind a causal convolution and silu, dt behind softplus, then y * silu(z) and an RMS norm in groups.
+//
+//  * conv_silu_kernel          convolution + silu of a multi-token chunk, sliding window in registers
+//  * ssd_token_kernel          token by token with the state in registers: single-token steps (convolution fused in,
+//                              the state makes one trip through HBM), f32 sessions, and shapes the chunked scan leaves out
+//  * gated_norm_kernel         the grouped RMS norm of y * silu(z)
+// The chunked tensor-core scan of long chunks is in ssd_scan.cu.
+#include <algorithm>
+
+#include "mixers.cuh"
+
+namespace tb {
+
+__device__ __forceinline__ float full_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+
+// ---- convolution + silu ----------------------------------------------------------------------
+// A thread owns one channel of a run of tokens.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, const float* __restrict__ conv_w,
+                 const float* __restrict__ conv_b, const T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= channels) return;
+    const uint32_t s = blockIdx.z, t0 = blockIdx.y * run, t1 = min(place.chunk, t0 + run);
+    const uint32_t p0 = place.pos(s);
+    const T* in = rows + (size_t)s * place.chunk * ld + c;
+    float w[TAPS], win[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+        const int src = j - (TAPS - (int)taps);
+        w[j] = src >= 0 ? conv_w[(size_t)c * taps + src] : 0.0f;
+        win[j] = 0.0f;
+        const int t = (int)t0 - TAPS + j;
+        if (j > 0 && (int)t0 - t < (int)taps) {
+            const long long pos = (long long)p0 + t;
+            if (t >= 0) win[j] = to_f32(in[(size_t)t * ld]);
+            else if (pos >= 0) win[j] = to_f32(ring[((size_t)s * taps + pos % taps) * channels + c]);
+        }
+    }
+    const float b = conv_b[c];
+    for (uint32_t t = t0; t < t1; ++t) {
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+        win[TAPS - 1] = to_f32(in[(size_t)t * ld]);
+        float y = b;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], win[j], y);
+        out[((size_t)s * place.chunk + t) * channels + c] = from_f32<T>(full_silu(y));
+    }
+}
+
+template <typename T>
+static void conv_silu_typed(const Mamba2& m, uint32_t inner, uint32_t channels, const StepPlace& place, cudaStream_t stream) {
+    const uint32_t run = std::min(place.chunk, 32u);
+    const dim3 grid(ceil_div(channels, 128u), ceil_div(place.chunk, run), place.sessions);
+    const T* rows = (const T*)m.proj + inner;
+    if (m.taps <= 4)
+        launch_kernel(conv_silu_kernel<T, 4>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b, (const T*)m.ring,
+                      (T*)m.xbc, place, run);
+    else
+        launch_kernel(conv_silu_kernel<T, kMaxConvTaps>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b,
+                      (const T*)m.ring, (T*)m.xbc, place, run);
+}
+
+// ---- token by token ----------------------------------------------------------------------------
+// Block = (slice of at most 64 columns of the state, head, session).  Thread (p, k) holds S[k + NG i, p] of its slice for
+// i < ROWS.  FUSED (single-token steps): x, B and C are convolved here from the projected row and the ring; the ring rows
+// are written by the block that is first to own the channel (x: the head's own slice, B and C: the group's first head).
+constexpr uint32_t SSD_THREADS = 256, SSD_SLICE = 64, SSD_MAX_STATE = 256;
+
+template <typename T, int ROWS, bool FUSED>
+__global__ void __launch_bounds__(SSD_THREADS)
+ssd_token_kernel(Mamba2 m, StepPlace place) {
+    __shared__ float sb[SSD_MAX_STATE], sc[SSD_MAX_STATE], sx[SSD_SLICE], red[SSD_THREADS];
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t tid = threadIdx.x;
+    const uint32_t p_first = blockIdx.x * SSD_SLICE, h = blockIdx.y, s = blockIdx.z;
+    const uint32_t width = min(SSD_SLICE, m.vdim - p_first);
+    const uint32_t ng = SSD_THREADS / width;                 // row groups
+    const uint32_t p = tid % width, k = tid / width;
+    const bool live = k < ng;
+    const uint32_t inner = m.heads * m.vdim, gn = m.groups * m.state, channels = inner + 2 * gn;
+    const uint32_t group = h / (m.heads / m.groups);
+    const uint32_t p0 = place.pos(s);
+    float* state = m.ssm + (((size_t)s * m.heads + h) * m.state) * m.vdim + p_first + p;
+    float S[ROWS];
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const uint32_t n = k + ng * i;
+        S[i] = live && n < m.state && p0 > 0 ? state[(size_t)n * m.vdim] : 0.0f;
+    }
+    const float a = -expf(m.a_log[h]), dt_bias = m.dt_bias[h], skip = m.d_skip[h];
+    for (uint32_t t = 0; t < place.chunk; ++t) {
+        const size_t row = (size_t)s * place.chunk + t;
+        const float dt = softplus(m.dt[row * m.dt_ld + h] + dt_bias);
+        // this token's x slice, B and C
+        const uint32_t count = width + 2 * m.state;
+        for (uint32_t i = tid; i < count; i += SSD_THREADS) {
+            const uint32_t ch = i < width ? h * m.vdim + p_first + i
+                              : i < width + m.state ? inner + group * m.state + (i - width)
+                                                    : inner + gn + group * m.state + (i - width - m.state);
+            float v;
+            if (FUSED) {
+                const T* in = reinterpret_cast<const T*>(m.proj) + row * m.ld + inner + ch;
+                T* ring = reinterpret_cast<T*>(m.ring) + (size_t)s * m.taps * channels + ch;
+                const float* w = m.conv_w + (size_t)ch * m.taps;
+                const T now = *in;
+                v = fmaf(w[m.taps - 1], to_f32(now), m.conv_b[ch]);
+                for (uint32_t lag = 1; lag < m.taps && lag <= p0; ++lag)
+                    v = fmaf(w[m.taps - 1 - lag], to_f32(ring[(size_t)((p0 - lag) % m.taps) * channels]), v);
+                v = full_silu(v);
+                v = to_f32(from_f32<T>(v));     // the value a longer chunk would have stored
+                if (i < width || (h % (m.heads / m.groups) == 0 && p_first == 0)) ring[(size_t)(p0 % m.taps) * channels] = now;
+            } else {
+                v = to_f32(reinterpret_cast<const T*>(m.xbc)[row * channels + ch]);
+            }
+            if (i < width) sx[i] = v;
+            else if (i < width + m.state) sb[i - width] = v;
+            else sc[i - width - m.state] = v;
+        }
+        __syncthreads();
+        const float decay = expf(a * dt);
+        float acc = 0.0f;
+        if (live) {
+            const float xdt = dt * sx[p];
+#pragma unroll
+            for (int i = 0; i < ROWS; ++i) {
+                const uint32_t n = k + ng * i;
+                if (n < m.state) {
+                    S[i] = fmaf(S[i], decay, sb[n] * xdt);
+                    acc = fmaf(S[i], sc[n], acc);
+                }
+            }
+        }
+        red[tid] = acc;
+        __syncthreads();
+        if (tid < width) {
+            float y = skip * sx[tid];
+            for (uint32_t j = 0; j < ng; ++j) y += red[j * width + tid];
+            const uint32_t col = h * m.vdim + p_first + tid;
+            const float z = to_f32(reinterpret_cast<const T*>(m.proj)[row * m.ld + col]);
+            reinterpret_cast<T*>(m.gated)[row * inner + col] = from_f32<T>(y * full_silu(z));
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const uint32_t n = k + ng * i;
+        if (live && n < m.state) state[(size_t)n * m.vdim] = S[i];
+    }
+}
+
+template <typename T, bool FUSED>
+static void ssd_token_rows(const Mamba2& m, const StepPlace& place, cudaStream_t stream) {
+    const uint32_t width = std::min(m.vdim, SSD_SLICE), rows = ceil_div(m.state, SSD_THREADS / width);
+    const dim3 grid(ceil_div(m.vdim, SSD_SLICE), m.heads, place.sessions), block(SSD_THREADS);
+    if (rows <= 8) launch_kernel(ssd_token_kernel<T, 8, FUSED>, grid, block, 0, stream, m, place);
+    else if (rows <= 32) launch_kernel(ssd_token_kernel<T, 32, FUSED>, grid, block, 0, stream, m, place);
+    else launch_kernel(ssd_token_kernel<T, 64, FUSED>, grid, block, 0, stream, m, place);
+}
+
+bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state) {
+    return heads > 0 && heads <= 65535u && vdim > 0 && state > 0 && state <= SSD_MAX_STATE;
+}
+
+// ---- grouped RMS norm ------------------------------------------------------------------------------
+// One block per (row, norm group).
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_norm_kernel(const T* __restrict__ gated, const float* __restrict__ w, T* __restrict__ out, uint32_t inner, uint32_t groups,
+                  uint32_t out_ld, uint32_t out_cols, float eps) {
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const size_t row = blockIdx.x;
+    const uint32_t part = inner / groups, c0 = blockIdx.y * part;
+    const T* in = gated + row * inner + c0;
+    float ss = 0.0f;
+    for (uint32_t c = threadIdx.x; c < part; c += blockDim.x) { const float v = to_f32(in[c]); ss = fmaf(v, v, ss); }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float sum = 0.0f;
+    for (uint32_t i = 0; i < blockDim.x / 32; ++i) sum += red[i];
+    const float inv = rsqrtf(sum / (float)part + eps);
+    T* o = out + row * out_ld + c0;
+    for (uint32_t c = threadIdx.x; c < part; c += blockDim.x) o[c] = from_f32<T>(to_f32(in[c]) * inv * w[c0 + c]);
+    if (blockIdx.y == 0)
+        for (uint32_t c = inner + threadIdx.x; c < out_cols; c += blockDim.x) out[row * out_ld + c] = from_f32<T>(0.0f);
+}
+
+int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream_t stream) {
+    if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
+    const uint32_t inner = m.heads * m.vdim, channels = inner + 2 * m.groups * m.state, rows = place.sessions * place.chunk;
+    if (!mamba2_supported(m.heads, m.vdim, m.state) || m.taps == 0 || m.taps > kMaxConvTaps || place.sessions > 65535u ||
+        ceil_div(place.chunk, 32u) > 65535u || m.norm_groups > 65535u) {
+        set_thread_error("mamba2: at most 256 state rows, 16 convolution taps, 65535 sessions");
+        return TNSR_B200_ERR_UNSUPPORTED;
+    }
+    const bool bf = dtype == TNSR_B200_BF16;
+    int rc;
+    if (place.chunk == 1) {
+        if (bf) ssd_token_rows<bf16, true>(m, place, stream); else ssd_token_rows<float, true>(m, place, stream);
+        count_launch();
+        if ((rc = check_launch("ssd_token"))) return rc;
+    } else {
+        if (bf) conv_silu_typed<bf16>(m, inner, channels, place, stream); else conv_silu_typed<float>(m, inner, channels, place, stream);
+        count_launch();
+        if ((rc = check_launch("conv_silu"))) return rc;
+        const uint8_t* raw = (const uint8_t*)m.proj + (size_t)inner * (bf ? 2 : 4);
+        if ((rc = launch_conv_ring(raw, m.ld, channels, m.taps, m.ring, place, dtype, stream))) return rc;
+        if (bf) ssd_token_rows<bf16, false>(m, place, stream); else ssd_token_rows<float, false>(m, place, stream);
+        count_launch();
+        if ((rc = check_launch("ssd_token"))) return rc;
+    }
+    const dim3 grid(rows, m.norm_groups);
+    if (bf)
+        launch_kernel(gated_norm_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)m.gated, m.norm_w, (bf16*)m.out, inner, m.norm_groups,
+                      m.out_ld, m.out_cols, m.eps);
+    else
+        launch_kernel(gated_norm_kernel<float>, grid, dim3(256), 0, stream, (const float*)m.gated, m.norm_w, (float*)m.out, inner,
+                      m.norm_groups, m.out_ld, m.out_cols, m.eps);
+    count_launch();
+    return check_launch("gated_norm");
+}
+
+}  // namespace tb

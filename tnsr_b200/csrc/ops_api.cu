@@ -53,7 +53,8 @@ int tnsr_b200_gemm_bf16_ws(const void* a, const void* bt, const float* bias, con
                            void* stream) {
     if (!a || !bt || !out) return bad("gemm_bf16: null pointer");
     if (out_dtype != TNSR_B200_F32 && out_dtype != TNSR_B200_BF16) return bad("gemm_bf16: bad output dtype");
-    if (activation < -1 || activation > TNSR_B200_ACT_GELU) return bad("gemm_bf16: activation must be -1, RELU or GELU");
+    if (activation < -1 || activation > TNSR_B200_ACT_GELU_TANH || activation == TNSR_B200_ACT_SWIGLU)
+        return bad("gemm_bf16: activation must be -1, RELU, GELU or GELU_TANH");
     if (residual && out_dtype != TNSR_B200_F32) return bad("gemm_bf16: a residual needs f32 output");
     GemmEpilogue ep;
     ep.bias = bias;

@@ -41,6 +41,11 @@ __device__ __forceinline__ float strict_gelu(float x) {
     return x * (a + b);
 }
 
+// tanh form of gelu in f32 with the full-precision tanh.
+__device__ __forceinline__ float strict_gelu_tanh(float x) {
+    return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * (x + 0.044715f * (x * x * x))));
+}
+
 // ---------------------------------------------------------------------------
 // GEMM: one thread per output element, K walked in order through 16-wide
 // shared tiles.  The tiling changes which thread loads what, not the order in
@@ -78,6 +83,7 @@ gemm_strict_kernel(const float* __restrict__ a, const float* __restrict__ b, voi
     if (ep.bias) v = v + ep.bias[col];
     if (ep.activation == ACT_RELU) v = fmaxf(v, 0.0f);
     else if (ep.activation == ACT_GELU) v = strict_gelu(v);
+    else if (ep.activation == ACT_GELU_TANH) v = strict_gelu_tanh(v);
     if (ep.residual) v = ep.residual[(size_t)row * ep.ldr + col] + v;
     if (ep.round_bf16) v = round_to_bf16(v);
     size_t orow = row;
@@ -127,6 +133,7 @@ gemm_strict_rows_kernel(const float* __restrict__ a, const float* __restrict__ b
     if (ep.bias) v = v + ep.bias[col];
     if (ep.activation == ACT_RELU) v = fmaxf(v, 0.0f);
     else if (ep.activation == ACT_GELU) v = strict_gelu(v);
+    else if (ep.activation == ACT_GELU_TANH) v = strict_gelu_tanh(v);
     if (ep.residual) v = ep.residual[(size_t)row * ep.ldr + col] + v;
     if (ep.round_bf16) v = round_to_bf16(v);
     size_t orow = row;

@@ -160,7 +160,87 @@ class TransformerBlock:
         self.epsilon = epsilon
 
 
-class Gpt:
+class CachedModel:
+    """What every decoder-only model here can do: open sessions on the library, evaluate a whole context and generate.
+    A model provides ``_config`` (``vocab_size``, ``max_sequence_length`` and what its session needs) and
+    ``parameters()`` in the order of the library's parameter table."""
+
+    # -- sessions (src/nn/kv_cache.rs:89-115) --------------------------------
+    def decoder(self, backend, batch_size: int) -> "GptDecoder":
+        return self.decoder_with_capacity(backend, batch_size, self._config.max_sequence_length)
+
+    def decoder_with_capacity(self, backend, batch_size: int, capacity: int) -> "GptDecoder":
+        return self.decoder_with_options(backend, batch_size, capacity, GptDecoderOptions())
+
+    def decoder_with_options(self, backend, batch_size: int, capacity: int,
+                             options: GptDecoderOptions, **extra) -> "GptDecoder":
+        return GptDecoder(self, backend, batch_size, capacity, options, **extra)
+
+    def _generation_capacity(self, needed: int) -> int:
+        """Rows a generation session gets: the whole context, so that the reference's sliding window applies."""
+        return self._config.max_sequence_length
+
+    # -- full-context paths (src/nn.rs:629-715) -------------------------------
+    def forward(self, backend, token_ids) -> np.ndarray:
+        """``Gpt::forward`` evaluated on the backend: logits ``[batch, sequence, vocabulary]``
+        of a whole ``[batch, sequence]`` id block (a fresh session decoding one chunk is the same graph:
+        src/nn/kv_cache/graph.rs with past = 0)."""
+        ids = np.asarray(token_ids)
+        if ids.ndim != 2:
+            raise TnsrError("GPT token IDs must have shape [batch, sequence]")
+        batch, sequence = ids.shape
+        if batch == 0:
+            raise TnsrError("GPT batch size must be non-zero")
+        if sequence == 0:
+            raise TnsrError("GPT sequence length must be non-zero")
+        if sequence > self._config.max_sequence_length:
+            raise TnsrError(f"GPT sequence length {sequence} exceeds configured maximum "
+                            f"{self._config.max_sequence_length}")
+        decoder = self.decoder_with_capacity(backend, batch, sequence)
+        logits = decoder.decode([int(t) for t in ids.reshape(-1)])
+        return logits.reshape(batch, sequence, self._config.vocab_size)
+
+    def generate(self, backend, prompt: Sequence[int], max_new_tokens: int) -> List[int]:
+        """``Gpt::generate``: greedy, re-running the whole retained context for every new token."""
+        if len(prompt) == 0:
+            raise TnsrError("GPT generation prompt must be non-empty")
+        if not all(0 <= t < self._config.vocab_size for t in prompt):
+            raise TnsrError("GPT generation prompt contains an out-of-range token")
+        tokens = [int(t) for t in prompt]
+        context = self._generation_capacity(len(tokens) + max_new_tokens)
+        decoder = None
+        for _ in range(max_new_tokens):
+            window = tokens[max(0, len(tokens) - context):]
+            if decoder is None:
+                decoder = self.decoder_with_capacity(backend, 1, context)
+            decoder.reset()
+            logits = decoder.decode(window)
+            tokens.append(argmax_last(logits[logits.size - self._config.vocab_size:]))
+        return tokens
+
+    # -- greedy generation (src/nn/kv_cache.rs:121-157) ----------------------
+    def generate_cached(self, backend, prompt: Sequence[int], max_new_tokens: int) -> List[int]:
+        if len(prompt) == 0:
+            raise TnsrError("GPT generation prompt must be non-empty")
+        if not all(0 <= t < self._config.vocab_size for t in prompt):
+            raise TnsrError("GPT generation prompt contains an out-of-range token")
+        tokens = [int(t) for t in prompt]
+        if max_new_tokens == 0:
+            return tokens
+        decoder = self.decoder_with_capacity(backend, 1, self._generation_capacity(len(tokens) + max_new_tokens))
+        vocab = self._config.vocab_size
+        for _ in range(max_new_tokens):
+            if decoder.is_empty() or decoder.len() == decoder.capacity():
+                decoder.reset()
+                start = max(0, len(tokens) - decoder.capacity())
+                logits = decoder.decode(tokens[start:])
+            else:
+                logits = decoder.decode(tokens[-1:])
+            tokens.append(argmax_last(logits[logits.size - vocab:]))
+        return tokens
+
+
+class Gpt(CachedModel):
     """Decoder-only transformer with learned positions and a tied LM head."""
 
     def __init__(self, config: GptConfig):
@@ -198,75 +278,8 @@ class Gpt:
     def config(self) -> GptConfig:
         return self._config
 
-    # -- sessions (src/nn/kv_cache.rs:89-115) --------------------------------
-    def decoder(self, backend, batch_size: int) -> "GptDecoder":
-        return self.decoder_with_capacity(backend, batch_size, self._config.max_sequence_length)
-
-    def decoder_with_capacity(self, backend, batch_size: int, capacity: int) -> "GptDecoder":
-        return self.decoder_with_options(backend, batch_size, capacity, GptDecoderOptions())
-
-    def decoder_with_options(self, backend, batch_size: int, capacity: int,
-                             options: GptDecoderOptions, **extra) -> "GptDecoder":
-        return GptDecoder(self, backend, batch_size, capacity, options, **extra)
-
-    # -- full-context paths (src/nn.rs:629-715) -------------------------------
-    def forward(self, backend, token_ids) -> np.ndarray:
-        """``Gpt::forward`` evaluated on the backend: logits ``[batch, sequence, vocabulary]``
-        of a whole ``[batch, sequence]`` id block (a fresh session decoding one chunk is the same graph:
-        src/nn/kv_cache/graph.rs with past = 0)."""
-        ids = np.asarray(token_ids)
-        if ids.ndim != 2:
-            raise TnsrError("GPT token IDs must have shape [batch, sequence]")
-        batch, sequence = ids.shape
-        if batch == 0:
-            raise TnsrError("GPT batch size must be non-zero")
-        if sequence == 0:
-            raise TnsrError("GPT sequence length must be non-zero")
-        if sequence > self._config.max_sequence_length:
-            raise TnsrError(f"GPT sequence length {sequence} exceeds configured maximum "
-                            f"{self._config.max_sequence_length}")
-        decoder = self.decoder_with_capacity(backend, batch, sequence)
-        logits = decoder.decode([int(t) for t in ids.reshape(-1)])
-        return logits.reshape(batch, sequence, self._config.vocab_size)
-
-    def generate(self, backend, prompt: Sequence[int], max_new_tokens: int) -> List[int]:
-        """``Gpt::generate``: greedy, re-running the whole retained context for every new token."""
-        if len(prompt) == 0:
-            raise TnsrError("GPT generation prompt must be non-empty")
-        if not all(0 <= t < self._config.vocab_size for t in prompt):
-            raise TnsrError("GPT generation prompt contains an out-of-range token")
-        tokens = [int(t) for t in prompt]
-        context = self._config.max_sequence_length
-        decoder = None
-        for _ in range(max_new_tokens):
-            window = tokens[max(0, len(tokens) - context):]
-            if decoder is None:
-                decoder = self.decoder(backend, 1)
-            decoder.reset()
-            logits = decoder.decode(window)
-            tokens.append(argmax_last(logits[logits.size - self._config.vocab_size:]))
-        return tokens
-
-    # -- greedy generation (src/nn/kv_cache.rs:121-157) ----------------------
-    def generate_cached(self, backend, prompt: Sequence[int], max_new_tokens: int) -> List[int]:
-        if len(prompt) == 0:
-            raise TnsrError("GPT generation prompt must be non-empty")
-        if not all(0 <= t < self._config.vocab_size for t in prompt):
-            raise TnsrError("GPT generation prompt contains an out-of-range token")
-        tokens = [int(t) for t in prompt]
-        if max_new_tokens == 0:
-            return tokens
-        decoder = self.decoder(backend, 1)
-        vocab = self._config.vocab_size
-        for _ in range(max_new_tokens):
-            if decoder.is_empty() or decoder.len() == decoder.capacity():
-                decoder.reset()
-                start = max(0, len(tokens) - decoder.capacity())
-                logits = decoder.decode(tokens[start:])
-            else:
-                logits = decoder.decode(tokens[-1:])
-            tokens.append(argmax_last(logits[logits.size - vocab:]))
-        return tokens
+    def parameters(self) -> List[Parameter]:
+        return model_parameters(self)
 
 
 def argmax_last(row: np.ndarray) -> int:
@@ -305,8 +318,8 @@ class GptDecoder:
     ``decode(tokens[batch, chunk], position) -> flat f32 logits``).
     """
 
-    def __init__(self, model: Gpt, backend, batch: int, capacity: int,
-                 options: GptDecoderOptions = GptDecoderOptions(), backend_impl=None, device: int = 0):
+    def __init__(self, model: CachedModel, backend, batch: int, capacity: int,
+                 options: GptDecoderOptions = GptDecoderOptions(), backend_impl=None, device: int = 0, **session):
         config = model.config()
         if not batch > 0:
             raise TnsrError("decoder batch size must be non-zero")
@@ -322,7 +335,7 @@ class GptDecoder:
         if elements * 4 * config.num_layers * 2 > USIZE_MAX:
             raise TnsrError("decoder total cache size overflow")
         self._model = model
-        self._parameters = model_parameters(model)
+        self._parameters = model.parameters()
         self._revisions = [p.revision() for p in self._parameters]
         self._uploaded: List[Optional[int]] = [None] * len(self._parameters)
         self._batch, self._capacity, self._length = batch, capacity, 0
@@ -332,7 +345,7 @@ class GptDecoder:
             self._backend = backend_impl
         elif backend in (Backend.Cuda, Backend.Ptx):
             from .session import B200Session
-            self._backend = B200Session(config, batch, capacity, options, device=device)
+            self._backend = B200Session(config, batch, capacity, options, device=device, **session)
         elif backend == Backend.Cpu:
             raise TnsrError("this library has no CPU executor; use Backend.Cuda")
         else:

@@ -132,6 +132,72 @@ class NamedParameters:
         os.replace(tmp, os.path.join(directory, "manifest.json"))
 
 
+# ---- safetensors ---------------------------------------------------------------------------------
+# u64 little-endian header length, a JSON header {name: {dtype, shape, data_offsets}}, then the tensor bytes.
+
+_SAFETENSORS_DTYPES = {"F32": "<f4", "F16": "<f2", "F64": "<f8", "I32": "<i4", "I64": "<i8", "U8": "u1", "I8": "i1"}
+
+
+def read_safetensors(path: str) -> Dict[str, np.ndarray]:
+    """Every tensor of a safetensors file by name; bf16 is widened to f32 (exact), other types keep theirs."""
+    try:
+        with open(path, "rb") as f:
+            blob = f.read()
+    except OSError as e:
+        raise TnsrError(f"read safetensors: {e}")
+    if len(blob) < 8:
+        raise TnsrError("truncated safetensors file")
+    length = int.from_bytes(blob[:8], "little")
+    if length > len(blob) - 8:
+        raise TnsrError("truncated safetensors header")
+    try:
+        header = json.loads(blob[8:8 + length])
+    except ValueError as e:
+        raise TnsrError(f"parse safetensors header: {e}")
+    tensors = {}
+    for name, entry in header.items():
+        if name == "__metadata__":
+            continue
+        begin, end = entry["data_offsets"]
+        if not 0 <= begin <= end <= len(blob) - 8 - length:
+            raise TnsrError(f"{name}: tensor data out of bounds")
+        raw, dtype = blob[8 + length + begin:8 + length + end], entry["dtype"]
+        if dtype == "BF16":
+            values = (np.frombuffer(raw, dtype="<u2").astype(np.uint32) << 16).view(np.float32)
+        elif dtype in _SAFETENSORS_DTYPES:
+            values = np.frombuffer(raw, dtype=_SAFETENSORS_DTYPES[dtype])
+        else:
+            raise TnsrError(f"{name}: unsupported dtype {dtype}")
+        if values.size != int(np.prod(entry["shape"], dtype=np.int64)):
+            raise TnsrError(f"{name}: tensor length disagrees with shape")
+        tensors[name] = values.reshape(entry["shape"])
+    return tensors
+
+
+def write_safetensors(path: str, tensors: Dict[str, np.ndarray]) -> None:
+    """f32 arrays whose values are exact in bf16 are stored as bf16, everything else as f32; integers as i32."""
+    header, parts, offset = OrderedDict(), [], 0
+    for name, values in tensors.items():
+        values = np.asarray(values)
+        if np.issubdtype(values.dtype, np.integer):
+            dtype, raw = "I32", values.astype("<i4").tobytes()
+        else:
+            bits = np.ascontiguousarray(values, dtype=np.float32).view(np.uint32)
+            if np.any(bits & 0xFFFF):
+                dtype, raw = "F32", bits.astype("<u4").tobytes()
+            else:
+                dtype, raw = "BF16", (bits >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": dtype, "shape": list(values.shape), "data_offsets": [offset, offset + len(raw)]}
+        parts.append(raw)
+        offset += len(raw)
+    text = json.dumps(header).encode()
+    text += b" " * (-len(text) % 8)
+    with open(path, "wb") as f:
+        f.write(len(text).to_bytes(8, "little") + text)
+        for raw in parts:
+            f.write(raw)
+
+
 _ATTENTION = ["query_weight", "query_bias", "key_weight", "key_bias", "value_weight", "value_bias", "output_weight",
               "output_bias"]
 _BLOCK = ["attention_norm_weight", "attention_norm_bias", "feed_forward_norm_weight", "feed_forward_norm_bias"]
@@ -195,9 +261,35 @@ def load_gpt(directory: str) -> Gpt:
 
 def decoder_state_config(decoder) -> dict:
     c = decoder._model.config()
-    return dict(kind="gpt_decoder_state", batch=decoder.batch_size(), capacity=decoder.capacity(), length=decoder.len(),
-                num_layers=c.num_layers, embed_dim=c.embed_dim, num_heads=c.num_heads,
-                attention_precision=decoder._options.attention_precision.value, weight_dtype=c.weight_dtype)
+    config = dict(kind="gpt_decoder_state", batch=decoder.batch_size(), capacity=decoder.capacity(), length=decoder.len(),
+                  num_layers=c.num_layers, embed_dim=c.embed_dim, num_heads=getattr(c, "num_heads", 0),
+                  attention_precision=decoder._options.attention_precision.value, weight_dtype=c.weight_dtype)
+    if getattr(c, "stack", None) is not None:
+        # caches and states of a described model travel whole: convolution rings and recurrent states have no length axis
+        config.update(kind="stack_decoder_state", architecture=c.architecture)
+    return config
+
+
+def _save_stack_state(decoder, directory: str, config: dict) -> None:
+    named = NamedParameters()
+    if decoder.len():
+        for index in range(decoder._backend.cache_count()):
+            values = decoder._backend.read_cache(index)
+            named.insert(f"cache.{index:04d}", values, values.shape, "decoder_state")
+    named.save(directory, config)
+
+
+def _load_stack_state(decoder, named, length: int) -> None:
+    count = decoder._backend.cache_count()
+    named.validate_names({f"cache.{i:04d}" for i in range(count)} if length else set())
+    decoder.reset()
+    decoder._failed = True
+    for index in range(count) if length else ():
+        parameter = dict((n, p) for n, p, _ in named.iter())[f"cache.{index:04d}"]
+        decoder._backend.write_cache(index, parameter.values())
+    decoder._length = length
+    decoder._revisions = [p.revision() for p in decoder._parameters]
+    decoder._failed = False
 
 
 def save_decoder_state(decoder, directory: str) -> None:
@@ -205,6 +297,8 @@ def save_decoder_state(decoder, directory: str) -> None:
     if decoder._failed:
         raise TnsrError("decoder execution failed; reset the cache before reuse")
     config = decoder_state_config(decoder)
+    if config["kind"] == "stack_decoder_state":
+        return _save_stack_state(decoder, directory, config)
     named = NamedParameters()
     length = decoder.len()
     if length:
@@ -220,15 +314,21 @@ def load_decoder_state(decoder, directory: str) -> None:
     width and precision and enough capacity; its previous contents are discarded.  The weights are the caller's
     business, exactly as with a live session: a state only continues correctly under the weights that produced it."""
     named, config = NamedParameters.load(directory)
-    if not isinstance(config, dict) or config.get("kind") != "gpt_decoder_state":
-        raise TnsrError("archive does not hold a decoder state")
     mine = decoder_state_config(decoder)
+    if not isinstance(config, dict) or config.get("kind") != mine["kind"]:
+        raise TnsrError("archive does not hold a decoder state")
+    stack = mine["kind"] == "stack_decoder_state"
+    for key in ("architecture", "capacity") if stack else ():
+        if config.get(key) != mine[key]:
+            raise TnsrError(f"decoder state mismatch: {key} is {config.get(key)!r}, this decoder has {mine[key]!r}")
     for key in ("batch", "num_layers", "embed_dim", "num_heads", "attention_precision", "weight_dtype"):
         if config.get(key) != mine[key]:
             raise TnsrError(f"decoder state mismatch: {key} is {config.get(key)!r}, this decoder has {mine[key]!r}")
     length = config.get("length")
     if not isinstance(length, int) or length < 0 or length > decoder.capacity():
         raise TnsrError("decoder context capacity exceeded")
+    if stack:
+        return _load_stack_state(decoder, named, length)
     names = {f"cache.{layer:04d}.{name}" for layer in range(mine["num_layers"]) for name in ("key", "value")} if length else set()
     named.validate_names(names)
     decoder.reset()

@@ -18,19 +18,29 @@ class B200Session:
         from .nn import GptAttentionPrecision, TnsrError
         weight_dtype = getattr(config, "weight_dtype", "f32")
         kv = "bf16" if weight_dtype == "bf16" else "f32"
-        if options is not None and options.attention_precision == GptAttentionPrecision.Bf16:
+        stack = getattr(config, "stack", None)          # models described layer by layer
+        bf16_attention = options is not None and options.attention_precision == GptAttentionPrecision.Bf16
+        if bf16_attention and stack is None:
             kv = "bf16"
-        self.cfg = Config(config.vocab_size, config.max_sequence_length, config.embed_dim, config.num_heads,
-                          config.feed_forward_dim, config.num_layers, config.layer_norm_epsilon,
-                          ACT[getattr(config, "activation", "relu")], DTYPE[weight_dtype], DTYPE[kv], batch,
-                          capacity, device, LOGITS[logits_mode],
-                          PREFILL[options.prefill.value] if options is not None else PREFILL["auto"], step_parts,
-                          kv_page_rows, kv_pool_pages, small_batch_mode)
+        prefill = PREFILL[options.prefill.value] if options is not None else PREFILL["auto"]
+        if stack is None:
+            shape = (config.embed_dim, config.num_heads, config.feed_forward_dim, config.num_layers, config.layer_norm_epsilon,
+                     ACT[getattr(config, "activation", "relu")])
+        else:
+            shape = (config.embed_dim, 1, 1, config.num_layers, config.layer_norm_epsilon, 0)
+        self.cfg = Config(config.vocab_size, config.max_sequence_length, *shape, DTYPE[weight_dtype], DTYPE[kv], batch,
+                          capacity, device, LOGITS[logits_mode], prefill, step_parts, kv_page_rows, kv_pool_pages,
+                          small_batch_mode)
         self.handle = C.c_void_p()
         self.batch, self.capacity, self.vocab = batch, capacity, config.vocab_size
         self.embed_dim = config.embed_dim
         self.logits_mode = logits_mode
-        code = lib().tnsr_b200_decoder_create(C.byref(self.cfg), C.byref(self.handle))
+        self.is_stack = stack is not None
+        if stack is None:
+            code = lib().tnsr_b200_decoder_create(C.byref(self.cfg), C.byref(self.handle))
+        else:
+            desc = stack()                              # keeps the layer array alive for the call
+            code = lib().tnsr_b200_decoder_create_stack(C.byref(self.cfg), C.byref(desc), C.byref(self.handle))
         if code != 0:
             self.handle = None
             raise TnsrError(f"initialize CUDA decoder: {_native.last_error(None)}")
@@ -124,12 +134,20 @@ class B200Session:
         self._check(lib().tnsr_b200_decoder_attention_profile(self.handle, C.byref(ms), C.byref(n)))
         return ms.value, int(n.value)
 
+    def cache_count(self) -> int:
+        """Cache and state tensors of the handle (GPT: keys and values of every layer)."""
+        return int(lib().tnsr_b200_decoder_cache_count(self.handle))
+
     def read_cache(self, index: int) -> np.ndarray:
-        out = np.empty((self.batch, self.capacity, self.embed_dim), dtype=np.float32)
+        """Cache tensor as f32: [batch, capacity, width]; [batch, elements per session] for a described model."""
+        if self.is_stack:
+            out = np.empty((self.batch, int(lib().tnsr_b200_decoder_cache_elems(self.handle, index)) // self.batch), dtype=np.float32)
+        else:
+            out = np.empty((self.batch, self.capacity, self.embed_dim), dtype=np.float32)
         self._check(lib().tnsr_b200_decoder_read_cache(self.handle, index, out.ctypes.data_as(C.POINTER(C.c_float))))
         return out
 
     def write_cache(self, index: int, values: np.ndarray) -> None:
         v = np.ascontiguousarray(values, dtype=np.float32)
-        assert v.size == self.batch * self.capacity * self.embed_dim
+        assert v.size == int(lib().tnsr_b200_decoder_cache_elems(self.handle, index))
         self._check(lib().tnsr_b200_decoder_write_cache(self.handle, index, v.ctypes.data_as(C.POINTER(C.c_float))))
