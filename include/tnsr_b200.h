@@ -524,6 +524,61 @@ TNSR_B200_API int tnsr_b200_add_f32(const float* a, const float* b, float* out, 
 TNSR_B200_API int tnsr_b200_swiglu_f32(const float* gate, const float* up, float* out, uint64_t elems,
                                        void* stream);
 
+/* ---- operators of models described layer by layer ------------------------------- */
+
+/* x / sqrt(mean(x^2) + epsilon) * (offset + weight), statistics in f32. */
+TNSR_B200_API int tnsr_b200_rmsnorm(const float* x, const float* weight, float offset, void* out, uint32_t rows,
+                                    uint32_t width, float epsilon, int out_dtype, void* stream);
+
+/* What a step of `chunk` tokens per session works on.  Session b stands at
+ * d_positions[b] if d_positions is set, else at `position`. */
+typedef struct tnsr_b200_place {
+    uint32_t sessions, chunk, position, pad0;
+    const uint32_t* d_positions;
+} tnsr_b200_place;
+
+/* Grouped-query causal attention over caches that already hold the new rows:
+ * out[row, h] = sigmoid(gate[row, h]) * softmax_j(cap(q . k_j * scale)) . v_j with
+ * cap(s) = softcap * tanh(s / softcap) (softcap 0: none; gate NULL: none).  q
+ * [sessions, chunk, heads, dim], k_cache [sessions, capacity, kv_heads, dim],
+ * v_cache [.., vdim], out [sessions, chunk, out_ld], columns from heads * vdim to
+ * out_cols are zeroed.  dtype: element type of q, caches and out.  engine: 0 =
+ * best kernel for the shape, 1 = one warp per (query, head).  workspace:
+ * tnsr_b200_grouped_attention_workspace() bytes, zeroed once (NULL: the keys of
+ * a session are not divided over CTAs). */
+typedef struct tnsr_b200_grouped_attention_args {
+    const void *q, *k_cache, *v_cache;
+    const float* gate;
+    void* out;
+    void* workspace;
+    uint64_t workspace_bytes;
+    uint32_t heads, kv_heads, dim, vdim, capacity, gate_ld, out_ld, out_cols;
+    float scale, softcap;
+    int32_t dtype, engine;
+} tnsr_b200_grouped_attention_args;
+TNSR_B200_API uint64_t tnsr_b200_grouped_attention_workspace(uint32_t dim, uint32_t vdim);
+TNSR_B200_API int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args,
+                                              const tnsr_b200_place* place, void* stream);
+
+/* The mamba2 mixer between its two projections: proj [rows, ld] holds z | x | B |
+ * C, dt [rows, dt_ld] the raw step sizes; ring [sessions, taps, channels] and ssm
+ * [sessions, heads, state, vdim] (f32) are the session's state, read and updated;
+ * xbc [rows, channels] and gated [rows, heads * vdim] are scratch; out [rows,
+ * out_ld].  dtype: element type of proj, ring, xbc, gated and out.  engine: 0 =
+ * best kernel for the chunk, 1 = token by token. */
+typedef struct tnsr_b200_mamba2_args {
+    const void* proj;
+    const float *dt, *conv_w, *conv_b, *dt_bias, *a_log, *d_skip, *norm_w;
+    void* ring;
+    float* ssm;
+    void *xbc, *gated, *out;
+    uint32_t ld, dt_ld, heads, vdim, state, groups, norm_groups, taps, out_ld, out_cols;
+    float eps;
+    int32_t dtype, engine;
+    uint32_t pad0;
+} tnsr_b200_mamba2_args;
+TNSR_B200_API int tnsr_b200_mamba2(const tnsr_b200_mamba2_args* args, const tnsr_b200_place* place, void* stream);
+
 /* Next-token sampling on the device (no reference counterpart: tnsr's decode
  * loop is greedy, src/nn/kv_cache.rs:121-157).  Per row: the top_k entries
  * under IEEE totalOrder with ties towards the larger index (so top_k = 1 is

@@ -50,6 +50,24 @@ class StackDesc(C.Structure):
                 ("num_layers", C.c_uint32)]
 
 
+class Place(C.Structure):
+    _fields_ = [("sessions", C.c_uint32), ("chunk", C.c_uint32), ("position", C.c_uint32), ("pad0", C.c_uint32),
+                ("d_positions", C.c_void_p)]
+
+
+class GroupedAttentionArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "gate", "out", "workspace")] + [("workspace_bytes", C.c_uint64)] + \
+        [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "capacity", "gate_ld", "out_ld", "out_cols")] + \
+        [("scale", C.c_float), ("softcap", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32)]
+
+
+class Mamba2Args(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "dt", "conv_w", "conv_b", "dt_bias", "a_log", "d_skip", "norm_w", "ring", "ssm", "xbc",
+                                          "gated", "out")] + \
+        [(n, C.c_uint32) for n in ("ld", "dt_ld", "heads", "vdim", "state", "groups", "norm_groups", "taps", "out_ld", "out_cols")] + \
+        [("eps", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32), ("pad0", C.c_uint32)]
+
+
 _vp, _u32, _u64, _i, _f = C.c_void_p, C.c_uint32, C.c_uint64, C.c_int, C.c_float
 _fp, _u32p = C.POINTER(C.c_float), C.POINTER(C.c_uint32)
 
@@ -99,6 +117,10 @@ SIGNATURES = {
     "tnsr_b200_encoder_attention": (_i, [_vp, _vp, _vp, _u32, _vp, _vp, _u32, _u32, _u32, _u32, _vp]),
     "tnsr_b200_add_f32": (_i, [_vp, _vp, _vp, _u64, _vp]),
     "tnsr_b200_swiglu_f32": (_i, [_vp, _vp, _vp, _u64, _vp]),
+    "tnsr_b200_rmsnorm": (_i, [_vp, _vp, _f, _vp, _u32, _u32, _f, _i, _vp]),
+    "tnsr_b200_grouped_attention_workspace": (_u64, [_u32, _u32]),
+    "tnsr_b200_grouped_attention": (_i, [C.POINTER(GroupedAttentionArgs), C.POINTER(Place), _vp]),
+    "tnsr_b200_mamba2": (_i, [C.POINTER(Mamba2Args), C.POINTER(Place), _vp]),
     "tnsr_b200_sample_top_k": (_i, [_vp, _vp, _u32, _u32, _f, _u32, _u64, _u32, _u32, _vp]),
     "tnsr_b200_decoder_set_sampler": (_i, [_vp, _f, _u32, _u64]),
     "tnsr_b200_decoder_release": (_i, [_vp, _u32]),

@@ -317,7 +317,7 @@ int stack_create(tnsr_b200_decoder* dec, const tnsr_b200_stack* st) {
             S->caches.push_back({L.k_cache, L.k_elems, dtype});
             S->caches.push_back({L.v_cache, L.v_elems, dtype});
             S->caches.push_back({L.ring, L.ring_elems, dtype});
-            S->attention_ws_bytes = std::max(S->attention_ws_bytes, grouped_attention_workspace_bytes(c.batch, l.heads, l.kv_heads, l.vdim));
+            S->attention_ws_bytes = std::max(S->attention_ws_bytes, grouped_attention_workspace_bytes(l.dim, l.vdim));
         } else {
             L.ssm_elems = (uint64_t)c.batch * l.heads * l.state * l.vdim;
             if ((rc = dev_alloc(dec, (void**)&L.ssm, L.ssm_elems * 4, true))) return rc;

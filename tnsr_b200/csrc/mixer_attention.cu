@@ -17,33 +17,6 @@ __device__ __forceinline__ float mx_warp_sum(float v) {
     return v;
 }
 
-template <typename T>
-__device__ __forceinline__ float2 load_pair(const T* p, bool vec, bool second);
-template <>
-__device__ __forceinline__ float2 load_pair<float>(const float* p, bool vec, bool second) {
-    if (vec) return *reinterpret_cast<const float2*>(p);
-    return make_float2(p[0], second ? p[1] : 0.0f);
-}
-template <>
-__device__ __forceinline__ float2 load_pair<bf16>(const bf16* p, bool vec, bool second) {
-    if (vec) return bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(p));
-    return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.0f);
-}
-template <typename T>
-__device__ __forceinline__ void store_pair(T* p, float2 v, bool vec, bool second);
-template <>
-__device__ __forceinline__ void store_pair<float>(float* p, float2 v, bool vec, bool second) {
-    if (vec) { *reinterpret_cast<float2*>(p) = v; return; }
-    p[0] = v.x;
-    if (second) p[1] = v.y;
-}
-template <>
-__device__ __forceinline__ void store_pair<bf16>(bf16* p, float2 v, bool vec, bool second) {
-    if (vec) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); return; }
-    p[0] = __float2bfloat16_rn(v.x);
-    if (second) p[1] = __float2bfloat16_rn(v.y);
-}
-
 // NP: channel pairs per lane (a head unit has at most 64 NP channels).  TAPS: compiled window length; shorter filters are
 // padded with zero weights at the old end and never touch the padded rows.
 template <typename T, int NP, int TAPS>

@@ -13,58 +13,83 @@
 
 namespace tb {
 
+int launch_ssd_scan(const Mamba2& m, const StepPlace& place, cudaStream_t stream);   // ssd_scan.cu
+
+// Shortest chunk that takes the chunked tensor-core scan; below it the token kernel's few steps are cheaper.
+constexpr uint32_t SSD_SCAN_MIN_TOKENS = 16;
+
 __device__ __forceinline__ float full_silu(float x) { return x / (1.0f + expf(-x)); }
+// silu of an activation that is stored in T: bf16 results come from the hardware exponential, f32 ones from expf.
+template <typename T>
+__device__ __forceinline__ float act_silu(float x);
+template <>
+__device__ __forceinline__ float act_silu<float>(float x) { return full_silu(x); }
+template <>
+__device__ __forceinline__ float act_silu<bf16>(float x) { return fast_silu(x); }
 __device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
 // ---- convolution + silu ----------------------------------------------------------------------
-// A thread owns one channel of a run of tokens.
+// A thread owns two neighbouring channels of a run of tokens.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, const float* __restrict__ conv_w,
-                 const float* __restrict__ conv_b, const T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run) {
+                 const float* __restrict__ conv_b, const T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run,
+                 uint32_t vec) {
     pdl_wait();
     pdl_trigger();
-    const uint32_t c = blockIdx.x * blockDim.x + threadIdx.x;
+    const uint32_t c = 2 * (blockIdx.x * blockDim.x + threadIdx.x);
     if (c >= channels) return;
+    const bool second = c + 1 < channels;
     const uint32_t s = blockIdx.z, t0 = blockIdx.y * run, t1 = min(place.chunk, t0 + run);
     const uint32_t p0 = place.pos(s);
     const T* in = rows + (size_t)s * place.chunk * ld + c;
-    float w[TAPS], win[TAPS];
+    T* dst = out + (size_t)s * place.chunk * channels + c;
+    float2 w[TAPS], win[TAPS];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
         const int src = j - (TAPS - (int)taps);
-        w[j] = src >= 0 ? conv_w[(size_t)c * taps + src] : 0.0f;
-        win[j] = 0.0f;
+        w[j] = make_float2(src >= 0 ? conv_w[(size_t)c * taps + src] : 0.0f, src >= 0 && second ? conv_w[(size_t)(c + 1) * taps + src] : 0.0f);
+        win[j] = make_float2(0.0f, 0.0f);
         const int t = (int)t0 - TAPS + j;
         if (j > 0 && (int)t0 - t < (int)taps) {
             const long long pos = (long long)p0 + t;
-            if (t >= 0) win[j] = to_f32(in[(size_t)t * ld]);
-            else if (pos >= 0) win[j] = to_f32(ring[((size_t)s * taps + pos % taps) * channels + c]);
+            if (t >= 0) win[j] = load_pair<T>(in + (size_t)t * ld, vec, second);
+            else if (pos >= 0) win[j] = load_pair<T>(ring + ((size_t)s * taps + pos % taps) * channels + c, vec, second);
         }
     }
-    const float b = conv_b[c];
-    for (uint32_t t = t0; t < t1; ++t) {
+    const float2 b = make_float2(conv_b[c], second ? conv_b[c + 1] : 0.0f);
+    // rows are asked for eight at a time, so that their round trips overlap
+    constexpr uint32_t AHEAD = 8;
+    for (uint32_t t = t0; t < t1; t += AHEAD) {
+        float2 next[AHEAD];
 #pragma unroll
-        for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
-        win[TAPS - 1] = to_f32(in[(size_t)t * ld]);
-        float y = b;
+        for (uint32_t i = 0; i < AHEAD; ++i)
+            next[i] = t + i < t1 ? load_pair<T>(in + (size_t)(t + i) * ld, vec, second) : make_float2(0.0f, 0.0f);
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], win[j], y);
-        out[((size_t)s * place.chunk + t) * channels + c] = from_f32<T>(full_silu(y));
+        for (uint32_t i = 0; i < AHEAD; ++i) {
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
+            win[TAPS - 1] = next[i];
+            float2 y = b;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) { y.x = fmaf(w[j].x, win[j].x, y.x); y.y = fmaf(w[j].y, win[j].y, y.y); }
+            if (t + i < t1) store_pair<T>(dst + (size_t)(t + i) * channels, make_float2(act_silu<T>(y.x), act_silu<T>(y.y)), vec, second);
+        }
     }
 }
 
 template <typename T>
 static void conv_silu_typed(const Mamba2& m, uint32_t inner, uint32_t channels, const StepPlace& place, cudaStream_t stream) {
     const uint32_t run = std::min(place.chunk, 32u);
-    const dim3 grid(ceil_div(channels, 128u), ceil_div(place.chunk, run), place.sessions);
+    const dim3 grid(ceil_div(ceil_div(channels, 2u), 128u), ceil_div(place.chunk, run), place.sessions);
     const T* rows = (const T*)m.proj + inner;
+    const uint32_t vec = inner % 2 == 0 && channels % 2 == 0 && m.ld % 2 == 0;
     if (m.taps <= 4)
         launch_kernel(conv_silu_kernel<T, 4>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b, (const T*)m.ring,
-                      (T*)m.xbc, place, run);
+                      (T*)m.xbc, place, run, vec);
     else
         launch_kernel(conv_silu_kernel<T, kMaxConvTaps>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b,
-                      (const T*)m.ring, (T*)m.xbc, place, run);
+                      (const T*)m.ring, (T*)m.xbc, place, run, vec);
 }
 
 // ---- token by token ----------------------------------------------------------------------------
@@ -114,7 +139,7 @@ ssd_token_kernel(Mamba2 m, StepPlace place) {
                 v = fmaf(w[m.taps - 1], to_f32(now), m.conv_b[ch]);
                 for (uint32_t lag = 1; lag < m.taps && lag <= p0; ++lag)
                     v = fmaf(w[m.taps - 1 - lag], to_f32(ring[(size_t)((p0 - lag) % m.taps) * channels]), v);
-                v = full_silu(v);
+                v = act_silu<T>(v);
                 v = to_f32(from_f32<T>(v));     // the value a longer chunk would have stored
                 if (i < width || (h % (m.heads / m.groups) == 0 && p_first == 0)) ring[(size_t)(p0 % m.taps) * channels] = now;
             } else {
@@ -145,7 +170,7 @@ ssd_token_kernel(Mamba2 m, StepPlace place) {
             for (uint32_t j = 0; j < ng; ++j) y += red[j * width + tid];
             const uint32_t col = h * m.vdim + p_first + tid;
             const float z = to_f32(reinterpret_cast<const T*>(m.proj)[row * m.ld + col]);
-            reinterpret_cast<T*>(m.gated)[row * inner + col] = from_f32<T>(y * full_silu(z));
+            reinterpret_cast<T*>(m.gated)[row * inner + col] = from_f32<T>(y * act_silu<T>(z));
         }
         __syncthreads();
     }
@@ -170,7 +195,8 @@ bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state) {
 }
 
 // ---- grouped RMS norm ------------------------------------------------------------------------------
-// One block per (row, norm group).
+// One block per (row, norm group): any width.  Parts of whole 16-byte chunks up to 1024 values take a warp each and stay in
+// registers between the sum and the scaling (gated_norm_warp_kernel).
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const T* __restrict__ gated, const float* __restrict__ w, T* __restrict__ out, uint32_t inner, uint32_t groups,
@@ -196,6 +222,46 @@ gated_norm_kernel(const T* __restrict__ gated, const float* __restrict__ w, T* _
         for (uint32_t c = inner + threadIdx.x; c < out_cols; c += blockDim.x) out[row * out_ld + c] = from_f32<T>(0.0f);
 }
 
+constexpr uint32_t GN_VEC = 4;   // 16-byte chunks per lane: parts of up to 1024 values, one warp each
+__global__ void __launch_bounds__(128)
+gated_norm_warp_kernel(const bf16* __restrict__ gated, const float* __restrict__ w, bf16* __restrict__ out, uint32_t rows, uint32_t inner,
+                       uint32_t groups, uint32_t out_ld, uint32_t out_cols, float eps) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t lane = threadIdx.x & 31, task = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (task >= rows * groups) return;
+    const uint32_t row = task / groups, grp = task % groups, part = inner / groups, chunks = part / 8, c0 = grp * part;
+    const uint4* in = reinterpret_cast<const uint4*>(gated + (size_t)row * inner + c0);
+    float v[GN_VEC][8], ss = 0.0f;
+#pragma unroll
+    for (uint32_t i = 0; i < GN_VEC; ++i) {
+        const uint32_t c = lane + 32 * i;
+        const uint4 q = c < chunks ? in[c] : make_uint4(0u, 0u, 0u, 0u);
+        const uint32_t words[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 f = bf16x2_to_f32(words[k]);
+            v[i][2 * k] = f.x;
+            v[i][2 * k + 1] = f.y;
+            ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = rsqrtf(ss / (float)part + eps);
+    uint4* o = reinterpret_cast<uint4*>(out + (size_t)row * out_ld + c0);
+#pragma unroll
+    for (uint32_t i = 0; i < GN_VEC; ++i) {
+        const uint32_t c = lane + 32 * i;
+        if (c >= chunks) continue;
+        const float4 w0 = *reinterpret_cast<const float4*>(w + c0 + c * 8), w1 = *reinterpret_cast<const float4*>(w + c0 + c * 8 + 4);
+        o[c] = make_uint4(pack_bf16x2(v[i][0] * inv * w0.x, v[i][1] * inv * w0.y), pack_bf16x2(v[i][2] * inv * w0.z, v[i][3] * inv * w0.w),
+                          pack_bf16x2(v[i][4] * inv * w1.x, v[i][5] * inv * w1.y), pack_bf16x2(v[i][6] * inv * w1.z, v[i][7] * inv * w1.w));
+    }
+    if (grp == 0)
+        for (uint32_t c = inner + lane; c < out_cols; c += 32) out[(size_t)row * out_ld + c] = __float2bfloat16_rn(0.0f);
+}
+
 int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream_t stream) {
     if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
     const uint32_t inner = m.heads * m.vdim, channels = inner + 2 * m.groups * m.state, rows = place.sessions * place.chunk;
@@ -216,12 +282,22 @@ int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream
         if ((rc = check_launch("conv_silu"))) return rc;
         const uint8_t* raw = (const uint8_t*)m.proj + (size_t)inner * (bf ? 2 : 4);
         if ((rc = launch_conv_ring(raw, m.ld, channels, m.taps, m.ring, place, dtype, stream))) return rc;
-        if (bf) ssd_token_rows<bf16, false>(m, place, stream); else ssd_token_rows<float, false>(m, place, stream);
-        count_launch();
-        if ((rc = check_launch("ssd_token"))) return rc;
+        if (bf && m.engine == 0 && place.chunk >= SSD_SCAN_MIN_TOKENS) {
+            if ((rc = launch_ssd_scan(m, place, stream))) return rc;
+        } else {
+            if (bf) ssd_token_rows<bf16, false>(m, place, stream); else ssd_token_rows<float, false>(m, place, stream);
+            count_launch();
+            if ((rc = check_launch("ssd_token"))) return rc;
+        }
     }
     const dim3 grid(rows, m.norm_groups);
-    if (bf)
+    const uint32_t part = inner / m.norm_groups;
+    const bool warp_norm = bf && part % 8 == 0 && part <= GN_VEC * 256 && m.out_ld % 8 == 0 && inner % 8 == 0 &&
+                           (reinterpret_cast<uintptr_t>(m.gated) | reinterpret_cast<uintptr_t>(m.out) | reinterpret_cast<uintptr_t>(m.norm_w)) % 16 == 0;
+    if (warp_norm)
+        launch_kernel(gated_norm_warp_kernel, dim3(ceil_div(rows * m.norm_groups, 4)), dim3(128), 0, stream, (const bf16*)m.gated, m.norm_w, (bf16*)m.out,
+                      rows, inner, m.norm_groups, m.out_ld, m.out_cols, m.eps);
+    else if (bf)
         launch_kernel(gated_norm_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)m.gated, m.norm_w, (bf16*)m.out, inner, m.norm_groups,
                       m.out_ld, m.out_cols, m.eps);
     else

@@ -67,7 +67,7 @@ struct GroupedAttention {
     uint64_t workspace_bytes = 0;
     int engine = 0;                       // 0: best kernel for the shape, 1: one warp per (row, head)
 };
-uint64_t grouped_attention_workspace_bytes(uint32_t sessions, uint32_t heads, uint32_t kv_heads, uint32_t vdim);
+uint64_t grouped_attention_workspace_bytes(uint32_t dim, uint32_t vdim);
 int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, int dtype, cudaStream_t stream);
 
 // ---- mamba2 ---------------------------------------------------------------------
@@ -94,5 +94,78 @@ struct Mamba2 {
 };
 bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state);
 int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream_t stream);
+
+// ---- device helpers ----------------------------------------------------------------
+#ifdef __CUDACC__
+// Two neighbouring channels as f32; one access when `vec` (even address), else element by element (`second`: the second
+// one exists).
+template <typename T>
+__device__ __forceinline__ float2 load_pair(const T* p, bool vec, bool second);
+template <>
+__device__ __forceinline__ float2 load_pair<float>(const float* p, bool vec, bool second) {
+    if (vec) return *reinterpret_cast<const float2*>(p);
+    return make_float2(p[0], second ? p[1] : 0.0f);
+}
+template <>
+__device__ __forceinline__ float2 load_pair<bf16>(const bf16* p, bool vec, bool second) {
+    if (vec) return bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(p));
+    return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.0f);
+}
+template <typename T>
+__device__ __forceinline__ void store_pair(T* p, float2 v, bool vec, bool second);
+template <>
+__device__ __forceinline__ void store_pair<float>(float* p, float2 v, bool vec, bool second) {
+    if (vec) { *reinterpret_cast<float2*>(p) = v; return; }
+    p[0] = v.x;
+    if (second) p[1] = v.y;
+}
+template <>
+__device__ __forceinline__ void store_pair<bf16>(bf16* p, float2 v, bool vec, bool second) {
+    if (vec) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y); return; }
+    p[0] = __float2bfloat16_rn(v.x);
+    if (second) p[1] = __float2bfloat16_rn(v.y);
+}
+
+// Warp-level tensor-core pieces shared by the grouped attention and the chunked scan: ldmatrix, mma.sync m16n8k16
+// (bf16 operands, f32 accumulators), 16-byte asynchronous copies.
+__device__ __forceinline__ uint32_t mx_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void mx_cp16(void* dst, const void* src, bool real) {
+    const uint32_t bytes = real ? 16u : 0u;   // zero-fill when the source is outside
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mx_smem(dst)), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void mx_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void mx_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void mx_ldsm(uint32_t addr, uint32_t* r) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mx_ldsm_t(uint32_t addr, uint32_t* r) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mx_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float mx_ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float mx_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// x = hi + lo with both halves bf16: two products with an exact bf16 operand then carry 16 bits of x.
+__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16x2(x, y);
+    const float2 h = bf16x2_to_f32(hi);
+    lo = pack_bf16x2(x - h.x, y - h.y);
+}
+#endif  // __CUDACC__
 
 }  // namespace tb

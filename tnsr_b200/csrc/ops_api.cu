@@ -2,6 +2,7 @@
 // include/tnsr_b200.h).  They queue work on the caller's stream and never
 // synchronise or allocate.
 #include "common.cuh"
+#include "mixers.cuh"
 
 using namespace tb;
 
@@ -153,6 +154,59 @@ int tnsr_b200_sample_top_k(const float* logits, uint32_t* out, uint32_t rows, ui
 int tnsr_b200_argmax(const float* logits, uint32_t* out, uint32_t rows, uint32_t vocab, void* stream) {
     if (!logits || !out || vocab == 0) return bad("argmax: null pointer or empty vocabulary");
     return launch_argmax(logits, out, rows, vocab, vocab, as_stream(stream));
+}
+
+int tnsr_b200_rmsnorm(const float* x, const float* weight, float offset, void* out, uint32_t rows, uint32_t width,
+                      float epsilon, int out_dtype, void* stream) {
+    if (!x || !weight || !out) return bad("rmsnorm: null pointer");
+    if (width == 0 || !(epsilon > 0.0f)) return bad("rmsnorm: width and epsilon must be positive");
+    if (out_dtype != TNSR_B200_F32 && out_dtype != TNSR_B200_BF16) return bad("rmsnorm: bad output dtype");
+    return launch_rmsnorm(x, weight, offset, out, rows, width, epsilon, out_dtype, as_stream(stream));
+}
+
+uint64_t tnsr_b200_grouped_attention_workspace(uint32_t dim, uint32_t vdim) { return grouped_attention_workspace_bytes(dim, vdim); }
+
+static StepPlace step_place(const tnsr_b200_place* p) {
+    StepPlace place;
+    place.sessions = p->sessions;
+    place.chunk = p->chunk;
+    place.position = p->position;
+    place.d_position = p->d_positions;
+    place.position_stride = p->d_positions ? 1u : 0u;
+    return place;
+}
+
+int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args, const tnsr_b200_place* place, void* stream) {
+    if (!args || !place || !args->q || !args->k_cache || !args->v_cache || !args->out) return bad("grouped_attention: null pointer");
+    if (args->dtype != TNSR_B200_F32 && args->dtype != TNSR_B200_BF16) return bad("grouped_attention: dtype must be f32 or bf16");
+    if (args->heads == 0 || args->dim == 0 || args->vdim == 0 || args->capacity == 0 || args->out_ld < args->out_cols ||
+        args->out_cols < args->heads * args->vdim)
+        return bad("grouped_attention: sizes must be positive and the output row must hold every head");
+    if (!place->d_positions && (uint64_t)place->position + place->chunk > args->capacity) return bad("grouped_attention: the chunk ends past the capacity");
+    GroupedAttention a;
+    a.q = args->q; a.k_cache = args->k_cache; a.v_cache = args->v_cache;
+    a.heads = args->heads; a.kv_heads = args->kv_heads; a.dim = args->dim; a.vdim = args->vdim; a.capacity = args->capacity;
+    a.scale = args->scale; a.softcap = args->softcap; a.gate = args->gate; a.gate_ld = args->gate_ld;
+    a.out = args->out; a.out_ld = args->out_ld; a.out_cols = args->out_cols;
+    a.workspace = args->workspace; a.workspace_bytes = args->workspace_bytes; a.engine = args->engine;
+    return launch_grouped_attention(a, step_place(place), args->dtype, as_stream(stream));
+}
+
+int tnsr_b200_mamba2(const tnsr_b200_mamba2_args* args, const tnsr_b200_place* place, void* stream) {
+    if (!args || !place || !args->proj || !args->dt || !args->conv_w || !args->conv_b || !args->dt_bias || !args->a_log || !args->d_skip ||
+        !args->norm_w || !args->ring || !args->ssm || !args->gated || !args->out || (place->chunk > 1 && !args->xbc))
+        return bad("mamba2: null pointer");
+    if (args->dtype != TNSR_B200_F32 && args->dtype != TNSR_B200_BF16) return bad("mamba2: dtype must be f32 or bf16");
+    if (args->groups == 0 || args->heads == 0 || args->heads % args->groups || args->norm_groups == 0 ||
+        (args->heads * args->vdim) % args->norm_groups || args->out_ld < args->out_cols || args->out_cols < args->heads * args->vdim)
+        return bad("mamba2: groups must divide heads, norm_groups the width, and the output row must hold every head");
+    Mamba2 m;
+    m.proj = args->proj; m.ld = args->ld; m.dt = args->dt; m.dt_ld = args->dt_ld;
+    m.heads = args->heads; m.vdim = args->vdim; m.state = args->state; m.groups = args->groups; m.norm_groups = args->norm_groups; m.taps = args->taps;
+    m.conv_w = args->conv_w; m.conv_b = args->conv_b; m.dt_bias = args->dt_bias; m.a_log = args->a_log; m.d_skip = args->d_skip; m.norm_w = args->norm_w;
+    m.eps = args->eps; m.ring = args->ring; m.ssm = args->ssm; m.xbc = args->xbc; m.gated = args->gated;
+    m.out = args->out; m.out_ld = args->out_ld; m.out_cols = args->out_cols; m.engine = args->engine;
+    return launch_mamba2(m, step_place(place), args->dtype, as_stream(stream));
 }
 
 }  // extern "C"
