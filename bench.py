@@ -24,7 +24,9 @@ of the operator configurations.
 
 `--workload c0|c1|c2|c3` measures the smaller configurations on one GPU (the f32
 4-layer model end to end, the GEMM sweep, the SwiGLU MLP, ragged decode attention),
-each with the CPU restatement timed beside it on a stated sample.
+each with the CPU restatement timed beside it on a stated sample.  `--workload bolonex`
+measures prefill and decode of Bolonex models at a few real-model sizes, each beside a
+GPT of the same width, depth and feed-forward weights (1 GPU).
 
 The CPU arm times this repository's restatement of the reference's CPU executor
 (oracle/) on the host cores: the reference is Rust and cannot be built here.
@@ -76,7 +78,7 @@ def parse_args():
     ap.add_argument("--prefill", type=int, default=PREFILL)
     ap.add_argument("--layers", type=int, default=12)
     ap.add_argument("--vocab", type=int, default=32000)
-    ap.add_argument("--workload", default="c4", choices=["c4", "c0", "c1", "c2", "c3"],
+    ap.add_argument("--workload", default="c4", choices=["c4", "c0", "c1", "c2", "c3", "bolonex"],
                     help="c4 (default): the serving decode benchmark; c0: the 4-layer d128 f32 model, 16-token prompt + 64 "
                          "greedy steps; c1: GEMM sweep; c2: SwiGLU MLP; c3: ragged decode attention -- each with the CPU "
                          "restatement timed beside it (1 GPU)")
@@ -403,7 +405,7 @@ def _percentile(xs, q):
     return float(np.percentile(np.asarray(xs, dtype=np.float64), q))
 
 
-def measure_decode(args, cfg, sessions, rank, local_rank, world, barrier, reduce_max, full):
+def measure_decode(args, cfg, sessions, rank, local_rank, world, barrier, reduce_max, full, arrays=None):
     """Prefill `sessions` sessions on this rank, then time K greedy steps from position `prefill`, `--repeats` times
     (every repeat starts over from the same position and ids).  Returns the per-repeat milliseconds (max over ranks)
     and, when `full`, the attention-kernel profile and the end-to-end loop as well."""
@@ -423,7 +425,8 @@ def measure_decode(args, cfg, sessions, rank, local_rank, world, barrier, reduce
     def position_of(step):
         return args.prefill + step % span
     lib = _native.lib()
-    arrays = normal_model_arrays(cfg, seed=5, std=0.02)
+    if arrays is None:
+        arrays = normal_model_arrays(cfg, seed=5, std=0.02)
     sess = B200Session(cfg, sessions, capacity, device=local_rank, logits_mode="none", step_parts=args.step_parts,
                        small_batch_mode=args.small_batch_mode)
     for i, a in enumerate(arrays):
@@ -529,6 +532,50 @@ def measure_decode(args, cfg, sessions, rank, local_rank, world, barrier, reduce
         out["e2e_same_tokens"] = bool(np.array_equal(cur, tokens_after_timed))
     sess.close()
     return out
+
+
+# (name, sessions, prefill, width, layers, heads, kv_heads, head_dim, mamba2 heads, mamba2 head width, state, feed-forward of the
+# two-matrix block, of the GPT's three-matrix block): equal feed-forward weights, every fourth layer attention
+BOLONEX_SIZES = [
+    ("12x768, 256 sessions", 256, 512, 768, 12, 12, 4, 64, 24, 64, 128, 3072, 2048),
+    ("12x768, 32 sessions", 32, 512, 768, 12, 12, 4, 64, 24, 64, 128, 3072, 2048),
+    ("12x1024, 64 sessions", 64, 1024, 1024, 12, 16, 4, 64, 32, 64, 128, 4224, 2816),
+    ("12x768, one session of 1792 tokens", 1, 1792, 768, 12, 12, 4, 64, 24, 64, 128, 3072, 2048),
+]
+
+
+def run_bolonex(args):
+    """Prefill and decode tokens/s of Bolonex beside the closest model here, a GPT of equal width, depth and feed-forward
+    weights; value = decode tokens/s of the first size."""
+    import copy
+    import torch
+    from tnsr_b200.nn import GptConfig
+    from tnsr_b200.synthetic import bolonex_arrays, bolonex_config
+    torch.cuda.set_device(0)
+    cases, clocks, launches = [], None, 0
+    barrier = torch.cuda.synchronize
+    for name, sessions, prefill, width, layers, heads, kv, hd, mh, mw, state, ff, gpt_ff in BOLONEX_SIZES:
+        a = copy.copy(args)
+        a.prefill, a.steps, a.repeats = prefill, min(args.steps, 64), min(args.repeats, 5)
+        model = bolonex_config(width, layers, heads, kv, hd, mh, mw, state, ff, args.vocab)
+        gpt = GptConfig(vocab_size=args.vocab, max_sequence_length=2048, embed_dim=width, num_heads=width // 64, feed_forward_dim=gpt_ff,
+                        num_layers=layers, layer_norm_epsilon=1e-5, activation="swiglu", weight_dtype="bf16")
+        case = {"case": name, "sessions": sessions, "prefill": prefill}
+        for label, cfg, arrays in (("bolonex", model, bolonex_arrays(model, seed=5)), ("gpt", gpt, None)):
+            r = measure_decode(a, cfg, sessions, 0, 0, 1, barrier, float, False, arrays)
+            ms = float(np.median(r["samples_ms"])) / a.steps
+            case[label] = {"decode_ms_per_step": ms, "decode_tokens_per_s": sessions / ms * 1e3, "prefill_ms": r["prefill_ms"],
+                           "prefill_tokens_per_s": sessions * prefill / r["prefill_ms"] * 1e3}
+            if label == "bolonex":
+                launches += r["launches"]
+                clocks = clocks or r["clocks"]
+        cases.append(case)
+    first = cases[0]["bolonex"]
+    line = _op_line(args, "bolonex_decode_tokens_per_s", "tokens/s", first["decode_tokens_per_s"], first["decode_ms_per_step"], "bf16",
+                    "Bolonex beside a GPT of equal width, depth and feed-forward weights; value = decode of " + cases[0]["case"], None, None,
+                    cases, launches, clocks)
+    line["steps"] = min(args.steps, 64)
+    print(json.dumps(line), flush=True)
 
 
 def operator_summary(samples):
@@ -687,6 +734,9 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         run_reference(args)
+    elif args.workload == "bolonex":
+        if int(os.environ.get("RANK", "0")) == 0:
+            run_bolonex(args)
     elif args.workload != "c4":
         if int(os.environ.get("RANK", "0")) == 0:
             run_ops(args)

@@ -8,6 +8,7 @@
     python -m tnsr_b200.opbench serving_attention  # configuration 4's decode attention: 256 x 12 x 64, 641 live keys
     python -m tnsr_b200.opbench elementwise # LayerNorm, SwiGLU, embedding, greedy pick
     python -m tnsr_b200.opbench prefill_attention  # configuration 4's prefill attention on both engines
+    python -m tnsr_b200.opbench mixers      # the mixers of described models: grouped attention, mamba2, RMS norm
     python -m tnsr_b200.opbench all
 
 Every line is one JSON object: algorithmic flops / bytes, CUDA-event time (median of `--samples`
@@ -293,20 +294,104 @@ def bench_elementwise(samples):
     emit(op="argmax", rows=rows, vocab=vocab, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
 
 
+def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads, hd, softcap, name):
+    """Grouped-query attention with capped scores and gates: `chunk` queries per session after `position` cached rows.
+    Algorithmic bytes: the live K/V rows and q / out once; flops: 4 hd per (query, head, visible key)."""
+    hbm, tf, kind = peaks()
+    capacity = position + chunk
+    g = torch.Generator(device="cuda").manual_seed(8)
+    randn = lambda *shape: torch.randn(shape, device="cuda", generator=g).to(torch.bfloat16)
+    nbytes = sessions * 2.0 * ((position + chunk) * kv_heads * 2 * hd + chunk * heads * 2 * hd)
+    sets = copies_for(int(nbytes))
+    q = [randn(sessions * chunk, heads * hd) for _ in range(sets)]
+    k = [randn(sessions, capacity, kv_heads * hd) for _ in range(sets)]
+    v = [randn(sessions, capacity, kv_heads * hd) for _ in range(sets)]
+    gate = torch.randn((sessions * chunk, 32), device="cuda", generator=g)
+    out = torch.empty((sessions * chunk, heads * hd), device="cuda", dtype=torch.bfloat16)
+    size = lib().tnsr_b200_grouped_attention_workspace(hd, hd)
+    ws = torch.zeros(size, dtype=torch.uint8, device="cuda")
+    where = _native.Place(sessions, chunk, position, 0, None)
+    args = [_native.GroupedAttentionArgs(q[i].data_ptr(), k[i].data_ptr(), v[i].data_ptr(), gate.data_ptr(), out.data_ptr(), ws.data_ptr(), size,
+                                         heads, kv_heads, hd, hd, capacity, 32, heads * hd, heads * hd, hd ** -0.5, softcap, 1, 0) for i in range(sets)]
+    ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_grouped_attention(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
+    pairs = sessions * heads * sum(position + t + 1 for t in range(chunk))
+    flops = 4.0 * hd * pairs
+    emit(op="grouped_attention", case=name, sessions=sessions, chunk=chunk, position=position, heads=heads, kv_heads=kv_heads, head_dim=hd,
+         softcap=softcap, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf,
+         peaks=kind)
+
+
+def bench_mamba2(samples, sessions, chunk, heads, vdim, state, groups, name):
+    """The mamba2 mixer between its projections.  Algorithmic bytes: projected rows in, mixer rows out, the f32 state in and
+    out; flops of the chunked form (chunks of 64): C B^T (causal half), weights x, C S and B x^T per head."""
+    hbm, tf, kind = peaks()
+    inner, gn = heads * vdim, groups * state
+    channels, proj = inner + 2 * gn, 2 * inner + 2 * gn
+    rows = sessions * chunk
+    g = torch.Generator(device="cuda").manual_seed(9)
+    nbytes = rows * 2.0 * (proj + inner) + rows * 4.0 * heads + sessions * heads * state * vdim * 8.0
+    sets = min(8, copies_for(int(nbytes)))
+    ld = (proj + 31) // 32 * 32
+    u = [torch.randn((rows, ld), device="cuda", generator=g).to(torch.bfloat16) for _ in range(sets)]
+    ssm = [torch.zeros((sessions, heads, state, vdim), device="cuda") for _ in range(sets)]
+    dt = torch.randn((rows, heads), device="cuda", generator=g)
+    f32 = lambda *shape: torch.rand(shape, device="cuda", generator=g)
+    conv, conv_b, vec, norm = f32(channels, 4), f32(channels), f32(heads), f32(inner)
+    ring = torch.zeros((sessions, 4, channels), device="cuda", dtype=torch.bfloat16)
+    xbc = torch.empty((rows, channels), device="cuda", dtype=torch.bfloat16)
+    gated = torch.empty((rows, inner), device="cuda", dtype=torch.bfloat16)
+    out = torch.empty((rows, inner), device="cuda", dtype=torch.bfloat16)
+    where = _native.Place(sessions, chunk, 64, 0, None)
+    args = [_native.Mamba2Args(u[i].data_ptr(), dt.data_ptr(), conv.data_ptr(), conv_b.data_ptr(), vec.data_ptr(), vec.data_ptr(), vec.data_ptr(),
+                               norm.data_ptr(), ring.data_ptr(), ssm[i].data_ptr(), xbc.data_ptr(), gated.data_ptr(), out.data_ptr(), ld, heads,
+                               heads, vdim, state, groups, groups, 4, inner, inner, 1e-5, 1, 0, 0) for i in range(sets)]
+    ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_mamba2(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
+    q = 64
+    flops = rows * (2.0 * q * state * groups / 2 + heads * (2.0 * q * vdim / 2 + 4.0 * state * vdim)) if chunk > 1 else rows * heads * 6.0 * state * vdim
+    emit(op="mamba2", case=name, sessions=sessions, chunk=chunk, heads=heads, vdim=vdim, state=state, groups=groups, ms=ms, gbs=nbytes / ms / 1e6,
+         frac_hbm=nbytes / ms / 1e6 / hbm, tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf, peaks=kind)
+
+
+def bench_mixers(samples):
+    """Beside the GPT kernels of the same sizes (serving_attention, prefill_attention, elementwise)."""
+    bench_attention(samples, serving=True)
+    bench_grouped_attention(samples, 256, 1, 640, 12, 12, 64, 30.0, "decode, a key/value head per head")
+    bench_grouped_attention(samples, 256, 1, 640, 12, 4, 64, 30.0, "decode, 3 heads per key/value head")
+    bench_grouped_attention(samples, 64, 1, 1536, 16, 2, 128, 30.0, "decode, 8 heads of 128 per key/value head")
+    bench_grouped_attention(samples, 1, 1, 8191, 12, 4, 64, 30.0, "decode, one long session")
+    bench_prefill_attention(samples)
+    bench_grouped_attention(samples, 64, 512, 0, 12, 12, 64, 30.0, "prefill, a key/value head per head")
+    bench_grouped_attention(samples, 64, 512, 0, 12, 12, 64, 0.0, "prefill, a key/value head per head, no cap")
+    bench_grouped_attention(samples, 64, 512, 0, 12, 4, 64, 30.0, "prefill, 3 heads per key/value head")
+    bench_grouped_attention(samples, 16, 1024, 0, 16, 2, 128, 30.0, "prefill, 8 heads of 128 per key/value head")
+    bench_mamba2(samples, 256, 1, 24, 64, 128, 1, "decode")
+    bench_mamba2(samples, 32, 1, 24, 64, 128, 1, "decode, 32 sessions")
+    bench_mamba2(samples, 64, 512, 24, 64, 128, 1, "prefill")
+    bench_mamba2(samples, 256, 512, 24, 64, 128, 1, "prefill, 256 sessions")
+    bench_mamba2(samples, 1, 4096, 24, 64, 128, 1, "prefill, one long prompt")
+    hbm, _, kind = peaks()
+    rows, d = 131072, 768
+    x, w = torch.randn((rows, d), device="cuda"), torch.ones(d, device="cuda")
+    y = torch.empty((rows, d), device="cuda", dtype=torch.bfloat16)
+    ms, _ = timed(lambda _: ok(lib().tnsr_b200_rmsnorm(ptr(x), ptr(w), 1.0, ptr(y), rows, d, 1e-5, 1, stream())), 1, samples)
+    nbytes = rows * d * 6.0
+    emit(op="rmsnorm_f32_to_bf16", rows=rows, width=d, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "skinny_gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "all"])
+    ap.add_argument("what", choices=["gemm", "skinny_gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers", "all"])
     ap.add_argument("--samples", type=int, default=20)
     args = ap.parse_args()
     if not torch.cuda.is_available():
         sys.exit("opbench needs a CUDA device")
-    todo = (["gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention"]
+    todo = (["gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers"]
             if args.what == "all" else [args.what])
     for name in todo:
         {"gemm": bench_gemm, "skinny_gemm": lambda n: bench_gemm(n, shapes=[(m, 4096, 4096) for m in (1, 8, 64)], outs=("bf16",)),
          "serving_gemms": bench_serving_gemms, "mlp": bench_mlp, "attention": bench_attention,
          "serving_attention": lambda n: bench_attention(n, serving=True),
-         "elementwise": bench_elementwise, "prefill_attention": bench_prefill_attention}[name](args.samples)
+         "elementwise": bench_elementwise, "prefill_attention": bench_prefill_attention, "mixers": bench_mixers}[name](args.samples)
 
 
 if __name__ == "__main__":

@@ -35,6 +35,41 @@ def normal_model_arrays(cfg: GptConfig, seed: int, std: float = 0.02, bias_std: 
     return arrays
 
 
+def bolonex_config(width, layers, heads, kv_heads, head_dim, ssm_heads, ssm_dim, state, feed_forward, vocab_size, attention_every=4,
+                   max_sequence_length=2048):
+    """A Bolonex of real-model proportions: every `attention_every`-th layer attention, the others mamba2, none sharing."""
+    from .bolonex import BolonexConfig, LayerConfig, RotaryConfig
+    rotary = RotaryConfig(head_dim, 500000.0, 8.0, 1.0, 4.0, 8192.0)
+    attention = LayerConfig("attention", heads, head_dim, 4, feed_forward, kv_heads=kv_heads, dim=head_dim, rotary=rotary,
+                            scale=head_dim ** -0.5, softcap=30.0)
+    mamba = LayerConfig("mamba2", ssm_heads, ssm_dim, 4, feed_forward, state=state, groups=1, norm_groups=1)
+    return BolonexConfig(vocab_size, width, tuple(attention if i % attention_every == 0 else mamba for i in range(layers)), 1.0, 1e-5, "bf16",
+                         max_sequence_length)
+
+
+def bolonex_arrays(cfg, seed: int, std: float = 0.02):
+    """Parameter arrays of a Bolonex in the order of its tensor table: matrices N(0, std), norms and skips one, decays and
+    step biases in the range a trained layer has."""
+    rng = np.random.default_rng(seed)
+    arrays = []
+    for name, shape in cfg.tensor_shapes().items():
+        leaf = name.split(".")[-1]
+        if name.endswith(("norm1", "final.norm")) or leaf == "b":
+            a = np.zeros(shape, np.float32)
+        elif leaf in ("norm", "D"):
+            a = np.ones(shape, np.float32)
+        elif leaf == "conv":
+            a = rng.uniform(-0.5, 0.5, shape).astype(np.float32)
+        elif leaf == "dt_bias":
+            a = rng.uniform(-4.0, -1.0, shape).astype(np.float32)
+        elif leaf == "A_log":
+            a = np.log(rng.uniform(1.0, 16.0, shape)).astype(np.float32)
+        else:
+            a = rng.standard_normal(shape, dtype=np.float32) * np.float32(std)
+        arrays.append(a)
+    return arrays
+
+
 def config0_model(activation="relu"):
     cfg = GptConfig(vocab_size=96, max_sequence_length=128, embed_dim=128, num_heads=4,
                     feed_forward_dim=512, num_layers=4, layer_norm_epsilon=1e-5, activation=activation)
