@@ -543,7 +543,10 @@ typedef struct tnsr_b200_place {
  * [sessions, chunk, heads, dim], k_cache [sessions, capacity, kv_heads, dim],
  * v_cache [.., vdim], out [sessions, chunk, out_ld], columns from heads * vdim to
  * out_cols are zeroed.  dtype: element type of q, caches and out.  engine: 0 =
- * best kernel for the shape, 1 = one warp per (query, head).  workspace:
+ * best kernel for the shape, 1 = one warp per (query, head), 2 = warp-level tensor
+ * cores only.  A host-known position (d_positions NULL) is what the tcgen05
+ * kernel of long chunks needs; d_status (may be NULL) receives 2 if one of its
+ * bounded waits gave up.  workspace:
  * tnsr_b200_grouped_attention_workspace() bytes, zeroed once (NULL: the keys of
  * a session are not divided over CTAs). */
 typedef struct tnsr_b200_grouped_attention_args {
@@ -551,6 +554,7 @@ typedef struct tnsr_b200_grouped_attention_args {
     const float* gate;
     void* out;
     void* workspace;
+    int* d_status;
     uint64_t workspace_bytes;
     uint32_t heads, kv_heads, dim, vdim, capacity, gate_ld, out_ld, out_cols;
     float scale, softcap;

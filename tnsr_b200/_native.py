@@ -56,7 +56,7 @@ class Place(C.Structure):
 
 
 class GroupedAttentionArgs(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "gate", "out", "workspace")] + [("workspace_bytes", C.c_uint64)] + \
+    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "gate", "out", "workspace", "d_status")] + [("workspace_bytes", C.c_uint64)] + \
         [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "capacity", "gate_ld", "out_ld", "out_cols")] + \
         [("scale", C.c_float), ("softcap", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32)]
 

@@ -55,6 +55,13 @@ embedding_kernel(const T* __restrict__ tok, const T* __restrict__ pos, const uin
     }
     const T* tr = tok + (size_t)id * width;
     if (!pos) {
+        if (width % 4 == 0) {
+            for (uint32_t c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
+                const float4 v = load4<T>(tr + c);
+                *reinterpret_cast<float4*>(o + c) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+            }
+            return;
+        }
         for (uint32_t c = threadIdx.x; c < width; c += blockDim.x) o[c] = load1<T>(tr + c) * scale;
         return;
     }

@@ -9,6 +9,7 @@
 //                           loop); warps merge through shared memory, splits through a workspace by whichever CTA is last,
 //                           in split order, so results do not depend on timing.
 //  * grouped_tile_kernel    many rows (prefill): 64 rows per CTA, all warps share double-buffered key tiles.
+// Prefill with heads of 64 at a position the host knows runs on the tcgen05 kernel of prefill_tc.cu instead.
 //
 // Scores, softmax statistics and accumulators are f32; the weights enter the value product as two bf16 halves
 // (split_bf16x2), so they keep 16 bits.  A capped score costs three special-function results instead of one:
@@ -109,24 +110,6 @@ grouped_split_kernel(GaParams P) {
     const uint32_t tiles = (keys + 15) / 16, per_split = (tiles + P.splits - 1) / P.splits;
     const uint32_t tile0 = min(tiles, split * per_split), tile1 = min(tiles, tile0 + per_split);
 
-    // query fragments straight from global memory: rows g8 and g8 + 8
-    uint32_t qa[DK / 16][4];
-    const bf16* q = reinterpret_cast<const bf16*>(a.q);
-    const size_t q_ld = (size_t)a.heads * a.dim;
-    auto q_pair = [&](uint32_t r, uint32_t c) -> uint32_t {
-        if (r >= n_rows || c >= a.dim) return 0u;
-        const uint32_t R = row0 + r;
-        const bf16* src = q + ((size_t)s * P.place.chunk + R / P.per) * q_ld + (size_t)(kvh * P.per + R % P.per) * a.dim + c;
-        const uint32_t lo = __bfloat16_as_ushort(src[0]), hi = c + 1 < a.dim ? __bfloat16_as_ushort(src[1]) : 0u;
-        return lo | (hi << 16);
-    };
-#pragma unroll
-    for (int kk = 0; kk < DK / 16; ++kk) {
-        qa[kk][0] = q_pair(g8, kk * 16 + t4 * 2);
-        qa[kk][1] = UPPER ? q_pair(g8 + 8, kk * 16 + t4 * 2) : 0u;
-        qa[kk][2] = q_pair(g8, kk * 16 + 8 + t4 * 2);
-        qa[kk][3] = UPPER ? q_pair(g8 + 8, kk * 16 + 8 + t4 * 2) : 0u;
-    }
     const uint32_t lim0 = p0 + (row0 + min(g8, n_rows - 1)) / P.per, lim1 = p0 + (row0 + min(g8 + 8, n_rows - 1)) / P.per;
 
     uint8_t* ring = smem + warp * (STAGES * S::STAGE);
@@ -142,12 +125,31 @@ grouped_split_kernel(GaParams P) {
         }
         mx_commit();
     };
+#pragma unroll
+    for (int i = 0; i < STAGES - 1; ++i) load(tile0 + warp + i * GA_WARPS, i);
+    // query fragments straight from global memory: rows g8 and g8 + 8
+    uint32_t qa[DK / 16][4];
+    const bf16* q = reinterpret_cast<const bf16*>(a.q);
+    const size_t q_ld = (size_t)a.heads * a.dim;
+    auto q_pair = [&](uint32_t r, uint32_t c) -> uint32_t {
+        if (r >= n_rows || c >= a.dim) return 0u;
+        const uint32_t R = row0 + r;
+        const bf16* src = q + ((size_t)s * P.place.chunk + R / P.per) * q_ld + (size_t)(kvh * P.per + R % P.per) * a.dim + c;
+        if (P.vec) return *reinterpret_cast<const uint32_t*>(src);
+        const uint32_t lo = __bfloat16_as_ushort(src[0]), hi = c + 1 < a.dim ? __bfloat16_as_ushort(src[1]) : 0u;
+        return lo | (hi << 16);
+    };
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+        qa[kk][0] = q_pair(g8, kk * 16 + t4 * 2);
+        qa[kk][1] = UPPER ? q_pair(g8 + 8, kk * 16 + t4 * 2) : 0u;
+        qa[kk][2] = q_pair(g8, kk * 16 + 8 + t4 * 2);
+        qa[kk][3] = UPPER ? q_pair(g8 + 8, kk * 16 + 8 + t4 * 2) : 0u;
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
-#pragma unroll
-    for (int i = 0; i < STAGES - 1; ++i) load(tile0 + warp + i * GA_WARPS, i);
     uint32_t stage = 0;
     for (uint32_t i = tile0 + warp; i < tile1; i += GA_WARPS) {
         mx_wait<STAGES - 2>();
@@ -503,9 +505,13 @@ uint32_t padded_width(uint32_t dim, uint32_t vdim) {
     return w <= 64 ? 64 : w <= 128 ? 128 : 256;
 }
 
-// Splits of the keys: three CTAs per SM if the (session, key/value head, row tile) triples do not give them already.
+// Splits of the keys: as many CTAs as fit the GPU at once (three, two or one per SM at padded widths 64, 128, 256) if the
+// (session, key/value head, row tile) triples do not give them already.
 constexpr uint64_t GA_CTAS = 444;
-uint32_t splits_for(uint64_t units) { return (uint32_t)std::min<uint64_t>(GA_MAX_SPLITS, std::max<uint64_t>(1, GA_CTAS / units)); }
+uint32_t splits_for(uint64_t units, uint32_t padded) {
+    const uint64_t slots = padded == 64 ? GA_CTAS : padded == 128 ? 296 : 148;
+    return (uint32_t)std::min<uint64_t>(GA_MAX_SPLITS, std::max<uint64_t>(1, slots / units));
+}
 // More than one split means at most GA_CTAS / 2 units and GA_CTAS partial tiles.
 constexpr uint64_t GA_COUNTER_BYTES = 1024;
 static_assert(GA_COUNTER_BYTES >= GA_CTAS / 2 * 4, "one merge counter per unit");
@@ -545,7 +551,7 @@ int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, 
     if (P.rows <= GA_SPLIT_ROWS || place.chunk == 1) {
         P.row_tiles = ceil_div(P.rows, 16u);
         const uint64_t units = (uint64_t)place.sessions * a.kv_heads * P.row_tiles;
-        P.splits = splits_for(units);
+        P.splits = splits_for(units, w);
         if (!a.workspace || a.workspace_bytes < grouped_attention_workspace_bytes(a.dim, a.vdim)) P.splits = 1;
         if (P.splits > 1) {
             P.done = reinterpret_cast<uint32_t*>(a.workspace);
@@ -555,6 +561,8 @@ int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, 
         if (w == 64) rc = upper ? launch_split<64, 64, 4, true>(P, stream) : launch_split<64, 64, 4, false>(P, stream);
         else if (w == 128) rc = upper ? launch_split<128, 128, 3, true>(P, stream) : launch_split<128, 128, 3, false>(P, stream);
         else rc = upper ? launch_split<256, 256, 2, true>(P, stream) : launch_split<256, 256, 2, false>(P, stream);
+    } else if (a.engine == 0 && grouped_attention_tc_eligible(a, place)) {
+        return launch_grouped_attention_tc(a, place, stream);
     } else {
         P.row_tiles = ceil_div(P.rows, 64u);
         if (w == 64) rc = launch_tile<64, 64, 64>(P, stream);

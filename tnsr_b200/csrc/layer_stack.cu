@@ -482,6 +482,7 @@ int stack_step(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t chunk,
             a.gate = S->tail; a.gate_ld = L.tail_cols;
             a.out = S->cat; a.out_ld = L.k_out; a.out_cols = L.mixer_cols;
             a.paging = pg;
+            a.d_status = dec->d_status;
             a.workspace = S->attention_ws; a.workspace_bytes = S->attention_ws_bytes;
             a.engine = chunk > 1 && c.prefill_mode == TNSR_B200_PREFILL_SCALAR ? 1 : 0;
             RUN(dec, launch_grouped_attention(a, place, dtype, st));

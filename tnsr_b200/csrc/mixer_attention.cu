@@ -44,78 +44,103 @@ attention_prep_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t r
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
         const uint32_t c = 2 * (lane + 32 * i);
+        const bool first = c < width, second = c + 1 < width;
         nw[i] = make_float2(1.0f, 1.0f);
-        if (which < 2 && c < width) {
+        if (which < 2 && first) {
             const float* g = which == 0 ? a.q_norm : a.k_norm;
-            nw[i] = make_float2(g[c], c + 1 < width ? g[c + 1] : 0.0f);
+            nw[i] = make_float2(g[c], second ? g[c + 1] : 0.0f);
+        }
+        const float* cw = a.conv_w + (size_t)(ch0 + c) * a.taps;
+        if (TAPS == 4 && a.taps == 4) {
+            const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            const float4 x = first ? *reinterpret_cast<const float4*>(cw) : zero, y = second ? *reinterpret_cast<const float4*>(cw + 4) : zero;
+            w[0][i] = make_float2(x.x, y.x);
+            w[TAPS > 1 ? 1 : 0][i] = make_float2(x.y, y.y);
+            w[TAPS > 2 ? 2 : 0][i] = make_float2(x.z, y.z);
+            w[TAPS > 3 ? 3 : 0][i] = make_float2(x.w, y.w);
+        } else {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                const int src = j - (TAPS - (int)a.taps);
+                w[j][i].x = src >= 0 && first ? cw[src] : 0.0f;
+                w[j][i].y = src >= 0 && second ? cw[a.taps + src] : 0.0f;
+            }
         }
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
-            const int src = j - (TAPS - (int)a.taps);
-            const bool ok = src >= 0 && c < width;
-            w[j][i].x = ok ? a.conv_w[(size_t)(ch0 + c) * a.taps + src] : 0.0f;
-            w[j][i].y = ok && c + 1 < width ? a.conv_w[(size_t)(ch0 + c + 1) * a.taps + src] : 0.0f;
             // the window holds tokens t - TAPS + 1 .. t; before the first token: t0 - TAPS + 1 .. t0 - 1 in slots 1 ..
             win[j][i] = make_float2(0.0f, 0.0f);
             const int t = (int)t0 - TAPS + j;      // token that slot j holds before the first shift
-            if (j > 0 && (int)t0 - t < (int)a.taps && c < width) {
+            if (j > 0 && (int)t0 - t < (int)a.taps && first) {
                 const long long pos = (long long)p0 + t;
-                if (t >= 0) win[j][i] = load_pair<T>(rows + (size_t)t * a.ld + c, vec, c + 1 < width);
-                else if (pos >= 0) win[j][i] = load_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, vec, c + 1 < width);
+                if (t >= 0) win[j][i] = load_pair<T>(rows + (size_t)t * a.ld + c, vec, second);
+                else if (pos >= 0) win[j][i] = load_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, vec, second);
             }
         }
     }
     const uint32_t pairs = a.rotary_dims / 2;
-    for (uint32_t t = t0; t < t1; ++t) {
-        float2 y[NP];
-        float ss = 0.0f;
+    // a few tokens' inputs and angles are asked for together, so that their round trips overlap
+    constexpr uint32_t AHEAD = NP == 1 ? 4 : NP == 2 ? 2 : 1;
+    for (uint32_t tb = t0; tb < t1; tb += AHEAD) {
+        float2 next[AHEAD][NP], angle[AHEAD][NP];
 #pragma unroll
-        for (int i = 0; i < NP; ++i) {
-            const uint32_t c = 2 * (lane + 32 * i);
+        for (uint32_t u = 0; u < AHEAD; ++u)
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
-            win[TAPS - 1][i] = c < width ? load_pair<T>(rows + (size_t)t * a.ld + c, vec, c + 1 < width) : make_float2(0.0f, 0.0f);
-            y[i] = make_float2(0.0f, 0.0f);
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) {
-                y[i].x = fmaf(w[j][i].x, win[j][i].x, y[i].x);
-                y[i].y = fmaf(w[j][i].y, win[j][i].y, y[i].y);
+            for (int i = 0; i < NP; ++i) {
+                const uint32_t pi = lane + 32 * i, c = 2 * pi;
+                const bool there = tb + u < t1;
+                next[u][i] = there && c < width ? load_pair<T>(rows + (size_t)(tb + u) * a.ld + c, vec, c + 1 < width) : make_float2(0.0f, 0.0f);
+                angle[u][i] = there && which < 2 && pi < pairs ? a.rotation[(size_t)(p0 + tb + u) * pairs + pi] : make_float2(1.0f, 0.0f);
             }
-            ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, ss));
-        }
-        const uint32_t pos = p0 + t;
-        if (place.chunk == 1) {
-            // the slot of this position held the oldest row, which no single-token step reads
+#pragma unroll
+        for (uint32_t u = 0; u < AHEAD; ++u) {
+            const uint32_t t = tb + u;
+            if (t >= t1) break;
+            float2 y[NP];
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
+                win[TAPS - 1][i] = next[u][i];
+                y[i] = make_float2(0.0f, 0.0f);
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    y[i].x = fmaf(w[j][i].x, win[j][i].x, y[i].x);
+                    y[i].y = fmaf(w[j][i].y, win[j][i].y, y[i].y);
+                }
+                ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, ss));
+            }
+            const uint32_t pos = p0 + t;
+            if (place.chunk == 1) {
+                // the slot of this position held the oldest row, which no single-token step reads
+#pragma unroll
+                for (int i = 0; i < NP; ++i) {
+                    const uint32_t c = 2 * (lane + 32 * i);
+                    if (c < width) store_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, win[TAPS - 1][i], vec, c + 1 < width);
+                }
+            }
+            if (which < 2) {
+                const float inv = rsqrtf(mx_warp_sum(ss) / (float)width + a.eps);
+#pragma unroll
+                for (int i = 0; i < NP; ++i) {
+                    const float2 v = make_float2(y[i].x * (inv * nw[i].x), y[i].y * (inv * nw[i].y)), cs = angle[u][i];
+                    // pairs past the rotated dimensions have the angle zero
+                    y[i] = make_float2(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y);
+                }
+            }
+            T* dst;
+            if (which == 0) dst = reinterpret_cast<T*>(a.q) + ((size_t)s * place.chunk + t) * nq + head * a.dim;
+            else {
+                const size_t row = kv_row(a.paging, s, pos, a.capacity);
+                dst = which == 1 ? reinterpret_cast<T*>(a.k_cache) + row * nk + head * a.dim
+                                 : reinterpret_cast<T*>(a.v_cache) + row * ((size_t)a.kv_heads * a.vdim) + head * a.vdim;
+            }
 #pragma unroll
             for (int i = 0; i < NP; ++i) {
                 const uint32_t c = 2 * (lane + 32 * i);
-                if (c < width) store_pair<T>(ring + (size_t)(pos % a.taps) * channels + c, win[TAPS - 1][i], vec, c + 1 < width);
+                if (c < width) store_pair<T>(dst + c, y[i], vec, c + 1 < width);
             }
-        }
-        if (which < 2) {
-            const float inv = rsqrtf(mx_warp_sum(ss) / (float)width + a.eps);
-#pragma unroll
-            for (int i = 0; i < NP; ++i) {
-                const uint32_t pi = lane + 32 * i;
-                y[i].x *= inv * nw[i].x;
-                y[i].y *= inv * nw[i].y;
-                if (pi < pairs) {
-                    const float2 cs = a.rotation[(size_t)pos * pairs + pi];
-                    y[i] = make_float2(y[i].x * cs.x - y[i].y * cs.y, y[i].y * cs.x + y[i].x * cs.y);
-                }
-            }
-        }
-        T* dst;
-        if (which == 0) dst = reinterpret_cast<T*>(a.q) + ((size_t)s * place.chunk + t) * nq + head * a.dim;
-        else {
-            const size_t row = kv_row(a.paging, s, pos, a.capacity);
-            dst = which == 1 ? reinterpret_cast<T*>(a.k_cache) + row * nk + head * a.dim
-                             : reinterpret_cast<T*>(a.v_cache) + row * ((size_t)a.kv_heads * a.vdim) + head * a.vdim;
-        }
-#pragma unroll
-        for (int i = 0; i < NP; ++i) {
-            const uint32_t c = 2 * (lane + 32 * i);
-            if (c < width) store_pair<T>(dst + c, y[i], vec, c + 1 < width);
         }
     }
 }
@@ -144,7 +169,7 @@ int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dt
         set_thread_error("attention: head widths up to 256, 1..16 convolution taps, an even number of rotated dimensions");
         return TNSR_B200_ERR_UNSUPPORTED;
     }
-    const uint32_t run = std::min(place.chunk, 16u), runs = ceil_div(place.chunk, run);
+    const uint32_t run = std::min(place.chunk, 32u), runs = ceil_div(place.chunk, run);
     const uint64_t total = (uint64_t)place.sessions * runs * (a.heads + 2 * a.kv_heads);
     if (total > 0x7fffffffull) { set_thread_error("attention: too many rows for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
     if (dtype == TNSR_B200_BF16) prep_width<bf16>(a, place, run, runs, (uint32_t)total, stream);

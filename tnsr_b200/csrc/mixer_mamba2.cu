@@ -2,9 +2,9 @@
 //     S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t
 // with x, B, C behind a causal convolution and silu, dt behind softplus, then y * silu(z) and an RMS norm in groups.
 //
-//  * conv_silu_kernel          convolution + silu of a multi-token chunk, sliding window in registers
-//  * ssd_token_kernel          token by token with the state in registers: single-token steps (convolution fused in,
-//                              the state makes one trip through HBM), f32 sessions, and shapes the chunked scan leaves out
+//  * conv_silu_kernel          convolution + silu, sliding window in registers (single-token steps also update the ring)
+//  * ssd_token_kernel          token by token with the state in registers: single-token steps (the state makes one trip
+//                              through HBM), short chunks, f32 sessions
 //  * gated_norm_kernel         the grouped RMS norm of y * silu(z)
 // The chunked tensor-core scan of long chunks is in ssd_scan.cu.
 #include <algorithm>
@@ -33,7 +33,7 @@ __device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, const float* __restrict__ conv_w,
-                 const float* __restrict__ conv_b, const T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run,
+                 const float* __restrict__ conv_b, T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run,
                  uint32_t vec) {
     pdl_wait();
     pdl_trigger();
@@ -58,6 +58,20 @@ conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uin
         }
     }
     const float2 b = make_float2(conv_b[c], second ? conv_b[c + 1] : 0.0f);
+    if (place.chunk == 1) {
+        // the slot of this position held the oldest row, which no single-token step reads
+        const float2 now = load_pair<T>(in, vec, second);
+        float2 y = b;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const float2 u = j + 1 < TAPS ? win[j + 1] : now;
+            y.x = fmaf(w[j].x, u.x, y.x);
+            y.y = fmaf(w[j].y, u.y, y.y);
+        }
+        store_pair<T>(dst, make_float2(act_silu<T>(y.x), act_silu<T>(y.y)), vec, second);
+        store_pair<T>(ring + ((size_t)s * taps + p0 % taps) * channels + c, now, vec, second);
+        return;
+    }
     // rows are asked for eight at a time, so that their round trips overlap
     constexpr uint32_t AHEAD = 8;
     for (uint32_t t = t0; t < t1; t += AHEAD) {
@@ -85,109 +99,116 @@ static void conv_silu_typed(const Mamba2& m, uint32_t inner, uint32_t channels, 
     const T* rows = (const T*)m.proj + inner;
     const uint32_t vec = inner % 2 == 0 && channels % 2 == 0 && m.ld % 2 == 0;
     if (m.taps <= 4)
-        launch_kernel(conv_silu_kernel<T, 4>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b, (const T*)m.ring,
+        launch_kernel(conv_silu_kernel<T, 4>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b, (T*)m.ring,
                       (T*)m.xbc, place, run, vec);
     else
         launch_kernel(conv_silu_kernel<T, kMaxConvTaps>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b,
-                      (const T*)m.ring, (T*)m.xbc, place, run, vec);
+                      (T*)m.ring, (T*)m.xbc, place, run, vec);
 }
 
 // ---- token by token ----------------------------------------------------------------------------
-// Block = (slice of at most 64 columns of the state, head, session).  Thread (p, k) holds S[k + NG i, p] of its slice for
-// i < ROWS.  FUSED (single-token steps): x, B and C are convolved here from the projected row and the ring; the ring rows
-// are written by the block that is first to own the channel (x: the head's own slice, B and C: the group's first head).
+// Block = (slice of at most 64 columns of the state, head, session).  A thread owns VEC neighbouring columns of every
+// (256 / (width / VEC))-th row of its slice; everything a token needs besides the state (x, B, C, step, gate input) is
+// asked for together with the state, one memory round trip per step.
 constexpr uint32_t SSD_THREADS = 256, SSD_SLICE = 64, SSD_MAX_STATE = 256;
 
-template <typename T, int ROWS, bool FUSED>
+template <typename T, int ROWS, int VEC>
 __global__ void __launch_bounds__(SSD_THREADS)
 ssd_token_kernel(Mamba2 m, StepPlace place) {
-    __shared__ float sb[SSD_MAX_STATE], sc[SSD_MAX_STATE], sx[SSD_SLICE], red[SSD_THREADS];
+    __shared__ float sb[SSD_MAX_STATE], sc[SSD_MAX_STATE], sx[SSD_SLICE], red[SSD_THREADS * VEC];
     pdl_wait();
     pdl_trigger();
     const uint32_t tid = threadIdx.x;
     const uint32_t p_first = blockIdx.x * SSD_SLICE, h = blockIdx.y, s = blockIdx.z;
     const uint32_t width = min(SSD_SLICE, m.vdim - p_first);
-    const uint32_t ng = SSD_THREADS / width;                 // row groups
-    const uint32_t p = tid % width, k = tid / width;
+    const uint32_t across = width / VEC, ng = SSD_THREADS / across;     // threads along a row, row groups
+    const uint32_t p = (tid % across) * VEC, k = tid / across;
     const bool live = k < ng;
     const uint32_t inner = m.heads * m.vdim, gn = m.groups * m.state, channels = inner + 2 * gn;
     const uint32_t group = h / (m.heads / m.groups);
     const uint32_t p0 = place.pos(s);
     float* state = m.ssm + (((size_t)s * m.heads + h) * m.state) * m.vdim + p_first + p;
-    float S[ROWS];
+    float S[ROWS][VEC];
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
         const uint32_t n = k + ng * i;
-        S[i] = live && n < m.state && p0 > 0 ? state[(size_t)n * m.vdim] : 0.0f;
+        const bool have = live && n < m.state && p0 > 0;
+        if (VEC == 4) {
+            const float4 v = have ? *reinterpret_cast<const float4*>(state + (size_t)n * m.vdim) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            S[i][0] = v.x; S[i][VEC > 1 ? 1 : 0] = v.y; S[i][VEC > 2 ? 2 : 0] = v.z; S[i][VEC > 3 ? 3 : 0] = v.w;
+        } else {
+            S[i][0] = have ? state[(size_t)n * m.vdim] : 0.0f;
+        }
     }
-    const float a = -expf(m.a_log[h]), dt_bias = m.dt_bias[h], skip = m.d_skip[h];
+    const T* xbc = reinterpret_cast<const T*>(m.xbc) + (size_t)s * place.chunk * channels;
+    const T* zrow = reinterpret_cast<const T*>(m.proj) + (size_t)s * place.chunk * m.ld + h * m.vdim + p_first;
+    const float a_log = m.a_log[h], dt_bias = m.dt_bias[h], skip = m.d_skip[h];
     for (uint32_t t = 0; t < place.chunk; ++t) {
         const size_t row = (size_t)s * place.chunk + t;
-        const float dt = softplus(m.dt[row * m.dt_ld + h] + dt_bias);
-        // this token's x slice, B and C
-        const uint32_t count = width + 2 * m.state;
-        for (uint32_t i = tid; i < count; i += SSD_THREADS) {
-            const uint32_t ch = i < width ? h * m.vdim + p_first + i
-                              : i < width + m.state ? inner + group * m.state + (i - width)
-                                                    : inner + gn + group * m.state + (i - width - m.state);
-            float v;
-            if (FUSED) {
-                const T* in = reinterpret_cast<const T*>(m.proj) + row * m.ld + inner + ch;
-                T* ring = reinterpret_cast<T*>(m.ring) + (size_t)s * m.taps * channels + ch;
-                const float* w = m.conv_w + (size_t)ch * m.taps;
-                const T now = *in;
-                v = fmaf(w[m.taps - 1], to_f32(now), m.conv_b[ch]);
-                for (uint32_t lag = 1; lag < m.taps && lag <= p0; ++lag)
-                    v = fmaf(w[m.taps - 1 - lag], to_f32(ring[(size_t)((p0 - lag) % m.taps) * channels]), v);
-                v = act_silu<T>(v);
-                v = to_f32(from_f32<T>(v));     // the value a longer chunk would have stored
-                if (i < width || (h % (m.heads / m.groups) == 0 && p_first == 0)) ring[(size_t)(p0 % m.taps) * channels] = now;
-            } else {
-                v = to_f32(reinterpret_cast<const T*>(m.xbc)[row * channels + ch]);
-            }
-            if (i < width) sx[i] = v;
-            else if (i < width + m.state) sb[i - width] = v;
-            else sc[i - width - m.state] = v;
+        const float dt_raw = m.dt[row * m.dt_ld + h];
+        const float z = tid < width ? to_f32(zrow[(size_t)t * m.ld + tid]) : 0.0f;
+        if (tid < m.state) {
+            sb[tid] = to_f32(xbc[(size_t)t * channels + inner + group * m.state + tid]);
+            sc[tid] = to_f32(xbc[(size_t)t * channels + inner + gn + group * m.state + tid]);
         }
+        if (tid < width) sx[tid] = to_f32(xbc[(size_t)t * channels + h * m.vdim + p_first + tid]);
+        const float dt = softplus(dt_raw + dt_bias);
+        const float decay = expf(-expf(a_log) * dt);
         __syncthreads();
-        const float decay = expf(a * dt);
-        float acc = 0.0f;
+        float acc[VEC], xdt[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { acc[e] = 0.0f; xdt[e] = live ? dt * sx[p + e] : 0.0f; }
         if (live) {
-            const float xdt = dt * sx[p];
 #pragma unroll
             for (int i = 0; i < ROWS; ++i) {
                 const uint32_t n = k + ng * i;
                 if (n < m.state) {
-                    S[i] = fmaf(S[i], decay, sb[n] * xdt);
-                    acc = fmaf(S[i], sc[n], acc);
+                    const float b = sb[n], c = sc[n];
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        S[i][e] = fmaf(S[i][e], decay, b * xdt[e]);
+                        acc[e] = fmaf(S[i][e], c, acc[e]);
+                    }
                 }
             }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) red[k * width + p + e] = acc[e];
         }
-        red[tid] = acc;
         __syncthreads();
         if (tid < width) {
             float y = skip * sx[tid];
             for (uint32_t j = 0; j < ng; ++j) y += red[j * width + tid];
-            const uint32_t col = h * m.vdim + p_first + tid;
-            const float z = to_f32(reinterpret_cast<const T*>(m.proj)[row * m.ld + col]);
-            reinterpret_cast<T*>(m.gated)[row * inner + col] = from_f32<T>(y * act_silu<T>(z));
+            reinterpret_cast<T*>(m.gated)[row * inner + h * m.vdim + p_first + tid] = from_f32<T>(y * act_silu<T>(z));
         }
-        __syncthreads();
+        if (t + 1 < place.chunk) __syncthreads();
     }
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
         const uint32_t n = k + ng * i;
-        if (live && n < m.state) state[(size_t)n * m.vdim] = S[i];
+        if (!(live && n < m.state)) continue;
+        if (VEC == 4)
+            *reinterpret_cast<float4*>(state + (size_t)n * m.vdim) = make_float4(S[i][0], S[i][VEC > 1 ? 1 : 0], S[i][VEC > 2 ? 2 : 0], S[i][VEC > 3 ? 3 : 0]);
+        else
+            state[(size_t)n * m.vdim] = S[i][0];
     }
 }
 
-template <typename T, bool FUSED>
-static void ssd_token_rows(const Mamba2& m, const StepPlace& place, cudaStream_t stream) {
-    const uint32_t width = std::min(m.vdim, SSD_SLICE), rows = ceil_div(m.state, SSD_THREADS / width);
+template <typename T>
+static void ssd_token(const Mamba2& m, const StepPlace& place, cudaStream_t stream) {
     const dim3 grid(ceil_div(m.vdim, SSD_SLICE), m.heads, place.sessions), block(SSD_THREADS);
-    if (rows <= 8) launch_kernel(ssd_token_kernel<T, 8, FUSED>, grid, block, 0, stream, m, place);
-    else if (rows <= 32) launch_kernel(ssd_token_kernel<T, 32, FUSED>, grid, block, 0, stream, m, place);
-    else launch_kernel(ssd_token_kernel<T, 64, FUSED>, grid, block, 0, stream, m, place);
+    const uint32_t width = std::min(m.vdim, SSD_SLICE);
+    if (m.vdim % 4 == 0 && reinterpret_cast<uintptr_t>(m.ssm) % 16 == 0) {
+        const uint32_t rows = ceil_div(m.state, SSD_THREADS / (width / 4));
+        if (rows <= 2) launch_kernel(ssd_token_kernel<T, 2, 4>, grid, block, 0, stream, m, place);
+        else if (rows <= 4) launch_kernel(ssd_token_kernel<T, 4, 4>, grid, block, 0, stream, m, place);
+        else if (rows <= 8) launch_kernel(ssd_token_kernel<T, 8, 4>, grid, block, 0, stream, m, place);
+        else launch_kernel(ssd_token_kernel<T, 16, 4>, grid, block, 0, stream, m, place);
+        return;
+    }
+    const uint32_t rows = ceil_div(m.state, SSD_THREADS / width);
+    if (rows <= 8) launch_kernel(ssd_token_kernel<T, 8, 1>, grid, block, 0, stream, m, place);
+    else if (rows <= 32) launch_kernel(ssd_token_kernel<T, 32, 1>, grid, block, 0, stream, m, place);
+    else launch_kernel(ssd_token_kernel<T, 64, 1>, grid, block, 0, stream, m, place);
 }
 
 bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state) {
@@ -195,7 +216,7 @@ bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state) {
 }
 
 // ---- grouped RMS norm ------------------------------------------------------------------------------
-// One block per (row, norm group): any width.  Parts of whole 16-byte chunks up to 1024 values take a warp each and stay in
+// One block per (row, norm group): any width.  Parts of whole 16-byte chunks up to 2048 values take a warp each and stay in
 // registers between the sum and the scaling (gated_norm_warp_kernel).
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -222,7 +243,7 @@ gated_norm_kernel(const T* __restrict__ gated, const float* __restrict__ w, T* _
         for (uint32_t c = inner + threadIdx.x; c < out_cols; c += blockDim.x) out[row * out_ld + c] = from_f32<T>(0.0f);
 }
 
-constexpr uint32_t GN_VEC = 4;   // 16-byte chunks per lane: parts of up to 1024 values, one warp each
+constexpr uint32_t GN_VEC = 8;   // 16-byte chunks per lane: parts of up to 2048 values, one warp each
 __global__ void __launch_bounds__(128)
 gated_norm_warp_kernel(const bf16* __restrict__ gated, const float* __restrict__ w, bf16* __restrict__ out, uint32_t rows, uint32_t inner,
                        uint32_t groups, uint32_t out_ld, uint32_t out_cols, float eps) {
@@ -272,23 +293,19 @@ int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream
     }
     const bool bf = dtype == TNSR_B200_BF16;
     int rc;
-    if (place.chunk == 1) {
-        if (bf) ssd_token_rows<bf16, true>(m, place, stream); else ssd_token_rows<float, true>(m, place, stream);
-        count_launch();
-        if ((rc = check_launch("ssd_token"))) return rc;
-    } else {
-        if (bf) conv_silu_typed<bf16>(m, inner, channels, place, stream); else conv_silu_typed<float>(m, inner, channels, place, stream);
-        count_launch();
-        if ((rc = check_launch("conv_silu"))) return rc;
+    if (bf) conv_silu_typed<bf16>(m, inner, channels, place, stream); else conv_silu_typed<float>(m, inner, channels, place, stream);
+    count_launch();
+    if ((rc = check_launch("conv_silu"))) return rc;
+    if (place.chunk > 1) {
         const uint8_t* raw = (const uint8_t*)m.proj + (size_t)inner * (bf ? 2 : 4);
         if ((rc = launch_conv_ring(raw, m.ld, channels, m.taps, m.ring, place, dtype, stream))) return rc;
-        if (bf && m.engine == 0 && place.chunk >= SSD_SCAN_MIN_TOKENS) {
-            if ((rc = launch_ssd_scan(m, place, stream))) return rc;
-        } else {
-            if (bf) ssd_token_rows<bf16, false>(m, place, stream); else ssd_token_rows<float, false>(m, place, stream);
-            count_launch();
-            if ((rc = check_launch("ssd_token"))) return rc;
-        }
+    }
+    if (bf && m.engine == 0 && place.chunk >= SSD_SCAN_MIN_TOKENS) {
+        if ((rc = launch_ssd_scan(m, place, stream))) return rc;
+    } else {
+        if (bf) ssd_token<bf16>(m, place, stream); else ssd_token<float>(m, place, stream);
+        count_launch();
+        if ((rc = check_launch("ssd_token"))) return rc;
     }
     const dim3 grid(rows, m.norm_groups);
     const uint32_t part = inner / m.norm_groups;

@@ -65,10 +65,15 @@ struct GroupedAttention {
     KvPaging paging;
     void* workspace = nullptr;            // grouped_attention_workspace_bytes(), zeroed once
     uint64_t workspace_bytes = 0;
-    int engine = 0;                       // 0: best kernel for the shape, 1: one warp per (row, head)
+    int* d_status = nullptr;              // device status word (a bounded wait of the tcgen05 kernel gave up), may be null
+    int engine = 0;                       // 0: best kernel for the shape, 1: one warp per (row, head), 2: not the tcgen05 kernel
 };
 uint64_t grouped_attention_workspace_bytes(uint32_t dim, uint32_t vdim);
 int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, int dtype, cudaStream_t stream);
+
+// Many rows, heads of 64, position on the host: the tcgen05 kernel of prefill_tc.cu.
+bool grouped_attention_tc_eligible(const GroupedAttention& a, const StepPlace& place);
+int launch_grouped_attention_tc(const GroupedAttention& a, const StepPlace& place, cudaStream_t stream);
 
 // ---- mamba2 ---------------------------------------------------------------------
 struct Mamba2 {
@@ -86,7 +91,7 @@ struct Mamba2 {
     float eps = 0.0f;
     void* ring = nullptr;              // [sessions, taps, inner + 2 groups * state]
     float* ssm = nullptr;              // [sessions, heads, state, vdim]
-    void* xbc = nullptr;               // [rows, inner + 2 groups * state] scratch (chunks of two tokens and more)
+    void* xbc = nullptr;               // [rows, inner + 2 groups * state] scratch: convolved x | B | C
     void* gated = nullptr;             // [rows, inner] scratch: y * silu(z)
     void* out = nullptr;               // [rows, out_ld]; columns [inner, out_cols) are zeroed
     uint32_t out_ld = 0, out_cols = 0;

@@ -188,13 +188,13 @@ int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args, co
     a.heads = args->heads; a.kv_heads = args->kv_heads; a.dim = args->dim; a.vdim = args->vdim; a.capacity = args->capacity;
     a.scale = args->scale; a.softcap = args->softcap; a.gate = args->gate; a.gate_ld = args->gate_ld;
     a.out = args->out; a.out_ld = args->out_ld; a.out_cols = args->out_cols;
-    a.workspace = args->workspace; a.workspace_bytes = args->workspace_bytes; a.engine = args->engine;
+    a.d_status = args->d_status; a.workspace = args->workspace; a.workspace_bytes = args->workspace_bytes; a.engine = args->engine;
     return launch_grouped_attention(a, step_place(place), args->dtype, as_stream(stream));
 }
 
 int tnsr_b200_mamba2(const tnsr_b200_mamba2_args* args, const tnsr_b200_place* place, void* stream) {
     if (!args || !place || !args->proj || !args->dt || !args->conv_w || !args->conv_b || !args->dt_bias || !args->a_log || !args->d_skip ||
-        !args->norm_w || !args->ring || !args->ssm || !args->gated || !args->out || (place->chunk > 1 && !args->xbc))
+        !args->norm_w || !args->ring || !args->ssm || !args->xbc || !args->gated || !args->out)
         return bad("mamba2: null pointer");
     if (args->dtype != TNSR_B200_F32 && args->dtype != TNSR_B200_BF16) return bad("mamba2: dtype must be f32 or bf16");
     if (args->groups == 0 || args->heads == 0 || args->heads % args->groups || args->norm_groups == 0 ||

@@ -36,10 +36,14 @@
 //                                                             upper P tile; the next P V overwrites O only after
 //                                                             the following p_full, i.e. after the fold)
 //
+// Grouped-query form (described models): query head h reads key/value head h / per, scores may be capped (cap tanh(s / cap),
+// monotonic, so the row maximum is still taken over raw scores), and a sigmoid gate per (row, head) scales the output.
+//
 // Every wait is bounded; a wait that gives up raises the CTA's abort flag, the
 // roles fall through to the common teardown and the status word is set.
 #include <algorithm>
 
+#include "mixers.cuh"
 #include "tc_common.cuh"
 
 namespace tb {
@@ -70,10 +74,16 @@ struct PtParams {
     bf16* out;
     uint32_t chunk, position, heads, q_tiles, sessions;
     float scale_log2;
+    uint32_t per;              // query heads per key/value head
+    uint32_t out_ld, out_cols; // output rows: pitch, columns (those past the heads are zeroed)
+    const float* gate;         // [rows, gate_ld] or nullptr
+    uint32_t gate_ld;
+    float cap_pre, cap_post;   // capped scores in log2 units: cap_post - 2 cap_post / (1 + exp2(s cap_pre))
     int* d_status;
     uint64_t wait_limit_ns;
 };
 
+template <bool CAPPED>
 __global__ void __launch_bounds__(PT_THREADS, 2)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PtParams prm) {
@@ -152,8 +162,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     if (!mbar_wait(kv_empty + stage, ((g / PT_KV_STAGES) & 1) ^ 1, abort_flag, prm.wait_limit_ns)) { ok = false; break; }
                     uint8_t* dst = kv_ring + stage * PT_KV_BYTES;
                     mbar_expect_tx(kv_full + stage, PT_KV_BYTES);
-                    tma_load_3d(dst, &map_k, (int32_t)(h * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
-                    tma_load_3d(dst + PT_TILE_BYTES, &map_v, (int32_t)(h * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
+                    tma_load_3d(dst, &map_k, (int32_t)(h / prm.per * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
+                    tma_load_3d(dst + PT_TILE_BYTES, &map_v, (int32_t)(h / prm.per * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
                 }
             }
         }
@@ -214,6 +224,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t row = quarter * 32 + lane;
         const uint32_t lane_taddr = tmem_base + ((quarter * 32u) << 16);
         const float sl2 = prm.scale_log2;
+        auto capped = [&](float v) { return fmaf(-2.0f * prm.cap_post, mx_rcp(pt_ex2(v * prm.cap_pre) + 1.0f), prm.cap_post); };
         uint32_t pair_uses = 0, g = 0;
         bool ok = true;
         // Both threads of a row publish a value and read the partner's.
@@ -273,9 +284,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (!exchange(mx, other)) { ok = false; break; }
                 mx = fmaxf(m, fmaxf(mx, other));
                 const float ms = (mx == -INFINITY) ? 0.0f : mx;
-                const float corr = pt_ex2((m - ms) * sl2);      // 0 for the first block
+                // the first block has nothing to rescale (its corr is 0, or finite when capped)
+                const float top = CAPPED ? capped(ms) : ms * sl2;
+                const float corr = CAPPED ? pt_ex2(capped(m) - top) : pt_ex2((m - ms) * sl2);
                 m = mx;
-                const float neg = -ms * sl2;
+                const float neg = -top;
                 // the previous block's output; once it is complete the upper P tile may be overwritten
                 if (j > 0 && !fold(b - 1, corr_pending)) { ok = false; break; }
                 corr_pending = corr;
@@ -295,7 +308,18 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     uint32_t packed[16];
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
-                        const float p0 = pt_ex2(fmaf(v[2 * i], sl2, neg)), p1 = pt_ex2(fmaf(v[2 * i + 1], sl2, neg));
+                        float p0, p1;
+                        if (CAPPED) {
+                            p0 = pt_ex2(capped(v[2 * i]) + neg);
+                            p1 = pt_ex2(capped(v[2 * i + 1]) + neg);
+                            if (need_mask) {      // a capped score is finite also for a hidden key
+                                if (kbase + c * 32 + 2 * i > limit) p0 = 0.0f;
+                                if (kbase + c * 32 + 2 * i + 1 > limit) p1 = 0.0f;
+                            }
+                        } else {
+                            p0 = pt_ex2(fmaf(v[2 * i], sl2, neg));
+                            p1 = pt_ex2(fmaf(v[2 * i + 1], sl2, neg));
+                        }
                         rs4[i & 3] += p0 + p1;
                         packed[i] = pack_bf16x2(p0, p1);
                     }
@@ -318,8 +342,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             float l_other = 0.0f;
             if (ok) ok = exchange(l, l_other);
             if (ok && q0 + row < prm.chunk) {
-                const float inv = 1.0f / (l + l_other);
-                bf16* og = prm.out + ((size_t)s * prm.chunk + q0 + row) * ((size_t)prm.heads * PT_HD) + (size_t)h * PT_HD + half * 32;
+                const size_t out_row = (size_t)s * prm.chunk + q0 + row;
+                float inv = 1.0f / (l + l_other);
+                if (prm.gate) inv *= 1.0f / (1.0f + __expf(-prm.gate[out_row * prm.gate_ld + h]));
+                bf16* og = prm.out + out_row * prm.out_ld + (size_t)h * PT_HD + half * 32;
+                if (h + 1 == prm.heads && half == 1)
+                    for (uint32_t c = prm.heads * PT_HD; c < prm.out_cols; ++c) prm.out[out_row * prm.out_ld + c] = __float2bfloat16_rn(0.0f);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     uint4 w;
@@ -376,14 +404,13 @@ bool prefill_attention_tc_eligible(uint32_t sessions, uint32_t chunk, uint32_t p
     return encode_fn() != nullptr;
 }
 
-int launch_prefill_attention_tc(const bf16* q, const bf16* k_cache, const bf16* v_cache, bf16* out, uint32_t sessions,
-                                uint32_t chunk, uint32_t position, uint32_t capacity, uint32_t heads, int* d_status,
-                                cudaStream_t stream) {
-    const uint64_t width = (uint64_t)heads * PT_HD;
+template <bool CAPPED>
+static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, uint32_t kv_heads, uint32_t capacity, PtParams& prm, cudaStream_t stream) {
+    const uint64_t width = (uint64_t)prm.heads * PT_HD, kv_width = (uint64_t)kv_heads * PT_HD;
     CUtensorMap mq, mk, mv;
-    if (!make_map3(&mq, q, width, chunk, sessions, chunk) ||
-        !make_map3(&mk, k_cache, width, (uint64_t)position + chunk, sessions, capacity) ||
-        !make_map3(&mv, v_cache, width, (uint64_t)position + chunk, sessions, capacity)) {
+    if (!make_map3(&mq, q, width, prm.chunk, prm.sessions, prm.chunk) ||
+        !make_map3(&mk, k_cache, kv_width, (uint64_t)prm.position + prm.chunk, prm.sessions, capacity) ||
+        !make_map3(&mv, v_cache, kv_width, (uint64_t)prm.position + prm.chunk, prm.sessions, capacity)) {
         set_thread_error("prefill attention: tensor map encoding failed");
         return TNSR_B200_ERR_CUDA;
     }
@@ -391,31 +418,68 @@ int launch_prefill_attention_tc(const bf16* q, const bf16* k_cache, const bf16* 
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-        if (cudaFuncSetAttribute(prefill_attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(prefill_attention_tc_kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
+        if (cudaFuncSetAttribute(prefill_attention_tc_kernel<CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(prefill_attention_tc_kernel<CAPPED>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  (int)cudaSharedmemCarveoutMaxShared) != cudaSuccess)
             return check_launch("prefill_attention_tc attribute");
         if (dev >= 0 && dev < 64) configured[dev] = true;
     }
-    PtParams prm;
-    prm.out = out;
-    prm.chunk = chunk;
-    prm.position = position;
-    prm.heads = heads;
-    prm.q_tiles = ceil_div(chunk, (uint32_t)PT_BQ);
-    prm.scale_log2 = (1.0f / sqrtf((float)PT_HD)) * 1.4426950408889634f;
-    prm.d_status = d_status;
+    prm.q_tiles = ceil_div(prm.chunk, (uint32_t)PT_BQ);
+    prm.per = prm.heads / kv_heads;
     prm.wait_limit_ns = g_wait_limit_ns.load(std::memory_order_relaxed);
-    prm.sessions = sessions;
     // persistent: two CTAs per SM walk the list of (query tile, head, session) items
     int dev_sms = 0;
     cudaDeviceGetAttribute(&dev_sms, cudaDevAttrMultiProcessorCount, dev);
     if (dev_sms <= 0) dev_sms = 148;
-    const uint64_t items = (uint64_t)prm.q_tiles * heads * sessions;
+    const uint64_t items = (uint64_t)prm.q_tiles * prm.heads * prm.sessions;
     dim3 grid((unsigned)std::min<uint64_t>(items, 2ull * dev_sms));
-    launch_kernel(prefill_attention_tc_kernel, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
+    launch_kernel(prefill_attention_tc_kernel<CAPPED>, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
     count_launch();
     return check_launch("prefill_attention_tc");
+}
+
+int launch_prefill_attention_tc(const bf16* q, const bf16* k_cache, const bf16* v_cache, bf16* out, uint32_t sessions,
+                                uint32_t chunk, uint32_t position, uint32_t capacity, uint32_t heads, int* d_status,
+                                cudaStream_t stream) {
+    PtParams prm = {};
+    prm.out = out;
+    prm.chunk = chunk;
+    prm.position = position;
+    prm.heads = heads;
+    prm.sessions = sessions;
+    prm.scale_log2 = (1.0f / sqrtf((float)PT_HD)) * 1.4426950408889634f;
+    prm.out_ld = prm.out_cols = heads * PT_HD;
+    prm.d_status = d_status;
+    return launch_pt<false>(q, k_cache, v_cache, heads, capacity, prm, stream);
+}
+
+bool grouped_attention_tc_eligible(const GroupedAttention& a, const StepPlace& place) {
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    return a.dim == (uint32_t)PT_HD && a.vdim == (uint32_t)PT_HD && !a.paging.table && a.scale > 0.0f && a.out_ld % 8 == 0 && aligned(a.q) &&
+           aligned(a.k_cache) && aligned(a.v_cache) && aligned(a.out) && (uint64_t)place.sessions * a.heads * ceil_div(place.chunk, (uint32_t)PT_BQ) < 0x7fffffffull &&
+           prefill_attention_tc_eligible(place.sessions, place.chunk, place.position, place.d_position, a.capacity, a.heads, a.dim);
+}
+
+int launch_grouped_attention_tc(const GroupedAttention& a, const StepPlace& place, cudaStream_t stream) {
+    PtParams prm = {};
+    prm.out = (bf16*)a.out;
+    prm.chunk = place.chunk;
+    prm.position = place.position;
+    prm.heads = a.heads;
+    prm.sessions = place.sessions;
+    prm.scale_log2 = a.scale * 1.4426950408889634f;
+    prm.out_ld = a.out_ld;
+    prm.out_cols = a.out_cols;
+    prm.gate = a.gate;
+    prm.gate_ld = a.gate_ld;
+    prm.d_status = a.d_status;
+    const bf16 *q = (const bf16*)a.q, *k = (const bf16*)a.k_cache, *v = (const bf16*)a.v_cache;
+    if (a.softcap > 0.0f) {
+        prm.cap_pre = 2.0f * 1.4426950408889634f * a.scale / a.softcap;
+        prm.cap_post = a.softcap * 1.4426950408889634f;
+        return launch_pt<true>(q, k, v, a.kv_heads, a.capacity, prm, stream);
+    }
+    return launch_pt<false>(q, k, v, a.kv_heads, a.capacity, prm, stream);
 }
 
 }  // namespace tb

@@ -3,10 +3,14 @@
 // Within a chunk of 64 tokens, with c_i the running sum of the log decays:
 //     y_i = exp(c_i) C_i S_in + sum_{j <= i} (C_i . B_j) exp(c_i - c_j) dt_j x_j + D x_i
 //     S_out = exp(c_63) S_in + sum_j B_j (exp(c_63 - c_j) dt_j x_j)^T
-// A CTA owns the whole sequence of one (session, head, slice of the state's columns) and carries S in accumulator
-// registers from chunk to chunk; columns of S do not couple, so slices are independent.  Four warps: 16 token rows each
-// for y, a quarter of the state's rows each for S.  Factors that are f32 -- the decayed weights, the state, the weighted
-// inputs -- enter the products as two bf16 halves (split_bf16x2), so that they keep 16 bits.
+// A CTA owns the whole sequence of one (session, head, 64 columns of the state) and carries S from chunk to chunk; columns
+// of S do not couple, so each of its four warps owns 16 of them.  A warp keeps S transposed in accumulator registers
+// (rows = its columns, from x^T . B): in that layout the accumulators of S^T are, register by register, the B operand of
+// C . S, so the state never passes through shared memory.  The decayed weights (C B^T with the decays applied) are made
+// once per CTA, 16 token rows per warp, and shared.  The next chunk's B, C and x arrive while this one is computed.
+//
+// Factors that are f32 -- the decayed weights, the state, the weighted inputs -- enter the products as two bf16 halves
+// (split_bf16x2), so that they keep 16 bits.
 #include <algorithm>
 
 #include "mixers.cuh"
@@ -14,72 +18,45 @@
 namespace tb {
 
 constexpr int SC_Q = 64;          // tokens per chunk
+constexpr uint32_t SC_P = 64;     // columns of the state per CTA, 16 per warp
 constexpr float SC_LOG2E = 1.4426950408889634f;
 
-template <int NP, int PT>
+template <int NP>
 struct ScanShape {
-    static constexpr uint32_t BP = NP * 2 + 16, XP = PT * 2 + 16;     // row pitches: conflict-free ldmatrix
-    static constexpr uint32_t B_BYTES = SC_Q * BP, X_BYTES = SC_Q * XP, S_BYTES = NP * XP;
-    static constexpr uint32_t BYTES = 2 * B_BYTES + 3 * X_BYTES + 2 * S_BYTES;
+    static constexpr uint32_t BP = NP * 2 + 16, XP = SC_P * 2 + 16, WP = SC_Q * 2 + 16;   // row pitches: conflict-free ldmatrix
+    static constexpr uint32_t B_BYTES = SC_Q * BP, X_BYTES = SC_Q * XP, W_BYTES = SC_Q * WP;
+    static constexpr uint32_t STAGE = 2 * B_BYTES + X_BYTES;          // B, C, x of one chunk
+    static constexpr uint32_t BYTES = 2 * STAGE + 2 * W_BYTES;
 };
 
-// NP: state rows padded to a multiple of 64, PT: columns of the slice (padded).
-template <int NP, int PT>
+// NP: state rows padded to a multiple of 64.
+template <int NP>
 __global__ void __launch_bounds__(128, NP <= 128 ? 2 : 1)
 ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
-    using S = ScanShape<NP, PT>;
-    constexpr int MT = NP / 64;                 // 16-row tiles of the state per warp
+    using S = ScanShape<NP>;
+    constexpr int NT = NP / 8;                  // 8-row tiles of the state
     extern __shared__ __align__(16) uint8_t smem[];
-    uint8_t* sb = smem;
-    uint8_t* sc = sb + S::B_BYTES;
-    uint8_t* sx = sc + S::B_BYTES;
-    uint8_t* sxh = sx + S::X_BYTES;
-    uint8_t* sxl = sxh + S::X_BYTES;
-    uint8_t* ssh = sxl + S::X_BYTES;
-    uint8_t* ssl = ssh + S::S_BYTES;
-    __shared__ float s_cum[SC_Q], s_dt[SC_Q];   // running log2 decay, step size
+    uint8_t* swh = smem + 2 * S::STAGE;
+    uint8_t* swl = swh + S::W_BYTES;
+    __shared__ float s_cum[2][SC_Q], s_dt[2][SC_Q];   // running log2 decay, step size
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
-    const uint32_t p_first = blockIdx.x * PT, h = blockIdx.y, s = blockIdx.z;
-    const uint32_t width = min((uint32_t)PT, m.vdim - p_first);
+    const uint32_t p_first = blockIdx.x * SC_P, h = blockIdx.y, s = blockIdx.z;
+    const uint32_t width = min(SC_P, m.vdim - p_first);
     const uint32_t inner = m.heads * m.vdim, gn = m.groups * m.state, channels = inner + 2 * gn;
     const uint32_t group = h / (m.heads / m.groups);
+    const uint32_t pw = warp * 16;              // the warp's columns
+    const bool owner = pw < width;
     pdl_wait();
     pdl_trigger();
     const uint32_t p0 = place.pos(s);
     const float a2 = -expf(m.a_log[h]) * SC_LOG2E, dt_bias = m.dt_bias[h], skip = m.d_skip[h];
     const size_t row_base = (size_t)s * place.chunk;
     const bf16* xbc = reinterpret_cast<const bf16*>(m.xbc) + row_base * channels;
+    const bf16* zb = reinterpret_cast<const bf16*>(m.proj) + row_base * m.ld + h * m.vdim + p_first;
+    bf16* gb = reinterpret_cast<bf16*>(m.gated) + row_base * inner + h * m.vdim + p_first;
     float* state = m.ssm + (((size_t)s * m.heads + h) * m.state) * m.vdim + p_first;
 
-    // S: rows n = (warp * MT + mt) * 16 + g8 (+ 8), columns nt * 8 + t4 * 2 (+ 1)
-    float acc[MT][PT / 8][4];
-    auto state_rows = [&](int mt, int half) { return (uint32_t)((warp * MT + mt) * 16) + g8 + half * 8; };
-    auto store_state_tiles = [&]() {
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-            for (int nt = 0; nt < PT / 8; ++nt)
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    uint32_t hi, lo;
-                    split_bf16x2(acc[mt][nt][2 * half], acc[mt][nt][2 * half + 1], hi, lo);
-                    const uint32_t off = state_rows(mt, half) * S::XP + (nt * 8 + t4 * 2) * 2;
-                    *reinterpret_cast<uint32_t*>(ssh + off) = hi;
-                    *reinterpret_cast<uint32_t*>(ssl + off) = lo;
-                }
-    };
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int nt = 0; nt < PT / 8; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const uint32_t n = state_rows(mt, e >> 1), p = nt * 8 + t4 * 2 + (e & 1);
-                acc[mt][nt][e] = p0 > 0 && n < m.state && p < width ? state[(size_t)n * m.vdim + p] : 0.0f;
-            }
-    store_state_tiles();
-
-    // one operand tile: 64 rows of `w` channels from channel c0 on, rows past the chunk's end and channels past w are zero
+    // one operand tile: 64 rows of `w` channels from channel c0 on; rows past the chunk's end and channels past w are zero
     auto load_tile = [&](uint8_t* dst, uint32_t pitch, uint32_t padded, uint32_t c0, uint32_t w, uint32_t t0) {
         const uint32_t live = min((uint32_t)SC_Q, place.chunk - t0);
         if (vec) {
@@ -97,183 +74,253 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
             }
         }
     };
-
-    for (uint32_t t0 = 0; t0 < place.chunk; t0 += SC_Q) {
-        load_tile(sb, S::BP, NP, inner + group * m.state, m.state, t0);
-        load_tile(sc, S::BP, NP, inner + gn + group * m.state, m.state, t0);
-        load_tile(sx, S::XP, PT, h * m.vdim + p_first, width, t0);
+    auto load_chunk = [&](uint32_t t0, uint32_t buf) {
+        if (t0 < place.chunk) {
+            uint8_t* dst = smem + buf * S::STAGE;
+            load_tile(dst, S::BP, NP, inner + group * m.state, m.state, t0);
+            load_tile(dst + S::B_BYTES, S::BP, NP, inner + gn + group * m.state, m.state, t0);
+            load_tile(dst + 2 * S::B_BYTES, S::XP, SC_P, h * m.vdim + p_first, width, t0);
+        }
         mx_commit();
-        if (warp == 0) {
-            // steps and running log decays of tokens 2 lane, 2 lane + 1; tokens past the end have step 0
-            float dt[2], d2[2];
+    };
+    // warp 0: raw steps of tokens 2 lane, 2 lane + 1 of the chunk at t0; -inf (step 0) past the end
+    float raw[2];
+    auto fetch_steps = [&](uint32_t t0) {
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const uint32_t t = t0 + 2 * lane + i;
-                dt[i] = 0.0f;
-                if (t < place.chunk) {
-                    const float u = m.dt[(row_base + t) * m.dt_ld + h] + dt_bias;
-                    dt[i] = u > 20.0f ? u : log1pf(expf(u));
-                }
-                d2[i] = a2 * dt[i];
-            }
-            float sum = d2[0] + d2[1];
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float up = __shfl_up_sync(0xffffffffu, sum, o);
-                if (lane >= (uint32_t)o) sum += up;
-            }
-            s_cum[2 * lane + 1] = sum;
-            s_cum[2 * lane] = sum - d2[1];
-            s_dt[2 * lane] = dt[0];
-            s_dt[2 * lane + 1] = dt[1];
+        for (int i = 0; i < 2; ++i) {
+            const uint32_t t = t0 + 2 * lane + i;
+            raw[i] = t < place.chunk ? m.dt[(row_base + t) * m.dt_ld + h] + dt_bias : -INFINITY;
         }
-        mx_wait<0>();
-        __syncthreads();
-        const float last = s_cum[SC_Q - 1];
-        // inputs weighted for the state at the end of the chunk
-        for (uint32_t i = tid; i < SC_Q * (PT / 2); i += 128) {
-            const uint32_t r = i / (PT / 2), c = (i % (PT / 2)) * 2;
-            const float w = mx_ex2(last - s_cum[r]) * s_dt[r];
-            const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(sx + r * S::XP + c * 2));
-            uint32_t hi, lo;
-            split_bf16x2(x.x * w, x.y * w, hi, lo);
-            *reinterpret_cast<uint32_t*>(sxh + r * S::XP + c * 2) = hi;
-            *reinterpret_cast<uint32_t*>(sxl + r * S::XP + c * 2) = lo;
+    };
+    auto make_decays = [&](uint32_t buf) {
+        float dt[2], d2[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            dt[i] = raw[i] > 20.0f ? raw[i] : log1pf(expf(raw[i]));
+            d2[i] = a2 * dt[i];
         }
-        // ---- C . B^T (columns up to the warp's own rows) and C . S_in ----
-        const uint32_t i0 = warp * 16 + g8, i1 = i0 + 8;
-        const float cum0 = s_cum[i0], cum1 = s_cum[i1];
-        float gm[SC_Q / 8][4], y[PT / 8][4];
+        float sum = d2[0] + d2[1];
 #pragma unroll
-        for (int i = 0; i < SC_Q / 8; ++i) gm[i][0] = gm[i][1] = gm[i][2] = gm[i][3] = 0.0f;
-#pragma unroll
-        for (int i = 0; i < PT / 8; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.0f;
-        const uint32_t a_addr = mx_smem(sc) + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::BP + (lane >> 4) * 16;
-        const uint32_t b_off = ((lane & 7) + (lane >> 4) * 8) * S::BP + ((lane >> 3) & 1) * 16;
-        const uint32_t t_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::XP + (lane >> 4) * 16;   // transposed [k][n] tiles
-        const uint32_t sb_a = mx_smem(sb), ssh_a = mx_smem(ssh), ssl_a = mx_smem(ssl), sx_a = mx_smem(sx);
-#pragma unroll
-        for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t ca[4], bb[4];
-            mx_ldsm(a_addr + kk * 32, ca);
-#pragma unroll
-            for (int n = 0; n < SC_Q / 16; ++n) {
-                if ((uint32_t)n > warp) continue;
-                mx_ldsm(sb_a + b_off + n * 16 * S::BP + kk * 32, bb);
-                mx_mma(gm[2 * n], ca, bb[0], bb[1]);
-                mx_mma(gm[2 * n + 1], ca, bb[2], bb[3]);
-            }
-#pragma unroll
-            for (int n = 0; n < PT / 16; ++n) {
-                mx_ldsm_t(ssh_a + t_off + kk * 16 * S::XP + n * 32, bb);
-                mx_mma(y[2 * n], ca, bb[0], bb[1]);
-                mx_mma(y[2 * n + 1], ca, bb[2], bb[3]);
-                mx_ldsm_t(ssl_a + t_off + kk * 16 * S::XP + n * 32, bb);
-                mx_mma(y[2 * n], ca, bb[0], bb[1]);
-                mx_mma(y[2 * n + 1], ca, bb[2], bb[3]);
-            }
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= (uint32_t)o) sum += up;
         }
-        const float e0 = mx_ex2(cum0), e1 = mx_ex2(cum1);
+        s_cum[buf][2 * lane + 1] = sum;
+        s_cum[buf][2 * lane] = sum - d2[1];
+        s_dt[buf][2 * lane] = dt[0];
+        s_dt[buf][2 * lane + 1] = dt[1];
+    };
+
+    load_chunk(0, 0);
+    if (warp == 0) fetch_steps(0);
+    // S^T: rows p = pw + g8 (+ 8), columns n = nt * 8 + t4 * 2 (+ 1)
+    float acc[NT][4];
 #pragma unroll
-        for (int i = 0; i < PT / 8; ++i) { y[i][0] *= e0; y[i][1] *= e0; y[i][2] *= e1; y[i][3] *= e1; }
-        // ---- decayed weights times x ----
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-        for (int kk = 0; kk < SC_Q / 16; ++kk) {
-            if ((uint32_t)kk > warp) continue;
-            uint32_t hi[4], lo[4], bb[4];
-#pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                const uint32_t j = (2 * kk + n) * 8 + t4 * 2;
-                const float cj0 = s_cum[j], cj1 = s_cum[j + 1], dj0 = s_dt[j], dj1 = s_dt[j + 1];
-                const float* v = gm[2 * kk + n];
-                const float w0 = j <= i0 ? v[0] * mx_ex2(cum0 - cj0) * dj0 : 0.0f;
-                const float w1 = j + 1 <= i0 ? v[1] * mx_ex2(cum0 - cj1) * dj1 : 0.0f;
-                const float w2 = j <= i1 ? v[2] * mx_ex2(cum1 - cj0) * dj0 : 0.0f;
-                const float w3 = j + 1 <= i1 ? v[3] * mx_ex2(cum1 - cj1) * dj1 : 0.0f;
-                split_bf16x2(w0, w1, hi[2 * n], lo[2 * n]);
-                split_bf16x2(w2, w3, hi[2 * n + 1], lo[2 * n + 1]);
-            }
-#pragma unroll
-            for (int n = 0; n < PT / 16; ++n) {
-                mx_ldsm_t(sx_a + t_off + kk * 16 * S::XP + n * 32, bb);
-                mx_mma(y[2 * n], hi, bb[0], bb[1]);
-                mx_mma(y[2 * n + 1], hi, bb[2], bb[3]);
-                mx_mma(y[2 * n], lo, bb[0], bb[1]);
-                mx_mma(y[2 * n + 1], lo, bb[2], bb[3]);
-            }
+        for (int e = 0; e < 4; ++e) {
+            const uint32_t p = pw + g8 + (e >> 1) * 8, n = nt * 8 + t4 * 2 + (e & 1);
+            acc[nt][e] = p0 > 0 && n < m.state && p < width ? state[(size_t)n * m.vdim + p] : 0.0f;
         }
-        // ---- skip, gate, store ----
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-            const uint32_t r = half ? i1 : i0, t = t0 + r;
-            if (t >= place.chunk) continue;
-            const bf16* z = reinterpret_cast<const bf16*>(m.proj) + (row_base + t) * m.ld + h * m.vdim + p_first;
-            bf16* out = reinterpret_cast<bf16*>(m.gated) + (row_base + t) * inner + h * m.vdim + p_first;
-#pragma unroll
-            for (int nt = 0; nt < PT / 8; ++nt) {
-                const uint32_t c = nt * 8 + t4 * 2;
-                if (c >= width) continue;
-                const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(sx + r * S::XP + c * 2));
-                const bool second = c + 1 < width;
-                const float2 zz = load_pair<bf16>(z + c, vec, second);
-                const float v0 = fmaf(skip, x.x, y[nt][2 * half]), v1 = fmaf(skip, x.y, y[nt][2 * half + 1]);
-                store_pair<bf16>(out + c, make_float2(v0 * fast_silu(zz.x), v1 * fast_silu(zz.y)), vec, second);
-            }
-        }
-        __syncthreads();     // weighted inputs are in place; the state tiles have been read
-        // ---- state at the end of the chunk ----
-        const float el = mx_ex2(last);
-        const uint32_t bt_off = ((lane & 7) + (lane >> 4) * 8) * S::BP + ((lane >> 3) & 1) * 16;   // B^T: rows n from [token][n] tiles
-        const uint32_t sxh_a = mx_smem(sxh), sxl_a = mx_smem(sxl);
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-            for (int nt = 0; nt < PT / 8; ++nt) { acc[mt][nt][0] *= el; acc[mt][nt][1] *= el; acc[mt][nt][2] *= el; acc[mt][nt][3] *= el; }
-#pragma unroll
-        for (int kk = 0; kk < SC_Q / 16; ++kk) {
-            uint32_t ba[MT][4];
-#pragma unroll
-            for (int mt = 0; mt < MT; ++mt) mx_ldsm_t(sb_a + bt_off + kk * 16 * S::BP + (warp * MT + mt) * 32, ba[mt]);
-#pragma unroll
-            for (int n = 0; n < PT / 16; ++n) {
-                uint32_t xh[4], xl[4];
-                mx_ldsm_t(sxh_a + t_off + kk * 16 * S::XP + n * 32, xh);
-                mx_ldsm_t(sxl_a + t_off + kk * 16 * S::XP + n * 32, xl);
-#pragma unroll
-                for (int mt = 0; mt < MT; ++mt) {
-                    mx_mma(acc[mt][2 * n], ba[mt], xh[0], xh[1]);
-                    mx_mma(acc[mt][2 * n + 1], ba[mt], xh[2], xh[3]);
-                    mx_mma(acc[mt][2 * n], ba[mt], xl[0], xl[1]);
-                    mx_mma(acc[mt][2 * n + 1], ba[mt], xl[2], xl[3]);
-                }
-            }
-        }
-        store_state_tiles();
-        __syncthreads();     // every tile may be refilled
+    if (warp == 0) {
+        make_decays(0);
+        fetch_steps(SC_Q);
     }
+
+    uint32_t buf = 0;
+    for (uint32_t t0 = 0; t0 < place.chunk; t0 += SC_Q, buf ^= 1) {
+        mx_wait<0>();
+        __syncthreads();     // this chunk's tiles and decays are in place; everyone is done with the other buffer and the weights
+        load_chunk(t0 + SC_Q, buf ^ 1);
+        const uint32_t sb = mx_smem(smem + buf * S::STAGE), sc = sb + S::B_BYTES;
+        const uint8_t* sx = smem + buf * S::STAGE + 2 * S::B_BYTES;
+        const uint32_t sx_a = mx_smem(sx);
+        const float *cum = s_cum[buf], *dts = s_dt[buf];
+        // gate inputs of this warp's outputs: rows mt * 16 + g8 (+ 8), columns pw + nt * 8 + t4 * 2
+        uint32_t z[4][2][2];
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
+        for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-        for (int nt = 0; nt < PT / 8; ++nt)
+            for (int half = 0; half < 2; ++half)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const uint32_t n = state_rows(mt, e >> 1), p = nt * 8 + t4 * 2 + (e & 1);
-                if (n < m.state && p < width) state[(size_t)n * m.vdim + p] = acc[mt][nt][e];
+                for (int nt = 0; nt < 2; ++nt) {
+                    const uint32_t t = t0 + mt * 16 + half * 8 + g8, c = pw + nt * 8 + t4 * 2;
+                    z[mt][half][nt] = 0u;
+                    if (t < place.chunk && c < width) {
+                        const bf16* src = zb + (size_t)t * m.ld + c;
+                        if (vec) z[mt][half][nt] = *reinterpret_cast<const uint32_t*>(src);
+                        else z[mt][half][nt] = (uint32_t)__bfloat16_as_ushort(src[0]) | (c + 1 < width ? (uint32_t)__bfloat16_as_ushort(src[1]) << 16 : 0u);
+                    }
+                }
+        const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::BP + (lane >> 4) * 16;      // A operand, row-major tiles
+        const uint32_t b_off = ((lane & 7) + (lane >> 4) * 8) * S::BP + ((lane >> 3) & 1) * 16;      // B operand, [n][k] tiles
+        // ---- decayed weights of the warp's 16 token rows: columns up to the diagonal block ----
+        {
+            float gm[SC_Q / 8][4];
+#pragma unroll
+            for (int i = 0; i < SC_Q / 8; ++i) gm[i][0] = gm[i][1] = gm[i][2] = gm[i][3] = 0.0f;
+#pragma unroll
+            for (int kk = 0; kk < NP / 16; ++kk) {
+                uint32_t ca[4], bb[4];
+                mx_ldsm(sc + a_off + warp * 16 * S::BP + kk * 32, ca);
+#pragma unroll
+                for (int n = 0; n < SC_Q / 16; ++n) {
+                    if ((uint32_t)n > warp) continue;
+                    mx_ldsm(sb + b_off + n * 16 * S::BP + kk * 32, bb);
+                    mx_mma(gm[2 * n], ca, bb[0], bb[1]);
+                    mx_mma(gm[2 * n + 1], ca, bb[2], bb[3]);
+                }
             }
+            const uint32_t i0 = warp * 16 + g8, i1 = i0 + 8;
+            const float cum0 = cum[i0], cum1 = cum[i1];
+#pragma unroll
+            for (int n = 0; n < SC_Q / 8; ++n) {
+                if ((uint32_t)(n >> 1) > warp) continue;
+                const uint32_t j = n * 8 + t4 * 2;
+                const float2 cj = *reinterpret_cast<const float2*>(cum + j), dj = *reinterpret_cast<const float2*>(dts + j);
+                const float w0 = j <= i0 ? gm[n][0] * mx_ex2(cum0 - cj.x) * dj.x : 0.0f;
+                const float w1 = j + 1 <= i0 ? gm[n][1] * mx_ex2(cum0 - cj.y) * dj.y : 0.0f;
+                const float w2 = j <= i1 ? gm[n][2] * mx_ex2(cum1 - cj.x) * dj.x : 0.0f;
+                const float w3 = j + 1 <= i1 ? gm[n][3] * mx_ex2(cum1 - cj.y) * dj.y : 0.0f;
+                uint32_t hi, lo;
+                split_bf16x2(w0, w1, hi, lo);
+                *reinterpret_cast<uint32_t*>(swh + i0 * S::WP + j * 2) = hi;
+                *reinterpret_cast<uint32_t*>(swl + i0 * S::WP + j * 2) = lo;
+                split_bf16x2(w2, w3, hi, lo);
+                *reinterpret_cast<uint32_t*>(swh + i1 * S::WP + j * 2) = hi;
+                *reinterpret_cast<uint32_t*>(swl + i1 * S::WP + j * 2) = lo;
+            }
+        }
+        // ---- C . S_in, scaled by the decay since the chunk's start ----
+        float y[4][2][4];
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) y[mt][nt][0] = y[mt][nt][1] = y[mt][nt][2] = y[mt][nt][3] = 0.0f;
+        if (owner) {
+#pragma unroll
+            for (int kk = 0; kk < NP / 16; ++kk) {
+                // state rows 16 kk .. + 15: accumulator tiles 2 kk (k 0-7) and 2 kk + 1 (k 8-15); registers 0, 1 are columns
+                // pw .. + 7, registers 2, 3 columns pw + 8 .. + 15
+                uint32_t h00, l00, h01, l01, h10, l10, h11, l11;
+                split_bf16x2(acc[2 * kk][0], acc[2 * kk][1], h00, l00);
+                split_bf16x2(acc[2 * kk + 1][0], acc[2 * kk + 1][1], h01, l01);
+                split_bf16x2(acc[2 * kk][2], acc[2 * kk][3], h10, l10);
+                split_bf16x2(acc[2 * kk + 1][2], acc[2 * kk + 1][3], h11, l11);
+#pragma unroll
+                for (int mt = 0; mt < 4; ++mt) {
+                    uint32_t ca[4];
+                    mx_ldsm(sc + a_off + mt * 16 * S::BP + kk * 32, ca);
+                    mx_mma(y[mt][0], ca, h00, h01);
+                    mx_mma(y[mt][1], ca, h10, h11);
+                    mx_mma(y[mt][0], ca, l00, l01);
+                    mx_mma(y[mt][1], ca, l10, l11);
+                }
+            }
+#pragma unroll
+            for (int mt = 0; mt < 4; ++mt) {
+                const float e0 = mx_ex2(cum[mt * 16 + g8]), e1 = mx_ex2(cum[mt * 16 + 8 + g8]);
+#pragma unroll
+                for (int nt = 0; nt < 2; ++nt) { y[mt][nt][0] *= e0; y[mt][nt][1] *= e0; y[mt][nt][2] *= e1; y[mt][nt][3] *= e1; }
+            }
+        }
+        __syncthreads();     // the weights of all rows are in place
+        if (owner) {
+            // ---- weights . x ----
+            const uint32_t w_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::WP + (lane >> 4) * 16;
+            const uint32_t x_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::XP + (lane >> 4) * 16 + pw * 2;    // [token][p]: B operand, transposed
+            const uint32_t swh_a = mx_smem(swh), swl_a = mx_smem(swl);
+#pragma unroll
+            for (int kk = 0; kk < SC_Q / 16; ++kk) {
+                uint32_t xb[4], wa[4];
+                mx_ldsm_t(sx_a + x_off + kk * 16 * S::XP, xb);
+#pragma unroll
+                for (int mt = kk; mt < 4; ++mt) {
+                    mx_ldsm(swh_a + w_off + mt * 16 * S::WP + kk * 32, wa);
+                    mx_mma(y[mt][0], wa, xb[0], xb[1]);
+                    mx_mma(y[mt][1], wa, xb[2], xb[3]);
+                    mx_ldsm(swl_a + w_off + mt * 16 * S::WP + kk * 32, wa);
+                    mx_mma(y[mt][0], wa, xb[0], xb[1]);
+                    mx_mma(y[mt][1], wa, xb[2], xb[3]);
+                }
+            }
+            // ---- skip, gate, store ----
+#pragma unroll
+            for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const uint32_t r = mt * 16 + half * 8 + g8, t = t0 + r;
+                    if (t >= place.chunk) continue;
+#pragma unroll
+                    for (int nt = 0; nt < 2; ++nt) {
+                        const uint32_t c = pw + nt * 8 + t4 * 2;
+                        if (c >= width) continue;
+                        const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(sx + r * S::XP + c * 2)), zz = bf16x2_to_f32(z[mt][half][nt]);
+                        const float v0 = fmaf(skip, x.x, y[mt][nt][2 * half]) * fast_silu(zz.x);
+                        const float v1 = fmaf(skip, x.y, y[mt][nt][2 * half + 1]) * fast_silu(zz.y);
+                        store_pair<bf16>(gb + (size_t)t * inner + c, make_float2(v0, v1), vec, c + 1 < width);
+                    }
+                }
+            // ---- S^T at the end of the chunk: decayed, plus (x_j weighted by what is left of it)^T . B ----
+            const float last = cum[SC_Q - 1], el = mx_ex2(last);
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) { acc[nt][0] *= el; acc[nt][1] *= el; acc[nt][2] *= el; acc[nt][3] *= el; }
+            const uint32_t xt_off = ((lane & 7) + (lane >> 4) * 8) * S::XP + ((lane >> 3) & 1) * 16 + pw * 2;   // x^T: A operand from [token][p]
+            const uint32_t bt_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::BP + (lane >> 4) * 16;            // B: B operand from [token][n]
+#pragma unroll
+            for (int kk = 0; kk < SC_Q / 16; ++kk) {
+                uint32_t xa[4], xh[4], xl[4];
+                mx_ldsm_t(sx_a + xt_off + kk * 16 * S::XP, xa);
+                // registers 0, 1 hold tokens t4 * 2 (+ 1), registers 2, 3 tokens 8 + t4 * 2 (+ 1)
+#pragma unroll
+                for (int r = 0; r < 2; ++r) {
+                    const uint32_t j = kk * 16 + r * 8 + t4 * 2;
+                    const float2 cj = *reinterpret_cast<const float2*>(cum + j), dj = *reinterpret_cast<const float2*>(dts + j);
+                    const float w0 = mx_ex2(last - cj.x) * dj.x, w1 = mx_ex2(last - cj.y) * dj.y;
+#pragma unroll
+                    for (int q = 0; q < 2; ++q) {
+                        const float2 x = bf16x2_to_f32(xa[2 * r + q]);
+                        split_bf16x2(x.x * w0, x.y * w1, xh[2 * r + q], xl[2 * r + q]);
+                    }
+                }
+#pragma unroll
+                for (int n = 0; n < NT / 2; ++n) {
+                    uint32_t bb[4];
+                    mx_ldsm_t(sb + bt_off + kk * 16 * S::BP + n * 32, bb);
+                    mx_mma(acc[2 * n], xh, bb[0], bb[1]);
+                    mx_mma(acc[2 * n + 1], xh, bb[2], bb[3]);
+                    mx_mma(acc[2 * n], xl, bb[0], bb[1]);
+                    mx_mma(acc[2 * n + 1], xl, bb[2], bb[3]);
+                }
+            }
+        }
+        if (warp == 0) {     // the other buffer's decays: last read before this iteration's first barrier
+            make_decays(buf ^ 1);
+            fetch_steps(t0 + 2 * SC_Q);
+        }
+    }
+    mx_wait<0>();
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const uint32_t p = pw + g8 + (e >> 1) * 8, n = nt * 8 + t4 * 2 + (e & 1);
+            if (n < m.state && p < width) state[(size_t)n * m.vdim + p] = acc[nt][e];
+        }
 }
 
-template <int NP, int PT>
+template <int NP>
 static int launch_scan(const Mamba2& m, const StepPlace& place, uint32_t vec, cudaStream_t stream) {
     static bool configured[64] = {};
-    const uint32_t bytes = ScanShape<NP, PT>::BYTES;
+    const uint32_t bytes = ScanShape<NP>::BYTES;
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-        if (cudaFuncSetAttribute(ssd_scan_kernel<NP, PT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
+        if (cudaFuncSetAttribute(ssd_scan_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess)
             return check_launch("ssd_scan attribute");
         if (dev >= 0 && dev < 64) configured[dev] = true;
     }
-    launch_kernel(ssd_scan_kernel<NP, PT>, dim3(ceil_div(m.vdim, (uint32_t)PT), m.heads, place.sessions), dim3(128), bytes, stream, m, place, vec);
+    launch_kernel(ssd_scan_kernel<NP>, dim3(ceil_div(m.vdim, SC_P), m.heads, place.sessions), dim3(128), bytes, stream, m, place, vec);
     count_launch();
     return check_launch("ssd_scan");
 }
@@ -283,10 +330,9 @@ int launch_ssd_scan(const Mamba2& m, const StepPlace& place, cudaStream_t stream
     const uint32_t inner = m.heads * m.vdim;
     auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
     const uint32_t vec = m.vdim % 8 == 0 && m.state % 8 == 0 && m.ld % 2 == 0 && inner % 8 == 0 && aligned(m.xbc) && aligned(m.proj) && aligned(m.gated);
-    const bool narrow = m.vdim <= 32;
-    if (m.state <= 64) return narrow ? launch_scan<64, 32>(m, place, vec, stream) : launch_scan<64, 64>(m, place, vec, stream);
-    if (m.state <= 128) return narrow ? launch_scan<128, 32>(m, place, vec, stream) : launch_scan<128, 64>(m, place, vec, stream);
-    return launch_scan<256, 32>(m, place, vec, stream);
+    if (m.state <= 64) return launch_scan<64>(m, place, vec, stream);
+    if (m.state <= 128) return launch_scan<128>(m, place, vec, stream);
+    return launch_scan<256>(m, place, vec, stream);
 }
 
 }  // namespace tb

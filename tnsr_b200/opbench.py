@@ -311,7 +311,7 @@ def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads,
     size = lib().tnsr_b200_grouped_attention_workspace(hd, hd)
     ws = torch.zeros(size, dtype=torch.uint8, device="cuda")
     where = _native.Place(sessions, chunk, position, 0, None)
-    args = [_native.GroupedAttentionArgs(q[i].data_ptr(), k[i].data_ptr(), v[i].data_ptr(), gate.data_ptr(), out.data_ptr(), ws.data_ptr(), size,
+    args = [_native.GroupedAttentionArgs(q[i].data_ptr(), k[i].data_ptr(), v[i].data_ptr(), gate.data_ptr(), out.data_ptr(), ws.data_ptr(), None, size,
                                          heads, kv_heads, hd, hd, capacity, 32, heads * hd, heads * hd, hd ** -0.5, softcap, 1, 0) for i in range(sets)]
     ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_grouped_attention(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
     pairs = sessions * heads * sum(position + t + 1 for t in range(chunk))
