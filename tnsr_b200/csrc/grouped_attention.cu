@@ -155,14 +155,21 @@ grouped_split_kernel(GaParams P) {
         mx_wait<STAGES - 2>();
         __syncwarp();
         const uint32_t sk = mx_smem(ring + stage * S::STAGE), sv = sk + 16 * S::KP;
-        float sc[2][4] = {};
+        float sc[2][4] = {}, odd[2][4] = {};       // even and odd k steps apart: shorter chains of dependent products
 #pragma unroll
-        for (int kk = 0; kk < DK / 16; ++kk) {
-            uint32_t b[4];
+        for (int kk = 0; kk < DK / 16; kk += 2) {
+            uint32_t b[4], c[4];
             mx_ldsm(sk + ((lane & 7) + (lane >> 4) * 8) * S::KP + (kk * 16 + ((lane >> 3) & 1) * 8) * 2, b);
+            mx_ldsm(sk + ((lane & 7) + (lane >> 4) * 8) * S::KP + (kk * 16 + 16 + ((lane >> 3) & 1) * 8) * 2, c);
             mx_mma(sc[0], qa[kk], b[0], b[1]);
             mx_mma(sc[1], qa[kk], b[2], b[3]);
+            mx_mma(odd[0], qa[kk + 1], c[0], c[1]);
+            mx_mma(odd[1], qa[kk + 1], c[2], c[3]);
         }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[n][e] += odd[n][e];
         float mx0 = m0, mx1 = m1;
 #pragma unroll
         for (int n = 0; n < 2; ++n)
@@ -202,14 +209,23 @@ grouped_split_kernel(GaParams P) {
         l1 = l1 * c1 + r1;
 #pragma unroll
         for (int n = 0; n < DV / 8; ++n) { o[n][0] *= c0; o[n][1] *= c0; if (UPPER) { o[n][2] *= c1; o[n][3] *= c1; } }
+        // 64 columns at a time, the two halves of a weight eight products apart: one accumulator's products wait for each other
 #pragma unroll
-        for (int n = 0; n < DV / 16; ++n) {
-            uint32_t b[4];
-            mx_ldsm_t(sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * S::VP + (n * 16 + (lane >> 4) * 8) * 2, b);
-            mx_mma(o[2 * n], hi, b[0], b[1]);
-            mx_mma(o[2 * n], lo, b[0], b[1]);
-            mx_mma(o[2 * n + 1], hi, b[2], b[3]);
-            mx_mma(o[2 * n + 1], lo, b[2], b[3]);
+        for (int n0 = 0; n0 < DV / 16; n0 += 4) {
+            uint32_t b[4][4];
+#pragma unroll
+            for (int n = 0; n < 4; ++n)
+                mx_ldsm_t(sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * S::VP + ((n0 + n) * 16 + (lane >> 4) * 8) * 2, b[n]);
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                mx_mma(o[2 * (n0 + n)], hi, b[n][0], b[n][1]);
+                mx_mma(o[2 * (n0 + n) + 1], hi, b[n][2], b[n][3]);
+            }
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                mx_mma(o[2 * (n0 + n)], lo, b[n][0], b[n][1]);
+                mx_mma(o[2 * (n0 + n) + 1], lo, b[n][2], b[n][3]);
+            }
         }
         __syncwarp();    // every lane is done with the stage that the next load may overwrite
         load(i + (STAGES - 1) * GA_WARPS, (stage + STAGES - 1) % STAGES);
@@ -424,13 +440,21 @@ grouped_tile_kernel(GaParams P) {
                     split_bf16x2(pc, pd, hi[2 * n + 1], lo[2 * n + 1]);
                 }
 #pragma unroll
-                for (int n = 0; n < DV / 16; ++n) {
-                    uint32_t bb[4];
-                    mx_ldsm_t(sv + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::VP + (n * 16 + (lane >> 4) * 8) * 2, bb);
-                    mx_mma(o[2 * n], hi, bb[0], bb[1]);
-                    mx_mma(o[2 * n + 1], hi, bb[2], bb[3]);
-                    mx_mma(o[2 * n], lo, bb[0], bb[1]);
-                    mx_mma(o[2 * n + 1], lo, bb[2], bb[3]);
+                for (int n0 = 0; n0 < DV / 16; n0 += 4) {
+                    uint32_t bb[4][4];
+#pragma unroll
+                    for (int n = 0; n < 4; ++n)
+                        mx_ldsm_t(sv + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::VP + ((n0 + n) * 16 + (lane >> 4) * 8) * 2, bb[n]);
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) {
+                        mx_mma(o[2 * (n0 + n)], hi, bb[n][0], bb[n][1]);
+                        mx_mma(o[2 * (n0 + n) + 1], hi, bb[n][2], bb[n][3]);
+                    }
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) {
+                        mx_mma(o[2 * (n0 + n)], lo, bb[n][0], bb[n][1]);
+                        mx_mma(o[2 * (n0 + n) + 1], lo, bb[n][2], bb[n][3]);
+                    }
                 }
             }
         }
@@ -505,15 +529,15 @@ uint32_t padded_width(uint32_t dim, uint32_t vdim) {
     return w <= 64 ? 64 : w <= 128 ? 128 : 256;
 }
 
-// Splits of the keys: as many CTAs as fit the GPU at once (three, two or one per SM at padded widths 64, 128, 256) if the
+// Splits of the keys: as many CTAs as fit the GPU at once (four, two or one per SM at padded widths 64, 128, 256) if the
 // (session, key/value head, row tile) triples do not give them already.
-constexpr uint64_t GA_CTAS = 444;
+constexpr uint64_t GA_CTAS = 592;
 uint32_t splits_for(uint64_t units, uint32_t padded) {
     const uint64_t slots = padded == 64 ? GA_CTAS : padded == 128 ? 296 : 148;
     return (uint32_t)std::min<uint64_t>(GA_MAX_SPLITS, std::max<uint64_t>(1, slots / units));
 }
 // More than one split means at most GA_CTAS / 2 units and GA_CTAS partial tiles.
-constexpr uint64_t GA_COUNTER_BYTES = 1024;
+constexpr uint64_t GA_COUNTER_BYTES = 2048;
 static_assert(GA_COUNTER_BYTES >= GA_CTAS / 2 * 4, "one merge counter per unit");
 
 // Rows (chunk * heads per group) up to which the split kernel runs: one tile per 16 of them re-reads the keys.
@@ -558,7 +582,7 @@ int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, 
             P.partial = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(a.workspace) + GA_COUNTER_BYTES);
         }
         const bool upper = P.rows > 8;
-        if (w == 64) rc = upper ? launch_split<64, 64, 4, true>(P, stream) : launch_split<64, 64, 4, false>(P, stream);
+        if (w == 64) rc = upper ? launch_split<64, 64, 3, true>(P, stream) : launch_split<64, 64, 3, false>(P, stream);
         else if (w == 128) rc = upper ? launch_split<128, 128, 3, true>(P, stream) : launch_split<128, 128, 3, false>(P, stream);
         else rc = upper ? launch_split<256, 256, 2, true>(P, stream) : launch_split<256, 256, 2, false>(P, stream);
     } else if (a.engine == 0 && grouped_attention_tc_eligible(a, place)) {

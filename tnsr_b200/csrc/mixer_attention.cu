@@ -145,6 +145,111 @@ attention_prep_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t r
     }
 }
 
+// The same for bf16 heads of whole 16-byte groups and at most four taps: a lane owns eight channels, LPU lanes a head unit,
+// so that a warp serves 32 / LPU units at once.
+template <int LPU>
+__global__ void __launch_bounds__(128, 5)
+attention_prep_wide_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t runs, uint32_t total) {
+    pdl_wait();
+    pdl_trigger();
+    const uint32_t lane = threadIdx.x & 31, sub = lane % LPU;
+    const uint32_t task = (blockIdx.x * 4 + (threadIdx.x >> 5)) * (32 / LPU) + lane / LPU;
+    const bool live_task = task < total;                       // idle groups take part in the shuffles
+    const uint32_t units = a.heads + 2 * a.kv_heads;
+    const uint32_t tk = live_task ? task : 0;
+    const uint32_t unit = tk % units, r = (tk / units) % runs, s = tk / (units * runs);
+    const uint32_t nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim, channels = nq + nk + nv;
+    const uint32_t which = unit < a.heads ? 0u : unit < a.heads + a.kv_heads ? 1u : 2u;
+    const uint32_t head = which == 0 ? unit : which == 1 ? unit - a.heads : unit - a.heads - a.kv_heads;
+    const uint32_t width = which == 2 ? a.vdim : a.dim;
+    const uint32_t c = sub * 8, ch = (which == 0 ? head * a.dim : which == 1 ? nq + head * a.dim : nq + nk + head * a.vdim) + c;
+    const bool mine = live_task && c < width;
+    const bf16* rows = reinterpret_cast<const bf16*>(a.proj) + (size_t)s * place.chunk * a.ld + ch;
+    bf16* ring = reinterpret_cast<bf16*>(a.ring) + (size_t)s * a.taps * channels + ch;
+    const uint32_t p0 = place.pos(s);
+    const uint32_t t0 = r * run, t1 = min(place.chunk, t0 + run);
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    float w[4][8], nw[8];
+    uint4 win[4];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        nw[e] = mine && which < 2 ? (which == 0 ? a.q_norm : a.k_norm)[c + e] : 1.0f;
+        const float* cw = a.conv_w + (size_t)(ch + e) * a.taps;
+        if (a.taps == 4) {
+            const float4 x = mine ? *reinterpret_cast<const float4*>(cw) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            w[0][e] = x.x; w[1][e] = x.y; w[2][e] = x.z; w[3][e] = x.w;
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { const int src = j - (4 - (int)a.taps); w[j][e] = mine && src >= 0 ? cw[src] : 0.0f; }
+        }
+    }
+#pragma unroll
+    for (int j = 1; j < 4; ++j) {           // slot j: token t0 - 4 + j until the first shift
+        win[j] = zero;
+        const int t = (int)t0 - 4 + j;
+        if (mine && (int)t0 - t < (int)a.taps) {
+            const long long pos = (long long)p0 + t;
+            if (t >= 0) win[j] = *reinterpret_cast<const uint4*>(rows + (size_t)t * a.ld);
+            else if (pos >= 0) win[j] = *reinterpret_cast<const uint4*>(ring + (size_t)(pos % a.taps) * channels);
+        }
+    }
+    const uint32_t pairs = a.rotary_dims / 2;
+    const bool turns = mine && which < 2 && c < a.rotary_dims;
+    bf16* dst = which == 0 ? reinterpret_cast<bf16*>(a.q) + (size_t)s * place.chunk * nq + head * a.dim + c
+              : which == 1 ? reinterpret_cast<bf16*>(a.k_cache) + head * a.dim + c : reinterpret_cast<bf16*>(a.v_cache) + head * a.vdim + c;
+    const uint32_t dst_ld = which == 0 ? nq : which == 1 ? nk : nv;
+    uint4 next = mine && t0 < t1 ? *reinterpret_cast<const uint4*>(rows + (size_t)t0 * a.ld) : zero;
+#pragma unroll 4
+    for (uint32_t u = 0; u < run; ++u) {      // the same trip count for every group of the warp: they shuffle together
+        const uint32_t t = t0 + u, pos = p0 + t;
+        const bool here = mine && t < t1;
+        win[0] = win[1]; win[1] = win[2]; win[2] = win[3]; win[3] = next;
+        next = mine && t + 1 < t1 ? *reinterpret_cast<const uint4*>(rows + (size_t)(t + 1) * a.ld) : zero;
+        float4 ang[2];
+        ang[0] = ang[1] = make_float4(1.0f, 0.0f, 1.0f, 0.0f);
+        if (turns && t < t1) {
+            const float4* at = reinterpret_cast<const float4*>(a.rotation + (size_t)pos * pairs + c / 2);
+            ang[0] = at[0];
+            ang[1] = at[1];
+        }
+        float y[8] = {};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const uint32_t words[4] = {win[j].x, win[j].y, win[j].z, win[j].w};
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                const float2 f = bf16x2_to_f32(words[q]);
+                y[2 * q] = fmaf(w[j][2 * q], f.x, y[2 * q]);
+                y[2 * q + 1] = fmaf(w[j][2 * q + 1], f.y, y[2 * q + 1]);
+            }
+        }
+        if (place.chunk == 1 && here) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.taps) * channels) = win[3];
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+        for (int o = LPU / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = which < 2 ? rsqrtf(ss / (float)width + a.eps) : 1.0f;
+        uint32_t out[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            const float cs = q & 1 ? ang[q >> 1].z : ang[q >> 1].x, sn = q & 1 ? ang[q >> 1].w : ang[q >> 1].y;
+            const float a0 = y[2 * q] * (inv * nw[2 * q]), a1 = y[2 * q + 1] * (inv * nw[2 * q + 1]);
+            out[q] = pack_bf16x2(a0 * cs - a1 * sn, a1 * cs + a0 * sn);
+        }
+        if (here) {
+            const size_t row = which == 0 ? t : kv_row(a.paging, s, pos, a.capacity);
+            *reinterpret_cast<uint4*>(dst + row * dst_ld) = make_uint4(out[0], out[1], out[2], out[3]);
+        }
+    }
+}
+
+static bool prep_wide_fits(const AttentionPrep& a) {
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    return a.taps <= 4 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.rotary_dims % 8 == 0 && aligned(a.proj) && aligned(a.ring) &&
+           aligned(a.q) && aligned(a.k_cache) && aligned(a.v_cache) && aligned(a.conv_w) && aligned(a.rotation);
+}
+
 template <typename T, int NP>
 static void prep_taps(const AttentionPrep& a, const StepPlace& place, uint32_t run, uint32_t runs, uint32_t total, uint32_t vec,
                       cudaStream_t stream) {
@@ -172,7 +277,13 @@ int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dt
     const uint32_t run = std::min(place.chunk, 32u), runs = ceil_div(place.chunk, run);
     const uint64_t total = (uint64_t)place.sessions * runs * (a.heads + 2 * a.kv_heads);
     if (total > 0x7fffffffull) { set_thread_error("attention: too many rows for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
-    if (dtype == TNSR_B200_BF16) prep_width<bf16>(a, place, run, runs, (uint32_t)total, stream);
+    if (dtype == TNSR_B200_BF16 && prep_wide_fits(a)) {
+        const uint32_t width = std::max(a.dim, a.vdim);
+        auto grid = [&](uint32_t lanes) { return dim3((uint32_t)ceil_div64(total, 4 * (32 / lanes))); };
+        if (width <= 64) launch_kernel(attention_prep_wide_kernel<8>, grid(8), dim3(128), 0, stream, a, place, run, runs, (uint32_t)total);
+        else if (width <= 128) launch_kernel(attention_prep_wide_kernel<16>, grid(16), dim3(128), 0, stream, a, place, run, runs, (uint32_t)total);
+        else launch_kernel(attention_prep_wide_kernel<32>, grid(32), dim3(128), 0, stream, a, place, run, runs, (uint32_t)total);
+    } else if (dtype == TNSR_B200_BF16) prep_width<bf16>(a, place, run, runs, (uint32_t)total, stream);
     else prep_width<float>(a, place, run, runs, (uint32_t)total, stream);
     count_launch();
     return check_launch("attention_prep");

@@ -25,7 +25,7 @@ __device__ __forceinline__ float act_silu(float x);
 template <>
 __device__ __forceinline__ float act_silu<float>(float x) { return full_silu(x); }
 template <>
-__device__ __forceinline__ float act_silu<bf16>(float x) { return fast_silu(x); }
+__device__ __forceinline__ float act_silu<bf16>(float x) { return mx_silu(x); }
 __device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
 // ---- convolution + silu ----------------------------------------------------------------------
@@ -45,10 +45,22 @@ conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uin
     const T* in = rows + (size_t)s * place.chunk * ld + c;
     T* dst = out + (size_t)s * place.chunk * channels + c;
     float2 w[TAPS], win[TAPS];
+    const float* cw = conv_w + (size_t)c * taps;
+    if (TAPS == 4 && taps == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(cw), y = second ? *reinterpret_cast<const float4*>(cw + 4) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        w[0] = make_float2(x.x, y.x);
+        w[TAPS > 1 ? 1 : 0] = make_float2(x.y, y.y);
+        w[TAPS > 2 ? 2 : 0] = make_float2(x.z, y.z);
+        w[TAPS > 3 ? 3 : 0] = make_float2(x.w, y.w);
+    } else {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const int src = j - (TAPS - (int)taps);
+            w[j] = make_float2(src >= 0 ? cw[src] : 0.0f, src >= 0 && second ? cw[taps + src] : 0.0f);
+        }
+    }
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-        const int src = j - (TAPS - (int)taps);
-        w[j] = make_float2(src >= 0 ? conv_w[(size_t)c * taps + src] : 0.0f, src >= 0 && second ? conv_w[(size_t)(c + 1) * taps + src] : 0.0f);
         win[j] = make_float2(0.0f, 0.0f);
         const int t = (int)t0 - TAPS + j;
         if (j > 0 && (int)t0 - t < (int)taps) {
@@ -113,7 +125,7 @@ static void conv_silu_typed(const Mamba2& m, uint32_t inner, uint32_t channels, 
 constexpr uint32_t SSD_THREADS = 256, SSD_SLICE = 64, SSD_MAX_STATE = 256;
 
 template <typename T, int ROWS, int VEC>
-__global__ void __launch_bounds__(SSD_THREADS)
+__global__ void __launch_bounds__(SSD_THREADS, ROWS * VEC <= 32 ? 4 : 2)
 ssd_token_kernel(Mamba2 m, StepPlace place) {
     __shared__ float sb[SSD_MAX_STATE], sc[SSD_MAX_STATE], sx[SSD_SLICE], red[SSD_THREADS * VEC];
     pdl_wait();

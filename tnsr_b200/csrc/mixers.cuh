@@ -165,6 +165,8 @@ __device__ __forceinline__ float mx_rcp(float x) {
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// silu by one exponential and one reciprocal of the special-function unit (for results that are stored as bf16).
+__device__ __forceinline__ float mx_silu(float x) { return x * mx_rcp(1.0f + mx_ex2(-1.4426950408889634f * x)); }
 // x = hi + lo with both halves bf16: two products with an exact bf16 operand then carry 16 bits of x.
 __device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16x2(x, y);

@@ -7,7 +7,8 @@
 // of S do not couple, so each of its four warps owns 16 of them.  A warp keeps S transposed in accumulator registers
 // (rows = its columns, from x^T . B): in that layout the accumulators of S^T are, register by register, the B operand of
 // C . S, so the state never passes through shared memory.  The decayed weights (C B^T with the decays applied) are made
-// once per CTA, 16 token rows per warp, and shared.  The next chunk's B, C and x arrive while this one is computed.
+// once per CTA, 16 token rows per warp, and shared.  Three CTAs per SM (states up to 128 rows) hide each other's waits; the
+// next chunk's C is asked for as soon as the current one is used up, its B and x at the end of the chunk.
 //
 // Factors that are f32 -- the decayed weights, the state, the weighted inputs -- enter the products as two bf16 halves
 // (split_bf16x2), so that they keep 16 bits.
@@ -26,17 +27,17 @@ struct ScanShape {
     static constexpr uint32_t BP = NP * 2 + 16, XP = SC_P * 2 + 16, WP = SC_Q * 2 + 16;   // row pitches: conflict-free ldmatrix
     static constexpr uint32_t B_BYTES = SC_Q * BP, X_BYTES = SC_Q * XP, W_BYTES = SC_Q * WP;
     static constexpr uint32_t STAGE = 2 * B_BYTES + X_BYTES;          // B, C, x of one chunk
-    static constexpr uint32_t BYTES = 2 * STAGE + 2 * W_BYTES;
+    static constexpr uint32_t BYTES = STAGE + 2 * W_BYTES;
 };
 
 // NP: state rows padded to a multiple of 64.
 template <int NP>
-__global__ void __launch_bounds__(128, NP <= 128 ? 2 : 1)
+__global__ void __launch_bounds__(128, NP <= 128 ? 3 : 1)
 ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
     using S = ScanShape<NP>;
     constexpr int NT = NP / 8;                  // 8-row tiles of the state
     extern __shared__ __align__(16) uint8_t smem[];
-    uint8_t* swh = smem + 2 * S::STAGE;
+    uint8_t* swh = smem + S::STAGE;
     uint8_t* swl = swh + S::W_BYTES;
     __shared__ float s_cum[2][SC_Q], s_dt[2][SC_Q];   // running log2 decay, step size
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
@@ -74,12 +75,14 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
             }
         }
     };
-    auto load_chunk = [&](uint32_t t0, uint32_t buf) {
+    auto load_c = [&](uint32_t t0) {
+        if (t0 < place.chunk) load_tile(smem + S::B_BYTES, S::BP, NP, inner + gn + group * m.state, m.state, t0);
+        mx_commit();
+    };
+    auto load_bx = [&](uint32_t t0) {
         if (t0 < place.chunk) {
-            uint8_t* dst = smem + buf * S::STAGE;
-            load_tile(dst, S::BP, NP, inner + group * m.state, m.state, t0);
-            load_tile(dst + S::B_BYTES, S::BP, NP, inner + gn + group * m.state, m.state, t0);
-            load_tile(dst + 2 * S::B_BYTES, S::XP, SC_P, h * m.vdim + p_first, width, t0);
+            load_tile(smem, S::BP, NP, inner + group * m.state, m.state, t0);
+            load_tile(smem + 2 * S::B_BYTES, S::XP, SC_P, h * m.vdim + p_first, width, t0);
         }
         mx_commit();
     };
@@ -111,7 +114,8 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
         s_dt[buf][2 * lane + 1] = dt[1];
     };
 
-    load_chunk(0, 0);
+    load_c(0);
+    load_bx(0);
     if (warp == 0) fetch_steps(0);
     // S^T: rows p = pw + g8 (+ 8), columns n = nt * 8 + t4 * 2 (+ 1)
     float acc[NT][4];
@@ -130,28 +134,11 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
     uint32_t buf = 0;
     for (uint32_t t0 = 0; t0 < place.chunk; t0 += SC_Q, buf ^= 1) {
         mx_wait<0>();
-        __syncthreads();     // this chunk's tiles and decays are in place; everyone is done with the other buffer and the weights
-        load_chunk(t0 + SC_Q, buf ^ 1);
-        const uint32_t sb = mx_smem(smem + buf * S::STAGE), sc = sb + S::B_BYTES;
-        const uint8_t* sx = smem + buf * S::STAGE + 2 * S::B_BYTES;
+        __syncthreads();     // this chunk's tiles and decays are in place; everyone is done with the weights of the last one
+        const uint32_t sb = mx_smem(smem), sc = sb + S::B_BYTES;
+        const uint8_t* sx = smem + 2 * S::B_BYTES;
         const uint32_t sx_a = mx_smem(sx);
         const float *cum = s_cum[buf], *dts = s_dt[buf];
-        // gate inputs of this warp's outputs: rows mt * 16 + g8 (+ 8), columns pw + nt * 8 + t4 * 2
-        uint32_t z[4][2][2];
-#pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-            for (int half = 0; half < 2; ++half)
-#pragma unroll
-                for (int nt = 0; nt < 2; ++nt) {
-                    const uint32_t t = t0 + mt * 16 + half * 8 + g8, c = pw + nt * 8 + t4 * 2;
-                    z[mt][half][nt] = 0u;
-                    if (t < place.chunk && c < width) {
-                        const bf16* src = zb + (size_t)t * m.ld + c;
-                        if (vec) z[mt][half][nt] = *reinterpret_cast<const uint32_t*>(src);
-                        else z[mt][half][nt] = (uint32_t)__bfloat16_as_ushort(src[0]) | (c + 1 < width ? (uint32_t)__bfloat16_as_ushort(src[1]) << 16 : 0u);
-                    }
-                }
         const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::BP + (lane >> 4) * 16;      // A operand, row-major tiles
         const uint32_t b_off = ((lane & 7) + (lane >> 4) * 8) * S::BP + ((lane >> 3) & 1) * 16;      // B operand, [n][k] tiles
         // ---- decayed weights of the warp's 16 token rows: columns up to the diagonal block ----
@@ -159,7 +146,7 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
             float gm[SC_Q / 8][4];
 #pragma unroll
             for (int i = 0; i < SC_Q / 8; ++i) gm[i][0] = gm[i][1] = gm[i][2] = gm[i][3] = 0.0f;
-#pragma unroll
+#pragma unroll 2
             for (int kk = 0; kk < NP / 16; ++kk) {
                 uint32_t ca[4], bb[4];
                 mx_ldsm(sc + a_off + warp * 16 * S::BP + kk * 32, ca);
@@ -207,14 +194,19 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
                 split_bf16x2(acc[2 * kk + 1][0], acc[2 * kk + 1][1], h01, l01);
                 split_bf16x2(acc[2 * kk][2], acc[2 * kk][3], h10, l10);
                 split_bf16x2(acc[2 * kk + 1][2], acc[2 * kk + 1][3], h11, l11);
+                // (products of one accumulator are kept eight apart: each waits for the one before it)
+                uint32_t ca[4][4];
+#pragma unroll
+                for (int mt = 0; mt < 4; ++mt) mx_ldsm(sc + a_off + mt * 16 * S::BP + kk * 32, ca[mt]);
 #pragma unroll
                 for (int mt = 0; mt < 4; ++mt) {
-                    uint32_t ca[4];
-                    mx_ldsm(sc + a_off + mt * 16 * S::BP + kk * 32, ca);
-                    mx_mma(y[mt][0], ca, h00, h01);
-                    mx_mma(y[mt][1], ca, h10, h11);
-                    mx_mma(y[mt][0], ca, l00, l01);
-                    mx_mma(y[mt][1], ca, l10, l11);
+                    mx_mma(y[mt][0], ca[mt], h00, h01);
+                    mx_mma(y[mt][1], ca[mt], h10, h11);
+                }
+#pragma unroll
+                for (int mt = 0; mt < 4; ++mt) {
+                    mx_mma(y[mt][0], ca[mt], l00, l01);
+                    mx_mma(y[mt][1], ca[mt], l10, l11);
                 }
             }
 #pragma unroll
@@ -224,21 +216,43 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
                 for (int nt = 0; nt < 2; ++nt) { y[mt][nt][0] *= e0; y[mt][nt][1] *= e0; y[mt][nt][2] *= e1; y[mt][nt][3] *= e1; }
             }
         }
-        __syncthreads();     // the weights of all rows are in place
+        __syncthreads();     // the weights of all rows are in place, C has been used up
+        load_c(t0 + SC_Q);
         if (owner) {
+            // gate inputs of this warp's outputs: rows mt * 16 + g8 (+ 8), columns pw + nt * 8 + t4 * 2
+            uint32_t z[4][2][2];
+#pragma unroll
+            for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+                for (int half = 0; half < 2; ++half)
+#pragma unroll
+                    for (int nt = 0; nt < 2; ++nt) {
+                        const uint32_t t = t0 + mt * 16 + half * 8 + g8, c = pw + nt * 8 + t4 * 2;
+                        z[mt][half][nt] = 0u;
+                        if (t < place.chunk && c < width) {
+                            const bf16* src = zb + (size_t)t * m.ld + c;
+                            if (vec) z[mt][half][nt] = *reinterpret_cast<const uint32_t*>(src);
+                            else z[mt][half][nt] = (uint32_t)__bfloat16_as_ushort(src[0]) | (c + 1 < width ? (uint32_t)__bfloat16_as_ushort(src[1]) << 16 : 0u);
+                        }
+                    }
             // ---- weights . x ----
             const uint32_t w_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::WP + (lane >> 4) * 16;
             const uint32_t x_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::XP + (lane >> 4) * 16 + pw * 2;    // [token][p]: B operand, transposed
             const uint32_t swh_a = mx_smem(swh), swl_a = mx_smem(swl);
-#pragma unroll
+#pragma unroll 1
             for (int kk = 0; kk < SC_Q / 16; ++kk) {
                 uint32_t xb[4], wa[4];
                 mx_ldsm_t(sx_a + x_off + kk * 16 * S::XP, xb);
 #pragma unroll
-                for (int mt = kk; mt < 4; ++mt) {
+                for (int mt = 0; mt < 4; ++mt) {
+                    if (mt < kk) continue;
                     mx_ldsm(swh_a + w_off + mt * 16 * S::WP + kk * 32, wa);
                     mx_mma(y[mt][0], wa, xb[0], xb[1]);
                     mx_mma(y[mt][1], wa, xb[2], xb[3]);
+                }
+#pragma unroll
+                for (int mt = 0; mt < 4; ++mt) {
+                    if (mt < kk) continue;
                     mx_ldsm(swl_a + w_off + mt * 16 * S::WP + kk * 32, wa);
                     mx_mma(y[mt][0], wa, xb[0], xb[1]);
                     mx_mma(y[mt][1], wa, xb[2], xb[3]);
@@ -256,8 +270,8 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
                         const uint32_t c = pw + nt * 8 + t4 * 2;
                         if (c >= width) continue;
                         const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(sx + r * S::XP + c * 2)), zz = bf16x2_to_f32(z[mt][half][nt]);
-                        const float v0 = fmaf(skip, x.x, y[mt][nt][2 * half]) * fast_silu(zz.x);
-                        const float v1 = fmaf(skip, x.y, y[mt][nt][2 * half + 1]) * fast_silu(zz.y);
+                        const float v0 = fmaf(skip, x.x, y[mt][nt][2 * half]) * mx_silu(zz.x);
+                        const float v1 = fmaf(skip, x.y, y[mt][nt][2 * half + 1]) * mx_silu(zz.y);
                         store_pair<bf16>(gb + (size_t)t * inner + c, make_float2(v0, v1), vec, c + 1 < width);
                     }
                 }
@@ -267,7 +281,7 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
             for (int nt = 0; nt < NT; ++nt) { acc[nt][0] *= el; acc[nt][1] *= el; acc[nt][2] *= el; acc[nt][3] *= el; }
             const uint32_t xt_off = ((lane & 7) + (lane >> 4) * 8) * S::XP + ((lane >> 3) & 1) * 16 + pw * 2;   // x^T: A operand from [token][p]
             const uint32_t bt_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::BP + (lane >> 4) * 16;            // B: B operand from [token][n]
-#pragma unroll
+#pragma unroll 1
             for (int kk = 0; kk < SC_Q / 16; ++kk) {
                 uint32_t xa[4], xh[4], xl[4];
                 mx_ldsm_t(sx_a + xt_off + kk * 16 * S::XP, xa);
@@ -284,13 +298,18 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
                     }
                 }
 #pragma unroll
-                for (int n = 0; n < NT / 2; ++n) {
-                    uint32_t bb[4];
-                    mx_ldsm_t(sb + bt_off + kk * 16 * S::BP + n * 32, bb);
-                    mx_mma(acc[2 * n], xh, bb[0], bb[1]);
-                    mx_mma(acc[2 * n + 1], xh, bb[2], bb[3]);
-                    mx_mma(acc[2 * n], xl, bb[0], bb[1]);
-                    mx_mma(acc[2 * n + 1], xl, bb[2], bb[3]);
+                for (int n = 0; n < NT / 4; ++n) {
+                    uint32_t b0[4], b1[4];
+                    mx_ldsm_t(sb + bt_off + kk * 16 * S::BP + n * 64, b0);
+                    mx_ldsm_t(sb + bt_off + kk * 16 * S::BP + n * 64 + 32, b1);
+                    mx_mma(acc[4 * n], xh, b0[0], b0[1]);
+                    mx_mma(acc[4 * n + 1], xh, b0[2], b0[3]);
+                    mx_mma(acc[4 * n + 2], xh, b1[0], b1[1]);
+                    mx_mma(acc[4 * n + 3], xh, b1[2], b1[3]);
+                    mx_mma(acc[4 * n], xl, b0[0], b0[1]);
+                    mx_mma(acc[4 * n + 1], xl, b0[2], b0[3]);
+                    mx_mma(acc[4 * n + 2], xl, b1[0], b1[1]);
+                    mx_mma(acc[4 * n + 3], xl, b1[2], b1[3]);
                 }
             }
         }
@@ -298,6 +317,8 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
             make_decays(buf ^ 1);
             fetch_steps(t0 + 2 * SC_Q);
         }
+        __syncthreads();     // B and x have been used up
+        load_bx(t0 + SC_Q);
     }
     mx_wait<0>();
 #pragma unroll
