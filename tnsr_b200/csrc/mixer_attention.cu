@@ -146,10 +146,12 @@ attention_prep_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t r
 }
 
 // The same for bf16 heads of whole 16-byte groups and at most four taps: a lane owns eight channels, LPU lanes a head unit,
-// so that a warp serves 32 / LPU units at once.
+// so that a warp serves 32 / LPU units at once; rows travel four tokens ahead of their use (the kernel lives on bytes in
+// flight), angles one.
 template <int LPU>
-__global__ void __launch_bounds__(128, 5)
+__global__ void __launch_bounds__(128, 4)
 attention_prep_wide_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint32_t runs, uint32_t total) {
+    constexpr uint32_t AHEAD = 4;
     pdl_wait();
     pdl_trigger();
     const uint32_t lane = threadIdx.x & 31, sub = lane % LPU;
@@ -164,13 +166,25 @@ attention_prep_wide_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint3
     const uint32_t width = which == 2 ? a.vdim : a.dim;
     const uint32_t c = sub * 8, ch = (which == 0 ? head * a.dim : which == 1 ? nq + head * a.dim : nq + nk + head * a.vdim) + c;
     const bool mine = live_task && c < width;
-    const bf16* rows = reinterpret_cast<const bf16*>(a.proj) + (size_t)s * place.chunk * a.ld + ch;
-    bf16* ring = reinterpret_cast<bf16*>(a.ring) + (size_t)s * a.taps * channels + ch;
     const uint32_t p0 = place.pos(s);
-    const uint32_t t0 = r * run, t1 = min(place.chunk, t0 + run);
+    const uint32_t t0 = r * run, n = mine ? min(place.chunk - t0, run) : 0u;     // this group's tokens: t0 .. t0 + n - 1
+    const bf16* rows = reinterpret_cast<const bf16*>(a.proj) + ((size_t)s * place.chunk + t0) * a.ld + ch;
+    bf16* ring = reinterpret_cast<bf16*>(a.ring) + (size_t)s * a.taps * channels + ch;
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-    float w[4][8], nw[8];
+    uint4 next[AHEAD];
+#pragma unroll
+    for (uint32_t i = 0; i < AHEAD; ++i) next[i] = i < n ? *reinterpret_cast<const uint4*>(rows + (size_t)i * a.ld) : zero;
     uint4 win[4];
+#pragma unroll
+    for (int j = 1; j < 4; ++j) {           // slot j: token t0 - 4 + j until the first shift
+        win[j] = zero;
+        const uint32_t lag = 4 - j;
+        if (mine && lag < a.taps) {
+            if (t0 >= lag) win[j] = *reinterpret_cast<const uint4*>(rows - (size_t)lag * a.ld);
+            else if (p0 + t0 >= lag) win[j] = *reinterpret_cast<const uint4*>(ring + (size_t)((p0 + t0 - lag) % a.taps) * channels);
+        }
+    }
+    float w[4][8], nw[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
         nw[e] = mine && which < 2 ? (which == 0 ? a.q_norm : a.k_norm)[c + e] : 1.0f;
@@ -183,71 +197,67 @@ attention_prep_wide_kernel(AttentionPrep a, StepPlace place, uint32_t run, uint3
             for (int j = 0; j < 4; ++j) { const int src = j - (4 - (int)a.taps); w[j][e] = mine && src >= 0 ? cw[src] : 0.0f; }
         }
     }
-#pragma unroll
-    for (int j = 1; j < 4; ++j) {           // slot j: token t0 - 4 + j until the first shift
-        win[j] = zero;
-        const int t = (int)t0 - 4 + j;
-        if (mine && (int)t0 - t < (int)a.taps) {
-            const long long pos = (long long)p0 + t;
-            if (t >= 0) win[j] = *reinterpret_cast<const uint4*>(rows + (size_t)t * a.ld);
-            else if (pos >= 0) win[j] = *reinterpret_cast<const uint4*>(ring + (size_t)(pos % a.taps) * channels);
-        }
-    }
     const uint32_t pairs = a.rotary_dims / 2;
-    const bool turns = mine && which < 2 && c < a.rotary_dims;
-    bf16* dst = which == 0 ? reinterpret_cast<bf16*>(a.q) + (size_t)s * place.chunk * nq + head * a.dim + c
+    const bool turns = which < 2 && c < a.rotary_dims;
+    const float4* angles = reinterpret_cast<const float4*>(a.rotation + (size_t)(p0 + t0) * pairs + c / 2);
+    const uint32_t angle_ld = pairs / 2;
+    const float4 still = make_float4(1.0f, 0.0f, 1.0f, 0.0f);      // no rotation
+    float4 ang[2];
+    ang[0] = turns && n > 0 ? __ldg(angles) : still;
+    ang[1] = turns && n > 0 ? __ldg(angles + 1) : still;
+    bf16* dst = which == 0 ? reinterpret_cast<bf16*>(a.q) + ((size_t)s * place.chunk + t0) * nq + head * a.dim + c
               : which == 1 ? reinterpret_cast<bf16*>(a.k_cache) + head * a.dim + c : reinterpret_cast<bf16*>(a.v_cache) + head * a.vdim + c;
     const uint32_t dst_ld = which == 0 ? nq : which == 1 ? nk : nv;
-    uint4 next = mine && t0 < t1 ? *reinterpret_cast<const uint4*>(rows + (size_t)t0 * a.ld) : zero;
-#pragma unroll 4
-    for (uint32_t u = 0; u < run; ++u) {      // the same trip count for every group of the warp: they shuffle together
-        const uint32_t t = t0 + u, pos = p0 + t;
-        const bool here = mine && t < t1;
-        win[0] = win[1]; win[1] = win[2]; win[2] = win[3]; win[3] = next;
-        next = mine && t + 1 < t1 ? *reinterpret_cast<const uint4*>(rows + (size_t)(t + 1) * a.ld) : zero;
-        float4 ang[2];
-        ang[0] = ang[1] = make_float4(1.0f, 0.0f, 1.0f, 0.0f);
-        if (turns && t < t1) {
-            const float4* at = reinterpret_cast<const float4*>(a.rotation + (size_t)pos * pairs + c / 2);
-            ang[0] = at[0];
-            ang[1] = at[1];
-        }
-        float y[8] = {};
+    const float inv_width = 1.0f / (float)width;
+    for (uint32_t u0 = 0; u0 < run; u0 += AHEAD) {      // the same trip count for every group of the warp: they shuffle together
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const uint32_t words[4] = {win[j].x, win[j].y, win[j].z, win[j].w};
+        for (uint32_t i = 0; i < AHEAD; ++i) {
+            const uint32_t u = u0 + i;
+            const bool here = u < n;
+            win[0] = win[1]; win[1] = win[2]; win[2] = win[3]; win[3] = next[i];
+            next[i] = u + AHEAD < n ? *reinterpret_cast<const uint4*>(rows + (size_t)(u + AHEAD) * a.ld) : zero;
+            const float4 now[2] = {ang[0], ang[1]};
+            if (turns && u + 1 < n) {
+                ang[0] = __ldg(angles + (size_t)(u + 1) * angle_ld);
+                ang[1] = __ldg(angles + (size_t)(u + 1) * angle_ld + 1);
+            }
+            float y[8] = {};
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const uint32_t words[4] = {win[j].x, win[j].y, win[j].z, win[j].w};
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const float2 f = bf16x2_to_f32(words[q]);
+                    y[2 * q] = fmaf(w[j][2 * q], f.x, y[2 * q]);
+                    y[2 * q + 1] = fmaf(w[j][2 * q + 1], f.y, y[2 * q + 1]);
+                }
+            }
+            if (place.chunk == 1 && here) *reinterpret_cast<uint4*>(ring + (size_t)((p0 + t0) % a.taps) * channels) = win[3];
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+#pragma unroll
+            for (int o = LPU / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = which < 2 ? rsqrtf(fmaf(ss, inv_width, a.eps)) : 1.0f;
+            uint32_t out[4];
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
-                const float2 f = bf16x2_to_f32(words[q]);
-                y[2 * q] = fmaf(w[j][2 * q], f.x, y[2 * q]);
-                y[2 * q + 1] = fmaf(w[j][2 * q + 1], f.y, y[2 * q + 1]);
+                const float cs = q & 1 ? now[q >> 1].z : now[q >> 1].x, sn = q & 1 ? now[q >> 1].w : now[q >> 1].y;
+                const float a0 = y[2 * q] * (inv * nw[2 * q]), a1 = y[2 * q + 1] * (inv * nw[2 * q + 1]);
+                out[q] = pack_bf16x2(a0 * cs - a1 * sn, a1 * cs + a0 * sn);
             }
-        }
-        if (place.chunk == 1 && here) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.taps) * channels) = win[3];
-        float ss = 0.0f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
-#pragma unroll
-        for (int o = LPU / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        const float inv = which < 2 ? rsqrtf(ss / (float)width + a.eps) : 1.0f;
-        uint32_t out[4];
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            const float cs = q & 1 ? ang[q >> 1].z : ang[q >> 1].x, sn = q & 1 ? ang[q >> 1].w : ang[q >> 1].y;
-            const float a0 = y[2 * q] * (inv * nw[2 * q]), a1 = y[2 * q + 1] * (inv * nw[2 * q + 1]);
-            out[q] = pack_bf16x2(a0 * cs - a1 * sn, a1 * cs + a0 * sn);
-        }
-        if (here) {
-            const size_t row = which == 0 ? t : kv_row(a.paging, s, pos, a.capacity);
-            *reinterpret_cast<uint4*>(dst + row * dst_ld) = make_uint4(out[0], out[1], out[2], out[3]);
+            if (here) {
+                const size_t row = which == 0 ? u : kv_row(a.paging, s, p0 + t0 + u, a.capacity);
+                *reinterpret_cast<uint4*>(dst + row * dst_ld) = make_uint4(out[0], out[1], out[2], out[3]);
+            }
         }
     }
 }
 
 static bool prep_wide_fits(const AttentionPrep& a) {
     auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-    return a.taps <= 4 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.rotary_dims % 8 == 0 && aligned(a.proj) && aligned(a.ring) &&
-           aligned(a.q) && aligned(a.k_cache) && aligned(a.v_cache) && aligned(a.conv_w) && aligned(a.rotation);
+    return a.taps <= 4 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.rotary_dims % 8 == 0 &&
+           aligned(a.proj) && aligned(a.ring) && aligned(a.q) && aligned(a.k_cache) && aligned(a.v_cache) && aligned(a.conv_w) && aligned(a.rotation);
 }
 
 template <typename T, int NP>

@@ -61,11 +61,16 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
     auto load_tile = [&](uint8_t* dst, uint32_t pitch, uint32_t padded, uint32_t c0, uint32_t w, uint32_t t0) {
         const uint32_t live = min((uint32_t)SC_Q, place.chunk - t0);
         if (vec) {
-            const uint32_t ch = padded / 8;
-            for (uint32_t i = tid; i < SC_Q * ch; i += 128) {
-                const uint32_t r = i / ch, c = (i % ch) * 8;
-                const bool real = r < live && c < w;
-                mx_cp16(dst + r * pitch + c * 2, real ? xbc + (size_t)(t0 + r) * channels + c0 + c : xbc, real);
+            // a thread keeps its 16-byte column and walks down the rows
+            const uint32_t ch = padded / 8, step = 128 / ch, r0 = tid / ch, c = (tid % ch) * 8;
+            const bf16* src = xbc + (size_t)(t0 + r0) * channels + c0 + c;
+            uint8_t* to = dst + r0 * pitch + c * 2;
+            const uint32_t n = c < w && live > r0 ? live - r0 : 0u;     // rows of this thread's column that exist, from r0 on
+#pragma unroll 8
+            for (uint32_t r = 0; r < SC_Q; r += step) {
+                mx_cp16(to, r < n ? src : xbc, r < n);
+                src += (size_t)step * channels;
+                to += step * pitch;
             }
         } else {
             for (uint32_t i = tid; i < SC_Q * padded; i += 128) {
@@ -219,22 +224,24 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
         __syncthreads();     // the weights of all rows are in place, C has been used up
         load_c(t0 + SC_Q);
         if (owner) {
-            // gate inputs of this warp's outputs: rows mt * 16 + g8 (+ 8), columns pw + nt * 8 + t4 * 2
+            // gate inputs of this warp's outputs: rows mt * 16 + half * 8 + g8, columns pw + nt * 8 + t4 * 2
             uint32_t z[4][2][2];
+            const uint32_t c0 = pw + t4 * 2, live = place.chunk - t0 > g8 ? place.chunk - t0 - g8 : 0u;   // rows from g8 on
+            {
+                const bf16* src = zb + (size_t)(t0 + g8) * m.ld + c0;
+                const size_t down = (size_t)8 * m.ld;
 #pragma unroll
-            for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-                for (int half = 0; half < 2; ++half)
+                for (int rr = 0; rr < 8; ++rr, src += down)
 #pragma unroll
                     for (int nt = 0; nt < 2; ++nt) {
-                        const uint32_t t = t0 + mt * 16 + half * 8 + g8, c = pw + nt * 8 + t4 * 2;
-                        z[mt][half][nt] = 0u;
-                        if (t < place.chunk && c < width) {
-                            const bf16* src = zb + (size_t)t * m.ld + c;
-                            if (vec) z[mt][half][nt] = *reinterpret_cast<const uint32_t*>(src);
-                            else z[mt][half][nt] = (uint32_t)__bfloat16_as_ushort(src[0]) | (c + 1 < width ? (uint32_t)__bfloat16_as_ushort(src[1]) << 16 : 0u);
+                        uint32_t v = 0u;
+                        if ((uint32_t)rr * 8 < live && c0 + nt * 8 < width) {
+                            if (vec) v = __ldg(reinterpret_cast<const uint32_t*>(src + nt * 8));
+                            else v = (uint32_t)__bfloat16_as_ushort(src[nt * 8]) | (c0 + nt * 8 + 1 < width ? (uint32_t)__bfloat16_as_ushort(src[nt * 8 + 1]) << 16 : 0u);
                         }
+                        z[rr >> 1][rr & 1][nt] = v;
                     }
+            }
             // ---- weights . x ----
             const uint32_t w_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::WP + (lane >> 4) * 16;
             const uint32_t x_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::XP + (lane >> 4) * 16 + pw * 2;    // [token][p]: B operand, transposed
@@ -259,22 +266,24 @@ ssd_scan_kernel(Mamba2 m, StepPlace place, uint32_t vec) {
                 }
             }
             // ---- skip, gate, store ----
+            {
+                bf16* out = gb + (size_t)(t0 + g8) * inner + c0;
+                const uint8_t* xr = sx + g8 * S::XP + c0 * 2;
+                const size_t down = (size_t)8 * inner;
 #pragma unroll
-            for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    const uint32_t r = mt * 16 + half * 8 + g8, t = t0 + r;
-                    if (t >= place.chunk) continue;
+                for (int rr = 0; rr < 8; ++rr, out += down) {
+                    if ((uint32_t)rr * 8 >= live) break;
 #pragma unroll
                     for (int nt = 0; nt < 2; ++nt) {
-                        const uint32_t c = pw + nt * 8 + t4 * 2;
-                        if (c >= width) continue;
-                        const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(sx + r * S::XP + c * 2)), zz = bf16x2_to_f32(z[mt][half][nt]);
-                        const float v0 = fmaf(skip, x.x, y[mt][nt][2 * half]) * mx_silu(zz.x);
-                        const float v1 = fmaf(skip, x.y, y[mt][nt][2 * half + 1]) * mx_silu(zz.y);
-                        store_pair<bf16>(gb + (size_t)t * inner + c, make_float2(v0, v1), vec, c + 1 < width);
+                        if (c0 + nt * 8 >= width) continue;
+                        const float2 x = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(xr + rr * 8 * S::XP + nt * 16));
+                        const float2 zz = bf16x2_to_f32(z[rr >> 1][rr & 1][nt]);
+                        const float v0 = fmaf(skip, x.x, y[rr >> 1][nt][2 * (rr & 1)]) * mx_silu(zz.x);
+                        const float v1 = fmaf(skip, x.y, y[rr >> 1][nt][2 * (rr & 1) + 1]) * mx_silu(zz.y);
+                        store_pair<bf16>(out + nt * 8, make_float2(v0, v1), vec, c0 + nt * 8 + 1 < width);
                     }
                 }
+            }
             // ---- S^T at the end of the chunk: decayed, plus (x_j weighted by what is left of it)^T . B ----
             const float last = cum[SC_Q - 1], el = mx_ex2(last);
 #pragma unroll
