@@ -44,7 +44,7 @@ CONFIGS = {
     "even": config(128, 320, [mamba2(4, 64, 128, groups=2, norm_groups=4, ff=192), attention(8, 2, 64, 64, base=5000.0, scaling=SCALING, ff=256),
                               mamba2(4, 64, 128, groups=2, norm_groups=4, ff=192, weights_of=0)], scale=1.5),
     # nothing divides anything: one head per key/value head, no cap, no frequency scaling, one tap, no feed-forward
-    "odd": config(72, 97, [attention(3, 3, 10, 7, conv=1, rot=6, softcap=None), mamba2(5, 7, 5, groups=5, norm_groups=5, conv=5),
+    "odd": config(70, 97, [attention(3, 3, 10, 7, conv=1, rot=6, softcap=None), mamba2(5, 7, 5, groups=5, norm_groups=5, conv=5),
                            attention(9, 1, 14, 22, conv=6, rot=14, softcap=7.0, ff=37)], scale=1.0, eps=1e-3),
     # wide heads and states: several slices of the state, two 128-column paddings
     "wide": config(160, 128, [attention(2, 1, 136, 200, rot=64, ff=96), mamba2(2, 136, 200, ff=64), attention(4, 2, 96, 80, ff=64)]),

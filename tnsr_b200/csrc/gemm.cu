@@ -819,13 +819,13 @@ static int launch_tc_e(const CUtensorMap& ma, const CUtensorMap& mb, const CUten
     return check_launch("gemm_tc");
 }
 
-// Wide tiles with a bf16 epilogue (QKV routing, SwiGLU) and a short K: the main loop of a K = 768 tile is shorter than
+// Wide tiles with a bf16 epilogue (QKV routing, SwiGLU, column ranges) and a short K: the main loop of a K = 768 tile is shorter than
 // 8 warps need to drain the previous accumulator, so these run 16 epilogue warps (and 3 ring stages instead of 4, which
 // is why longer K keeps 8: there the deeper ring is worth more).
 template <int BN, int MODE>
 static int launch_tc_t(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap* mo, const TcParams& prm, cudaStream_t stream) {
-    if (BN == 256 && (MODE == GEMM_QKV || MODE == GEMM_SWIGLU) && prm.k <= 1024)
-        return launch_tc_e<BN, MODE, (BN == 256 && (MODE == GEMM_QKV || MODE == GEMM_SWIGLU)) ? 16 : 8>(ma, mb, mo, prm, stream);
+    constexpr bool many_warps = BN == 256 && (MODE == GEMM_QKV || MODE == GEMM_SWIGLU || MODE == GEMM_SEGMENTS);
+    if (many_warps && prm.k <= 1024) return launch_tc_e<BN, MODE, many_warps ? 16 : 8>(ma, mb, mo, prm, stream);
     // narrow tiles: one epilogue warp per TMEM lane quarter is all a 32- or 64-column tile can use
     if (BN <= 64 && MODE != GEMM_ARGMAX) return launch_tc_e<BN, MODE, BN <= 64 ? 4 : 8>(ma, mb, mo, prm, stream);
     return launch_tc_e<BN, MODE, 8>(ma, mb, mo, prm, stream);
