@@ -57,7 +57,8 @@ typedef enum tnsr_b200_activation {
     TNSR_B200_ACT_RELU = 0,
     TNSR_B200_ACT_GELU = 1,
     TNSR_B200_ACT_SWIGLU = 2,
-    TNSR_B200_ACT_GELU_TANH = 3   /* 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))): operator calls and described models */
+    TNSR_B200_ACT_GELU_TANH = 3,  /* 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))): operator calls and described models */
+    TNSR_B200_ACT_RELU_SQUARED = 4   /* grouped products */
 } tnsr_b200_activation;
 
 typedef enum tnsr_b200_dtype {
@@ -143,10 +144,20 @@ typedef struct tnsr_b200_decoder tnsr_b200_decoder;
 
 /* Models described layer by layer (no reference counterpart: tnsr has one GPT
  * block).  A described model is an embedding table, a list of layers and an
- * output head; every layer is one pre-norm block whose mixer and feed-forward
- * read the same normalised rows and are added to the residual together:
- *     h = rms(x) * (norm_offset + w);   x <- x + mixer(h) + feed_forward(h)
- * (feed_forward(h) = W_down gelu_tanh(W_up h), left out when feed_forward is 0).
+ * output head.  A layer is a pre-norm block of one of two forms, with
+ * norm(x) = rms(x) * (norm_offset + w):
+ * BLOCK_PARALLEL: mixer and feed-forward read the same rows and are added to the
+ *     residual together:  h = norm(x);  x <- x + mixer(h) + feed_forward(h)
+ * BLOCK_SEQUENTIAL: each has a norm and a layer scale (one factor per channel):
+ *     x <- x + s1 * mixer(norm1(x));  x <- x + s2 * feed_forward(norm2(x))
+ * The feed-forward is left out when feed_forward is 0.  FF_GELU_TANH (parallel
+ * blocks): W_down gelu_tanh(W_up h).  FF_POLYNORM (sequential): W_down p(W_up h),
+ * p(z) = a N(z) + b N(z^2) + c N(z^3) + e with elementwise powers and N(v) =
+ * v / rms(v) over the row.  FF_EXPERTS (sequential): the `top` of experts +
+ * identity_experts with the largest softmax(W_router h) + correction, weighted by
+ * their softmax values divided by the chosen ones' sum, times router_scale; an
+ * expert is W_down relu(W_up h)^2 of width feed_forward, an identity expert
+ * returns h.
  *
  * MIXER_ATTENTION: projections with bias, a causal per-channel convolution of
  * conv_taps taps on q, k and v, per-head RMS norm of q and k, interleaved rotary
@@ -158,13 +169,35 @@ typedef struct tnsr_b200_decoder tnsr_b200_decoder;
  * x|B|C, dt = softplus(dt + bias), a [state, vdim] f32 state per head with scalar
  * decay exp(-exp(A_log) dt), skip D x, gate silu(z), RMS norm in norm_groups
  * parts.
+ * MIXER_ATTENTION_HGRN2: two mixers side by side, their results added with the
+ * gains attention_gain and recurrent_gain.  Attention as above without biases,
+ * convolutions, norms and gate; with window > 0 a position sees itself and the
+ * window - 1 before it; with score_kind SCORE_SIGMOID a visible key counts with
+ * sigmoid(score + bias of the head), not normalised over keys.  HGRN2: per head a
+ * [rec_dim, rec_vdim] f32 state, f = l + (1 - l) sigmoid(W_f h + b),
+ * S <- diag(f) S + (1 - f) v^T, o = S^T silu(W_q h), then an RMS norm per head.
+ * MIXER_RGLRU: y = gelu_tanh(W_y h + b) beside u = convolution of W_x h + b over
+ * `width` channels in `blocks` equal parts; gates r, i = sigmoid of a square matrix
+ * per part; a = exp(-8 r softplus(lambda)), S <- a S + sqrt(1 - a^2) i u (f32);
+ * output W_o (S y).
  *
  * weights_of >= 0: the layer has no tensors of its own and uses those of that
  * layer (same sizes), with a cache or state of its own. */
 typedef enum tnsr_b200_mixer {
     TNSR_B200_MIXER_ATTENTION = 0,
-    TNSR_B200_MIXER_MAMBA2 = 1
+    TNSR_B200_MIXER_MAMBA2 = 1,
+    TNSR_B200_MIXER_ATTENTION_HGRN2 = 2,
+    TNSR_B200_MIXER_RGLRU = 3
 } tnsr_b200_mixer;
+typedef enum tnsr_b200_block_form { TNSR_B200_BLOCK_PARALLEL = 0, TNSR_B200_BLOCK_SEQUENTIAL = 1 } tnsr_b200_block_form;
+typedef enum tnsr_b200_feed_forward {
+    TNSR_B200_FF_GELU_TANH = 0,
+    TNSR_B200_FF_POLYNORM = 1,
+    TNSR_B200_FF_EXPERTS = 2
+} tnsr_b200_feed_forward;
+typedef enum tnsr_b200_score_kind { TNSR_B200_SCORE_SOFTMAX = 0, TNSR_B200_SCORE_SIGMOID = 1 } tnsr_b200_score_kind;
+/* Which dimensions of a head turn together: 2i and 2i + 1, or i and i + rotary_dims / 2. */
+typedef enum tnsr_b200_rotary_layout { TNSR_B200_ROTARY_INTERLEAVED = 0, TNSR_B200_ROTARY_HALVES = 1 } tnsr_b200_rotary_layout;
 
 typedef struct tnsr_b200_layer {
     uint32_t mixer;         /* tnsr_b200_mixer */
@@ -177,7 +210,7 @@ typedef struct tnsr_b200_layer {
     uint32_t kv_heads;      /* divides heads */
     uint32_t dim;           /* query / key width per head, <= 256 */
     uint32_t rotary_dims;   /* even, <= dim */
-    uint32_t pad0;
+    uint32_t rotary_layout; /* tnsr_b200_rotary_layout; interleaved for MIXER_ATTENTION */
     double rotary_base;
     double rotary_factor;   /* 0: frequencies as they are */
     double rotary_low, rotary_high, rotary_original;
@@ -187,7 +220,20 @@ typedef struct tnsr_b200_layer {
     uint32_t state;         /* <= 256 */
     uint32_t groups;        /* divides heads */
     uint32_t norm_groups;   /* divides heads * vdim */
-    uint32_t pad1;
+    uint32_t block_form;    /* tnsr_b200_block_form */
+    uint32_t feed_forward_kind;  /* tnsr_b200_feed_forward */
+    /* attention beside HGRN2 (heads, vdim, kv_heads, dim, rotary and score fields: the attention's) */
+    uint32_t window;        /* 0: every earlier position is visible */
+    uint32_t score_kind;    /* tnsr_b200_score_kind */
+    uint32_t rec_heads, rec_dim, rec_vdim;   /* rec_dim <= 256 */
+    double attention_gain, recurrent_gain;
+    /* rglru (conv_taps; heads and vdim do not apply) */
+    uint32_t width;
+    uint32_t blocks;        /* divides width */
+    /* experts */
+    uint32_t experts, identity_experts, top;
+    uint32_t pad0;
+    double router_scale;
 } tnsr_b200_layer;
 
 typedef struct tnsr_b200_stack {
@@ -248,8 +294,14 @@ TNSR_B200_API int tnsr_b200_decoder_create(const tnsr_b200_config* config, tnsr_
  * [vocab, d], head [vocab, d], final norm [d], then for every layer with tensors
  * of its own: norm [d]; attention: q, q bias, k, k bias, v, v bias, q norm, k
  * norm, q conv, k conv, v conv, gate, output; mamba2: in, conv, conv bias, dt
- * bias, A_log, D, norm, output; then up, down if it has a feed-forward.  Matrices
- * are [out, in] here, convolutions [channels, taps].  The attention caches are
+ * bias, A_log, D, norm, output; attention beside HGRN2: q, k, v, head bias
+ * (sigmoid scores only), output, then q, f, f bias, lower bound, v, norm, output of
+ * the recurrent half; rglru: y, y bias, x, x bias, conv, conv bias, r, r bias, i, i
+ * bias, lambda, output; then the feed-forward, if there is one: up, down;
+ * polynorm: up, down, the four constants; experts: up and down of every expert,
+ * router, correction.  Sequential blocks have the scale s1 after the mixer's
+ * tensors, and norm2 before and s2 after the feed-forward's.  Matrices are [out,
+ * in] here, convolutions [channels, taps], gate matrices [blocks, out, in].  The attention caches are
  * [batch, capacity, kv_heads * width]; paging applies to them only.  Sessions at
  * position 0 start from empty states whatever their slot held before. */
 TNSR_B200_API int tnsr_b200_decoder_create_stack(const tnsr_b200_config* config, const tnsr_b200_stack* stack,
@@ -559,6 +611,11 @@ typedef struct tnsr_b200_grouped_attention_args {
     uint32_t heads, kv_heads, dim, vdim, capacity, gate_ld, out_ld, out_cols;
     float scale, softcap;
     int32_t dtype, engine;
+    const float* head_bias; /* [heads], sigmoid scores */
+    uint32_t window;        /* > 0: a query sees itself and the window - 1 keys before it */
+    uint32_t score_kind;    /* tnsr_b200_score_kind; SIGMOID: out = gain * sum_j sigmoid(q . k_j * scale + head_bias) v_j */
+    float gain;             /* factor of the result; 0 counts as 1 */
+    uint32_t pad0;
 } tnsr_b200_grouped_attention_args;
 TNSR_B200_API uint64_t tnsr_b200_grouped_attention_workspace(uint32_t dim, uint32_t vdim);
 TNSR_B200_API int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args,
@@ -582,6 +639,98 @@ typedef struct tnsr_b200_mamba2_args {
     uint32_t pad0;
 } tnsr_b200_mamba2_args;
 TNSR_B200_API int tnsr_b200_mamba2(const tnsr_b200_mamba2_args* args, const tnsr_b200_place* place, void* stream);
+
+/* Rotary positions without a convolution or norm before them: proj [rows, ld]
+ * holds q | k | v; the first rotary_dims dimensions of every q and k head turn by
+ * position * rotary_base^(-2i/rotary_dims); q rows go to q, k and v rows to the
+ * caches at their positions.  rotation: [capacity, rotary_dims / 2] (cos, sin)
+ * pairs, NULL when rotary_dims is 0. */
+typedef struct tnsr_b200_rotary_args {
+    const void* proj;
+    const float* rotation;
+    void *q, *k_cache, *v_cache;
+    uint32_t ld, heads, kv_heads, dim, vdim, rotary_dims, rotary_layout, capacity;
+    int32_t dtype;
+    uint32_t pad0;
+} tnsr_b200_rotary_args;
+TNSR_B200_API int tnsr_b200_rotary(const tnsr_b200_rotary_args* args, const tnsr_b200_place* place, void* stream);
+
+/* HGRN2 between its projections: q [rows, ld] before silu, v [rows, ld], f
+ * [rows, f_ld] f32 before bias and sigmoid; state [sessions, heads, dim, vdim] f32
+ * is read and updated; out [rows, out_ld] = gain * norm_w * rms-normed o, columns
+ * from heads * vdim to out_cols are zeroed.  raw: [rows, heads * vdim] f32 scratch,
+ * used when vdim > 128.  engine: 0 = best kernel for the chunk, 1 = token by token. */
+typedef struct tnsr_b200_hgrn2_args {
+    const void *q, *v;
+    const float *f, *f_bias, *lower, *norm_w;
+    float *state, *raw;
+    void* out;
+    uint32_t ld, f_ld, heads, dim, vdim, out_ld, out_cols;
+    float eps, gain;
+    int32_t dtype, engine;
+    uint32_t pad0;
+} tnsr_b200_hgrn2_args;
+TNSR_B200_API int tnsr_b200_hgrn2(const tnsr_b200_hgrn2_args* args, const tnsr_b200_place* place, void* stream);
+
+/* The real-gated linear recurrent unit between its projections: proj [rows, ld]
+ * holds y (after gelu) in columns [0, width) and x from column x_col on; gate_w
+ * [blocks, 2 n, n] (rows r, then i; n = width / blocks; type dtype), r_bias and
+ * i_bias [width]; ring [sessions, taps, width] and state [sessions, width] f32 are
+ * read and updated; u [blocks, rows, n] and gates [blocks, rows, 2 n] f32 are
+ * scratch; out [rows, out_ld], columns from width to out_cols are zeroed. */
+typedef struct tnsr_b200_rglru_args {
+    const void *proj, *gate_w;
+    const float *conv_w, *conv_b, *r_bias, *i_bias, *lambda;
+    void* ring;
+    float* state;
+    void* u;
+    float* gates;
+    void* out;
+    int* d_status;
+    uint32_t ld, x_col, width, blocks, taps, out_ld, out_cols;
+    int32_t dtype;
+} tnsr_b200_rglru_args;
+TNSR_B200_API int tnsr_b200_rglru(const tnsr_b200_rglru_args* args, const tnsr_b200_place* place, void* stream);
+
+/* out[r, c] = p(z[r, :])[c] with p as in FF_POLYNORM; act = {a, b, c, e} on the
+ * device; columns from `width` to out_cols are zeroed. */
+TNSR_B200_API int tnsr_b200_polynorm(const void* z, const float* act, void* out, uint32_t rows, uint32_t width,
+                                     uint32_t out_ld, uint32_t out_cols, float epsilon, int dtype, void* stream);
+
+/* Products of row groups with a matrix each: rows offsets[g] .. offsets[g + 1] of a
+ * [rows, k] times w[g] [n, k] transposed, into out [rows, n].  offsets: groups + 1
+ * device values; NULL: every group has rows / groups rows.  activation:
+ * tnsr_b200_activation, -1 none, 4 relu squared.  engine: 0 = tcgen05 where the
+ * shape allows it, 1 = CUDA cores. */
+TNSR_B200_API int tnsr_b200_gemm_grouped(const void* a, const void* w, void* out, const uint32_t* offsets,
+                                         uint32_t groups, uint32_t rows, uint32_t n, uint32_t k, int activation,
+                                         int dtype, int out_dtype, int engine, int* d_status, void* stream);
+
+/* Mixture of experts on rows h [rows, d] whose router logits [rows, logits_ld] are
+ * given: x [rows, d] (f32) += layer_scale * sum over the chosen experts, and, if
+ * norm_out is set, norm_out [rows, d] = rms-normed x * (norm_offset + norm_w).  up
+ * [experts, ff, d], down [experts, d, ff]; h and norm_out may be the same rows.
+ * workspace: tnsr_b200_experts_workspace() bytes, 256-byte aligned.  chosen
+ * [rows, top] and weights [rows, top] (may be NULL) receive the routing. */
+typedef struct tnsr_b200_experts_args {
+    const float* logits;
+    const float* correction;
+    const void *h, *up, *down;
+    float* x;
+    const float *layer_scale, *norm_w;
+    void* norm_out;
+    void* workspace;
+    uint64_t workspace_bytes;
+    uint32_t* chosen;
+    float* weights;
+    int* d_status;
+    uint32_t rows, logits_ld, d, ff, experts, identity_experts, top;
+    float router_scale, norm_offset, eps;
+    int32_t dtype, engine;
+} tnsr_b200_experts_args;
+TNSR_B200_API uint64_t tnsr_b200_experts_workspace(uint32_t rows, uint32_t d, uint32_t ff, uint32_t experts,
+                                                   uint32_t top, int dtype);
+TNSR_B200_API int tnsr_b200_experts(const tnsr_b200_experts_args* args, void* stream);
 
 /* Next-token sampling on the device (no reference counterpart: tnsr's decode
  * loop is greedy, src/nn/kv_cache.rs:121-157).  Per row: the top_k entries

@@ -17,8 +17,12 @@ STATUS = {
     0: "OK", -1: "ERR_INVALID_ARGUMENT", -2: "ERR_CUDA", -3: "ERR_OUT_OF_MEMORY", -4: "ERR_CAPACITY",
     -5: "ERR_TOKEN_RANGE", -6: "ERR_FAILED_STATE", -7: "ERR_TIMEOUT", -8: "ERR_UNSUPPORTED", -9: "ERR_NO_DEVICE",
 }
-ACT = {"relu": 0, "gelu": 1, "swiglu": 2, "gelu_tanh": 3}
-MIXER = {"attention": 0, "mamba2": 1}
+ACT = {"relu": 0, "gelu": 1, "swiglu": 2, "gelu_tanh": 3, "relu_squared": 4}
+MIXER = {"attention": 0, "mamba2": 1, "attention+hgrn2": 2, "rglru": 3}
+BLOCK = {"parallel": 0, "sequential": 1}
+FEED_FORWARD = {"gelu_tanh": 0, "polynorm": 1, "experts": 2}
+SCORE = {"softmax": 0, "sigmoid": 1}
+ROTARY = {"interleaved": 0, "halves": 1}
 DTYPE = {"f32": 0, "bf16": 1}
 LOGITS = {"all": 0, "last": 1, "none": 2}
 PREFILL = {"auto": 0, "scalar": 1}
@@ -38,10 +42,13 @@ class Config(C.Structure):
 class LayerDesc(C.Structure):
     _fields_ = [
         ("mixer", C.c_uint32), ("weights_of", C.c_int32), ("heads", C.c_uint32), ("vdim", C.c_uint32), ("conv_taps", C.c_uint32),
-        ("feed_forward", C.c_uint32), ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("rotary_dims", C.c_uint32), ("pad0", C.c_uint32),
+        ("feed_forward", C.c_uint32), ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("rotary_dims", C.c_uint32), ("rotary_layout", C.c_uint32),
         ("rotary_base", C.c_double), ("rotary_factor", C.c_double), ("rotary_low", C.c_double), ("rotary_high", C.c_double),
         ("rotary_original", C.c_double), ("score_scale", C.c_double), ("score_softcap", C.c_double), ("state", C.c_uint32),
-        ("groups", C.c_uint32), ("norm_groups", C.c_uint32), ("pad1", C.c_uint32),
+        ("groups", C.c_uint32), ("norm_groups", C.c_uint32), ("block_form", C.c_uint32), ("feed_forward_kind", C.c_uint32),
+        ("window", C.c_uint32), ("score_kind", C.c_uint32), ("rec_heads", C.c_uint32), ("rec_dim", C.c_uint32), ("rec_vdim", C.c_uint32),
+        ("attention_gain", C.c_double), ("recurrent_gain", C.c_double), ("width", C.c_uint32), ("blocks", C.c_uint32),
+        ("experts", C.c_uint32), ("identity_experts", C.c_uint32), ("top", C.c_uint32), ("pad0", C.c_uint32), ("router_scale", C.c_double),
     ]
 
 
@@ -58,7 +65,33 @@ class Place(C.Structure):
 class GroupedAttentionArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "gate", "out", "workspace", "d_status")] + [("workspace_bytes", C.c_uint64)] + \
         [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "capacity", "gate_ld", "out_ld", "out_cols")] + \
-        [("scale", C.c_float), ("softcap", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32)]
+        [("scale", C.c_float), ("softcap", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32), ("head_bias", C.c_void_p),
+         ("window", C.c_uint32), ("score_kind", C.c_uint32), ("gain", C.c_float), ("pad0", C.c_uint32)]
+
+
+class RotaryArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "rotation", "q", "k_cache", "v_cache")] + \
+        [(n, C.c_uint32) for n in ("ld", "heads", "kv_heads", "dim", "vdim", "rotary_dims", "rotary_layout", "capacity")] + \
+        [("dtype", C.c_int32), ("pad0", C.c_uint32)]
+
+
+class Hgrn2Args(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("q", "v", "f", "f_bias", "lower", "norm_w", "state", "raw", "out")] + \
+        [(n, C.c_uint32) for n in ("ld", "f_ld", "heads", "dim", "vdim", "out_ld", "out_cols")] + \
+        [("eps", C.c_float), ("gain", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32), ("pad0", C.c_uint32)]
+
+
+class RglruArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "gate_w", "conv_w", "conv_b", "r_bias", "i_bias", "lambda_", "ring", "state", "u", "gates", "out",
+                                          "d_status")] + \
+        [(n, C.c_uint32) for n in ("ld", "x_col", "width", "blocks", "taps", "out_ld", "out_cols")] + [("dtype", C.c_int32)]
+
+
+class ExpertsArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("logits", "correction", "h", "up", "down", "x", "layer_scale", "norm_w", "norm_out", "workspace")] + \
+        [("workspace_bytes", C.c_uint64)] + [(n, C.c_void_p) for n in ("chosen", "weights", "d_status")] + \
+        [(n, C.c_uint32) for n in ("rows", "logits_ld", "d", "ff", "experts", "identity_experts", "top")] + \
+        [("router_scale", C.c_float), ("norm_offset", C.c_float), ("eps", C.c_float), ("dtype", C.c_int32), ("engine", C.c_int32)]
 
 
 class Mamba2Args(C.Structure):
@@ -121,6 +154,13 @@ SIGNATURES = {
     "tnsr_b200_grouped_attention_workspace": (_u64, [_u32, _u32]),
     "tnsr_b200_grouped_attention": (_i, [C.POINTER(GroupedAttentionArgs), C.POINTER(Place), _vp]),
     "tnsr_b200_mamba2": (_i, [C.POINTER(Mamba2Args), C.POINTER(Place), _vp]),
+    "tnsr_b200_rotary": (_i, [C.POINTER(RotaryArgs), C.POINTER(Place), _vp]),
+    "tnsr_b200_hgrn2": (_i, [C.POINTER(Hgrn2Args), C.POINTER(Place), _vp]),
+    "tnsr_b200_rglru": (_i, [C.POINTER(RglruArgs), C.POINTER(Place), _vp]),
+    "tnsr_b200_polynorm": (_i, [_vp, _vp, _vp, _u32, _u32, _u32, _u32, _f, _i, _vp]),
+    "tnsr_b200_gemm_grouped": (_i, [_vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _i, _i, _i, _i, _vp, _vp]),
+    "tnsr_b200_experts_workspace": (_u64, [_u32, _u32, _u32, _u32, _u32, _i]),
+    "tnsr_b200_experts": (_i, [C.POINTER(ExpertsArgs), _vp]),
     "tnsr_b200_sample_top_k": (_i, [_vp, _vp, _u32, _u32, _f, _u32, _u64, _u32, _u32, _vp]),
     "tnsr_b200_decoder_set_sampler": (_i, [_vp, _f, _u32, _u64]),
     "tnsr_b200_decoder_release": (_i, [_vp, _u32]),

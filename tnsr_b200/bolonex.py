@@ -7,16 +7,11 @@ of layers and tensor sharing all come from its config.json.
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Tuple
-
-import numpy as np
+from typing import Dict, Optional, Tuple
 
 from . import _native
-from .nn import CachedModel, MAX_EXACT_F32_INTEGER, Parameter, TnsrError
-
-# Longest context unless the caller says otherwise: rotary positions have no table to run out of, but a session's
-# positions stay exact f32 integers.
-DEFAULT_CONTEXT = 1 << 20
+from .described import DEFAULT_CONTEXT, DescribedModel
+from .nn import TnsrError
 
 
 @dataclass(frozen=True)
@@ -162,30 +157,6 @@ class BolonexConfig:
         return shapes
 
 
-class Bolonex(CachedModel):
-    def __init__(self, config: BolonexConfig, tensors: Dict[str, np.ndarray]):
-        assert 0 < config.vocab_size <= MAX_EXACT_F32_INTEGER and config.embed_dim > 0 and config.layers
-        assert 0 < config.max_sequence_length <= MAX_EXACT_F32_INTEGER
-        assert config.weight_dtype in ("f32", "bf16")
-        self._config = config
-        shapes = config.tensor_shapes()
-        missing, unexpected = sorted(set(shapes) - set(tensors)), sorted(set(tensors) - set(shapes))
-        if missing or unexpected:
-            raise TnsrError(f"parameter keys mismatch; missing: {missing}; unexpected: {unexpected}")
-        self._parameters = {}
-        for name, shape in shapes.items():
-            if tuple(tensors[name].shape) != shape:
-                raise TnsrError(f"{name}: expected shape {list(shape)}, got {list(tensors[name].shape)}")
-            self._parameters[name] = Parameter(tensors[name], shape)
-
-    def config(self) -> BolonexConfig:
-        return self._config
-
-    def parameters(self) -> List[Parameter]:
-        return list(self._parameters.values())
-
-    def named(self) -> Dict[str, Parameter]:
-        return dict(self._parameters)
-
-    def _generation_capacity(self, needed: int) -> int:
-        return min(needed, self._config.max_sequence_length)
+class Bolonex(DescribedModel):
+    def __init__(self, config: BolonexConfig, tensors):
+        super().__init__(config, tensors)

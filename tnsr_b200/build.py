@@ -25,7 +25,8 @@ LIB = os.path.join(CSRC, "libtnsr_b200.so")
 
 SOURCES = ["decoder.cu", "ops_api.cu", "elementwise.cu", "strict.cu", "gemm.cu", "gemm_skinny.cu", "attention.cu", "prefill.cu", "prefill_tc.cu",
            "decode_attention_static.cu", "sampler.cu", "encoder.cu", "decode_tail.cu", "gemm_stream.cu",
-           "layer_stack.cu", "mixer_attention.cu", "grouped_attention.cu", "mixer_mamba2.cu", "ssd_scan.cu"]
+           "layer_stack.cu", "mixer_attention.cu", "grouped_attention.cu", "mixer_mamba2.cu", "ssd_scan.cu", "mixer_hgrn2.cu", "hgrn2_scan.cu",
+           "mixer_rglru.cu", "feed_forward.cu", "gemm_grouped.cu"]
 EXTRA = {"strict.cu": ["--fmad=false"], "encoder.cu": ["--fmad=false"]}
 
 BASE_FLAGS = [

@@ -84,7 +84,7 @@ inline uint32_t ceil_div(uint32_t a, uint32_t b) { return (a + b - 1) / b; }
 inline uint64_t ceil_div64(uint64_t a, uint64_t b) { return (a + b - 1) / b; }
 
 // FFN / epilogue activation codes shared by host and device.
-enum : int { ACT_NONE = -1, ACT_RELU = 0, ACT_GELU = 1, ACT_GELU_TANH = 3 };   // values of tnsr_b200_activation
+enum : int { ACT_NONE = -1, ACT_RELU = 0, ACT_GELU = 1, ACT_GELU_TANH = 3, ACT_RELU_SQUARED = 4 };   // values of tnsr_b200_activation
 
 // Device-side status word: kernels never trap; they record the first problem
 // here and carry on with harmless values.
@@ -102,6 +102,7 @@ enum : int {
 
 struct GemmEpilogue {
     const float* bias = nullptr;      // [n] f32, added after accumulation
+    const float* scale = nullptr;     // [n] f32, factor of act(acc + bias) before the residual (f32 output; a layer scale)
     const float* residual = nullptr;  // [m, ldr] f32, added last (f32 output only)
     uint32_t ldr = 0;
     int activation = ACT_NONE;        // applied to acc + bias
@@ -378,6 +379,7 @@ __device__ __forceinline__ float apply_activation(float x, int act) {
     if (act == ACT_RELU) return fmaxf(x, 0.0f);
     if (act == ACT_GELU) return fast_gelu(x);
     if (act == ACT_GELU_TANH) return fast_gelu_tanh(x);
+    if (act == ACT_RELU_SQUARED) { const float y = fmaxf(x, 0.0f); return y * y; }
     return x;
 }
 

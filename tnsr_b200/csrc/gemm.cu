@@ -49,6 +49,7 @@ __device__ __forceinline__ void store_plain(const EpiParams& P, uint32_t row, ui
     if (P.ep.out_dtype == TNSR_B200_BF16) {
         reinterpret_cast<bf16*>(P.out)[orow * P.ldc + col] = __float2bfloat16_rn(v);
     } else {
+        if (P.ep.scale) v *= P.ep.scale[col];
         if (P.ep.residual) v += P.ep.residual[(size_t)row * P.ep.ldr + col];
         reinterpret_cast<float*>(P.out)[orow * P.ldc + col] = v;
     }
@@ -281,7 +282,7 @@ __device__ __forceinline__ float4 act4(float4 v, int act) {
 // pointers and leading dimensions).
 __device__ __forceinline__ bool f32_vector_path(const EpiParams& P, uint32_t col0) {
     const float* res = P.ep.residual;
-    return col0 + 32 <= P.n && (reinterpret_cast<uintptr_t>(P.ep.bias) & 15) == 0 && P.ldc % 4 == 0 &&
+    return col0 + 32 <= P.n && ((reinterpret_cast<uintptr_t>(P.ep.bias) | reinterpret_cast<uintptr_t>(P.ep.scale)) & 15) == 0 && P.ldc % 4 == 0 &&
            (reinterpret_cast<uintptr_t>(P.out) & 15) == 0 &&
            (!res || (P.ep.ldr % 4 == 0 && (reinterpret_cast<uintptr_t>(res) & 15) == 0));
 }
@@ -312,6 +313,7 @@ __device__ __forceinline__ void epilogue_block_reduce(const EpiParams& P, const 
     __syncwarp();
     float4* row = reinterpret_cast<float4*>(stage) + lane * 8;
     const bool bias_vec = with_bias && P.ep.bias && (reinterpret_cast<uintptr_t>(P.ep.bias) & 15) == 0 && col0 + 32 <= P.n;
+    const bool scale_vec = (reinterpret_cast<uintptr_t>(P.ep.scale) & 15) == 0 && col0 + 32 <= P.n;
 #pragma unroll
     for (int g = 0; g < 8; ++g) {
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -322,8 +324,17 @@ __device__ __forceinline__ void epilogue_block_reduce(const EpiParams& P, const 
             b = make_float4(c < P.n ? P.ep.bias[c] : 0.f, c + 1 < P.n ? P.ep.bias[c + 1] : 0.f,
                             c + 2 < P.n ? P.ep.bias[c + 2] : 0.f, c + 3 < P.n ? P.ep.bias[c + 3] : 0.f);
         }
-        const float4 v = act4(make_float4(acc[4 * g] + b.x, acc[4 * g + 1] + b.y, acc[4 * g + 2] + b.z, acc[4 * g + 3] + b.w),
-                              P.ep.activation);
+        float4 v = act4(make_float4(acc[4 * g] + b.x, acc[4 * g + 1] + b.y, acc[4 * g + 2] + b.z, acc[4 * g + 3] + b.w), P.ep.activation);
+        if (P.ep.scale) {
+            const uint32_t c = col0 + 4 * g;
+            if (scale_vec) {
+                const float4 f = __ldg(reinterpret_cast<const float4*>(P.ep.scale + c));
+                v = make_float4(v.x * f.x, v.y * f.y, v.z * f.z, v.w * f.w);
+            } else {
+                v = make_float4(c < P.n ? v.x * P.ep.scale[c] : 0.f, c + 1 < P.n ? v.y * P.ep.scale[c + 1] : 0.f,
+                                c + 2 < P.n ? v.z * P.ep.scale[c + 2] : 0.f, c + 3 < P.n ? v.w * P.ep.scale[c + 3] : 0.f);
+            }
+        }
         row[(g ^ lane) & 7] = v;     // 16-byte chunk g of row r sits at g ^ (r & 7)
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -547,13 +558,15 @@ __device__ __forceinline__ void epilogue_block(const EpiParams& P, float* stage,
             }
             float4 bv = make_float4(0.f, 0.f, 0.f, 0.f);
             if (P.ep.bias) bv = __ldg(reinterpret_cast<const float4*>(P.ep.bias + col0 + c4));
+            float4 sv = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (P.ep.scale) sv = __ldg(reinterpret_cast<const float4*>(P.ep.scale + col0 + c4));
 #pragma unroll
             for (uint32_t it = 0; it < 8; ++it) {
                 const uint32_t rr = it * 4 + rsub;
                 if (rr < rows) {
                     float4 v = stage_load4(stage, rr, c4);
                     v = act4(make_float4(v.x + bv.x, v.y + bv.y, v.z + bv.z, v.w + bv.w), P.ep.activation);
-                    v = make_float4(v.x + r4[it].x, v.y + r4[it].y, v.z + r4[it].z, v.w + r4[it].w);
+                    v = make_float4(fmaf(v.x, sv.x, r4[it].x), fmaf(v.y, sv.y, r4[it].y), fmaf(v.z, sv.z, r4[it].z), fmaf(v.w, sv.w, r4[it].w));
                     *reinterpret_cast<float4*>(out + map_out_row(P.ep, row0 + rr) * P.ldc + col0 + c4) = v;
                 }
             }
@@ -565,10 +578,11 @@ __device__ __forceinline__ void epilogue_block(const EpiParams& P, float* stage,
             for (int rr = 0; rr < 32; ++rr)
                 rv[rr] = (res && col_ok && (uint32_t)rr < rows) ? res[(size_t)(row0 + rr) * P.ep.ldr + col] : 0.0f;
             const float bv = (P.ep.bias && col_ok) ? __ldg(P.ep.bias + col) : 0.0f;
+            const float sv = (P.ep.scale && col_ok) ? __ldg(P.ep.scale + col) : 1.0f;
 #pragma unroll
             for (int rr = 0; rr < 32; ++rr)
                 if (col_ok && (uint32_t)rr < rows)
-                    out[map_out_row(P.ep, row0 + rr) * P.ldc + col] = apply_activation(stage[stage_index(rr, lane)] + bv, P.ep.activation) + rv[rr];
+                    out[map_out_row(P.ep, row0 + rr) * P.ldc + col] = fmaf(apply_activation(stage[stage_index(rr, lane)] + bv, P.ep.activation), sv, rv[rr]);
         }
     }
     __syncwarp();  // the buffer is reused by the next block

@@ -46,6 +46,7 @@ struct SkShape {
 
 struct SkParams {
     const float* bias;
+    const float* scale;
     const float* residual;
     uint32_t ldr;
     int activation, out_dtype;
@@ -66,6 +67,7 @@ __device__ __forceinline__ void sk_store(const SkParams& P, uint32_t row, uint32
     if (P.out_dtype == TNSR_B200_BF16) {
         reinterpret_cast<bf16*>(P.out)[(size_t)row * P.ldc + col] = __float2bfloat16_rn(v);
     } else {
+        if (P.scale) v *= __ldg(P.scale + col);
         if (P.residual) v += P.residual[(size_t)row * P.ldr + col];
         reinterpret_cast<float*>(P.out)[(size_t)row * P.ldc + col] = v;
     }
@@ -283,6 +285,7 @@ int launch_gemm_skinny(const bf16* a, const bf16* bt, void* out, uint32_t ldc, u
     const uint32_t tiles = ceil_div(n, (uint32_t)SK_ROWS), num_kb = ceil_div(k, (uint32_t)SK_BK);
     SkParams prm;
     prm.bias = ep.bias;
+    prm.scale = ep.scale;
     prm.residual = ep.residual;
     prm.ldr = ep.ldr;
     prm.activation = ep.activation;

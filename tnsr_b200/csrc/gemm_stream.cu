@@ -36,6 +36,7 @@ struct GsParams {
     void* out;
     uint32_t ldc, m, n, k;
     const float* bias;
+    const float* scale;
     const float* residual;
     uint32_t ldr;
     int activation, out_dtype;
@@ -179,6 +180,7 @@ gemm_stream_kernel(GsParams P) {
                     if (P.out_dtype == TNSR_B200_BF16) {
                         reinterpret_cast<bf16*>(P.out)[(size_t)m * P.ldc + colg] = __float2bfloat16_rn(v);
                     } else {
+                        if (P.scale) v *= __ldg(P.scale + colg);
                         if (P.residual) v += P.residual[(size_t)m * P.ldr + colg];
                         reinterpret_cast<float*>(P.out)[(size_t)m * P.ldc + colg] = v;
                     }
@@ -239,7 +241,7 @@ int launch_gemm_stream(const bf16* a, const bf16* bt, void* out, uint32_t ldc, u
     (void)d_status;      // nothing in this kernel waits on another agent: there is no time-out to report
     GsParams P = {};
     P.a = a; P.w = bt; P.out = out; P.ldc = ldc; P.m = m; P.n = n; P.k = k;
-    P.bias = ep.bias; P.residual = ep.residual; P.ldr = ep.ldr; P.activation = ep.activation; P.out_dtype = ep.out_dtype;
+    P.bias = ep.bias; P.scale = ep.scale; P.residual = ep.residual; P.ldr = ep.ldr; P.activation = ep.activation; P.out_dtype = ep.out_dtype;
     return m <= 8 ? gs_launch<8>(P, stream) : gs_launch<16>(P, stream);
 }
 

@@ -1,4 +1,5 @@
-// Grouped-query attention with capped scores and a sigmoid gate per head, bf16 caches, any widths up to 256.
+// Grouped-query attention with capped scores and a sigmoid gate per head, or with sigmoid weights that are not normalised
+// over keys, over all earlier keys or a window of them; bf16 caches, any widths up to 256.
 //
 // The query heads that share a key/value head are rows of one matrix product: row r of a (session, key/value head) is
 // query token r / per and head r % per of the group (per = heads / kv_heads), so a K/V tile is loaded once for the whole
@@ -13,7 +14,8 @@
 //
 // Scores, softmax statistics and accumulators are f32; the weights enter the value product as two bf16 halves
 // (split_bf16x2), so they keep 16 bits.  A capped score costs three special-function results instead of one:
-// cap tanh(u) = cap (1 - 2 / (1 + exp(2u))).
+// cap tanh(u) = cap (1 - 2 / (1 + exp(2u))).  Sigmoid weights (SIGMOID) need neither maximum nor sum: partial results of
+// warps and splits are added as they are.  With a window, tiles before the first row's window are never read.
 #include <algorithm>
 
 #include "mixers.cuh"
@@ -35,6 +37,10 @@ __device__ __forceinline__ float ga_score(float s, const GaScore& f) {
     const float e = mx_ex2(s * f.pre);                   // exp(2u)
     return fmaf(-2.0f * f.post, mx_rcp(e + 1.0f), f.post);
 }
+// Weight of a key with sigmoid scores: s = q . k, pre = -scale log2(e), bias2 = -bias log2(e).
+__device__ __forceinline__ float ga_sigmoid(float s, float pre, float bias2) { return mx_rcp(1.0f + mx_ex2(fmaf(s, pre, bias2))); }
+// First visible key of a query at position `limit`.
+__device__ __forceinline__ uint32_t ga_first(uint32_t limit, uint32_t window) { return window && limit >= window ? limit + 1 - window : 0u; }
 static GaScore make_score(float scale, float softcap) {
     GaScore f;
     f.capped = softcap > 0.0f;
@@ -74,7 +80,7 @@ __device__ __forceinline__ void ga_copy(uint8_t* dst, const bf16* src, size_t sr
 }
 
 __device__ __forceinline__ float ga_gate(const GroupedAttention& a, size_t row, uint32_t h) {
-    return a.gate ? 1.0f / (1.0f + __expf(-a.gate[row * a.gate_ld + h])) : 1.0f;
+    return a.gate ? a.gain / (1.0f + __expf(-a.gate[row * a.gate_ld + h])) : a.gain;
 }
 // Columns of the output rows past the last head.
 __device__ __forceinline__ void ga_zero_pad(const GroupedAttention& a, size_t row, uint32_t tid, uint32_t threads) {
@@ -93,7 +99,7 @@ struct SplitShape {
 };
 
 // UPPER: rows 8 .. 15 of the tile are in use (more than 8 rows).
-template <int DK, int DV, int STAGES, bool UPPER>
+template <int DK, int DV, int STAGES, bool UPPER, bool SIGMOID>
 __global__ void __launch_bounds__(GA_WARPS * 32)
 grouped_split_kernel(GaParams P) {
     using S = SplitShape<DK, DV, STAGES>;
@@ -107,10 +113,17 @@ grouped_split_kernel(GaParams P) {
     const uint32_t p0 = P.place.pos(s), row0 = tile * 16;
     const uint32_t n_rows = min(16u, P.rows - row0);
     const uint32_t keys = min(p0 + (row0 + n_rows - 1) / P.per + 1, a.capacity);    // visible to the tile's last row
-    const uint32_t tiles = (keys + 15) / 16, per_split = (tiles + P.splits - 1) / P.splits;
-    const uint32_t tile0 = min(tiles, split * per_split), tile1 = min(tiles, tile0 + per_split);
+    const uint32_t tiles = (keys + 15) / 16, first_tile = ga_first(p0 + row0 / P.per, a.window) / 16;      // of the tile's first row
+    const uint32_t per_split = (tiles - first_tile + P.splits - 1) / P.splits;
+    const uint32_t tile0 = min(tiles, first_tile + split * per_split), tile1 = min(tiles, tile0 + per_split);
 
     const uint32_t lim0 = p0 + (row0 + min(g8, n_rows - 1)) / P.per, lim1 = p0 + (row0 + min(g8 + 8, n_rows - 1)) / P.per;
+    const uint32_t low0 = ga_first(lim0, a.window), low1 = ga_first(lim1, a.window);
+    float bias0 = 0.0f, bias1 = 0.0f;      // of the two rows' heads, SIGMOID
+    if (SIGMOID && a.head_bias) {
+        bias0 = -GA_LOG2E * a.head_bias[kvh * P.per + (row0 + min(g8, n_rows - 1)) % P.per];
+        bias1 = -GA_LOG2E * a.head_bias[kvh * P.per + (row0 + min(g8 + 8, n_rows - 1)) % P.per];
+    }
 
     uint8_t* ring = smem + warp * (STAGES * S::STAGE);
     const size_t k_ld = (size_t)a.kv_heads * a.dim, v_ld = (size_t)a.kv_heads * a.vdim;
@@ -170,13 +183,29 @@ grouped_split_kernel(GaParams P) {
         for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) sc[n][e] += odd[n][e];
+        uint32_t hi[4] = {0u, 0u, 0u, 0u}, lo[4] = {0u, 0u, 0u, 0u};
+        if (SIGMOID) {
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                float w[4];
+#pragma unroll
+                for (int e = 0; e < (UPPER ? 4 : 2); ++e) {
+                    const uint32_t key = i * 16 + n * 8 + t4 * 2 + (e & 1);
+                    const bool seen = key <= (e < 2 ? lim0 : lim1) && key >= (e < 2 ? low0 : low1);
+                    w[e] = seen ? ga_sigmoid(sc[n][e], P.score.pre, e < 2 ? bias0 : bias1) : 0.0f;
+                }
+                split_bf16x2(w[0], w[1], hi[2 * n], lo[2 * n]);
+                if (UPPER) split_bf16x2(w[2], w[3], hi[2 * n + 1], lo[2 * n + 1]);
+            }
+        } else {
         float mx0 = m0, mx1 = m1;
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < (UPPER ? 4 : 2); ++e) {
                 const uint32_t key = i * 16 + n * 8 + t4 * 2 + (e & 1);
-                const float v = key <= (e < 2 ? lim0 : lim1) ? ga_score(sc[n][e], P.score) : -INFINITY;
+                const bool seen = key <= (e < 2 ? lim0 : lim1) && key >= (e < 2 ? low0 : low1);
+                const float v = seen ? ga_score(sc[n][e], P.score) : -INFINITY;
                 sc[n][e] = v;
                 if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
             }
@@ -192,7 +221,6 @@ grouped_split_kernel(GaParams P) {
             c1 = mx_ex2(m1 - ms1);
             m1 = mx1;
         }
-        uint32_t hi[4] = {0u, 0u, 0u, 0u}, lo[4] = {0u, 0u, 0u, 0u};
         float r0 = 0.0f, r1 = 0.0f;
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
@@ -209,6 +237,7 @@ grouped_split_kernel(GaParams P) {
         l1 = l1 * c1 + r1;
 #pragma unroll
         for (int n = 0; n < DV / 8; ++n) { o[n][0] *= c0; o[n][1] *= c0; if (UPPER) { o[n][2] *= c1; o[n][3] *= c1; } }
+        }
         // 64 columns at a time, the two halves of a weight eight products apart: one accumulator's products wait for each other
 #pragma unroll
         for (int n0 = 0; n0 < DV / 16; n0 += 4) {
@@ -261,6 +290,14 @@ grouped_split_kernel(GaParams P) {
     };
     for (uint32_t i = threadIdx.x; i < n_rows * a.vdim; i += blockDim.x) {
         const uint32_t r = i / a.vdim, c = i % a.vdim;
+        if (SIGMOID) {
+            float sum = 0.0f;
+#pragma unroll
+            for (uint32_t w = 0; w < GA_WARPS; ++w) sum += mg[(w * 16 + r) * RW + c];
+            if (P.splits == 1) finish(r, c, sum);
+            else P.partial[((slot * P.splits + split) * 16 + r) * RW + c] = sum;
+            continue;
+        }
         float mx = -INFINITY;
 #pragma unroll
         for (uint32_t w = 0; w < GA_WARPS; ++w) mx = fmaxf(mx, mg[(w * 16 + r) * RW + DV]);
@@ -292,6 +329,12 @@ grouped_split_kernel(GaParams P) {
     for (uint32_t i = threadIdx.x; i < n_rows * a.vdim; i += blockDim.x) {
         const uint32_t r = i / a.vdim, c = i % a.vdim;
         const float* src = P.partial + (slot * P.splits * 16 + r) * RW;
+        if (SIGMOID) {
+            float sum = 0.0f;
+            for (uint32_t w = 0; w < P.splits; ++w) sum += __ldcg(src + (size_t)w * 16 * RW + c);
+            finish(r, c, sum);
+            continue;
+        }
         float mx = -INFINITY;
         for (uint32_t w = 0; w < P.splits; ++w) mx = fmaxf(mx, __ldcg(src + (size_t)w * 16 * RW + DV));
         float num = 0.0f, den = 0.0f;
@@ -314,7 +357,7 @@ struct TileShape {
     static constexpr uint32_t BYTES = Q_BYTES + 2 * (K_BYTES + V_BYTES);
 };
 
-template <int DK, int DV, int BK>
+template <int DK, int DV, int BK, bool SIGMOID>
 __global__ void __launch_bounds__(128)
 grouped_tile_kernel(GaParams P) {
     using S = TileShape<DK, DV, BK>;
@@ -329,7 +372,7 @@ grouped_tile_kernel(GaParams P) {
     const uint32_t tile = P.row_tiles - 1 - blockIdx.x, kvh = blockIdx.y, s = blockIdx.z;
     const uint32_t p0 = P.place.pos(s), row0 = tile * 64, n_rows = min(64u, P.rows - row0);
     const uint32_t keys = min(p0 + (row0 + n_rows - 1) / P.per + 1, a.capacity);
-    const uint32_t blocks = (keys + BK - 1) / BK;
+    const uint32_t blocks = (keys + BK - 1) / BK, block0 = ga_first(p0 + row0 / P.per, a.window) / BK;
     const size_t k_ld = (size_t)a.kv_heads * a.dim, v_ld = (size_t)a.kv_heads * a.vdim, q_ld = (size_t)a.heads * a.dim;
 
     {   // query rows: row r is token r / per, head r % per of the group
@@ -360,7 +403,7 @@ grouped_tile_kernel(GaParams P) {
                         a.vdim, P.vec, threadIdx.x, 128);
         }
     };
-    load(0, 0);
+    load(block0, block0 & 1);
     mx_commit();
 
     constexpr bool KEEP_Q = DK <= 128;
@@ -374,18 +417,25 @@ grouped_tile_kernel(GaParams P) {
     const uint32_t lim0 = p0 + (row0 + min(r0, n_rows - 1)) / P.per, lim1 = p0 + (row0 + min(r1, n_rows - 1)) / P.per;
     const uint32_t warp_first = p0 + (row0 + min(warp * 16, n_rows - 1)) / P.per;          // limit of the warp's first row
     const uint32_t warp_last = p0 + (row0 + min(warp * 16 + 15, n_rows - 1)) / P.per;
+    const uint32_t low0 = ga_first(lim0, a.window), low1 = ga_first(lim1, a.window);
+    const uint32_t warp_low = ga_first(warp_first, a.window), warp_low_last = ga_first(warp_last, a.window);
+    float bias0 = 0.0f, bias1 = 0.0f;      // of the two rows' heads, SIGMOID
+    if (SIGMOID && a.head_bias) {
+        bias0 = -GA_LOG2E * a.head_bias[kvh * P.per + (row0 + min(r0, n_rows - 1)) % P.per];
+        bias1 = -GA_LOG2E * a.head_bias[kvh * P.per + (row0 + min(r1, n_rows - 1)) % P.per];
+    }
 
-    for (uint32_t b = 0; b < blocks; ++b) {
+    for (uint32_t b = block0; b < blocks; ++b) {
         if (b + 1 < blocks) load(b + 1, (b + 1) & 1);
         mx_commit();
         mx_wait<1>();
         __syncthreads();
-        if (KEEP_Q && b == 0) {
+        if (KEEP_Q && b == block0) {
 #pragma unroll
             for (int kk = 0; kk < (KEEP_Q ? DK / 16 : 1); ++kk) mx_ldsm(q_addr + kk * 32, qa[kk]);
         }
         const uint32_t sk = mx_smem(skv + (b & 1) * (S::K_BYTES + S::V_BYTES)), sv = sk + S::K_BYTES;
-        if (b * BK <= warp_last) {
+        if (b * BK <= warp_last && b * BK + BK > warp_low) {
             float sc[BK / 8][4];
 #pragma unroll
             for (int i = 0; i < BK / 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
@@ -402,14 +452,29 @@ grouped_tile_kernel(GaParams P) {
                     mx_mma(sc[2 * n + 1], q4, bb[2], bb[3]);
                 }
             }
-            const bool mask = b * BK + BK - 1 > warp_first;
+            const bool mask = b * BK + BK - 1 > warp_first || b * BK < warp_low_last;
+            auto hidden = [&](int i, int e) {
+                const uint32_t key = b * BK + i * 8 + t4 * 2 + (e & 1);
+                return key > (e < 2 ? lim0 : lim1) || key < (e < 2 ? low0 : low1);
+            };
+            if (SIGMOID) {
+#pragma unroll
+                for (int i = 0; i < BK / 8; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float w = ga_sigmoid(sc[i][e], P.score.pre, e < 2 ? bias0 : bias1);
+                        sc[i][e] = mask && hidden(i, e) ? 0.0f : w;
+                    }
+            }
+            float ms0 = 0.0f, ms1 = 0.0f;
+            if (!SIGMOID) {
             float mx0 = m0, mx1 = m1;
 #pragma unroll
             for (int i = 0; i < BK / 8; ++i) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     float v = ga_score(sc[i][e], P.score);
-                    if (mask && b * BK + i * 8 + t4 * 2 + (e & 1) > (e < 2 ? lim0 : lim1)) v = -INFINITY;
+                    if (mask && hidden(i, e)) v = -INFINITY;
                     sc[i][e] = v;
                 }
                 mx0 = fmaxf(mx0, fmaxf(sc[i][0], sc[i][1]));
@@ -419,7 +484,8 @@ grouped_tile_kernel(GaParams P) {
             mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
             mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-            const float ms0 = mx0 == -INFINITY ? 0.0f : mx0, ms1 = mx1 == -INFINITY ? 0.0f : mx1;
+            ms0 = mx0 == -INFINITY ? 0.0f : mx0;
+            ms1 = mx1 == -INFINITY ? 0.0f : mx1;
             const float c0 = mx_ex2(m0 - ms0), c1 = mx_ex2(m1 - ms1);
             m0 = mx0;
             m1 = mx1;
@@ -427,15 +493,16 @@ grouped_tile_kernel(GaParams P) {
             l1 *= c1;
 #pragma unroll
             for (int i = 0; i < DV / 8; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+            }
 #pragma unroll
             for (int kk = 0; kk < BK / 16; ++kk) {
                 uint32_t hi[4], lo[4];
 #pragma unroll
                 for (int n = 0; n < 2; ++n) {
                     const float* v = sc[2 * kk + n];
-                    const float pa = mx_ex2(v[0] - ms0), pb = mx_ex2(v[1] - ms0), pc = mx_ex2(v[2] - ms1), pd = mx_ex2(v[3] - ms1);
-                    l0 += pa + pb;
-                    l1 += pc + pd;
+                    const float pa = SIGMOID ? v[0] : mx_ex2(v[0] - ms0), pb = SIGMOID ? v[1] : mx_ex2(v[1] - ms0);
+                    const float pc = SIGMOID ? v[2] : mx_ex2(v[2] - ms1), pd = SIGMOID ? v[3] : mx_ex2(v[3] - ms1);
+                    if (!SIGMOID) { l0 += pa + pb; l1 += pc + pd; }
                     split_bf16x2(pa, pb, hi[2 * n], lo[2 * n]);
                     split_bf16x2(pc, pd, hi[2 * n + 1], lo[2 * n + 1]);
                 }
@@ -472,7 +539,7 @@ grouped_tile_kernel(GaParams P) {
         if (r >= n_rows) continue;
         const uint32_t R = row0 + r, h = kvh * P.per + R % P.per;
         const size_t row = (size_t)s * P.place.chunk + R / P.per;
-        const float f = ga_gate(a, row, h) / (half ? l1 : l0);
+        const float f = SIGMOID ? ga_gate(a, row, h) : ga_gate(a, row, h) / (half ? l1 : l0);
         bf16* dst = out + row * a.out_ld + (size_t)h * a.vdim;
 #pragma unroll
         for (int i = 0; i < DV / 8; ++i) {
@@ -503,25 +570,35 @@ int allow_smem(K kernel, uint32_t bytes, bool* configured) {
     return TNSR_B200_OK;
 }
 
-template <int DK, int DV, int STAGES, bool UPPER>
-int launch_split(const GaParams& P, cudaStream_t stream) {
+template <int DK, int DV, int STAGES, bool UPPER, bool SIGMOID>
+int launch_split_kind(const GaParams& P, cudaStream_t stream) {
     static bool configured[64] = {};
     const uint32_t bytes = SplitShape<DK, DV, STAGES>::BYTES;
-    int rc = allow_smem(grouped_split_kernel<DK, DV, STAGES, UPPER>, bytes, configured);
+    int rc = allow_smem(grouped_split_kernel<DK, DV, STAGES, UPPER, SIGMOID>, bytes, configured);
     if (rc) return rc;
-    launch_kernel(grouped_split_kernel<DK, DV, STAGES, UPPER>, dim3(P.splits, P.a.kv_heads * P.row_tiles, P.place.sessions), dim3(GA_WARPS * 32), bytes,
+    launch_kernel(grouped_split_kernel<DK, DV, STAGES, UPPER, SIGMOID>, dim3(P.splits, P.a.kv_heads * P.row_tiles, P.place.sessions), dim3(GA_WARPS * 32), bytes,
                   stream, P);
+    return TNSR_B200_OK;
+}
+
+template <int DK, int DV, int STAGES, bool UPPER>
+int launch_split(const GaParams& P, cudaStream_t stream) {
+    return P.a.score_kind == TNSR_B200_SCORE_SIGMOID ? launch_split_kind<DK, DV, STAGES, UPPER, true>(P, stream) : launch_split_kind<DK, DV, STAGES, UPPER, false>(P, stream);
+}
+
+template <int DK, int DV, int BK, bool SIGMOID>
+int launch_tile_kind(const GaParams& P, cudaStream_t stream) {
+    static bool configured[64] = {};
+    const uint32_t bytes = TileShape<DK, DV, BK>::BYTES;
+    int rc = allow_smem(grouped_tile_kernel<DK, DV, BK, SIGMOID>, bytes, configured);
+    if (rc) return rc;
+    launch_kernel(grouped_tile_kernel<DK, DV, BK, SIGMOID>, dim3(P.row_tiles, P.a.kv_heads, P.place.sessions), dim3(128), bytes, stream, P);
     return TNSR_B200_OK;
 }
 
 template <int DK, int DV, int BK>
 int launch_tile(const GaParams& P, cudaStream_t stream) {
-    static bool configured[64] = {};
-    const uint32_t bytes = TileShape<DK, DV, BK>::BYTES;
-    int rc = allow_smem(grouped_tile_kernel<DK, DV, BK>, bytes, configured);
-    if (rc) return rc;
-    launch_kernel(grouped_tile_kernel<DK, DV, BK>, dim3(P.row_tiles, P.a.kv_heads, P.place.sessions), dim3(128), bytes, stream, P);
-    return TNSR_B200_OK;
+    return P.a.score_kind == TNSR_B200_SCORE_SIGMOID ? launch_tile_kind<DK, DV, BK, true>(P, stream) : launch_tile_kind<DK, DV, BK, false>(P, stream);
 }
 
 uint32_t padded_width(uint32_t dim, uint32_t vdim) {
@@ -561,6 +638,7 @@ int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, 
     P.a = a;
     P.place = place;
     P.score = make_score(a.scale, a.softcap);
+    if (a.score_kind == TNSR_B200_SCORE_SIGMOID) P.score.pre = -GA_LOG2E * a.scale;
     P.per = a.heads / a.kv_heads;
     const uint64_t rows = (uint64_t)place.chunk * P.per;
     if (rows > 0x7fffffffull) { set_thread_error("grouped attention: too many rows"); return TNSR_B200_ERR_UNSUPPORTED; }
@@ -576,6 +654,7 @@ int launch_grouped_attention(const GroupedAttention& a, const StepPlace& place, 
         P.row_tiles = ceil_div(P.rows, 16u);
         const uint64_t units = (uint64_t)place.sessions * a.kv_heads * P.row_tiles;
         P.splits = splits_for(units, w);
+        if (a.window) P.splits = std::min(P.splits, std::max(1u, ceil_div(a.window + place.chunk, 16 * GA_WARPS)));   // a tile per warp at least
         if (!a.workspace || a.workspace_bytes < grouped_attention_workspace_bytes(a.dim, a.vdim)) P.splits = 1;
         if (P.splits > 1) {
             P.done = reinterpret_cast<uint32_t*>(a.workspace);

@@ -3,6 +3,7 @@
 //
 //  * attention_prep_kernel     one warp per (head unit, run of tokens): the convolution slides over the run in
 //                              registers, so every projected value is read once; q rows and cache rows come out.
+//  * attention_rotary_kernel   the same without convolution and norm: rotation (either layout) of q and k, cache rows.
 //  * grouped_attention_rows    one warp per (session, head, query), keys in order: f32 sessions, and every shape the
 //                              tensor-core kernels (grouped_attention.cu) leave out.
 #include <algorithm>
@@ -278,10 +279,100 @@ static void prep_width(const AttentionPrep& a, const StepPlace& place, uint32_t 
     else prep_taps<T, 4>(a, place, run, runs, total, vec, stream);
 }
 
+// ---- rotation alone --------------------------------------------------------------------------------
+// A thread owns EPT rotated pairs (or 2 EPT plain channels) of one head of one row: with EPT 8 in the layout of halves,
+// 16 bytes of the first half and 16 bytes of the second.  Heads of q, k and v are units of one row; a unit has `tasks`
+// threads.  VEC: 16-byte accesses (bf16, EPT 8) or single elements (EPT 1).
+template <typename T, int EPT>
+__global__ void __launch_bounds__(256)
+attention_rotary_kernel(AttentionPrep a, StepPlace place, uint32_t tasks, uint64_t total) {
+    pdl_wait();
+    pdl_trigger();
+    const uint64_t id = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (id >= total) return;
+    const uint32_t units = a.heads + 2 * a.kv_heads;
+    const uint32_t task = (uint32_t)(id % tasks), unit = (uint32_t)(id / tasks % units);
+    const uint32_t row = (uint32_t)(id / ((uint64_t)tasks * units)), s = row / place.chunk, t = row % place.chunk;
+    const uint32_t nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+    const uint32_t which = unit < a.heads ? 0u : unit < a.heads + a.kv_heads ? 1u : 2u;
+    const uint32_t head = which == 0 ? unit : which == 1 ? unit - a.heads : unit - a.heads - a.kv_heads;
+    const uint32_t width = which == 2 ? a.vdim : a.dim, turned = which == 2 ? 0u : a.rotary_dims, half = turned / 2;
+    const uint32_t pos = place.pos(s) + t;
+    const T* src = reinterpret_cast<const T*>(a.proj) + (size_t)row * a.ld + (which == 0 ? head * a.dim : which == 1 ? nq + head * a.dim : nq + nk + head * a.vdim);
+    T* dst;
+    if (which == 0) {
+        dst = reinterpret_cast<T*>(a.q) + (size_t)row * nq + head * a.dim;
+    } else {
+        const size_t kr = kv_row(a.paging, s, pos, a.capacity);
+        dst = which == 1 ? reinterpret_cast<T*>(a.k_cache) + kr * nk + head * a.dim : reinterpret_cast<T*>(a.v_cache) + kr * nv + head * a.vdim;
+    }
+    // tasks [0, half / EPT) turn pairs; the rest copies channels from `turned` on, 2 EPT at a time
+    const uint32_t pair_tasks = half / EPT;
+    if (task < pair_tasks) {
+        const uint32_t i0 = task * EPT;
+        const float2* angle = a.rotation + (size_t)pos * half + i0;
+        const bool halves = a.rotary_layout == TNSR_B200_ROTARY_HALVES;
+        const uint32_t c0 = halves ? i0 : 2 * i0, c1 = halves ? i0 + half : 2 * i0 + EPT;
+        if (EPT == 8) {
+            const uint4 x4 = *reinterpret_cast<const uint4*>(src + c0), y4 = *reinterpret_cast<const uint4*>(src + c1);
+            const uint32_t x[4] = {x4.x, x4.y, x4.z, x4.w}, y[4] = {y4.x, y4.y, y4.z, y4.w};
+            uint32_t ox[4], oy[4];
+#pragma unroll
+            for (int w = 0; w < 4; ++w) {
+                const float2 u = bf16x2_to_f32(x[w]), v = bf16x2_to_f32(y[w]);
+                if (halves) {        // word w: pairs 2w and 2w + 1, u from the first half, v from the second
+                    const float4 cs = __ldg(reinterpret_cast<const float4*>(angle) + w);
+                    ox[w] = pack_bf16x2(u.x * cs.x - v.x * cs.y, u.y * cs.z - v.y * cs.w);
+                    oy[w] = pack_bf16x2(v.x * cs.x + u.x * cs.y, v.y * cs.z + u.y * cs.w);
+                } else {             // word w of the first 16 bytes: pair w; of the second: pair 4 + w
+                    const float2 ca = __ldg(angle + w), cb = __ldg(angle + 4 + w);
+                    ox[w] = pack_bf16x2(u.x * ca.x - u.y * ca.y, u.y * ca.x + u.x * ca.y);
+                    oy[w] = pack_bf16x2(v.x * cb.x - v.y * cb.y, v.y * cb.x + v.x * cb.y);
+                }
+            }
+            *reinterpret_cast<uint4*>(dst + c0) = make_uint4(ox[0], ox[1], ox[2], ox[3]);
+            *reinterpret_cast<uint4*>(dst + c1) = make_uint4(oy[0], oy[1], oy[2], oy[3]);
+        } else {
+            const float2 cs = *angle;
+            const float u = to_f32(src[c0]), v = to_f32(src[c1]);
+            dst[c0] = from_f32<T>(u * cs.x - v * cs.y);
+            dst[c1] = from_f32<T>(v * cs.x + u * cs.y);
+        }
+        return;
+    }
+    const uint32_t c = turned + (task - pair_tasks) * 2 * EPT;
+    if (EPT == 8) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+            if (c + 8 * i < width) *reinterpret_cast<uint4*>(dst + c + 8 * i) = *reinterpret_cast<const uint4*>(src + c + 8 * i);
+    } else {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+            if (c + i < width) dst[c + i] = src[c + i];
+    }
+}
+
+static int launch_attention_rotary(const AttentionPrep& a, const StepPlace& place, int dtype, cudaStream_t stream) {
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool wide = dtype == TNSR_B200_BF16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.rotary_dims % 16 == 0 && aligned(a.proj) &&
+                      aligned(a.q) && aligned(a.k_cache) && aligned(a.v_cache) && aligned(a.rotation);
+    const uint32_t ept = wide ? 8 : 1;
+    const uint32_t tasks = std::max(a.rotary_dims / 2 / ept + ceil_div(a.dim - a.rotary_dims, 2 * ept), ceil_div(a.vdim, 2 * ept));
+    const uint64_t total = (uint64_t)place.sessions * place.chunk * (a.heads + 2 * a.kv_heads) * tasks;
+    if (ceil_div64(total, 256) > 0x7fffffffull) { set_thread_error("attention: too many rows for one launch"); return TNSR_B200_ERR_UNSUPPORTED; }
+    const dim3 grid((uint32_t)ceil_div64(total, 256)), block(256);
+    if (wide) launch_kernel(attention_rotary_kernel<bf16, 8>, grid, block, 0, stream, a, place, tasks, total);
+    else if (dtype == TNSR_B200_BF16) launch_kernel(attention_rotary_kernel<bf16, 1>, grid, block, 0, stream, a, place, tasks, total);
+    else launch_kernel(attention_rotary_kernel<float, 1>, grid, block, 0, stream, a, place, tasks, total);
+    count_launch();
+    return check_launch("attention_rotary");
+}
+
 int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dtype, cudaStream_t stream) {
     if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
-    if (a.dim > 256 || a.vdim > 256 || a.taps == 0 || a.taps > kMaxConvTaps || a.rotary_dims > a.dim || a.rotary_dims % 2) {
-        set_thread_error("attention: head widths up to 256, 1..16 convolution taps, an even number of rotated dimensions");
+    if (!a.conv_w && a.dim <= 256 && a.vdim <= 256 && a.rotary_dims <= a.dim && a.rotary_dims % 2 == 0) return launch_attention_rotary(a, place, dtype, stream);
+    if (a.rotary_layout != TNSR_B200_ROTARY_INTERLEAVED || a.dim > 256 || a.vdim > 256 || a.taps == 0 || a.taps > kMaxConvTaps || a.rotary_dims > a.dim || a.rotary_dims % 2) {
+        set_thread_error("attention: head widths up to 256, 1..16 convolution taps (behind one the interleaved rotation), an even number of rotated dimensions");
         return TNSR_B200_ERR_UNSUPPORTED;
     }
     const uint32_t run = std::min(place.chunk, 32u), runs = ceil_div(place.chunk, run);
@@ -344,7 +435,9 @@ grouped_attention_rows_kernel(GroupedAttention a, StepPlace place, uint32_t tota
     const T* kb = reinterpret_cast<const T*>(a.k_cache) + (size_t)g * a.dim;
     const T* vb = reinterpret_cast<const T*>(a.v_cache) + (size_t)g * a.vdim;
     const size_t k_ld = (size_t)a.kv_heads * a.dim, v_ld = (size_t)a.kv_heads * a.vdim;
-    const uint32_t keys = min(place.pos(s) + t + 1, a.capacity);
+    const uint32_t keys = min(place.pos(s) + t + 1, a.capacity), first = a.window && keys > a.window ? keys - a.window : 0u;
+    const bool sigmoid = a.score_kind == TNSR_B200_SCORE_SIGMOID;
+    const float bias = sigmoid && a.head_bias ? a.head_bias[h] : 0.0f;
     float q[GR_SLOTS], acc[GR_SLOTS];
 #pragma unroll
     for (int i = 0; i < GR_SLOTS; ++i) {
@@ -353,7 +446,7 @@ grouped_attention_rows_kernel(GroupedAttention a, StepPlace place, uint32_t tota
         acc[i] = 0.0f;
     }
     float m = -INFINITY, l = 0.0f;
-    for (uint32_t j = 0; j < keys; ++j) {
+    for (uint32_t j = first; j < keys; ++j) {
         const size_t kr = kv_row(a.paging, s, j, a.capacity);
         float part = 0.0f;
 #pragma unroll
@@ -362,6 +455,15 @@ grouped_attention_rows_kernel(GroupedAttention a, StepPlace place, uint32_t tota
             if (c < a.dim) part = fmaf(q[i], to_f32(kb[kr * k_ld + c]), part);
         }
         float sc = mx_warp_sum(part) * a.scale;
+        if (sigmoid) {
+            const float p = 1.0f / (1.0f + expf(-(sc + bias)));
+#pragma unroll
+            for (int i = 0; i < GR_SLOTS; ++i) {
+                const uint32_t c = lane + 32 * i;
+                if (c < a.vdim) acc[i] = fmaf(p, to_f32(vb[kr * v_ld + c]), acc[i]);
+            }
+            continue;
+        }
         if (a.softcap > 0.0f) sc = a.softcap * tanhf(sc / a.softcap);
         const float m_new = fmaxf(m, sc);
         const float corr = expf(m - m_new), p = expf(sc - m_new);
@@ -373,7 +475,8 @@ grouped_attention_rows_kernel(GroupedAttention a, StepPlace place, uint32_t tota
         }
         m = m_new;
     }
-    const float gate = a.gate ? 1.0f / (1.0f + expf(-a.gate[row * a.gate_ld + h])) : 1.0f;
+    const float gate = a.gain * (a.gate ? 1.0f / (1.0f + expf(-a.gate[row * a.gate_ld + h])) : 1.0f);
+    if (sigmoid) l = 1.0f;
     T* orow = reinterpret_cast<T*>(a.out) + row * a.out_ld;
 #pragma unroll
     for (int i = 0; i < GR_SLOTS; ++i) {

@@ -2,7 +2,7 @@
 //     S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t
 // with x, B, C behind a causal convolution and silu, dt behind softplus, then y * silu(z) and an RMS norm in groups.
 //
-//  * conv_silu_kernel          convolution + silu, sliding window in registers (single-token steps also update the ring)
+//  * short_conv_kernel         convolution (+ silu), sliding window in registers (single-token steps also update the ring)
 //  * ssd_token_kernel          token by token with the state in registers: single-token steps (the state makes one trip
 //                              through HBM), short chunks, f32 sessions
 //  * gated_norm_kernel         the grouped RMS norm of y * silu(z)
@@ -18,7 +18,6 @@ int launch_ssd_scan(const Mamba2& m, const StepPlace& place, cudaStream_t stream
 // Shortest chunk that takes the chunked tensor-core scan; below it the token kernel's few steps are cheaper.
 constexpr uint32_t SSD_SCAN_MIN_TOKENS = 16;
 
-__device__ __forceinline__ float full_silu(float x) { return x / (1.0f + expf(-x)); }
 // silu of an activation that is stored in T: bf16 results come from the hardware exponential, f32 ones from expf.
 template <typename T>
 __device__ __forceinline__ float act_silu(float x);
@@ -26,15 +25,14 @@ template <>
 __device__ __forceinline__ float act_silu<float>(float x) { return full_silu(x); }
 template <>
 __device__ __forceinline__ float act_silu<bf16>(float x) { return mx_silu(x); }
-__device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 
-// ---- convolution + silu ----------------------------------------------------------------------
+// ---- convolution (+ silu) --------------------------------------------------------------------
 // A thread owns two neighbouring channels of a run of tokens.
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool SILU>
 __global__ void __launch_bounds__(128)
-conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, const float* __restrict__ conv_w,
-                 const float* __restrict__ conv_b, T* __restrict__ ring, T* __restrict__ out, StepPlace place, uint32_t run,
-                 uint32_t vec) {
+short_conv_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uint32_t taps, const float* __restrict__ conv_w,
+                  const float* __restrict__ conv_b, T* __restrict__ ring, T* __restrict__ out, uint32_t part, StepPlace place,
+                  uint32_t run, uint32_t vec) {
     pdl_wait();
     pdl_trigger();
     const uint32_t c = 2 * (blockIdx.x * blockDim.x + threadIdx.x);
@@ -43,7 +41,16 @@ conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uin
     const uint32_t s = blockIdx.z, t0 = blockIdx.y * run, t1 = min(place.chunk, t0 + run);
     const uint32_t p0 = place.pos(s);
     const T* in = rows + (size_t)s * place.chunk * ld + c;
-    T* dst = out + (size_t)s * place.chunk * channels + c;
+    // output parts of `part` channels, each [rows, part]; the two channels of a thread may lie in different ones
+    const size_t part_elems = (size_t)place.sessions * place.chunk * part;
+    T* dst = out + c / part * part_elems + (size_t)s * place.chunk * part + c % part;
+    T* dst1 = out + (c + 1) / part * part_elems + (size_t)s * place.chunk * part + (c + 1) % part;
+    auto put = [&](uint32_t t, float2 y) {
+        if (SILU) y = make_float2(act_silu<T>(y.x), act_silu<T>(y.y));
+        if (vec) { store_pair<T>(dst + (size_t)t * part, y, true, true); return; }
+        dst[(size_t)t * part] = from_f32<T>(y.x);
+        if (second) dst1[(size_t)t * part] = from_f32<T>(y.y);
+    };
     float2 w[TAPS], win[TAPS];
     const float* cw = conv_w + (size_t)c * taps;
     if (TAPS == 4 && taps == 4) {
@@ -80,7 +87,7 @@ conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uin
             y.x = fmaf(w[j].x, u.x, y.x);
             y.y = fmaf(w[j].y, u.y, y.y);
         }
-        store_pair<T>(dst, make_float2(act_silu<T>(y.x), act_silu<T>(y.y)), vec, second);
+        put(0, y);
         store_pair<T>(ring + ((size_t)s * taps + p0 % taps) * channels + c, now, vec, second);
         return;
     }
@@ -99,23 +106,40 @@ conv_silu_kernel(const T* __restrict__ rows, uint32_t ld, uint32_t channels, uin
             float2 y = b;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) { y.x = fmaf(w[j].x, win[j].x, y.x); y.y = fmaf(w[j].y, win[j].y, y.y); }
-            if (t + i < t1) store_pair<T>(dst + (size_t)(t + i) * channels, make_float2(act_silu<T>(y.x), act_silu<T>(y.y)), vec, second);
+            if (t + i < t1) put(t + i, y);
         }
     }
 }
 
-template <typename T>
-static void conv_silu_typed(const Mamba2& m, uint32_t inner, uint32_t channels, const StepPlace& place, cudaStream_t stream) {
+template <typename T, bool SILU>
+static void short_conv_typed(const ShortConv& c, const StepPlace& place, cudaStream_t stream) {
     const uint32_t run = std::min(place.chunk, 32u);
-    const dim3 grid(ceil_div(ceil_div(channels, 2u), 128u), ceil_div(place.chunk, run), place.sessions);
-    const T* rows = (const T*)m.proj + inner;
-    const uint32_t vec = inner % 2 == 0 && channels % 2 == 0 && m.ld % 2 == 0;
-    if (m.taps <= 4)
-        launch_kernel(conv_silu_kernel<T, 4>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b, (T*)m.ring,
-                      (T*)m.xbc, place, run, vec);
+    const dim3 grid(ceil_div(ceil_div(c.channels, 2u), 128u), ceil_div(place.chunk, run), place.sessions);
+    auto even = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % (2 * sizeof(T)) == 0; };
+    const uint32_t vec = c.channels % 2 == 0 && c.ld % 2 == 0 && c.part % 2 == 0 && even(c.rows) && even(c.ring) && even(c.out);
+    if (c.taps <= 4)
+        launch_kernel(short_conv_kernel<T, 4, SILU>, grid, dim3(128), 0, stream, (const T*)c.rows, c.ld, c.channels, c.taps, c.w, c.b, (T*)c.ring,
+                      (T*)c.out, c.part, place, run, vec);
     else
-        launch_kernel(conv_silu_kernel<T, kMaxConvTaps>, grid, dim3(128), 0, stream, rows, m.ld, channels, m.taps, m.conv_w, m.conv_b,
-                      (T*)m.ring, (T*)m.xbc, place, run, vec);
+        launch_kernel(short_conv_kernel<T, kMaxConvTaps, SILU>, grid, dim3(128), 0, stream, (const T*)c.rows, c.ld, c.channels, c.taps, c.w, c.b,
+                      (T*)c.ring, (T*)c.out, c.part, place, run, vec);
+}
+
+int launch_short_conv(const ShortConv& c, const StepPlace& place, int dtype, cudaStream_t stream) {
+    if (place.sessions == 0 || place.chunk == 0) return TNSR_B200_OK;
+    if (c.taps == 0 || c.taps > kMaxConvTaps || c.part == 0 || c.channels % c.part || place.sessions > 65535u || ceil_div(place.chunk, 32u) > 65535u) {
+        set_thread_error("convolution: 1..16 taps, parts that divide the channels, at most 65535 sessions");
+        return TNSR_B200_ERR_UNSUPPORTED;
+    }
+    const bool bf = dtype == TNSR_B200_BF16;
+    if (bf && c.silu) short_conv_typed<bf16, true>(c, place, stream);
+    else if (bf) short_conv_typed<bf16, false>(c, place, stream);
+    else if (c.silu) short_conv_typed<float, true>(c, place, stream);
+    else short_conv_typed<float, false>(c, place, stream);
+    count_launch();
+    int rc = check_launch("short_conv");
+    if (rc) return rc;
+    return place.chunk > 1 ? launch_conv_ring(c.rows, c.ld, c.channels, c.taps, c.ring, place, dtype, stream) : TNSR_B200_OK;
 }
 
 // ---- token by token ----------------------------------------------------------------------------
@@ -305,13 +329,10 @@ int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream
     }
     const bool bf = dtype == TNSR_B200_BF16;
     int rc;
-    if (bf) conv_silu_typed<bf16>(m, inner, channels, place, stream); else conv_silu_typed<float>(m, inner, channels, place, stream);
-    count_launch();
-    if ((rc = check_launch("conv_silu"))) return rc;
-    if (place.chunk > 1) {
-        const uint8_t* raw = (const uint8_t*)m.proj + (size_t)inner * (bf ? 2 : 4);
-        if ((rc = launch_conv_ring(raw, m.ld, channels, m.taps, m.ring, place, dtype, stream))) return rc;
-    }
+    ShortConv c;
+    c.rows = (const uint8_t*)m.proj + (size_t)inner * (bf ? 2 : 4);
+    c.ld = m.ld; c.channels = c.part = channels; c.taps = m.taps; c.w = m.conv_w; c.b = m.conv_b; c.ring = m.ring; c.out = m.xbc; c.silu = true;
+    if ((rc = launch_short_conv(c, place, dtype, stream))) return rc;
     if (bf && m.engine == 0 && place.chunk >= SSD_SCAN_MIN_TOKENS) {
         if ((rc = launch_ssd_scan(m, place, stream))) return rc;
     } else {

@@ -31,6 +31,7 @@ int launch_conv_ring(const void* rows, uint32_t ld, uint32_t channels, uint32_t 
 
 // ---- attention ------------------------------------------------------------------
 // Projected rows [q | k | v] -> convolution over time -> per-head RMS norm of q and k -> rotation -> q rows and cache rows.
+// conv_w == nullptr: rotation alone (no convolution, no norm, no ring), in either layout.
 struct AttentionPrep {
     const void* proj = nullptr;        // [rows, ld], channels q | k | v
     uint32_t ld = 0;
@@ -40,6 +41,7 @@ struct AttentionPrep {
     const float* k_norm = nullptr;
     float eps = 0.0f;
     uint32_t rotary_dims = 0;
+    uint32_t rotary_layout = TNSR_B200_ROTARY_INTERLEAVED;   // halves: without a convolution only
     const float2* rotation = nullptr;  // [position][rotary_dims / 2] (cos, sin)
     void* ring = nullptr;              // [sessions, taps, channels]
     void* q = nullptr;                 // [rows, heads * dim]
@@ -51,13 +53,18 @@ struct AttentionPrep {
 int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dtype, cudaStream_t stream);
 
 // Grouped-query causal attention with capped scores and a sigmoid gate per head:
-// out[row, h * vdim ..] = sigmoid(gate[row, h]) * softmax(cap(q . k * scale)) . v ; columns [heads * vdim, out_cols) are zeroed.
+// out[row, h * vdim ..] = gain * sigmoid(gate[row, h]) * softmax(cap(q . k * scale)) . v ; columns [heads * vdim, out_cols)
+// are zeroed.  window > 0: a query sees itself and the window - 1 keys before it.  score_kind SIGMOID: the weight of a
+// visible key is sigmoid(q . k * scale + head_bias[h]), not normalised over keys (softcap does not apply).
 struct GroupedAttention {
     const void* q = nullptr;
     const void* k_cache = nullptr;
     const void* v_cache = nullptr;
     uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, capacity = 0;
     float scale = 0.0f, softcap = 0.0f;   // softcap 0: scores as they are
+    float gain = 1.0f;
+    uint32_t window = 0, score_kind = TNSR_B200_SCORE_SOFTMAX;
+    const float* head_bias = nullptr;     // [heads], sigmoid scores
     const float* gate = nullptr;          // [rows, gate_ld], nullptr: no gate
     uint32_t gate_ld = 0;
     void* out = nullptr;
@@ -100,8 +107,68 @@ struct Mamba2 {
 bool mamba2_supported(uint32_t heads, uint32_t vdim, uint32_t state);
 int launch_mamba2(const Mamba2& m, const StepPlace& place, int dtype, cudaStream_t stream);
 
+// ---- convolution alone ------------------------------------------------------------
+// out = [silu](conv(rows) + bias), reading and updating the session's ring.  Output channels may be cut into parts of
+// `part` channels, each a matrix [rows, part] of its own.
+struct ShortConv {
+    const void* rows = nullptr;        // [rows, ld]
+    uint32_t ld = 0, channels = 0, taps = 0, part = 0;   // part: channels, or a divisor of it
+    const float* w = nullptr;          // [channels, taps]
+    const float* b = nullptr;
+    void* ring = nullptr;              // [sessions, taps, channels]
+    void* out = nullptr;               // [channels / part][rows][part]
+    bool silu = false;
+};
+int launch_short_conv(const ShortConv& c, const StepPlace& place, int dtype, cudaStream_t stream);
+
+// ---- HGRN2 ------------------------------------------------------------------------
+// f = l + (1 - l) sigmoid(f_raw + b);  S <- diag(f) S + (1 - f) v^T;  o = S^T silu(q);  out = gain * norm_w * o / rms(o)
+struct Hgrn2 {
+    const void* q = nullptr;           // [rows, ld], before silu
+    const void* v = nullptr;           // [rows, ld]
+    uint32_t ld = 0;
+    const float* f = nullptr;          // [rows, f_ld], before bias and sigmoid
+    uint32_t f_ld = 0;
+    uint32_t heads = 0, dim = 0, vdim = 0;
+    const float* f_bias = nullptr;     // [heads * dim]
+    const float* lower = nullptr;      // [heads * dim]
+    const float* norm_w = nullptr;     // [vdim]
+    float eps = 0.0f, gain = 1.0f;
+    float* state = nullptr;            // [sessions, heads, dim, vdim]
+    float* raw = nullptr;              // [rows, heads * vdim] scratch, used when vdim > HGRN2_FUSED_VDIM
+    void* out = nullptr;               // [rows, out_ld]; columns [heads * vdim, out_cols) are zeroed
+    uint32_t out_ld = 0, out_cols = 0;
+    int engine = 0;                    // 0: best kernel for the shape, 1: token by token
+};
+constexpr uint32_t HGRN2_FUSED_VDIM = 128;   // value width up to which the kernels norm their own output
+bool hgrn2_supported(uint32_t heads, uint32_t dim, uint32_t vdim);
+int launch_hgrn2(const Hgrn2& m, const StepPlace& place, int dtype, cudaStream_t stream);
+
+// ---- real-gated linear recurrent unit ------------------------------------------------
+struct Rglru {
+    const void* proj = nullptr;        // [rows, ld]: y (after gelu) from column 0, x from column x_col
+    uint32_t ld = 0, x_col = 0;
+    uint32_t width = 0, blocks = 0, taps = 0;
+    const float* conv_w = nullptr;     // [width, taps]
+    const float* conv_b = nullptr;
+    const void* gate_w = nullptr;      // [blocks, 2 n, n]: rows of r, then of i; n = width / blocks
+    const float* r_bias = nullptr;     // [width]
+    const float* i_bias = nullptr;
+    const float* lambda = nullptr;     // [width]
+    void* ring = nullptr;              // [sessions, taps, width]
+    float* state = nullptr;            // [sessions, width]
+    void* u = nullptr;                 // [blocks, rows, n] scratch: convolved x
+    float* gates = nullptr;            // [blocks, rows, 2 n] scratch
+    void* out = nullptr;               // [rows, out_ld]; columns [width, out_cols) are zeroed
+    uint32_t out_ld = 0, out_cols = 0;
+    int* d_status = nullptr;
+};
+int launch_rglru(const Rglru& m, const StepPlace& place, int dtype, cudaStream_t stream);
+
 // ---- device helpers ----------------------------------------------------------------
 #ifdef __CUDACC__
+__device__ __forceinline__ float full_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 // Two neighbouring channels as f32; one access when `vec` (even address), else element by element (`second`: the second
 // one exists).
 template <typename T>

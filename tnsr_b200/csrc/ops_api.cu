@@ -2,6 +2,7 @@
 // include/tnsr_b200.h).  They queue work on the caller's stream and never
 // synchronise or allocate.
 #include "common.cuh"
+#include "feed_forward.cuh"
 #include "mixers.cuh"
 
 using namespace tb;
@@ -179,6 +180,7 @@ static StepPlace step_place(const tnsr_b200_place* p) {
 int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args, const tnsr_b200_place* place, void* stream) {
     if (!args || !place || !args->q || !args->k_cache || !args->v_cache || !args->out) return bad("grouped_attention: null pointer");
     if (args->dtype != TNSR_B200_F32 && args->dtype != TNSR_B200_BF16) return bad("grouped_attention: dtype must be f32 or bf16");
+    if (args->score_kind > TNSR_B200_SCORE_SIGMOID) return bad("grouped_attention: unknown score kind");
     if (args->heads == 0 || args->dim == 0 || args->vdim == 0 || args->capacity == 0 || args->out_ld < args->out_cols ||
         args->out_cols < args->heads * args->vdim)
         return bad("grouped_attention: sizes must be positive and the output row must hold every head");
@@ -189,6 +191,7 @@ int tnsr_b200_grouped_attention(const tnsr_b200_grouped_attention_args* args, co
     a.scale = args->scale; a.softcap = args->softcap; a.gate = args->gate; a.gate_ld = args->gate_ld;
     a.out = args->out; a.out_ld = args->out_ld; a.out_cols = args->out_cols;
     a.d_status = args->d_status; a.workspace = args->workspace; a.workspace_bytes = args->workspace_bytes; a.engine = args->engine;
+    a.head_bias = args->head_bias; a.window = args->window; a.score_kind = args->score_kind; a.gain = args->gain != 0.0f ? args->gain : 1.0f;
     return launch_grouped_attention(a, step_place(place), args->dtype, as_stream(stream));
 }
 
@@ -207,6 +210,88 @@ int tnsr_b200_mamba2(const tnsr_b200_mamba2_args* args, const tnsr_b200_place* p
     m.eps = args->eps; m.ring = args->ring; m.ssm = args->ssm; m.xbc = args->xbc; m.gated = args->gated;
     m.out = args->out; m.out_ld = args->out_ld; m.out_cols = args->out_cols; m.engine = args->engine;
     return launch_mamba2(m, step_place(place), args->dtype, as_stream(stream));
+}
+
+static bool two_types(int32_t dtype) { return dtype == TNSR_B200_F32 || dtype == TNSR_B200_BF16; }
+
+int tnsr_b200_rotary(const tnsr_b200_rotary_args* args, const tnsr_b200_place* place, void* stream) {
+    if (!args || !place || !args->proj || !args->q || !args->k_cache || !args->v_cache || (args->rotary_dims && !args->rotation)) return bad("rotary: null pointer");
+    if (!two_types(args->dtype) || args->rotary_layout > TNSR_B200_ROTARY_HALVES) return bad("rotary: bad dtype or layout");
+    if (args->heads == 0 || args->kv_heads == 0 || args->dim == 0 || args->vdim == 0 || args->rotary_dims > args->dim || args->rotary_dims % 2 ||
+        args->ld < args->heads * args->dim + args->kv_heads * (args->dim + args->vdim))
+        return bad("rotary: sizes must be positive, rotated dimensions even and the rows must hold q, k and v");
+    if (!place->d_positions && (uint64_t)place->position + place->chunk > args->capacity) return bad("rotary: the chunk ends past the capacity");
+    AttentionPrep p;
+    p.proj = args->proj; p.ld = args->ld; p.heads = args->heads; p.kv_heads = args->kv_heads; p.dim = args->dim; p.vdim = args->vdim;
+    p.rotary_dims = args->rotary_dims; p.rotary_layout = args->rotary_layout; p.rotation = (const float2*)args->rotation;
+    p.q = args->q; p.k_cache = args->k_cache; p.v_cache = args->v_cache; p.capacity = args->capacity;
+    return launch_attention_prep(p, step_place(place), args->dtype, as_stream(stream));
+}
+
+int tnsr_b200_hgrn2(const tnsr_b200_hgrn2_args* args, const tnsr_b200_place* place, void* stream) {
+    if (!args || !place || !args->q || !args->v || !args->f || !args->f_bias || !args->lower || !args->norm_w || !args->state || !args->out)
+        return bad("hgrn2: null pointer");
+    if (!two_types(args->dtype)) return bad("hgrn2: dtype must be f32 or bf16");
+    if (args->heads == 0 || args->dim == 0 || args->vdim == 0 || args->f_ld < args->heads * args->dim || args->out_ld < args->out_cols ||
+        args->out_cols < args->heads * args->vdim)
+        return bad("hgrn2: sizes must be positive and the rows must hold every head");
+    Hgrn2 m;
+    m.q = args->q; m.v = args->v; m.ld = args->ld; m.f = args->f; m.f_ld = args->f_ld; m.heads = args->heads; m.dim = args->dim; m.vdim = args->vdim;
+    m.f_bias = args->f_bias; m.lower = args->lower; m.norm_w = args->norm_w; m.eps = args->eps; m.gain = args->gain; m.state = args->state; m.raw = args->raw;
+    m.out = args->out; m.out_ld = args->out_ld; m.out_cols = args->out_cols; m.engine = args->engine;
+    return launch_hgrn2(m, step_place(place), args->dtype, as_stream(stream));
+}
+
+int tnsr_b200_rglru(const tnsr_b200_rglru_args* args, const tnsr_b200_place* place, void* stream) {
+    if (!args || !place || !args->proj || !args->gate_w || !args->conv_w || !args->conv_b || !args->r_bias || !args->i_bias || !args->lambda ||
+        !args->ring || !args->state || !args->u || !args->gates || !args->out)
+        return bad("rglru: null pointer");
+    if (!two_types(args->dtype)) return bad("rglru: dtype must be f32 or bf16");
+    if (args->width == 0 || args->x_col < args->width || args->ld < args->x_col + args->width || args->out_ld < args->out_cols || args->out_cols < args->width)
+        return bad("rglru: the rows must hold y, x and the output");
+    Rglru m;
+    m.proj = args->proj; m.ld = args->ld; m.x_col = args->x_col; m.width = args->width; m.blocks = args->blocks; m.taps = args->taps;
+    m.conv_w = args->conv_w; m.conv_b = args->conv_b; m.gate_w = args->gate_w; m.r_bias = args->r_bias; m.i_bias = args->i_bias; m.lambda = args->lambda;
+    m.ring = args->ring; m.state = args->state; m.u = args->u; m.gates = args->gates; m.out = args->out; m.out_ld = args->out_ld; m.out_cols = args->out_cols;
+    m.d_status = args->d_status;
+    return launch_rglru(m, step_place(place), args->dtype, as_stream(stream));
+}
+
+int tnsr_b200_polynorm(const void* z, const float* act, void* out, uint32_t rows, uint32_t width, uint32_t out_ld, uint32_t out_cols, float epsilon,
+                       int dtype, void* stream) {
+    if (!z || !act || !out) return bad("polynorm: null pointer");
+    if (!two_types(dtype) || width == 0 || out_cols < width || out_ld < out_cols || !(epsilon > 0.0f)) return bad("polynorm: bad dtype, sizes or epsilon");
+    return launch_polynorm(z, act, out, rows, width, out_ld, out_cols, epsilon, dtype, as_stream(stream));
+}
+
+int tnsr_b200_gemm_grouped(const void* a, const void* w, void* out, const uint32_t* offsets, uint32_t groups, uint32_t rows, uint32_t n, uint32_t k,
+                           int activation, int dtype, int out_dtype, int engine, int* d_status, void* stream) {
+    if (!a || !w || !out) return bad("gemm_grouped: null pointer");
+    if (!two_types(dtype) || !two_types(out_dtype)) return bad("gemm_grouped: dtype must be f32 or bf16");
+    GroupedGemm g;
+    g.a = a; g.w = w; g.out = out; g.offsets = offsets; g.groups = groups; g.rows = rows; g.n = n; g.k = k; g.activation = activation;
+    g.out_dtype = out_dtype; g.d_status = d_status; g.engine = engine;
+    return launch_gemm_grouped(g, dtype, as_stream(stream));
+}
+
+uint64_t tnsr_b200_experts_workspace(uint32_t rows, uint32_t d, uint32_t ff, uint32_t experts, uint32_t top, int dtype) {
+    return experts_workspace_bytes(rows, d, ff, experts, top, dtype);
+}
+
+int tnsr_b200_experts(const tnsr_b200_experts_args* args, void* stream) {
+    if (!args || !args->logits || !args->correction || !args->h || !args->up || !args->down || !args->x || !args->workspace ||
+        (args->norm_out && !args->norm_w))
+        return bad("experts: null pointer");
+    if (!two_types(args->dtype)) return bad("experts: dtype must be f32 or bf16");
+    if (args->d == 0 || args->ff == 0 || args->logits_ld < args->experts + args->identity_experts) return bad("experts: bad sizes");
+    Experts e;
+    e.logits = args->logits; e.correction = args->correction; e.h = args->h; e.up = args->up; e.down = args->down; e.x = args->x;
+    e.layer_scale = args->layer_scale; e.norm_w = args->norm_w; e.norm_out = args->norm_out; e.workspace = args->workspace;
+    e.workspace_bytes = args->workspace_bytes; e.chosen = args->chosen; e.weights = args->weights; e.d_status = args->d_status; e.rows = args->rows;
+    e.logits_ld = args->logits_ld; e.d = args->d; e.ff = args->ff; e.experts = args->experts; e.identity = args->identity_experts; e.top = args->top;
+    e.router_scale = args->router_scale; e.norm_offset = args->norm_offset; e.eps = args->eps; e.engine = args->engine;
+    int rc = launch_experts(e, args->dtype, as_stream(stream));
+    return rc ? rc : launch_experts_combine(e, args->dtype, as_stream(stream));
 }
 
 }  // extern "C"

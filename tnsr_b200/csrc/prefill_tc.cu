@@ -37,7 +37,9 @@
 //                                                             the following p_full, i.e. after the fold)
 //
 // Grouped-query form (described models): query head h reads key/value head h / per, scores may be capped (cap tanh(s / cap),
-// monotonic, so the row maximum is still taken over raw scores), and a sigmoid gate per (row, head) scales the output.
+// monotonic, so the row maximum is still taken over raw scores), and a sigmoid gate per (row, head) scales the output.  With
+// a window the key blocks of an item start at the first one its first query sees.  Sigmoid weights (PT_SIGMOID) are not
+// normalised over keys: there is no maximum, no rescaling, and P V of all blocks accumulates in TMEM, read once per item.
 //
 // Every wait is bounded; a wait that gives up raises the CTA's abort flag, the
 // roles fall through to the common teardown and the status word is set.
@@ -78,15 +80,21 @@ struct PtParams {
     uint32_t out_ld, out_cols; // output rows: pitch, columns (those past the heads are zeroed)
     const float* gate;         // [rows, gate_ld] or nullptr
     uint32_t gate_ld;
+    uint32_t window;           // 0: all earlier keys; else a query sees itself and the window - 1 keys before it
+    float gain;                // factor of the output
+    const float* head_bias;    // sigmoid scores: added to q . k * scale, may be null
     float cap_pre, cap_post;   // capped scores in log2 units: cap_post - 2 cap_post / (1 + exp2(s cap_pre))
     int* d_status;
     uint64_t wait_limit_ns;
 };
 
-template <bool CAPPED>
+enum : int { PT_SOFTMAX = 0, PT_CAPPED = 1, PT_SIGMOID = 2 };
+
+template <int KIND>
 __global__ void __launch_bounds__(PT_THREADS, 2)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PtParams prm) {
+    constexpr bool CAPPED = KIND == PT_CAPPED, SIGMOID = KIND == PT_SIGMOID;
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw_addr = smem_u32(smem_raw);
     uint8_t* smem = smem_raw + ((1024u - (raw_addr & 1023u)) & 1023u);
@@ -113,14 +121,16 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // (a running count of key blocks for the K/V ring, S, P and O; a running count of items for Q) stay in step.
     const uint32_t per_tile = prm.heads * prm.sessions;
     const uint32_t total_items = prm.q_tiles * per_tile;
-    auto item_coords = [&](uint32_t item, uint32_t& q0, uint32_t& h, uint32_t& s, uint32_t& n_blocks) {
+    auto item_coords = [&](uint32_t item, uint32_t& q0, uint32_t& h, uint32_t& s, uint32_t& block0, uint32_t& n_blocks) {
         const uint32_t q_tile_index = prm.q_tiles - 1 - item / per_tile, rem = item % per_tile;
         q0 = q_tile_index * PT_BQ;
         h = rem % prm.heads;
         s = rem / prm.heads;
         const uint32_t last_q = min(q0 + PT_BQ, prm.chunk) - 1;
         const uint32_t total = prm.position + last_q + 1;          // keys visible to the tile's last query
-        n_blocks = (total + PT_BK - 1) / PT_BK;
+        const uint32_t first = prm.position + q0 + 1;              // keys up to the tile's first query
+        block0 = prm.window && first > prm.window ? (first - prm.window) / PT_BK : 0u;
+        n_blocks = (total + PT_BK - 1) / PT_BK - block0;
     };
 
     if (threadIdx.x == 0) {
@@ -151,8 +161,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             uint32_t g = 0, it = 0;     // key blocks and items so far
             bool ok = true;
             for (uint32_t item = blockIdx.x; ok && item < total_items; item += gridDim.x, ++it) {
-                uint32_t q0, h, s, n_blocks;
-                item_coords(item, q0, h, s, n_blocks);
+                uint32_t q0, h, s, block0, n_blocks;
+                item_coords(item, q0, h, s, block0, n_blocks);
                 // the Q tile is free once every S product of the previous item has been computed
                 if (it > 0 && !mbar_wait(q_empty, (it - 1) & 1, abort_flag, prm.wait_limit_ns)) break;
                 mbar_expect_tx(q_full, PT_TILE_BYTES);
@@ -162,8 +172,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     if (!mbar_wait(kv_empty + stage, ((g / PT_KV_STAGES) & 1) ^ 1, abort_flag, prm.wait_limit_ns)) { ok = false; break; }
                     uint8_t* dst = kv_ring + stage * PT_KV_BYTES;
                     mbar_expect_tx(kv_full + stage, PT_KV_BYTES);
-                    tma_load_3d(dst, &map_k, (int32_t)(h / prm.per * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
-                    tma_load_3d(dst + PT_TILE_BYTES, &map_v, (int32_t)(h / prm.per * PT_HD), (int32_t)(j * PT_BK), (int32_t)s, kv_full + stage);
+                    tma_load_3d(dst, &map_k, (int32_t)(h / prm.per * PT_HD), (int32_t)((block0 + j) * PT_BK), (int32_t)s, kv_full + stage);
+                    tma_load_3d(dst + PT_TILE_BYTES, &map_v, (int32_t)(h / prm.per * PT_HD), (int32_t)((block0 + j) * PT_BK), (int32_t)s, kv_full + stage);
                 }
             }
         }
@@ -181,8 +191,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             uint32_t g = 0, it = 0;
             bool ok = true;
             for (uint32_t item = blockIdx.x; ok && item < total_items; item += gridDim.x, ++it) {
-                uint32_t q0, h, s, n_blocks;
-                item_coords(item, q0, h, s, n_blocks);
+                uint32_t q0, h, s, block0, n_blocks;
+                item_coords(item, q0, h, s, block0, n_blocks);
                 if (!mbar_wait(q_full, it & 1, abort_flag, prm.wait_limit_ns)) break;
                 if (!mbar_wait(kv_full + g % PT_KV_STAGES, (g / PT_KV_STAGES) & 1, abort_flag, prm.wait_limit_ns)) break;
                 // the score buffer is free: its last reader signalled p_full of the previous block, which was waited for below
@@ -210,7 +220,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     for (uint32_t kk = 0; kk < PT_BK / 16; ++kk) {
                         const uint64_t pdesc = make_kmajor_sw128_desc(kk < 4 ? p_lower : smem_u32(p_upper)) + (kk & 3) * 2;
                         const uint64_t vdesc = make_mnmajor_sw128_desc(v_addr + kk * 2048, PT_TILE_BYTES, 1024);
-                        umma_bf16(tmem_base + PT_O_COL, pdesc, vdesc, PT_IDESC_O, kk != 0);
+                        umma_bf16(tmem_base + PT_O_COL, pdesc, vdesc, PT_IDESC_O, kk != 0 || (SIGMOID && j > 0));
                     }
                     umma_commit(o_full);
                     umma_commit(kv_empty + stage);   // both products of this ring stage are done
@@ -239,10 +249,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             return true;
         };
         for (uint32_t item = blockIdx.x; ok && item < total_items; item += gridDim.x) {
-            uint32_t q0, h, s, n_blocks;
-            item_coords(item, q0, h, s, n_blocks);
+            uint32_t q0, h, s, block0, n_blocks;
+            item_coords(item, q0, h, s, block0, n_blocks);
             const uint32_t q_idx = min(q0 + row, prm.chunk - 1);
             const uint32_t limit = prm.position + q_idx;             // last visible key of this row
+            const uint32_t low = prm.window && limit >= prm.window ? limit + 1 - prm.window : 0u;   // first one
+            const float bias2 = SIGMOID && prm.head_bias ? -1.4426950408889634f * prm.head_bias[h] : 0.0f;
             float acc[32];                                           // output columns [32 half, 32 half + 32)
 #pragma unroll
             for (int i = 0; i < 32; ++i) acc[i] = 0.0f;
@@ -264,8 +276,15 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (!mbar_wait(s_full, b & 1, abort_flag, prm.wait_limit_ns)) { ok = false; break; }
                 tc_fence_after();
                 const uint32_t taddr = lane_taddr + half * 64;
-                const uint32_t kbase = j * PT_BK + half * 64;           // first key of this thread's columns
-                const bool need_mask = kbase + 63 > limit;
+                const uint32_t kbase = (block0 + j) * PT_BK + half * 64;           // first key of this thread's columns
+                const bool need_mask = kbase + 63 > limit || kbase < low;
+                auto hidden = [&](uint32_t key) { return key > limit || key < low; };
+                float corr = 0.0f, neg = 0.0f;
+                if (SIGMOID) {
+                    // the previous P V must have read the upper P tile; its result stays in TMEM
+                    if (j > 0 && !mbar_wait(o_full, (b - 1) & 1, abort_flag, prm.wait_limit_ns)) { ok = false; break; }
+                    tc_fence_after();
+                } else {
                 // pass 1: maximum of the raw scores of the own 64 columns (four independent chains)
                 float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -275,7 +294,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     tmem_ld_wait();
                     if (need_mask) {
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) if (kbase + c * 32 + i > limit) v[i] = -INFINITY;
+                        for (int i = 0; i < 32; ++i) if (hidden(kbase + c * 32 + i)) v[i] = -INFINITY;
                     }
 #pragma unroll
                     for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], v[i]);
@@ -286,12 +305,13 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 const float ms = (mx == -INFINITY) ? 0.0f : mx;
                 // the first block has nothing to rescale (its corr is 0, or finite when capped)
                 const float top = CAPPED ? capped(ms) : ms * sl2;
-                const float corr = CAPPED ? pt_ex2(capped(m) - top) : pt_ex2((m - ms) * sl2);
+                corr = CAPPED ? pt_ex2(capped(m) - top) : pt_ex2((m - ms) * sl2);
                 m = mx;
-                const float neg = -top;
+                neg = -top;
                 // the previous block's output; once it is complete the upper P tile may be overwritten
                 if (j > 0 && !fold(b - 1, corr_pending)) { ok = false; break; }
                 corr_pending = corr;
+                }
                 // pass 2: p = exp2(s * scale - m * scale) as bf16 into this thread's 128-byte row of the P tile
                 // (16-byte chunk c of row r at c ^ (r & 7))
                 uint8_t* p_row = (half ? p_upper : kv_ring + (b % PT_KV_STAGES) * PT_KV_BYTES) + row * 128u;
@@ -301,26 +321,33 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     float v[32];
                     tmem_ld32(taddr + c * 32, v);
                     tmem_ld_wait();
-                    if (need_mask) {
+                    if (need_mask && !SIGMOID) {
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) if (kbase + c * 32 + i > limit) v[i] = -INFINITY;
+                        for (int i = 0; i < 32; ++i) if (hidden(kbase + c * 32 + i)) v[i] = -INFINITY;
                     }
                     uint32_t packed[16];
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         float p0, p1;
-                        if (CAPPED) {
+                        if (SIGMOID) {           // sl2 = -scale log2(e)
+                            p0 = mx_rcp(1.0f + pt_ex2(fmaf(v[2 * i], sl2, bias2)));
+                            p1 = mx_rcp(1.0f + pt_ex2(fmaf(v[2 * i + 1], sl2, bias2)));
+                            if (need_mask) {
+                                if (hidden(kbase + c * 32 + 2 * i)) p0 = 0.0f;
+                                if (hidden(kbase + c * 32 + 2 * i + 1)) p1 = 0.0f;
+                            }
+                        } else if (CAPPED) {
                             p0 = pt_ex2(capped(v[2 * i]) + neg);
                             p1 = pt_ex2(capped(v[2 * i + 1]) + neg);
                             if (need_mask) {      // a capped score is finite also for a hidden key
-                                if (kbase + c * 32 + 2 * i > limit) p0 = 0.0f;
-                                if (kbase + c * 32 + 2 * i + 1 > limit) p1 = 0.0f;
+                                if (hidden(kbase + c * 32 + 2 * i)) p0 = 0.0f;
+                                if (hidden(kbase + c * 32 + 2 * i + 1)) p1 = 0.0f;
                             }
                         } else {
                             p0 = pt_ex2(fmaf(v[2 * i], sl2, neg));
                             p1 = pt_ex2(fmaf(v[2 * i + 1], sl2, neg));
                         }
-                        rs4[i & 3] += p0 + p1;
+                        if (!SIGMOID) rs4[i & 3] += p0 + p1;
                         packed[i] = pack_bf16x2(p0, p1);
                     }
 #pragma unroll
@@ -340,10 +367,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (!ok) break;
             ok = fold(g + n_blocks - 1, corr_pending);
             float l_other = 0.0f;
-            if (ok) ok = exchange(l, l_other);
+            if (ok && !SIGMOID) ok = exchange(l, l_other);
             if (ok && q0 + row < prm.chunk) {
                 const size_t out_row = (size_t)s * prm.chunk + q0 + row;
-                float inv = 1.0f / (l + l_other);
+                float inv = SIGMOID ? prm.gain : prm.gain / (l + l_other);
                 if (prm.gate) inv *= 1.0f / (1.0f + __expf(-prm.gate[out_row * prm.gate_ld + h]));
                 bf16* og = prm.out + out_row * prm.out_ld + (size_t)h * PT_HD + half * 32;
                 if (h + 1 == prm.heads && half == 1)
@@ -404,7 +431,7 @@ bool prefill_attention_tc_eligible(uint32_t sessions, uint32_t chunk, uint32_t p
     return encode_fn() != nullptr;
 }
 
-template <bool CAPPED>
+template <int KIND>
 static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, uint32_t kv_heads, uint32_t capacity, PtParams& prm, cudaStream_t stream) {
     const uint64_t width = (uint64_t)prm.heads * PT_HD, kv_width = (uint64_t)kv_heads * PT_HD;
     CUtensorMap mq, mk, mv;
@@ -418,8 +445,8 @@ static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, ui
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-        if (cudaFuncSetAttribute(prefill_attention_tc_kernel<CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(prefill_attention_tc_kernel<CAPPED>, cudaFuncAttributePreferredSharedMemoryCarveout,
+        if (cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  (int)cudaSharedmemCarveoutMaxShared) != cudaSuccess)
             return check_launch("prefill_attention_tc attribute");
         if (dev >= 0 && dev < 64) configured[dev] = true;
@@ -433,7 +460,7 @@ static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, ui
     if (dev_sms <= 0) dev_sms = 148;
     const uint64_t items = (uint64_t)prm.q_tiles * prm.heads * prm.sessions;
     dim3 grid((unsigned)std::min<uint64_t>(items, 2ull * dev_sms));
-    launch_kernel(prefill_attention_tc_kernel<CAPPED>, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
+    launch_kernel(prefill_attention_tc_kernel<KIND>, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
     count_launch();
     return check_launch("prefill_attention_tc");
 }
@@ -449,8 +476,9 @@ int launch_prefill_attention_tc(const bf16* q, const bf16* k_cache, const bf16* 
     prm.sessions = sessions;
     prm.scale_log2 = (1.0f / sqrtf((float)PT_HD)) * 1.4426950408889634f;
     prm.out_ld = prm.out_cols = heads * PT_HD;
+    prm.gain = 1.0f;
     prm.d_status = d_status;
-    return launch_pt<false>(q, k_cache, v_cache, heads, capacity, prm, stream);
+    return launch_pt<PT_SOFTMAX>(q, k_cache, v_cache, heads, capacity, prm, stream);
 }
 
 bool grouped_attention_tc_eligible(const GroupedAttention& a, const StepPlace& place) {
@@ -470,16 +498,23 @@ int launch_grouped_attention_tc(const GroupedAttention& a, const StepPlace& plac
     prm.scale_log2 = a.scale * 1.4426950408889634f;
     prm.out_ld = a.out_ld;
     prm.out_cols = a.out_cols;
+    prm.gain = a.gain;
+    prm.window = a.window;
     prm.gate = a.gate;
     prm.gate_ld = a.gate_ld;
     prm.d_status = a.d_status;
     const bf16 *q = (const bf16*)a.q, *k = (const bf16*)a.k_cache, *v = (const bf16*)a.v_cache;
+    if (a.score_kind == TNSR_B200_SCORE_SIGMOID) {
+        prm.scale_log2 = -a.scale * 1.4426950408889634f;
+        prm.head_bias = a.head_bias;
+        return launch_pt<PT_SIGMOID>(q, k, v, a.kv_heads, a.capacity, prm, stream);
+    }
     if (a.softcap > 0.0f) {
         prm.cap_pre = 2.0f * 1.4426950408889634f * a.scale / a.softcap;
         prm.cap_post = a.softcap * 1.4426950408889634f;
-        return launch_pt<true>(q, k, v, a.kv_heads, a.capacity, prm, stream);
+        return launch_pt<PT_CAPPED>(q, k, v, a.kv_heads, a.capacity, prm, stream);
     }
-    return launch_pt<false>(q, k, v, a.kv_heads, a.capacity, prm, stream);
+    return launch_pt<PT_SOFTMAX>(q, k, v, a.kv_heads, a.capacity, prm, stream);
 }
 
 }  // namespace tb

@@ -84,6 +84,7 @@ gemm_strict_kernel(const float* __restrict__ a, const float* __restrict__ b, voi
     if (ep.activation == ACT_RELU) v = fmaxf(v, 0.0f);
     else if (ep.activation == ACT_GELU) v = strict_gelu(v);
     else if (ep.activation == ACT_GELU_TANH) v = strict_gelu_tanh(v);
+    if (ep.scale) v = v * ep.scale[col];
     if (ep.residual) v = ep.residual[(size_t)row * ep.ldr + col] + v;
     if (ep.round_bf16) v = round_to_bf16(v);
     size_t orow = row;
@@ -134,6 +135,7 @@ gemm_strict_rows_kernel(const float* __restrict__ a, const float* __restrict__ b
     if (ep.activation == ACT_RELU) v = fmaxf(v, 0.0f);
     else if (ep.activation == ACT_GELU) v = strict_gelu(v);
     else if (ep.activation == ACT_GELU_TANH) v = strict_gelu_tanh(v);
+    if (ep.scale) v = v * ep.scale[col];
     if (ep.residual) v = ep.residual[(size_t)row * ep.ldr + col] + v;
     if (ep.round_bf16) v = round_to_bf16(v);
     size_t orow = row;

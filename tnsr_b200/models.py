@@ -9,7 +9,9 @@ import json
 import os
 from typing import Callable, Dict
 
-from .bolonex import DEFAULT_CONTEXT, Bolonex, BolonexConfig
+from .bolonex import Bolonex, BolonexConfig
+from .described import DEFAULT_CONTEXT
+from .ganupel import Ganupel, GanupelConfig
 from .nn import CachedModel, TnsrError
 from .parameters import load_gpt, read_safetensors
 
@@ -20,8 +22,12 @@ def _bolonex(config: dict, tensors: dict, weight_dtype: str, max_sequence_length
     return Bolonex(BolonexConfig.from_dict(config, weight_dtype, max_sequence_length), tensors)
 
 
+def _ganupel(config: dict, tensors: dict, weight_dtype: str, max_sequence_length: int) -> CachedModel:
+    return Ganupel(GanupelConfig.from_dict(config, weight_dtype, max_sequence_length), tensors)
+
+
 # architecture name in config.json -> builder(config, tensors, weight_dtype, max_sequence_length)
-ARCHITECTURES: Dict[str, Callable[[dict, dict, str, int], CachedModel]] = {"Bolonex": _bolonex}
+ARCHITECTURES: Dict[str, Callable[[dict, dict, str, int], CachedModel]] = {"Bolonex": _bolonex, "Ganupel": _ganupel}
 
 
 def load_model(directory: str, dtype: str = "bfloat16", max_sequence_length: int = DEFAULT_CONTEXT) -> CachedModel:
