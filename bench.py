@@ -26,7 +26,8 @@ of the operator configurations.
 4-layer model end to end, the GEMM sweep, the SwiGLU MLP, ragged decode attention),
 each with the CPU restatement timed beside it on a stated sample.  `--workload bolonex`
 measures prefill and decode of Bolonex models at a few real-model sizes, each beside a
-GPT of the same width, depth and feed-forward weights (1 GPU).
+GPT of the same width, depth and feed-forward weights (1 GPU), `--workload ganupel` Ganupel
+models, each beside a Bolonex.
 
 The CPU arm times this repository's restatement of the reference's CPU executor
 (oracle/) on the host cores: the reference is Rust and cannot be built here.
@@ -78,7 +79,7 @@ def parse_args():
     ap.add_argument("--prefill", type=int, default=PREFILL)
     ap.add_argument("--layers", type=int, default=12)
     ap.add_argument("--vocab", type=int, default=32000)
-    ap.add_argument("--workload", default="c4", choices=["c4", "c0", "c1", "c2", "c3", "bolonex"],
+    ap.add_argument("--workload", default="c4", choices=["c4", "c0", "c1", "c2", "c3", "bolonex", "ganupel"],
                     help="c4 (default): the serving decode benchmark; c0: the 4-layer d128 f32 model, 16-token prompt + 64 "
                          "greedy steps; c1: GEMM sweep; c2: SwiGLU MLP; c3: ragged decode attention -- each with the CPU "
                          "restatement timed beside it (1 GPU)")
@@ -544,38 +545,72 @@ BOLONEX_SIZES = [
 ]
 
 
-def run_bolonex(args):
-    """Prefill and decode tokens/s of Bolonex beside the closest model here, a GPT of equal width, depth and feed-forward
-    weights; value = decode tokens/s of the first size."""
+def run_beside(args, name, sizes, note):
+    """Prefill and decode tokens/s of a described model beside the closest models of equal width, depth and feed-forward
+    weights; sizes: (case, sessions, prefill, {label: (config, arrays)}).  value = decode tokens/s of the first size."""
     import copy
     import torch
-    from tnsr_b200.nn import GptConfig
-    from tnsr_b200.synthetic import bolonex_arrays, bolonex_config
     torch.cuda.set_device(0)
     cases, clocks, launches = [], None, 0
     barrier = torch.cuda.synchronize
-    for name, sessions, prefill, width, layers, heads, kv, hd, mh, mw, state, ff, gpt_ff in BOLONEX_SIZES:
+    for case_name, sessions, prefill, models in sizes:
         a = copy.copy(args)
         a.prefill, a.steps, a.repeats = prefill, min(args.steps, 64), min(args.repeats, 5)
-        model = bolonex_config(width, layers, heads, kv, hd, mh, mw, state, ff, args.vocab)
-        gpt = GptConfig(vocab_size=args.vocab, max_sequence_length=2048, embed_dim=width, num_heads=width // 64, feed_forward_dim=gpt_ff,
-                        num_layers=layers, layer_norm_epsilon=1e-5, activation="swiglu", weight_dtype="bf16")
-        case = {"case": name, "sessions": sessions, "prefill": prefill}
-        for label, cfg, arrays in (("bolonex", model, bolonex_arrays(model, seed=5)), ("gpt", gpt, None)):
+        case = {"case": case_name, "sessions": sessions, "prefill": prefill}
+        for label, (cfg, arrays) in models.items():
             r = measure_decode(a, cfg, sessions, 0, 0, 1, barrier, float, False, arrays)
             ms = float(np.median(r["samples_ms"])) / a.steps
             case[label] = {"decode_ms_per_step": ms, "decode_tokens_per_s": sessions / ms * 1e3, "prefill_ms": r["prefill_ms"],
                            "prefill_tokens_per_s": sessions * prefill / r["prefill_ms"] * 1e3}
-            if label == "bolonex":
+            if label == name:
                 launches += r["launches"]
                 clocks = clocks or r["clocks"]
         cases.append(case)
-    first = cases[0]["bolonex"]
-    line = _op_line(args, "bolonex_decode_tokens_per_s", "tokens/s", first["decode_tokens_per_s"], first["decode_ms_per_step"], "bf16",
-                    "Bolonex beside a GPT of equal width, depth and feed-forward weights; value = decode of " + cases[0]["case"], None, None,
-                    cases, launches, clocks)
+    first = cases[0][name]
+    line = _op_line(args, name + "_decode_tokens_per_s", "tokens/s", first["decode_tokens_per_s"], first["decode_ms_per_step"], "bf16",
+                    note + "; value = decode of " + cases[0]["case"], None, None, cases, launches, clocks)
     line["steps"] = min(args.steps, 64)
     print(json.dumps(line), flush=True)
+
+
+def bolonex_of_size(args, width, layers, heads, kv, hd, mh, mw, state, ff):
+    from tnsr_b200.synthetic import bolonex_arrays, bolonex_config
+    cfg = bolonex_config(width, layers, heads, kv, hd, mh, mw, state, ff, args.vocab)
+    return cfg, bolonex_arrays(cfg, seed=5)
+
+
+def run_bolonex(args):
+    """Bolonex beside a GPT."""
+    from tnsr_b200.nn import GptConfig
+
+    def sizes():
+        for name, sessions, prefill, width, layers, heads, kv, hd, mh, mw, state, ff, gpt_ff in BOLONEX_SIZES:
+            gpt = GptConfig(vocab_size=args.vocab, max_sequence_length=2048, embed_dim=width, num_heads=width // 64, feed_forward_dim=gpt_ff,
+                            num_layers=layers, layer_norm_epsilon=1e-5, activation="swiglu", weight_dtype="bf16")
+            yield name, sessions, prefill, {"bolonex": bolonex_of_size(args, width, layers, heads, kv, hd, mh, mw, state, ff), "gpt": (gpt, None)}
+    run_beside(args, "bolonex", sizes(), "Bolonex beside a GPT of equal width, depth and feed-forward weights")
+
+
+# (name, sessions, prefill, width, layers, heads, kv_heads, head_dim, window, hgrn2 heads, dim, vdim, unit width, blocks, dense
+# feed-forward, experts, identity experts, chosen, width of one expert): the chosen experts have the dense one's weights
+GANUPEL_SIZES = [
+    ("12x768, 256 sessions", 256, 512, 768, 12, 12, 4, 64, 256, 12, 64, 64, 1024, 8, 3072, 16, 2, 4, 768),
+    ("12x768, 32 sessions", 32, 512, 768, 12, 12, 4, 64, 256, 12, 64, 64, 1024, 8, 3072, 16, 2, 4, 768),
+    ("12x1024, 64 sessions", 64, 1024, 1024, 12, 16, 4, 64, 512, 8, 128, 128, 1536, 12, 4096, 32, 4, 4, 1024),
+    ("12x768, one session of 1792 tokens", 1, 1792, 768, 12, 12, 4, 64, 256, 12, 64, 64, 1024, 8, 3072, 16, 2, 4, 768),
+]
+
+
+def run_ganupel(args):
+    """Ganupel beside Bolonex, the closest model here."""
+    from tnsr_b200.synthetic import ganupel_arrays, ganupel_config
+
+    def sizes():
+        for name, sessions, prefill, width, layers, heads, kv, hd, window, rh, rd, rv, uw, ub, ff, ex, ident, top, eff in GANUPEL_SIZES:
+            cfg = ganupel_config(width, layers, heads, kv, hd, window, rh, rd, rv, uw, ub, ff, ex, ident, top, eff, args.vocab)
+            yield name, sessions, prefill, {"ganupel": (cfg, ganupel_arrays(cfg, seed=5)),
+                                            "bolonex": bolonex_of_size(args, width, layers, heads, kv, hd, width // 32, 64, 128, ff)}
+    run_beside(args, "ganupel", sizes(), "Ganupel beside Bolonex of equal width, depth and feed-forward weights per token")
 
 
 def operator_summary(samples):
@@ -734,9 +769,9 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         run_reference(args)
-    elif args.workload == "bolonex":
+    elif args.workload in ("bolonex", "ganupel"):
         if int(os.environ.get("RANK", "0")) == 0:
-            run_bolonex(args)
+            {"bolonex": run_bolonex, "ganupel": run_ganupel}[args.workload](args)
     elif args.workload != "c4":
         if int(os.environ.get("RANK", "0")) == 0:
             run_ops(args)

@@ -9,6 +9,7 @@
     python -m tnsr_b200.opbench elementwise # LayerNorm, SwiGLU, embedding, greedy pick
     python -m tnsr_b200.opbench prefill_attention  # configuration 4's prefill attention on both engines
     python -m tnsr_b200.opbench mixers      # the mixers of described models: grouped attention, mamba2, RMS norm
+    python -m tnsr_b200.opbench ganupel     # windowed sigmoid attention, HGRN2, linear recurrent unit, PolyNorm, experts
     python -m tnsr_b200.opbench all
 
 Every line is one JSON object: algorithmic flops / bytes, CUDA-event time (median of `--samples`
@@ -294,14 +295,15 @@ def bench_elementwise(samples):
     emit(op="argmax", rows=rows, vocab=vocab, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
 
 
-def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads, hd, softcap, name):
+def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads, hd, softcap, name, window=0, kind="softmax"):
     """Grouped-query attention with capped scores and gates: `chunk` queries per session after `position` cached rows.
     Algorithmic bytes: the live K/V rows and q / out once; flops: 4 hd per (query, head, visible key)."""
     hbm, tf, kind = peaks()
     capacity = position + chunk
     g = torch.Generator(device="cuda").manual_seed(8)
     randn = lambda *shape: torch.randn(shape, device="cuda", generator=g).to(torch.bfloat16)
-    nbytes = sessions * 2.0 * ((position + chunk) * kv_heads * 2 * hd + chunk * heads * 2 * hd)
+    live = min(position + chunk, window + chunk - 1) if window else position + chunk
+    nbytes = sessions * 2.0 * (live * kv_heads * 2 * hd + chunk * heads * 2 * hd)
     sets = copies_for(int(nbytes))
     q = [randn(sessions * chunk, heads * hd) for _ in range(sets)]
     k = [randn(sessions, capacity, kv_heads * hd) for _ in range(sets)]
@@ -312,11 +314,15 @@ def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads,
     ws = torch.zeros(size, dtype=torch.uint8, device="cuda")
     where = _native.Place(sessions, chunk, position, 0, None)
     args = [_native.GroupedAttentionArgs(q[i].data_ptr(), k[i].data_ptr(), v[i].data_ptr(), gate.data_ptr(), out.data_ptr(), ws.data_ptr(), None, size,
-                                         heads, kv_heads, hd, hd, capacity, 32, heads * hd, heads * hd, hd ** -0.5, softcap, 1, 0) for i in range(sets)]
+                                         heads, kv_heads, hd, hd, capacity, 32, heads * hd, heads * hd, hd ** -0.5, softcap, 1, 0,
+                                         gate.data_ptr() if kind == "sigmoid" else None, window, _native.SCORE[kind], 1.0, 0) for i in range(sets)]
+    if kind == "sigmoid":
+        for a in args:
+            a.gate = None
     ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_grouped_attention(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
-    pairs = sessions * heads * sum(position + t + 1 for t in range(chunk))
+    pairs = sessions * heads * sum(min(position + t + 1, window or position + t + 1) for t in range(chunk))
     flops = 4.0 * hd * pairs
-    emit(op="grouped_attention", case=name, sessions=sessions, chunk=chunk, position=position, heads=heads, kv_heads=kv_heads, head_dim=hd,
+    emit(op="grouped_attention", window=window, scores=kind, case=name, sessions=sessions, chunk=chunk, position=position, heads=heads, kv_heads=kv_heads, head_dim=hd,
          softcap=softcap, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf,
          peaks=kind)
 
@@ -378,20 +384,165 @@ def bench_mixers(samples):
     emit(op="rmsnorm_f32_to_bf16", rows=rows, width=d, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
 
 
+def bench_hgrn2(samples, sessions, chunk, heads, dim, vdim, name):
+    """HGRN2 between its projections.  Algorithmic bytes: q, v (bf16) and gates (f32) in, bf16 rows out, the f32 state in and
+    out; flops: q S and k v^T per token and head (the inner weights of a chunk are small beside them)."""
+    hbm, tf, kind = peaks()
+    k, inner, rows = heads * dim, heads * vdim, sessions * chunk
+    nbytes = rows * (2.0 * (k + inner) + 4.0 * k + 2.0 * inner) + sessions * heads * dim * vdim * 8.0
+    sets = min(8, copies_for(int(nbytes)))
+    g = torch.Generator(device="cuda").manual_seed(10)
+    u = [torch.randn((rows, k + inner), device="cuda", generator=g).to(torch.bfloat16) for _ in range(sets)]
+    f = [torch.randn((rows, k), device="cuda", generator=g) for _ in range(sets)]
+    state = [torch.zeros((sessions, heads, dim, vdim), device="cuda") for _ in range(sets)]
+    bias, lower, norm = torch.full((k,), 3.0, device="cuda"), torch.rand(k, device="cuda", generator=g) * 0.9, torch.ones(vdim, device="cuda")
+    out = torch.empty((rows, inner), device="cuda", dtype=torch.bfloat16)
+    raw = torch.empty((rows, inner), device="cuda")
+    where = _native.Place(sessions, chunk, 64, 0, None)
+    args = [_native.Hgrn2Args(u[i].data_ptr(), u[i].data_ptr() + 2 * k, f[i].data_ptr(), bias.data_ptr(), lower.data_ptr(), norm.data_ptr(), state[i].data_ptr(),
+                              raw.data_ptr(), out.data_ptr(), k + inner, k, heads, dim, vdim, inner, inner, 1e-5, 1.0, 1, 0, 0) for i in range(sets)]
+    ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_hgrn2(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
+    flops = rows * heads * 4.0 * dim * vdim
+    emit(op="hgrn2", case=name, sessions=sessions, chunk=chunk, heads=heads, dim=dim, vdim=vdim, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm,
+         tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf, peaks=kind)
+
+
+def bench_rglru(samples, sessions, chunk, width, blocks, name):
+    """The recurrent unit between its projections: convolution, gate products, scan.  Algorithmic bytes: y and x in, rows out,
+    the convolved rows and the f32 gates out and in, the state in and out."""
+    hbm, _, kind = peaks()
+    rows, part = sessions * chunk, width // blocks
+    nbytes = rows * width * (2.0 * 3 + 2.0 * 3 + 8.0 * 2) + sessions * width * 8.0 + 4.0 * width * part
+    sets = min(8, copies_for(int(nbytes)))
+    g = torch.Generator(device="cuda").manual_seed(11)
+    u = [torch.randn((rows, 2 * width), device="cuda", generator=g).to(torch.bfloat16) for _ in range(sets)]
+    w = (torch.randn((blocks, 2 * part, part), device="cuda", generator=g) * part ** -0.5).to(torch.bfloat16)
+    conv, vec, lam = torch.rand((width, 4), device="cuda", generator=g), torch.zeros(width, device="cuda"), torch.full((width,), -5.0, device="cuda")
+    ring, state = torch.zeros((sessions, 4, width), device="cuda", dtype=torch.bfloat16), torch.zeros((sessions, width), device="cuda")
+    conv_out, gates = torch.empty((rows, width), device="cuda", dtype=torch.bfloat16), torch.empty((rows, 2 * width), device="cuda")
+    out = torch.empty((rows, width), device="cuda", dtype=torch.bfloat16)
+    where = _native.Place(sessions, chunk, 64, 0, None)
+    args = [_native.RglruArgs(u[i].data_ptr(), w.data_ptr(), conv.data_ptr(), vec.data_ptr(), vec.data_ptr(), vec.data_ptr(), lam.data_ptr(), ring.data_ptr(),
+                              state.data_ptr(), conv_out.data_ptr(), gates.data_ptr(), out.data_ptr(), None, 2 * width, width, width, blocks, 4, width, width,
+                              1) for i in range(sets)]
+    ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_rglru(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
+    emit(op="rglru", case=name, sessions=sessions, chunk=chunk, width=width, blocks=blocks, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm,
+         peaks=kind)
+
+
+def bench_grouped_gemm(samples, groups, rows, n, k, activation, name):
+    """One product per group of rows (sizes of a uniform routing).  Flops of the real rows; bytes: rows, weights, results."""
+    hbm, tf, kind = peaks()
+    rng = np.random.default_rng(12)
+    counts = np.bincount(rng.integers(0, groups, rows), minlength=groups)
+    offsets = torch.from_numpy(np.concatenate([[0], np.cumsum(counts)]).astype(np.int32)).cuda()
+    nbytes = 2.0 * (rows * (n + k) + (counts > 0).sum() * n * k)
+    sets = min(16, copies_for(int(nbytes)))
+    g = torch.Generator(device="cuda").manual_seed(13)
+    a = [torch.randn((rows, k), device="cuda", generator=g).to(torch.bfloat16) for _ in range(sets)]
+    w = [(torch.randn((groups, n, k), device="cuda", generator=g) * 0.02).to(torch.bfloat16) for _ in range(sets)]
+    out = torch.empty((rows, n), device="cuda", dtype=torch.bfloat16)
+    status = torch.zeros(1, device="cuda", dtype=torch.int32)
+    ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_gemm_grouped(ptr(a[i]), ptr(w[i]), ptr(out), ptr(offsets), groups, rows, n, k, activation, 1, 1, 0,
+                                                                  ptr(status), stream())), sets, samples, reps=8)
+    flops = 2.0 * rows * n * k
+    emit(op="gemm_grouped", case=name, groups=groups, rows=rows, n=n, k=k, ms=ms, tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf,
+         gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
+
+
+def bench_experts(samples, rows, d, ff, experts, identity, top, name):
+    """Routing, gather, both products and the weighted sum with the next norm.  Flops of the products of real experts."""
+    hbm, tf, kind = peaks()
+    total = experts + identity
+    g = torch.Generator(device="cuda").manual_seed(14)
+    logits, correction = torch.randn((rows, total), device="cuda", generator=g), torch.zeros(total, device="cuda")
+    h = torch.randn((rows, d), device="cuda", generator=g).to(torch.bfloat16)
+    up = (torch.randn((experts, ff, d), device="cuda", generator=g) * 0.02).to(torch.bfloat16)
+    down = (torch.randn((experts, d, ff), device="cuda", generator=g) * 0.02).to(torch.bfloat16)
+    x, one, normed = torch.zeros((rows, d), device="cuda"), torch.ones(d, device="cuda"), torch.empty((rows, d), device="cuda", dtype=torch.bfloat16)
+    size = lib().tnsr_b200_experts_workspace(rows, d, ff, experts, top, 1)
+    ws = torch.empty(size, dtype=torch.uint8, device="cuda")
+    status = torch.zeros(1, device="cuda", dtype=torch.int32)
+    args = _native.ExpertsArgs(logits.data_ptr(), correction.data_ptr(), h.data_ptr(), up.data_ptr(), down.data_ptr(), x.data_ptr(), one.data_ptr(),
+                               one.data_ptr(), normed.data_ptr(), ws.data_ptr(), size, None, None, status.data_ptr(), rows, total, d, ff, experts, identity,
+                               top, 1.0, 1.0, 1e-5, 1, 0)
+    ms, _ = timed_graph(lambda _: ok(lib().tnsr_b200_experts(C.byref(args), stream())), 1, samples, reps=8)
+    pairs = rows * top * experts / total
+    flops, weights = pairs * 4.0 * d * ff, min(experts, pairs) * 4.0 * d * ff
+    nbytes = weights + rows * (2.0 * d * 2 + 4.0 * d * 2) + pairs * (2.0 * d * 4 + 2.0 * ff * 2)
+    emit(op="experts", case=name, rows=rows, d=d, ff=ff, experts=experts, identity=identity, top=top, ms=ms, tflops=flops / ms / 1e9,
+         frac_tensor=flops / ms / 1e9 / tf, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
+
+
+def bench_polynorm(samples, rows, width):
+    hbm, _, kind = peaks()
+    z, act = torch.randn((rows, width), device="cuda").to(torch.bfloat16), torch.tensor([0.5, 0.3, 0.2, 0.0], device="cuda")
+    out = torch.empty_like(z)
+    ms, _ = timed(lambda _: ok(lib().tnsr_b200_polynorm(ptr(z), ptr(act), ptr(out), rows, width, width, width, 1e-5, 1, stream())), 1, samples)
+    nbytes = rows * width * 4.0
+    emit(op="polynorm", rows=rows, width=width, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
+
+
+def bench_rotary(samples, sessions, chunk, heads, kv_heads, hd):
+    hbm, _, kind = peaks()
+    rows, cols = sessions * chunk, (heads + 2 * kv_heads) * hd
+    u = torch.randn((rows, cols), device="cuda").to(torch.bfloat16)
+    table = torch.rand((chunk, hd), device="cuda")
+    q = torch.empty((rows, heads * hd), device="cuda", dtype=torch.bfloat16)
+    k, v = (torch.empty((rows, kv_heads * hd), device="cuda", dtype=torch.bfloat16) for _ in range(2))
+    args = _native.RotaryArgs(u.data_ptr(), table.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), cols, heads, kv_heads, hd, hd, hd, 1, chunk, 1, 0)
+    where = _native.Place(sessions, chunk, 0, 0, None)
+    ms, _ = timed(lambda _: ok(lib().tnsr_b200_rotary(C.byref(args), C.byref(where), stream())), 1, samples)
+    nbytes = rows * cols * 4.0
+    emit(op="rotary", rows=rows, heads=heads, kv_heads=kv_heads, head_dim=hd, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
+
+
+def bench_ganupel(samples):
+    """Beside the like kernels of Bolonex (mixers) and of the GPT (serving_gemms, elementwise)."""
+    bench_grouped_attention(samples, 256, 1, 640, 12, 4, 64, 30.0, "Bolonex decode")
+    bench_grouped_attention(samples, 256, 1, 640, 12, 4, 64, 0.0, "decode, window 256", 256, "sigmoid")
+    bench_grouped_attention(samples, 256, 1, 640, 12, 4, 64, 0.0, "decode, no window", 0, "sigmoid")
+    bench_grouped_attention(samples, 64, 512, 0, 12, 4, 64, 30.0, "Bolonex prefill")
+    bench_grouped_attention(samples, 64, 512, 0, 12, 4, 64, 0.0, "prefill, window 256", 256, "sigmoid")
+    bench_grouped_attention(samples, 64, 512, 0, 12, 4, 64, 0.0, "prefill, no window", 0, "sigmoid")
+    bench_mamba2(samples, 256, 1, 24, 64, 128, 1, "Bolonex decode")
+    bench_hgrn2(samples, 256, 1, 12, 64, 64, "decode")
+    bench_hgrn2(samples, 256, 1, 8, 128, 128, "decode, 128 x 128")
+    bench_hgrn2(samples, 32, 1, 12, 64, 64, "decode, 32 sessions")
+    bench_mamba2(samples, 256, 512, 24, 64, 128, 1, "Bolonex prefill, 256 sessions")
+    bench_hgrn2(samples, 256, 512, 12, 64, 64, "prefill, 256 sessions")
+    bench_hgrn2(samples, 64, 1024, 8, 128, 128, "prefill, 128 x 128")
+    bench_hgrn2(samples, 64, 512, 12, 128, 64, "prefill, 128 x 64")
+    bench_hgrn2(samples, 1, 4096, 12, 64, 64, "prefill, one long prompt")
+    bench_rglru(samples, 256, 1, 1024, 8, "decode")
+    bench_rglru(samples, 256, 512, 1024, 8, "prefill, 256 sessions")
+    bench_rglru(samples, 1, 4096, 1024, 8, "prefill, one long prompt")
+    bench_polynorm(samples, 131072, 3072)
+    bench_rotary(samples, 256, 512, 12, 4, 64)
+    bench_grouped_gemm(samples, 16, 131072 * 4, 768, 768, 4, "up, prefill")
+    bench_grouped_gemm(samples, 16, 131072 * 4, 768, 768, -1, "down, prefill")
+    bench_grouped_gemm(samples, 32, 65536 * 4, 1024, 1024, 4, "up, prefill, 32 experts")
+    bench_grouped_gemm(samples, 16, 256 * 4, 768, 768, 4, "up, decode of 256")
+    bench_grouped_gemm(samples, 64, 64 * 4, 1024, 1024, 4, "up, decode of 64, 64 experts")
+    bench_experts(samples, 131072, 768, 768, 16, 2, 4, "prefill")
+    bench_experts(samples, 256, 768, 768, 16, 2, 4, "decode of 256")
+    bench_experts(samples, 32, 768, 768, 16, 2, 4, "decode of 32")
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemm", "skinny_gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers", "all"])
+    ap.add_argument("what", choices=["gemm", "skinny_gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers", "ganupel", "all"])
     ap.add_argument("--samples", type=int, default=20)
     args = ap.parse_args()
     if not torch.cuda.is_available():
         sys.exit("opbench needs a CUDA device")
-    todo = (["gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers"]
+    todo = (["gemm", "serving_gemms", "mlp", "attention", "serving_attention", "elementwise", "prefill_attention", "mixers", "ganupel"]
             if args.what == "all" else [args.what])
     for name in todo:
         {"gemm": bench_gemm, "skinny_gemm": lambda n: bench_gemm(n, shapes=[(m, 4096, 4096) for m in (1, 8, 64)], outs=("bf16",)),
          "serving_gemms": bench_serving_gemms, "mlp": bench_mlp, "attention": bench_attention,
          "serving_attention": lambda n: bench_attention(n, serving=True),
-         "elementwise": bench_elementwise, "prefill_attention": bench_prefill_attention, "mixers": bench_mixers}[name](args.samples)
+         "elementwise": bench_elementwise, "prefill_attention": bench_prefill_attention, "mixers": bench_mixers, "ganupel": bench_ganupel}[name](args.samples)
 
 
 if __name__ == "__main__":

@@ -70,6 +70,45 @@ def bolonex_arrays(cfg, seed: int, std: float = 0.02):
     return arrays
 
 
+def ganupel_config(width, layers, heads, kv_heads, head_dim, window, rec_heads, rec_dim, rec_vdim, unit_width, unit_blocks, feed_forward,
+                   experts, identity, top, expert_ff, vocab_size, max_sequence_length=2048):
+    """A Ganupel of real-model proportions: two layers of attention beside HGRN2, then one linear recurrent unit, and so on;
+    dense feed-forwards in the even layers, experts in the odd ones."""
+    from .ganupel import Dense, Experts, GanupelConfig, Hgrn2, LayerConfig, ParallelMixer, RgLru, WindowedAttention
+    mixer = ParallelMixer(WindowedAttention(heads, kv_heads, head_dim, head_dim, head_dim ** -0.5, window, head_dim, 10000.0),
+                          Hgrn2(rec_heads, rec_dim, rec_vdim), 1.0, 1.0)
+    unit, dense, sparse = RgLru(unit_width, unit_blocks, 4), Dense(feed_forward), Experts(expert_ff, experts, identity, top, 1.0)
+    return GanupelConfig(vocab_size, width, tuple(LayerConfig(unit if i % 3 == 2 else mixer, sparse if i % 2 else dense) for i in range(layers)), 1e-5, "bf16",
+                         max_sequence_length)
+
+
+def ganupel_arrays(cfg, seed: int, std: float = 0.02):
+    """Parameter arrays of a Ganupel in the order of its tensor table: matrices N(0, std), norms, scales and biases neutral,
+    gates and decays in the range a trained layer has."""
+    rng = np.random.default_rng(seed)
+    arrays = []
+    for name, shape in cfg.tensor_shapes().items():
+        leaf = name.split(".")[-1]
+        if name.endswith(("norm1", "norm2", "final.norm")) or leaf in ("b", "correction"):
+            a = np.full(shape, 3.0 if name.endswith("f.b") else 0.0, np.float32)
+        elif leaf in ("norm", "ls1", "ls2"):
+            a = np.ones(shape, np.float32)
+        elif leaf == "act":
+            a = np.float32([0.5, 0.3, 0.2, 0.0])
+        elif leaf == "pb":
+            a = np.full(shape, -5.0, np.float32)
+        elif leaf == "lower":
+            a = rng.uniform(0.0, 0.9, shape).astype(np.float32)
+        elif leaf == "lam":
+            a = rng.uniform(-8.0, -3.0, shape).astype(np.float32)
+        elif leaf == "conv":
+            a = rng.uniform(-0.5, 0.5, shape).astype(np.float32)
+        else:
+            a = rng.standard_normal(shape, dtype=np.float32) * np.float32(std)
+        arrays.append(a)
+    return arrays
+
+
 def config0_model(activation="relu"):
     cfg = GptConfig(vocab_size=96, max_sequence_length=128, embed_dim=128, num_heads=4,
                     feed_forward_dim=512, num_layers=4, layer_norm_epsilon=1e-5, activation=activation)
