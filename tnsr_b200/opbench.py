@@ -295,7 +295,7 @@ def bench_elementwise(samples):
     emit(op="argmax", rows=rows, vocab=vocab, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, peaks=kind)
 
 
-def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads, hd, softcap, name, window=0, kind="softmax"):
+def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads, hd, softcap, name, window=0, scores="softmax"):
     """Grouped-query attention with capped scores and gates: `chunk` queries per session after `position` cached rows.
     Algorithmic bytes: the live K/V rows and q / out once; flops: 4 hd per (query, head, visible key)."""
     hbm, tf, kind = peaks()
@@ -315,14 +315,14 @@ def bench_grouped_attention(samples, sessions, chunk, position, heads, kv_heads,
     where = _native.Place(sessions, chunk, position, 0, None)
     args = [_native.GroupedAttentionArgs(q[i].data_ptr(), k[i].data_ptr(), v[i].data_ptr(), gate.data_ptr(), out.data_ptr(), ws.data_ptr(), None, size,
                                          heads, kv_heads, hd, hd, capacity, 32, heads * hd, heads * hd, hd ** -0.5, softcap, 1, 0,
-                                         gate.data_ptr() if kind == "sigmoid" else None, window, _native.SCORE[kind], 1.0, 0) for i in range(sets)]
-    if kind == "sigmoid":
+                                         gate.data_ptr() if scores == "sigmoid" else None, window, _native.SCORE[scores], 1.0, 0) for i in range(sets)]
+    if scores == "sigmoid":
         for a in args:
             a.gate = None
     ms, _ = timed_graph(lambda i: ok(lib().tnsr_b200_grouped_attention(C.byref(args[i]), C.byref(where), stream())), sets, samples, reps=8)
     pairs = sessions * heads * sum(min(position + t + 1, window or position + t + 1) for t in range(chunk))
     flops = 4.0 * hd * pairs
-    emit(op="grouped_attention", window=window, scores=kind, case=name, sessions=sessions, chunk=chunk, position=position, heads=heads, kv_heads=kv_heads, head_dim=hd,
+    emit(op="grouped_attention", window=window, scores=scores, case=name, sessions=sessions, chunk=chunk, position=position, heads=heads, kv_heads=kv_heads, head_dim=hd,
          softcap=softcap, ms=ms, gbs=nbytes / ms / 1e6, frac_hbm=nbytes / ms / 1e6 / hbm, tflops=flops / ms / 1e9, frac_tensor=flops / ms / 1e9 / tf,
          peaks=kind)
 
