@@ -47,9 +47,16 @@ struct Experts {
     uint32_t rows = 0, logits_ld = 0, d = 0, ff = 0, experts = 0, identity = 0, top = 0;
     float router_scale = 1.0f, norm_offset = 0.0f, eps = 0.0f;
     int engine = 0;
+    // Set `router` to have launch_experts also norm x into h and form the router logits (steps of few rows, see
+    // experts_fused_router); `logits` is not read then.
+    const void* router = nullptr;         // [experts + identity, d]
+    const float* router_norm = nullptr;   // [d]
+    const float* partials = nullptr;      // partial sums of a split product, added to x first (launch_layernorm_fold)
+    uint32_t parts = 0, split_rows = 0;   // at most 4
 };
 constexpr uint32_t kMaxExperts = 1024;    // experts and identity experts together
 constexpr uint32_t kMaxTop = 32;
+bool experts_fused_router(const Experts& e);
 uint64_t experts_workspace_bytes(uint32_t rows, uint32_t d, uint32_t ff, uint32_t experts, uint32_t top, int dtype);
 // Routing, both grouped products and the gather between them; the result stays in the workspace.
 int launch_experts(const Experts& e, int dtype, cudaStream_t stream);

@@ -947,6 +947,7 @@ static int launch_gemm_impl(const bf16* a, const bf16* bt, void* out, uint32_t l
     uint32_t bn = 256;
     while (bn > 64 && (uint64_t)tiles_m * ceil_div(n, bn) < (uint64_t)sm_count()) bn >>= 1;
     if (bn == 64 && 2ull * tiles_m * ceil_div(n, 64) <= (uint64_t)sm_count()) bn = 32;  // very few tiles: halve once more
+    while (bn > 32 && bn / 2 >= n) bn >>= 1;      // no wider than the matrix (a router's few columns)
     if (split_req) bn = 32;   // many small tiles: every CTA takes in as little of both operands as possible
     TcParams prm;
     prm.k = k;

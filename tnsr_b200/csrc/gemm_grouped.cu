@@ -344,12 +344,17 @@ int launch_gemm_grouped(const GroupedGemm& g, int dtype, cudaStream_t stream) {
     const bool tc = dtype == TNSR_B200_BF16 && g.engine == 0 && g_gemm_engine != 1 && g.k % 8 == 0 && aligned(g.a, 16) && aligned(g.w, 16) &&
                     aligned(g.out, 4) && encode_fn() != nullptr;
     if (tc) {
+        // token rows per tile: a group's mean, less while there are fewer tiles than SMs
         const uint32_t per = ceil_div(g.rows, g.groups);
-        if (per <= 16) return launch_tc<16>(g, prm, stream);
-        if (per <= 32) return launch_tc<32>(g, prm, stream);
-        if (per <= 64) return launch_tc<64>(g, prm, stream);
-        if (per <= 128) return launch_tc<128>(g, prm, stream);
-        return launch_tc<256>(g, prm, stream);
+        uint32_t nt = per <= 16 ? 16 : per <= 32 ? 32 : per <= 64 ? 64 : per <= 128 ? 128 : 256;
+        while (nt > 32 && (uint64_t)ceil_div(g.n, (uint32_t)GG_ROWS) * g.groups * ceil_div(per, nt) < (uint64_t)gg_sms()) nt >>= 1;
+        switch (nt) {
+            case 16: return launch_tc<16>(g, prm, stream);
+            case 32: return launch_tc<32>(g, prm, stream);
+            case 64: return launch_tc<64>(g, prm, stream);
+            case 128: return launch_tc<128>(g, prm, stream);
+            default: return launch_tc<256>(g, prm, stream);
+        }
     }
     const uint64_t tiles = (uint64_t)ceil_div(g.n, 32u) * (g.rows / 32 + std::min(g.groups, g.rows));
     const dim3 grid((uint32_t)std::min<uint64_t>(std::max<uint64_t>(tiles, 1), 148ull * 8));

@@ -44,7 +44,7 @@ __device__ __forceinline__ void hs_gate(float z, float lower, float& f, float& k
 
 // NP: channels padded to a multiple of 64; WARPS: 16 columns each.
 template <int NP, int WARPS>
-__global__ void __launch_bounds__(WARPS * 32, NP <= 64 ? (WARPS == 4 ? 4 : 2) : NP <= 128 ? (WARPS == 4 ? 3 : 1) : 1)
+__global__ void __launch_bounds__(WARPS * 32, NP <= 64 ? (WARPS == 4 ? 4 : 2) : NP <= 128 ? (WARPS == 4 ? 2 : 1) : 1)
 hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     using S = HsShape<NP, WARPS>;
     constexpr int NT = NP / 8, GROUPS = NP / 16, MINE = (GROUPS + WARPS - 1) / WARPS;    // 16-channel groups, per warp
@@ -229,6 +229,7 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     load_v(0, smem);
     __syncthreads();       // s_tiny is clear
     prepare(0, smem, 0);
+    fetch(HS_Q);
 
     const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::NPITCH + (lane >> 4) * 16;     // A operand, [token][channel]
     const uint32_t b_off = ((lane & 7) + (lane >> 4) * 8) * S::NPITCH + ((lane >> 3) & 1) * 16;     // B operand, [n = token][k = channel]
@@ -274,7 +275,6 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
         __syncthreads();       // this chunk's operands are in place, the last one's have been used up
         if (t0 > 0) finish(t0 - HS_Q);
         const bool more = t0 + HS_Q < place.chunk;
-        if (more) fetch(t0 + HS_Q);
         load_v(t0 + HS_Q, next);
         const bool slow = s_tiny[buf] != 0;
         // ---- inner weights over this warp's channels ----
@@ -329,7 +329,10 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
                 mx_mma(y[1], ql, h10, h11);
             }
         }
-        if (more) prepare(t0 + HS_Q, next, buf ^ 1);
+        if (more) {
+            prepare(t0 + HS_Q, next, buf ^ 1);
+            fetch(t0 + 2 * HS_Q);       // a whole chunk ahead of its use
+        }
         __syncthreads();       // the inner weights of all warps are in place
         if (tid == 0) s_tiny[buf] = 0;
         if (owner) {

@@ -630,7 +630,12 @@ int stack_step(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t chunk,
     auto product = [&](const void* w, uint32_t n, void* out, uint32_t ld, int activation, int out_dtype) -> int {
         GemmEpilogue ep;
         ep.activation = activation; ep.out_dtype = out_dtype;
-        if (bf) RUN(dec, launch_gemm_bf16((const bf16*)dec->n, (const bf16*)w, out, ld, rows, n, d, GEMM_PLAIN, ep, nullptr, dec->d_status, st));
+        if (bf && out_dtype == TNSR_B200_BF16 && n % 32 == 0 && rows > 16) {     // one column range: its epilogue is the faster one for a short K
+            GemmSegments one;
+            one.count = 1;
+            one.s[0].out = out; one.s[0].ld = ld; one.s[0].activation = activation;
+            RUN(dec, launch_gemm_segments((const bf16*)dec->n, (const bf16*)w, rows, n, d, nullptr, one, dec->d_status, st));
+        } else if (bf) RUN(dec, launch_gemm_bf16((const bf16*)dec->n, (const bf16*)w, out, ld, rows, n, d, GEMM_PLAIN, ep, nullptr, dec->d_status, st));
         else RUN(dec, launch_gemm_strict((const float*)dec->n, (const float*)w, out, ld, rows, d, n, true, ep, st));
         return TNSR_B200_OK;
     };
@@ -720,16 +725,27 @@ int stack_step(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t chunk,
         if ((rc = add_product(S->cat, W.w_out, L.k_out, W.scale1))) return rc;
         if (!sequential(l) || !l.feed_forward) continue;
         // ---- feed-forward of a sequential block ----
-        if ((rc = norm(W.norm2))) return rc;
+        if (l.feed_forward_kind != TNSR_B200_FF_EXPERTS)
+            if ((rc = norm(W.norm2))) return rc;
         if (l.feed_forward_kind == TNSR_B200_FF_EXPERTS) {
             const uint32_t total = l.experts + l.identity_experts;
-            if ((rc = product(W.router, total, S->router, total, ACT_NONE, TNSR_B200_F32))) return rc;
             experts = Experts();
             experts.logits = S->router; experts.logits_ld = total; experts.correction = W.correction;
             experts.h = dec->n; experts.up = W.w_up; experts.down = W.w_down; experts.x = dec->h; experts.layer_scale = W.scale2;
             experts.workspace = S->experts_ws; experts.workspace_bytes = S->experts_ws_bytes; experts.d_status = dec->d_status;
             experts.rows = rows; experts.d = d; experts.ff = l.feed_forward; experts.experts = l.experts; experts.identity = l.identity_experts;
             experts.top = l.top; experts.router_scale = (float)l.router_scale; experts.norm_offset = S->norm_offset; experts.eps = eps;
+            if (chunk == 1) {       // few rows: norm and router in the choosing kernel
+                experts.router = W.router; experts.router_norm = W.norm2;
+                experts.partials = dec->split_ws; experts.parts = pending; experts.split_rows = dec->split_rows;
+            }
+            if (experts_fused_router(experts)) {
+                pending = 0;
+            } else {
+                experts.router = nullptr;
+                if ((rc = norm(W.norm2))) return rc;
+                if ((rc = product(W.router, total, S->router, total, ACT_NONE, TNSR_B200_F32))) return rc;
+            }
             RUN(dec, launch_experts(experts, dtype, st));
             pending_experts = true;
         } else {
