@@ -261,13 +261,13 @@ def test_hgrn2_portions_and_tokens(shape):
     want = expected_hgrn2(shape, u, t)
     for portions in ([n], [64, 64, 22], [15, 17, 33, 16, 69], [1] * 9 + [2, 3, 16, 17, 40, 1, 1, 61], [2] * 75):
         got, state = run_hgrn2(shape, u, t, portions, BF16)
-        assert np.sqrt(np.mean((got - want) ** 2)) < 4e-3 * np.std(want) and rel_err(got, want) < 1e-2, portions
+        assert np.sqrt(np.mean((got - want) ** 2)) < 4e-3 * np.std(want) and rel_err(got, want) < 2e-2, portions
         got32, state32 = run_hgrn2(shape, u, t, portions, F32)
         assert rel_err(got32, want) < 1e-5, portions
         # inputs are bf16-exact here, so the carried f32 states agree far below bf16's rounding
         assert rel_err(state.cpu().numpy(), state32.cpu().numpy()) < 1e-4
     token_by_token, _ = run_hgrn2(shape, u, t, [n], BF16, engine=1)
-    assert rel_err(token_by_token, want) < 1e-2
+    assert rel_err(token_by_token, want) < 2e-2
 
 
 @pytest.mark.parametrize("shape", [(2, 64, 64), (2, 20, 28), (1, 128, 128)])
@@ -283,7 +283,7 @@ def test_hgrn2_gates_that_all_but_vanish(shape):
     want = expected_hgrn2(shape, u, t)
     for portions in ([100], [50, 50], [37, 1, 62]):
         got, state = run_hgrn2(shape, u, t, portions, BF16)
-        assert np.isfinite(got).all() and np.sqrt(np.mean((got - want) ** 2)) < 4e-3 * np.std(want) and rel_err(got, want) < 1e-2, portions
+        assert np.isfinite(got).all() and np.sqrt(np.mean((got - want) ** 2)) < 4e-3 * np.std(want) and rel_err(got, want) < 2e-2, portions
         got32, state32 = run_hgrn2(shape, u, t, portions, F32)
         assert rel_err(got32, want) < 1e-5
         assert rel_err(state.cpu().numpy(), state32.cpu().numpy()) < 1e-4

@@ -10,12 +10,13 @@
 //
 // A CTA owns the whole sequence of one (session, head, up to 128 columns of the state).  Each warp owns 16 columns and keeps
 // its part of S transposed in accumulator registers (rows = its columns, from v^T . k): in that layout the accumulators of
-// S^T are, register by register, the B operand of q . S, so the state never passes through shared memory.  All warps make
-// the operands of the next chunk (gates, running products, silu) while this chunk's products run; the 16 x 16 inner weights
-// are split over the warps by channels and added through shared memory.  Two barriers per chunk.  The RMS norm of the
-// output waits in registers for the next chunk's first barrier, behind which the other warps' sums of squares are in place.
+// S^T are, register by register, the B operand of q . S, so the state never passes through shared memory.  Every warp forms
+// the 16 x 16 inner weights itself (their accumulators are the A operand of the product with v), and all warps make the
+// operands of the next chunk (gates, running products, silu), so one barrier per chunk is enough.  The RMS norm of the
+// output waits in registers for the next chunk's barrier, behind which the other warps' sums of squares are in place.
 //
-// Every f32 factor enters the products as two bf16 halves (split_bf16x2), so that it keeps 16 bits; v is bf16.
+// The state, the written k R, k / P and the inner weights enter the products as two bf16 halves (split_bf16x2), so that they
+// keep 16 bits; the readout's q P is rounded to bf16 like q itself, v is bf16.
 #include <algorithm>
 
 #include "mixers.cuh"
@@ -23,23 +24,24 @@
 namespace tb {
 
 constexpr int HS_Q = 16;
-constexpr float HS_TINY = 1e-30f;
+constexpr float HS_TINY = 1e-30f, HS_LOG2E = 1.4426950408889634f;
 
 template <int NP, int WARPS>
 struct HsShape {
     static constexpr uint32_t NPITCH = NP * 2 + 16, VPITCH = WARPS * 32 + 16;     // bytes; conflict-free ldmatrix
     static constexpr uint32_t OP = HS_Q * NPITCH;                                 // one operand half
     static constexpr uint32_t V_BYTES = HS_Q * VPITCH;
-    static constexpr uint32_t STAGE = 6 * OP + V_BYTES + NP * 4;                  // qP, k/P, kR (two halves each), v, P_15
-    static constexpr uint32_t APITCH = 18;                                        // floats
-    static constexpr uint32_t A_BYTES = WARPS * HS_Q * APITCH * 4;
-    static constexpr uint32_t BYTES = 2 * STAGE + A_BYTES;
+    static constexpr uint32_t STAGE = 5 * OP + V_BYTES + NP * 4;                  // qP, k/P and kR in two halves, v, P_15
+    static constexpr uint32_t SPITCH = 18;                                        // floats: weights formed gate by gate, per warp
+    static constexpr uint32_t BYTES = 2 * STAGE + WARPS * HS_Q * SPITCH * 4;
 };
 
-__device__ __forceinline__ void hs_gate(float z, float lower, float& f, float& k) {
-    const float e = mx_ex2(-1.4426950408889634f * fabsf(z)), big = mx_rcp(1.0f + e), small = e * big;     // sigmoid(|z|), sigmoid(-|z|)
-    f = fmaf(1.0f - lower, z >= 0.0f ? big : small, lower);
-    k = (1.0f - lower) * (z >= 0.0f ? small : big);
+// f = l + (1 - l) sigmoid(z) and k = (1 - l) sigmoid(-z) from t = exp(-z): sigmoid(-z) = t sigmoid(z), so that neither end
+// loses digits.  z2 = -log2(e) z; the bound keeps t finite (sigmoid(z) is zero to f32 long before).
+__device__ __forceinline__ void hs_gate(float z2, float lower, float rest, float& f, float& k) {
+    const float t = mx_ex2(fminf(z2, 120.0f)), s = mx_rcp(1.0f + t);
+    f = fmaf(rest, s, lower);
+    k = rest * (t * s);
 }
 
 // NP: channels padded to a multiple of 64; WARPS: 16 columns each.
@@ -49,15 +51,14 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     using S = HsShape<NP, WARPS>;
     constexpr int NT = NP / 8, GROUPS = NP / 16, MINE = (GROUPS + WARPS - 1) / WARPS;    // 16-channel groups, per warp
     extern __shared__ __align__(16) uint8_t smem[];
-    float* inner = reinterpret_cast<float*>(smem + 2 * S::STAGE);         // [WARPS][16][APITCH]
-    __shared__ float s_sq[WARPS][HS_Q];
-    __shared__ uint32_t s_tiny[2];
+    __shared__ float s_sq[2][WARPS][HS_Q];
+    __shared__ uint32_t s_tiny[4];            // by chunk modulo 4: one is set, one read and one cleared between two barriers
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     const uint32_t c_first = blockIdx.x * (WARPS * 16), h = blockIdx.y, s = blockIdx.z;
     const uint32_t width = min((uint32_t)(WARPS * 16), m.vdim - c_first);
     const uint32_t pw = warp * 16;              // the warp's columns
     const bool owner = pw < width, fused = m.vdim <= HGRN2_FUSED_VDIM;
-    if (tid < 2) s_tiny[tid] = 0;
+    if (tid < 4) s_tiny[tid] = 0;
     pdl_wait();
     pdl_trigger();
     const uint32_t p0 = place.pos(s);
@@ -69,14 +70,14 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
 
     // ---- operands of a chunk: a lane owns two channels of four tokens of a 16-channel group ----
     const uint32_t p8 = lane & 7, tq = lane >> 3;
-    float bias[MINE][2], lower[MINE][2];
+    float bias2[MINE][2], lower[MINE][2];       // channels past the last one: lower 1, that is f = 1 and k = 0
 #pragma unroll
     for (int i = 0; i < MINE; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const uint32_t c = (warp + i * WARPS) * 16 + p8 * 2 + e;
-            bias[i][e] = c < m.dim ? m.f_bias[h * m.dim + c] : 0.0f;
-            lower[i][e] = c < m.dim ? m.lower[h * m.dim + c] : 0.0f;
+            bias2[i][e] = c < m.dim ? -HS_LOG2E * m.f_bias[h * m.dim + c] : 0.0f;
+            lower[i][e] = c < m.dim ? m.lower[h * m.dim + c] : 1.0f;
         }
     float2 raw_f[MINE][4];
     uint32_t raw_q[MINE][4];
@@ -103,7 +104,7 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
             }
     };
     auto load_v = [&](uint32_t t0, uint8_t* stage) {
-        uint8_t* dst = stage + 6 * S::OP;
+        uint8_t* dst = stage + 5 * S::OP;
         if (t0 < place.chunk) {
             if (vec) {
                 for (uint32_t i = tid; i < HS_Q * WARPS * 2; i += WARPS * 32) {
@@ -121,7 +122,8 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
         }
         mx_commit();
     };
-    auto prepare = [&](uint32_t t0, uint8_t* stage, uint32_t buf) {
+    auto prepare = [&](uint32_t t0, uint8_t* stage) {
+        const bool whole = t0 + HS_Q <= place.chunk;
 #pragma unroll
         for (int i = 0; i < MINE; ++i) {
             const uint32_t grp = warp + i * WARPS, c = grp * 16 + p8 * 2;
@@ -129,15 +131,14 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
             float f[4][2], k[4][2], q[4][2], run[4][2], left[4][2], before[2], after[2], all[2];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const bool here = t0 + tq * 4 + j < place.chunk;
                 const float2 qv = bf16x2_to_f32(raw_q[i][j]);
                 const float z[2] = {raw_f[i][j].x, raw_f[i][j].y}, qq[2] = {qv.x, qv.y};
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    hs_gate(z[e] + bias[i][e], lower[i][e], f[j][e], k[j][e]);
-                    q[j][e] = mx_silu(qq[e]);
-                    if (!here || c + e >= m.dim) { f[j][e] = 1.0f; k[j][e] = 0.0f; q[j][e] = 0.0f; }
+                    hs_gate(fmaf(z[e], -HS_LOG2E, bias2[i][e]), lower[i][e], 1.0f - lower[i][e], f[j][e], k[j][e]);
+                    q[j][e] = mx_silu(qq[e]);      // 0 past the end and past the last channel
                 }
+                if (!whole && t0 + tq * 4 + j >= place.chunk) { f[j][0] = f[j][1] = 1.0f; k[j][0] = k[j][1] = 0.0f; }
             }
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
@@ -161,9 +162,8 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
                 u = __shfl_down_sync(0xffffffffu, y, 8);
                 after[e] = tq <= 2 ? u : 1.0f;
             }
-            const bool tiny = all[0] < HS_TINY || all[1] < HS_TINY;
-            if (tiny) s_tiny[buf] = 1u;        // every writer stores the same
-            if (tq == 0) *reinterpret_cast<float2*>(stage + 6 * S::OP + S::V_BYTES + c * 4) = make_float2(all[0], all[1]);
+            if (fminf(all[0], all[1]) < HS_TINY) s_tiny[t0 / HS_Q & 3] = 1u;        // every writer stores the same
+            if (tq == 0) *reinterpret_cast<float2*>(stage + 5 * S::OP + S::V_BYTES + c * 4) = make_float2(all[0], all[1]);
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 uint8_t* dst = stage + (tq * 4 + j) * S::NPITCH + c * 2;
@@ -172,42 +172,50 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
                 for (int e = 0; e < 2; ++e) {
                     const float p = before[e] * run[j][e];
                     qp[e] = q[j][e] * p;
-                    kp[e] = p < HS_TINY ? 0.0f : k[j][e] * mx_rcp(p);
+                    kp[e] = k[j][e] * mx_rcp(p);          // not used when the chunk is marked tiny
                     kr[e] = k[j][e] * (left[j][e] * after[e]);
                 }
                 uint32_t hi, lo;
-                split_bf16x2(qp[0], qp[1], hi, lo);
-                *reinterpret_cast<uint32_t*>(dst) = hi;
-                *reinterpret_cast<uint32_t*>(dst + S::OP) = lo;
+                *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(qp[0], qp[1]);
                 split_bf16x2(kp[0], kp[1], hi, lo);
-                *reinterpret_cast<uint32_t*>(dst + 2 * S::OP) = hi;
-                *reinterpret_cast<uint32_t*>(dst + 3 * S::OP) = lo;
+                *reinterpret_cast<uint32_t*>(dst + S::OP) = hi;
+                *reinterpret_cast<uint32_t*>(dst + 2 * S::OP) = lo;
                 split_bf16x2(kr[0], kr[1], hi, lo);
-                *reinterpret_cast<uint32_t*>(dst + 4 * S::OP) = hi;
-                *reinterpret_cast<uint32_t*>(dst + 5 * S::OP) = lo;
+                *reinterpret_cast<uint32_t*>(dst + 3 * S::OP) = hi;
+                *reinterpret_cast<uint32_t*>(dst + 4 * S::OP) = lo;
             }
         }
     };
-    // Inner weights of a chunk gate by gate: warp w forms columns j = w, w + WARPS, ... of the first partial matrix.
-    auto slow_weights = [&](uint32_t t0) {
-        for (uint32_t j = warp; j < HS_Q; j += WARPS) {
+    // Inner weights of a chunk gate by gate, in the layout of the product's accumulators.
+    auto slow_weights = [&](uint32_t t0, float (&gm)[2][4]) {
+        float* mine = reinterpret_cast<float*>(smem + 2 * S::STAGE) + warp * HS_Q * S::SPITCH;
+        for (uint32_t j = 0; j < HS_Q; ++j) {
             float g[NP / 32];
-            for (uint32_t i = 0; i < HS_Q; ++i) {
+#pragma unroll
+            for (int n = 0; n < NP / 32; ++n) g[n] = 0.0f;
+            for (uint32_t i = j; i < HS_Q; ++i) {
                 float sum = 0.0f;
 #pragma unroll
                 for (int n = 0; n < NP / 32; ++n) {
                     const uint32_t c = lane + 32 * n, t = t0 + i;
-                    if (c >= m.dim || t >= place.chunk || i < j) { if (i <= j) g[n] = 0.0f; continue; }
+                    if (c >= m.dim || t >= place.chunk) continue;
+                    const float lo = m.lower[h * m.dim + c];
                     float f, k;
-                    hs_gate(fb[(size_t)t * m.f_ld + c] + m.f_bias[h * m.dim + c], m.lower[h * m.dim + c], f, k);
+                    hs_gate(-HS_LOG2E * (fb[(size_t)t * m.f_ld + c] + m.f_bias[h * m.dim + c]), lo, 1.0f - lo, f, k);
                     g[n] = i == j ? k : g[n] * f;
                     sum = fmaf(mx_silu(__bfloat162float(qb[(size_t)t * m.ld + c])), g[n], sum);
                 }
 #pragma unroll
                 for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-                if (lane < WARPS) inner[(lane * HS_Q + i) * S::APITCH + j] = lane == 0 ? sum : 0.0f;
+                if (lane == 0) mine[i * S::SPITCH + j] = sum;
             }
         }
+        __syncwarp();
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) gm[nt][e] = mine[(g8 + (e >> 1) * 8) * S::SPITCH + nt * 8 + t4 * 2 + (e & 1)];      // above the diagonal: anything
+        __syncwarp();
     };
 
     // S^T: rows p = pw + g8 (+ 8), columns n = nt * 8 + t4 * 2 (+ 1)
@@ -228,7 +236,7 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     fetch(0);
     load_v(0, smem);
     __syncthreads();       // s_tiny is clear
-    prepare(0, smem, 0);
+    prepare(0, smem);
     fetch(HS_Q);
 
     const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::NPITCH + (lane >> 4) * 16;     // A operand, [token][channel]
@@ -237,7 +245,9 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     const uint32_t v_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * S::VPITCH + (lane >> 4) * 16 + pw * 2;     // [k = token][n = column], transposed
     const uint32_t vt_off = ((lane & 7) + (lane >> 4) * 8) * S::VPITCH + ((lane >> 3) & 1) * 16 + pw * 2;    // v^T: A operand from [token][column]
     float y[2][4];         // outputs: rows g8 (+ 8), columns pw + nt * 8 + t4 * 2 (+ 1); kept until the next chunk's norm
+    const float inv_vdim = 1.0f / (float)m.vdim;
     auto finish = [&](uint32_t t0) {
+        const uint32_t at = t0 / HS_Q & 1;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const uint32_t t = t0 + g8 + half * 8;
@@ -254,8 +264,8 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
             }
             float total = 0.0f;
 #pragma unroll
-            for (int w = 0; w < WARPS; ++w) total += s_sq[w][g8 + half * 8];
-            const float inv = rsqrtf(total / (float)m.vdim + m.eps);
+            for (int w = 0; w < WARPS; ++w) total += s_sq[at][w][g8 + half * 8];
+            const float inv = rsqrtf(fmaf(total, inv_vdim, m.eps));
             bf16* out = reinterpret_cast<bf16*>(m.out) + (row_base + t) * m.out_ld + h * m.vdim;
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
@@ -270,97 +280,62 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
     for (uint32_t t0 = 0; t0 < place.chunk; t0 += HS_Q, buf ^= 1) {
         uint8_t* stage = smem + buf * S::STAGE;
         uint8_t* next = smem + (buf ^ 1) * S::STAGE;
-        const uint32_t sb = mx_smem(stage), sv = sb + 6 * S::OP;
+        const uint32_t sb = mx_smem(stage), sv = sb + 5 * S::OP;
         mx_wait<0>();
-        __syncthreads();       // this chunk's operands are in place, the last one's have been used up
+        __syncthreads();       // this chunk's operands and the last one's sums are in place, the last one's operands used up
         if (t0 > 0) finish(t0 - HS_Q);
-        const bool more = t0 + HS_Q < place.chunk;
         load_v(t0 + HS_Q, next);
-        const bool slow = s_tiny[buf] != 0;
-        // ---- inner weights over this warp's channels ----
-        if (!slow) {
-            float gm[2][4] = {};
-#pragma unroll
-            for (int i = 0; i < MINE; ++i) {
-                const uint32_t kk = warp + i * WARPS;
-                if (kk >= GROUPS) continue;
-                uint32_t qh[4], ql[4], kh[4], kl[4];
-                mx_ldsm(sb + a_off + kk * 32, qh);
-                mx_ldsm(sb + S::OP + a_off + kk * 32, ql);
-                mx_ldsm(sb + 2 * S::OP + b_off + kk * 32, kh);
-                mx_ldsm(sb + 3 * S::OP + b_off + kk * 32, kl);
-                mx_mma(gm[0], qh, kh[0], kh[1]);
-                mx_mma(gm[1], qh, kh[2], kh[3]);
-                mx_mma(gm[0], ql, kh[0], kh[1]);
-                mx_mma(gm[1], ql, kh[2], kh[3]);
-                mx_mma(gm[0], qh, kl[0], kl[1]);
-                mx_mma(gm[1], qh, kl[2], kl[3]);
-            }
-            float* dst = inner + warp * HS_Q * S::APITCH;
-#pragma unroll
-            for (int nt = 0; nt < 2; ++nt) {
-                *reinterpret_cast<float2*>(dst + g8 * S::APITCH + nt * 8 + t4 * 2) = make_float2(gm[nt][0], gm[nt][1]);
-                *reinterpret_cast<float2*>(dst + (g8 + 8) * S::APITCH + nt * 8 + t4 * 2) = make_float2(gm[nt][2], gm[nt][3]);
-            }
-        } else {
-            slow_weights(t0);
-        }
-        // ---- q P . S_in ----
-        float yl[2][4];        // a second accumulator: shorter chains of dependent products
+        const uint32_t turn = t0 / HS_Q;
+        const bool slow = s_tiny[turn & 3] != 0;
+        if (tid == 0) s_tiny[(turn + 3) & 3] = 0;
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) y[nt][e] = yl[nt][e] = 0.0f;
+            for (int e = 0; e < 4; ++e) y[nt][e] = 0.0f;
         if (owner) {
+            // ---- q P . S_in and the inner weights q P . k / P ----
+            float yl[2][4] = {}, gm[2][4] = {};        // yl: a second accumulator, shorter chains of dependent products
 #pragma unroll
             for (int kk = 0; kk < GROUPS; ++kk) {
-                uint32_t h00, l00, h01, l01, h10, l10, h11, l11, qh[4], ql[4];
+                uint32_t h00, l00, h01, l01, h10, l10, h11, l11, qh[4], kh[4], kl[4];
                 mx_ldsm(sb + a_off + kk * 32, qh);
-                mx_ldsm(sb + S::OP + a_off + kk * 32, ql);
+                mx_ldsm(sb + S::OP + b_off + kk * 32, kh);
+                mx_ldsm(sb + 2 * S::OP + b_off + kk * 32, kl);
                 split_bf16x2(acc[2 * kk][0], acc[2 * kk][1], h00, l00);
                 split_bf16x2(acc[2 * kk + 1][0], acc[2 * kk + 1][1], h01, l01);
                 split_bf16x2(acc[2 * kk][2], acc[2 * kk][3], h10, l10);
                 split_bf16x2(acc[2 * kk + 1][2], acc[2 * kk + 1][3], h11, l11);
+                mx_mma(gm[0], qh, kh[0], kh[1]);
+                mx_mma(gm[1], qh, kh[2], kh[3]);
                 mx_mma(y[0], qh, h00, h01);
                 mx_mma(y[1], qh, h10, h11);
                 mx_mma(yl[0], qh, l00, l01);
                 mx_mma(yl[1], qh, l10, l11);
-                mx_mma(y[0], ql, h00, h01);
-                mx_mma(y[1], ql, h10, h11);
+                mx_mma(gm[0], qh, kl[0], kl[1]);
+                mx_mma(gm[1], qh, kl[2], kl[3]);
             }
-        }
-        if (more) {
-            prepare(t0 + HS_Q, next, buf ^ 1);
-            fetch(t0 + 2 * HS_Q);       // a whole chunk ahead of its use
-        }
-        __syncthreads();       // the inner weights of all warps are in place
-        if (tid == 0) s_tiny[buf] = 0;
-        if (owner) {
-            // ---- inner weights . v : A operand rows g8 (+ 8), columns t4 * 2 (+ 1, + 8, + 9) ----
+            if (slow) slow_weights(t0, gm);
+            // ---- inner weights . v ----
             uint32_t wh[4], wl[4], vb4[4];
-#pragma unroll
-            for (int r = 0; r < 4; ++r) {
-                const uint32_t i = g8 + (r & 1) * 8, j = t4 * 2 + (r >> 1) * 8;
-                float2 w = make_float2(0.0f, 0.0f);
-#pragma unroll
-                for (int k = 0; k < WARPS; ++k) {
-                    const float2 part = *reinterpret_cast<const float2*>(inner + (k * HS_Q + i) * S::APITCH + j);
-                    w.x += part.x;
-                    w.y += part.y;
-                }
-                if (j > i) w.x = 0.0f;
-                if (j + 1 > i) w.y = 0.0f;
-                split_bf16x2(w.x, w.y, wh[r], wl[r]);
-            }
             mx_ldsm_t(sv + v_off, vb4);
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {      // A operand: rows g8 (+ 8), columns t4 * 2 (+ 1, + 8, + 9)
+                const uint32_t i = g8 + (r & 1) * 8, j = t4 * 2 + (r >> 1) * 8;
+                const float w0 = j <= i ? gm[r >> 1][2 * (r & 1)] : 0.0f, w1 = j + 1 <= i ? gm[r >> 1][2 * (r & 1) + 1] : 0.0f;
+                split_bf16x2(w0, w1, wh[r], wl[r]);
+            }
             mx_mma(y[0], wh, vb4[0], vb4[1]);
             mx_mma(y[1], wh, vb4[2], vb4[3]);
             mx_mma(yl[0], wl, vb4[0], vb4[1]);
             mx_mma(yl[1], wl, vb4[2], vb4[3]);
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[nt][e] += yl[nt][e];
             // ---- S^T: decayed, plus v^T . (k R) ----
             uint32_t va[4];
             mx_ldsm_t(sv + vt_off, va);
-            const float* all = reinterpret_cast<const float*>(stage + 6 * S::OP + S::V_BYTES);
+            const float* all = reinterpret_cast<const float*>(stage + 5 * S::OP + S::V_BYTES);
 #pragma unroll
             for (int nt = 0; nt < NT; ++nt) {
                 const float2 d = *reinterpret_cast<const float2*>(all + nt * 8 + t4 * 2);
@@ -369,8 +344,8 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
 #pragma unroll
             for (int n = 0; n < NT / 2; ++n) {
                 uint32_t kh[4], kl[4];
-                mx_ldsm_t(sb + 4 * S::OP + bt_off + n * 32, kh);
-                mx_ldsm_t(sb + 5 * S::OP + bt_off + n * 32, kl);
+                mx_ldsm_t(sb + 3 * S::OP + bt_off + n * 32, kh);
+                mx_ldsm_t(sb + 4 * S::OP + bt_off + n * 32, kl);
                 mx_mma(acc[2 * n], va, kh[0], kh[1]);
                 mx_mma(acc[2 * n + 1], va, kh[2], kh[3]);
                 mx_mma(acc[2 * n], va, kl[0], kl[1]);
@@ -379,17 +354,19 @@ hgrn2_scan_kernel(Hgrn2 m, StepPlace place, uint32_t vec) {
         }
         float sq0 = 0.0f, sq1 = 0.0f;
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) y[nt][e] += yl[nt][e];
-            sq0 = fmaf(y[nt][0], y[nt][0], fmaf(y[nt][1], y[nt][1], sq0));      // columns past the width are zero: v is
+        for (int nt = 0; nt < 2; ++nt) {      // columns past the width are zero: v is
+            sq0 = fmaf(y[nt][0], y[nt][0], fmaf(y[nt][1], y[nt][1], sq0));
             sq1 = fmaf(y[nt][2], y[nt][2], fmaf(y[nt][3], y[nt][3], sq1));
         }
         sq0 += __shfl_xor_sync(0xffffffffu, sq0, 1);
         sq0 += __shfl_xor_sync(0xffffffffu, sq0, 2);
         sq1 += __shfl_xor_sync(0xffffffffu, sq1, 1);
         sq1 += __shfl_xor_sync(0xffffffffu, sq1, 2);
-        if (t4 == 0) { s_sq[warp][g8] = sq0; s_sq[warp][g8 + 8] = sq1; }
+        if (t4 == 0) { s_sq[turn & 1][warp][g8] = sq0; s_sq[turn & 1][warp][g8 + 8] = sq1; }
+        if (t0 + HS_Q < place.chunk) {
+            prepare(t0 + HS_Q, next);
+            fetch(t0 + 2 * HS_Q);       // a whole chunk ahead of its use
+        }
     }
     mx_wait<0>();
     __syncthreads();
