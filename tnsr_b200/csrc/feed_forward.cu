@@ -398,27 +398,39 @@ experts_choose_kernel(ChooseParams P) {
     }
     __syncthreads();
     const T* w = reinterpret_cast<const T*>(P.router);
-    for (uint32_t e = warp; e < P.route.total; e += EX_THREADS / 32) {
-        const T* we = w + (size_t)e * d;
-        float acc = 0.0f;
+    constexpr uint32_t WARPS = EX_THREADS / 32, SIDE = 4;          // a warp forms SIDE dot products side by side
+    for (uint32_t e0 = warp; e0 < P.route.total; e0 += WARPS * SIDE) {
+        float acc[SIDE] = {};
         if (sizeof(T) == 2 && d % 8 == 0) {
-#pragma unroll 4
+#pragma unroll 2
             for (uint32_t c = lane; c < d / 8; c += 32) {
-                const uint4 q = __ldg(reinterpret_cast<const uint4*>(we) + c);
-                const uint32_t words[4] = {q.x, q.y, q.z, q.w};
+                uint4 q[SIDE];
+#pragma unroll
+                for (uint32_t i = 0; i < SIDE; ++i)
+                    q[i] = e0 + i * WARPS < P.route.total ? __ldg(reinterpret_cast<const uint4*>(w + (size_t)(e0 + i * WARPS) * d) + c) : make_uint4(0u, 0u, 0u, 0u);
                 const float4 a = *reinterpret_cast<const float4*>(row_s + 8 * c), b = *reinterpret_cast<const float4*>(row_s + 8 * c + 4);
                 const float hv[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const float2 f = bf16x2_to_f32(words[i]);
-                    acc = fmaf(f.x, hv[2 * i], fmaf(f.y, hv[2 * i + 1], acc));
+                for (uint32_t i = 0; i < SIDE; ++i) {
+                    const uint32_t words[4] = {q[i].x, q[i].y, q[i].z, q[i].w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const float2 f = bf16x2_to_f32(words[j]);
+                        acc[i] = fmaf(f.x, hv[2 * j], fmaf(f.y, hv[2 * j + 1], acc[i]));
+                    }
                 }
             }
         } else {
-            for (uint32_t c = lane; c < d; c += 32) acc = fmaf(to_f32(we[c]), row_s[c], acc);
+            for (uint32_t c = lane; c < d; c += 32)
+#pragma unroll
+                for (uint32_t i = 0; i < SIDE; ++i)
+                    if (e0 + i * WARPS < P.route.total) acc[i] = fmaf(to_f32(w[(size_t)(e0 + i * WARPS) * d + c]), row_s[c], acc[i]);
         }
-        acc = ff_warp_sum(acc);
-        if (lane == 0) z[e] = acc;
+#pragma unroll
+        for (uint32_t i = 0; i < SIDE; ++i) {
+            const float v = ff_warp_sum(acc[i]);
+            if (lane == 0 && e0 + i * WARPS < P.route.total) z[e0 + i * WARPS] = v;
+        }
     }
     __syncthreads();
     if (warp != 0) return;

@@ -427,7 +427,7 @@ int stack_create(tnsr_b200_decoder* dec, const tnsr_b200_stack* st) {
                     const uint32_t total = l.experts + l.identity_experts;
                     if ((rc = dev_alloc(dec, &W.w_up, (size_t)l.experts * ff * d * e, true))) return rc;
                     if ((rc = dev_alloc(dec, &W.w_down, (size_t)l.experts * ff * d * e, true))) return rc;
-                    if ((rc = dev_alloc(dec, &W.router, (size_t)total * d * e, true))) return rc;
+                    if ((rc = dev_alloc(dec, &W.router, (size_t)round_up(total, 32) * d * e, true))) return rc;     // whole column blocks
                     if ((rc = floats(&W.correction, total))) return rc;
                     for (uint32_t x = 0; x < l.experts; ++x) {
                         matrix(ff, D, {StackPiece{W.w_up, 0, ff, x * ff, 0, D}});
@@ -552,7 +552,7 @@ int stack_alloc_rows(tnsr_b200_decoder* dec, uint32_t rows) {
         if (l.mixer == TNSR_B200_MIXER_RGLRU) u = std::max<uint64_t>(u, l.width);
         if (!sequential(l) || !l.feed_forward) continue;
         if (l.feed_forward_kind == TNSR_B200_FF_EXPERTS) {
-            router = std::max<uint64_t>(router, l.experts + l.identity_experts);
+            router = std::max<uint64_t>(router, round_up(l.experts + l.identity_experts, 32));
             experts = std::max(experts, experts_workspace_bytes(rows, dec->cfg.embed_dim, l.feed_forward, l.experts, l.top, dec->bf16_path ? TNSR_B200_BF16 : TNSR_B200_F32));
         } else {
             ff_z = std::max<uint64_t>(ff_z, l.feed_forward);
@@ -728,9 +728,9 @@ int stack_step(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t chunk,
         if (l.feed_forward_kind != TNSR_B200_FF_EXPERTS)
             if ((rc = norm(W.norm2))) return rc;
         if (l.feed_forward_kind == TNSR_B200_FF_EXPERTS) {
-            const uint32_t total = l.experts + l.identity_experts;
+            const uint32_t logit_cols = round_up(l.experts + l.identity_experts, 32);
             experts = Experts();
-            experts.logits = S->router; experts.logits_ld = total; experts.correction = W.correction;
+            experts.logits = S->router; experts.logits_ld = logit_cols; experts.correction = W.correction;
             experts.h = dec->n; experts.up = W.w_up; experts.down = W.w_down; experts.x = dec->h; experts.layer_scale = W.scale2;
             experts.workspace = S->experts_ws; experts.workspace_bytes = S->experts_ws_bytes; experts.d_status = dec->d_status;
             experts.rows = rows; experts.d = d; experts.ff = l.feed_forward; experts.experts = l.experts; experts.identity = l.identity_experts;
@@ -744,7 +744,7 @@ int stack_step(tnsr_b200_decoder* dec, const uint32_t* d_tokens, uint32_t chunk,
             } else {
                 experts.router = nullptr;
                 if ((rc = norm(W.norm2))) return rc;
-                if ((rc = product(W.router, total, S->router, total, ACT_NONE, TNSR_B200_F32))) return rc;
+                if ((rc = product(W.router, logit_cols, S->router, logit_cols, ACT_NONE, TNSR_B200_F32))) return rc;
             }
             RUN(dec, launch_experts(experts, dtype, st));
             pending_experts = true;

@@ -8,8 +8,8 @@
 //                        segments of 8 tokens each, which are scanned side by side from zero, joined through shared memory
 //                        (each segment is S -> A S + H) and finished from registers: every value is read once.
 //  * rglru_fused_step_kernel  single-token steps, bf16, parts of a multiple of 32 channels up to 256: convolution, both gates
-//                        and the recurrence of a part for 16 sessions in one block.  The gates of a part need its own
-//                        channels only, so nothing passes between blocks.
+//                        and the recurrence in one launch.  The gates of a part need its own channels only, so nothing
+//                        passes between parts.
 //  * rglru_step_kernel   the recurrence of the other single-token steps.
 // Gates, decays and the state are f32 in both precisions; 1 - a^2 is formed as -expm1(2 log a).
 #include <algorithm>
@@ -166,80 +166,126 @@ rglru_step_kernel(Rglru m, StepPlace place) {
     out[c] = from_f32<T>(S * y);
 }
 
-// Block = (part, 16 sessions).  u of the part goes to shared memory in bf16 and is the A operand of mma.sync; the gate matrix
-// is read from global memory as its B operand.  Of every 32 k values a lane loads eight consecutive ones (16 bytes): both
-// operands use the same order of k, so the sum does not notice.
-constexpr uint32_t RF_SESSIONS = 16, RF_MAX_PART = 256;
-__global__ void __launch_bounds__(256)
+// Block = (8 output channels of a part per warp, 16 sessions).  u of the whole part goes to shared memory in bf16
+// (every block of a part makes it; the ring slot they all write held the oldest row, which nobody reads) and is the A operand
+// of mma.sync; the gate rows are the B operand.  Of every 32 k values a lane takes eight consecutive ones (16 bytes): both
+// operands use the same order of k, so the sum does not notice.  Everything the block needs is asked for before the first use:
+// the weights even before the previous kernel has finished.
+constexpr uint32_t RF_SESSIONS = 16, RF_MAX_PART = 256, RF_MAX_WARPS = 16;
+template <int KS>      // part / 32, rounded up to 2, 4 or 8
+__global__ void __launch_bounds__(RF_MAX_WARPS * 32)
 rglru_fused_step_kernel(Rglru m, StepPlace place) {
-    constexpr uint32_t PITCH = RF_MAX_PART + 8;                 // elements
+    constexpr uint32_t PITCH = KS * 32 + 8;                 // elements
     __shared__ __align__(16) bf16 su[RF_SESSIONS * PITCH];
+    const uint32_t part = m.width / m.blocks, outs = blockDim.x / 4, subs = part / outs, blk = blockIdx.x / subs, c_first = blk * part, s0 = blockIdx.y * RF_SESSIONS;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
+    const uint32_t n0 = blockIdx.x % subs * outs + warp * 8;
+    uint4 br[KS], bi[KS];
+    {
+        const bf16* wr = reinterpret_cast<const bf16*>(m.gate_w) + (size_t)blk * 2 * part * part + (size_t)(n0 + g8) * part + t4 * 8;
+        const bf16* wi = wr + (size_t)part * part;
+#pragma unroll
+        for (int i = 0; i < KS; ++i) {
+            const bool there = i * 32 < part;
+            br[i] = there ? __ldg(reinterpret_cast<const uint4*>(wr + i * 32)) : make_uint4(0u, 0u, 0u, 0u);
+            bi[i] = there ? __ldg(reinterpret_cast<const uint4*>(wi + i * 32)) : make_uint4(0u, 0u, 0u, 0u);
+        }
+    }
+    const uint32_t c = n0 + t4 * 2, ch = c_first + c;
+    const RgChannel ca = rg_channel(m, ch), cb = rg_channel(m, ch + 1);
     pdl_wait();
     pdl_trigger();
-    const uint32_t part = m.width / m.blocks, blk = blockIdx.x, c_first = blk * part, s0 = blockIdx.y * RF_SESSIONS;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
     const bf16* proj = reinterpret_cast<const bf16*>(m.proj);
     bf16* ring = reinterpret_cast<bf16*>(m.ring);
-    // ---- convolution of two neighbouring channels per thread and turn; the slot of this position held the oldest row ----
-    for (uint32_t i = threadIdx.x; i < RF_SESSIONS * part / 2; i += 256) {
-        const uint32_t r = i / (part / 2), c = i % (part / 2) * 2, ch = c_first + c, s = s0 + r;
-        float2 y = make_float2(0.0f, 0.0f);
-        if (s < place.sessions) {
-            const uint32_t pos = place.pos(s);
-            const uint32_t now = *reinterpret_cast<const uint32_t*>(proj + (size_t)s * m.ld + m.x_col + ch);
-            uint32_t* slots = reinterpret_cast<uint32_t*>(ring + (size_t)s * m.taps * m.width + ch);
-            const float *w0 = m.conv_w + (size_t)ch * m.taps, *w1 = w0 + m.taps;
-            y = make_float2(m.conv_b[ch], m.conv_b[ch + 1]);
-            for (uint32_t j = 0; j < m.taps; ++j) {
-                const uint32_t lag = m.taps - 1 - j;
-                const uint32_t q = lag == 0 ? now : pos >= lag ? slots[(size_t)((pos - lag) % m.taps) * (m.width / 2)] : 0u;
-                const float2 v = bf16x2_to_f32(q);
-                y.x = fmaf(w0[j], v.x, y.x);
-                y.y = fmaf(w1[j], v.y, y.y);
+    float2 old[2], y[2];
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const uint32_t s = s0 + g8 + half * 8;
+        const bool here = s < place.sessions;
+        old[half] = here && place.pos(s) > 0 ? *reinterpret_cast<const float2*>(m.state + (size_t)s * m.width + ch) : make_float2(0.0f, 0.0f);
+        y[half] = here ? bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(proj + (size_t)s * m.ld + ch)) : make_float2(0.0f, 0.0f);
+    }
+    // ---- convolution: a thread owns two neighbouring channels and asks for eight sessions' rows at a time ----
+    const uint32_t pairs = part / 2, groups = blockDim.x / pairs, group = threadIdx.x / pairs, cc = threadIdx.x % pairs * 2, x = c_first + cc;
+    if (group < groups) {
+        constexpr uint32_t AT_ONCE = 8, LAGS = 3;          // rows up to LAGS back travel together, older ones one by one
+        const float *w0 = m.conv_w + (size_t)x * m.taps + m.taps - 1, *w1 = w0 + m.taps;       // of the current token; lag l at [-l]
+        const float2 bias = make_float2(m.conv_b[x], m.conv_b[x + 1]), wn = make_float2(*w0, *w1);
+        float2 wl[LAGS];
+#pragma unroll
+        for (uint32_t l = 0; l < LAGS; ++l) wl[l] = l + 1 < m.taps ? make_float2(w0[-(int)l - 1], w1[-(int)l - 1]) : make_float2(0.0f, 0.0f);
+        for (uint32_t r0 = group; r0 < RF_SESSIONS; r0 += AT_ONCE * groups) {
+            uint32_t now[AT_ONCE], back[LAGS][AT_ONCE], pos[AT_ONCE];
+#pragma unroll
+            for (uint32_t k = 0; k < AT_ONCE; ++k) {
+                const uint32_t r = r0 + k * groups, s = s0 + r;
+                const bool here = r < RF_SESSIONS && s < place.sessions;
+                pos[k] = here ? place.pos(s) : 0u;
+                now[k] = here ? *reinterpret_cast<const uint32_t*>(proj + (size_t)s * m.ld + m.x_col + x) : 0u;
+                const uint32_t slot = pos[k] % m.taps;
+#pragma unroll
+                for (uint32_t l = 1; l <= LAGS; ++l) {
+                    const uint32_t at = slot >= l ? slot - l : slot + m.taps - l;
+                    back[l - 1][k] = here && l < m.taps && pos[k] >= l
+                                         ? *reinterpret_cast<const uint32_t*>(ring + ((size_t)s * m.taps + at) * m.width + x) : 0u;
+                }
             }
-            slots[(size_t)(pos % m.taps) * (m.width / 2)] = now;
+#pragma unroll
+            for (uint32_t k = 0; k < AT_ONCE; ++k) {
+                const uint32_t r = r0 + k * groups, s = s0 + r;
+                if (r >= RF_SESSIONS) continue;
+                const float2 f = bf16x2_to_f32(now[k]);
+                float2 v = make_float2(fmaf(wn.x, f.x, bias.x), fmaf(wn.y, f.y, bias.y));
+#pragma unroll
+                for (uint32_t l = 0; l < LAGS; ++l) {
+                    const float2 g = bf16x2_to_f32(back[l][k]);
+                    v.x = fmaf(wl[l].x, g.x, v.x);
+                    v.y = fmaf(wl[l].y, g.y, v.y);
+                }
+                if (s < place.sessions) {
+                    const uint32_t slot = pos[k] % m.taps;
+                    for (uint32_t l = LAGS + 1; l < m.taps && l <= pos[k]; ++l) {
+                        const uint32_t at = slot >= l ? slot - l : slot + m.taps - l;
+                        const float2 g = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(ring + ((size_t)s * m.taps + at) * m.width + x));
+                        v.x = fmaf(w0[-(int)l], g.x, v.x);
+                        v.y = fmaf(w1[-(int)l], g.y, v.y);
+                    }
+                    *reinterpret_cast<uint32_t*>(ring + ((size_t)s * m.taps + slot) * m.width + x) = now[k];
+                }
+                *reinterpret_cast<uint32_t*>(su + r * PITCH + cc) = pack_bf16x2(v.x, v.y);
+            }
         }
-        *reinterpret_cast<uint32_t*>(su + r * PITCH + c) = pack_bf16x2(y.x, y.y);
     }
     __syncthreads();
-    // ---- gates and recurrence, eight channels per warp and turn ----
-    const bf16* w = reinterpret_cast<const bf16*>(m.gate_w) + (size_t)blk * 2 * part * part;
-    for (uint32_t n0 = warp * 8; n0 < part; n0 += 64) {
-        float gr[4] = {0.0f, 0.0f, 0.0f, 0.0f}, gi[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        const bf16 *wr = w + (size_t)(n0 + g8) * part + t4 * 8, *wi = wr + (size_t)part * part;
-#pragma unroll 4
-        for (uint32_t k0 = 0; k0 < part; k0 += 32) {
-            const uint4 br = __ldg(reinterpret_cast<const uint4*>(wr + k0)), bi = __ldg(reinterpret_cast<const uint4*>(wi + k0));
-            const uint4 lo = *reinterpret_cast<const uint4*>(su + g8 * PITCH + k0 + t4 * 8), hi = *reinterpret_cast<const uint4*>(su + (g8 + 8) * PITCH + k0 + t4 * 8);
-            const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
-            mx_mma(gr, a0, br.x, br.y);
-            mx_mma(gi, a0, bi.x, bi.y);
-            mx_mma(gr, a1, br.z, br.w);
-            mx_mma(gi, a1, bi.z, bi.w);
-        }
-        const uint32_t c = n0 + t4 * 2, ch = c_first + c;
-        const RgChannel ca = rg_channel(m, ch), cb = rg_channel(m, ch + 1);
+    // ---- gates and recurrence ----
+    float gr[4] = {0.0f, 0.0f, 0.0f, 0.0f}, gi[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-            const uint32_t r = g8 + half * 8, s = s0 + r;
-            if (s >= place.sessions) continue;
-            float2* state = reinterpret_cast<float2*>(m.state + (size_t)s * m.width + ch);
-            const float2 old = place.pos(s) > 0 ? *state : make_float2(0.0f, 0.0f);
-            const float2 y = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(proj + (size_t)s * m.ld + ch));
-            const float2 u = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(su + r * PITCH + c));
-            float a, b;
-            float2 S;
-            rg_token<bf16>(ca, gr[2 * half], gi[2 * half], u.x, a, b);
-            S.x = fmaf(a, old.x, b);
-            rg_token<bf16>(cb, gr[2 * half + 1], gi[2 * half + 1], u.y, a, b);
-            S.y = fmaf(a, old.y, b);
-            *state = S;
-            *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(m.out) + (size_t)s * m.out_ld + ch) = pack_bf16x2(S.x * y.x, S.y * y.y);
-        }
+    for (int i = 0; i < KS; ++i) {
+        if (i * 32 >= part) continue;
+        const uint4 lo = *reinterpret_cast<const uint4*>(su + g8 * PITCH + i * 32 + t4 * 8), hi = *reinterpret_cast<const uint4*>(su + (g8 + 8) * PITCH + i * 32 + t4 * 8);
+        const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+        mx_mma(gr, a0, br[i].x, br[i].y);
+        mx_mma(gi, a0, bi[i].x, bi[i].y);
+        mx_mma(gr, a1, br[i].z, br[i].w);
+        mx_mma(gi, a1, bi[i].z, bi[i].w);
     }
-    if (blk == 0 && m.out_cols > m.width) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const uint32_t r = g8 + half * 8, s = s0 + r;
+        if (s >= place.sessions) continue;
+        const float2 u = bf16x2_to_f32(*reinterpret_cast<const uint32_t*>(su + r * PITCH + c));
+        float a, b;
+        float2 S;
+        rg_token<bf16>(ca, gr[2 * half], gi[2 * half], u.x, a, b);
+        S.x = fmaf(a, old[half].x, b);
+        rg_token<bf16>(cb, gr[2 * half + 1], gi[2 * half + 1], u.y, a, b);
+        S.y = fmaf(a, old[half].y, b);
+        *reinterpret_cast<float2*>(m.state + (size_t)s * m.width + ch) = S;
+        *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(m.out) + (size_t)s * m.out_ld + ch) = pack_bf16x2(S.x * y[half].x, S.y * y[half].y);
+    }
+    if (blockIdx.x == 0 && m.out_cols > m.width) {
         const uint32_t pad = m.out_cols - m.width;
-        for (uint32_t i = threadIdx.x; i < pad * RF_SESSIONS; i += 256) {
+        for (uint32_t i = threadIdx.x; i < pad * RF_SESSIONS; i += blockDim.x) {
             const uint32_t s = s0 + i / pad;
             if (s < place.sessions) reinterpret_cast<bf16*>(m.out)[(size_t)s * m.out_ld + m.width + i % pad] = __float2bfloat16_rn(0.0f);
         }
@@ -276,7 +322,14 @@ int launch_rglru(const Rglru& m, const StepPlace& place, int dtype, cudaStream_t
     const bool bf = dtype == TNSR_B200_BF16;
     const uint32_t part = m.width / m.blocks, rows = place.sessions * place.chunk;
     if (bf && place.chunk == 1 && rglru_fused_fits(m)) {
-        launch_kernel(rglru_fused_step_kernel, dim3(m.blocks, ceil_div(place.sessions, RF_SESSIONS)), dim3(256), 0, stream, m, place);
+        // as many output channels per block as leave every SM a block: blocks of a part repeat its convolution
+        const uint32_t tiles = ceil_div(place.sessions, RF_SESSIONS);
+        uint32_t outs = 32;
+        while (outs * 2 <= 8 * RF_MAX_WARPS && part % (outs * 2) == 0 && m.width / (outs * 2) * tiles >= 128) outs *= 2;
+        const dim3 grid(m.width / outs, tiles), block(outs * 4);
+        if (part <= 64) launch_kernel(rglru_fused_step_kernel<2>, grid, block, 0, stream, m, place);
+        else if (part <= 128) launch_kernel(rglru_fused_step_kernel<4>, grid, block, 0, stream, m, place);
+        else launch_kernel(rglru_fused_step_kernel<8>, grid, block, 0, stream, m, place);
         count_launch();
         return check_launch("rglru_fused_step");
     }
