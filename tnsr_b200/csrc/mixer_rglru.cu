@@ -4,7 +4,7 @@
 //
 // The convolution writes u in the layout [blocks][rows][part], in which the gates are one grouped product with a [2 part,
 // part] matrix per block (r rows, then i rows), f32 out.
-//  * rglru_scan_kernel   many tokens: a block owns a strip of channels of one session; its 16 warps take consecutive
+//  * rglru_scan_kernel   many tokens: a block owns a strip of channels of one session; its eight warps take consecutive
 //                        segments of 8 tokens each, which are scanned side by side from zero, joined through shared memory
 //                        (each segment is S -> A S + H) and finished from registers: every value is read once.
 //  * rglru_fused_step_kernel  single-token steps, bf16, parts of a multiple of 32 channels up to 256: convolution, both gates
@@ -47,14 +47,26 @@ __device__ __forceinline__ void rg_token<float>(const RgChannel& ch, float r_raw
     b = sqrtf(-expm1f(2.0f * log_a)) * rg_sigmoid(i_raw + ch.i_bias) * u;
 }
 
-constexpr uint32_t RG_WARPS = 16, RG_SEG = 8;
+constexpr uint32_t RG_WARPS = 8, RG_SEG = 8;
 
-// VEC channels per lane (two when parts, pitches and pointers are even).
+// VEC channels per lane: two when parts, pitches and pointers are even.  y stays as it was stored until it is used.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(RG_WARPS * 32)
+struct RgRaw { typedef T type; };
+template <>
+struct RgRaw<bf16, 2> { typedef uint32_t type; };
+template <>
+struct RgRaw<float, 2> { typedef float2 type; };
+__device__ __forceinline__ float2 rg_values(uint32_t v) { return bf16x2_to_f32(v); }
+__device__ __forceinline__ float2 rg_values(float2 v) { return v; }
+__device__ __forceinline__ float2 rg_values(bf16 v) { return make_float2(__bfloat162float(v), 0.0f); }
+__device__ __forceinline__ float2 rg_values(float v) { return make_float2(v, 0.0f); }
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(RG_WARPS * 32, 3)
 rglru_scan_kernel(Rglru m, StepPlace place) {
     constexpr uint32_t STRIP = 32 * VEC;
-    __shared__ float seg_a[2][RG_WARPS][STRIP], seg_h[2][RG_WARPS][STRIP];
+    typedef typename RgRaw<T, VEC>::type Raw;
+    __shared__ float4 seg[2][RG_WARPS][32];          // per lane: A of its channels, H of its channels
     pdl_wait();
     pdl_trigger();
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, s = blockIdx.y;
@@ -77,58 +89,59 @@ rglru_scan_kernel(Rglru m, StepPlace place) {
     uint32_t buf = 0;
     for (uint32_t t0 = 0; t0 < place.chunk; t0 += RG_WARPS * RG_SEG, buf ^= 1) {
         const uint32_t first = t0 + warp * RG_SEG;
-        float a[RG_SEG][VEC], b[RG_SEG][VEC], yy[RG_SEG][VEC], uu[RG_SEG][VEC];
+        float a[RG_SEG][VEC], b[RG_SEG][VEC];
+        Raw yy[RG_SEG], uu[RG_SEG];
 #pragma unroll
         for (uint32_t i = 0; i < RG_SEG; ++i) {
             const uint32_t t = first + i;
             const bool here = live && t < place.chunk;
+            const Raw* up = reinterpret_cast<const Raw*>(u + (size_t)t * part);
+            const Raw* yp = reinterpret_cast<const Raw*>(y + (size_t)t * m.ld);
+            uu[i] = here ? *up : Raw();
+            yy[i] = here ? *yp : Raw();
             if (VEC == 2) {
                 const float2 z = make_float2(0.0f, 0.0f);
                 const float2 r = here ? *reinterpret_cast<const float2*>(gates + (size_t)t * 2 * part) : z;
                 const float2 g = here ? *reinterpret_cast<const float2*>(gates + (size_t)t * 2 * part + part) : z;
-                const float2 uv = here ? load_pair<T>(u + (size_t)t * part, true, true) : z, yv = here ? load_pair<T>(y + (size_t)t * m.ld, true, true) : z;
                 a[i][0] = r.x; a[i][VEC - 1] = r.y; b[i][0] = g.x; b[i][VEC - 1] = g.y;
-                uu[i][0] = uv.x; uu[i][VEC - 1] = uv.y; yy[i][0] = yv.x; yy[i][VEC - 1] = yv.y;
             } else {
                 a[i][0] = here ? gates[(size_t)t * 2 * part] : 0.0f;
                 b[i][0] = here ? gates[(size_t)t * 2 * part + part] : 0.0f;
-                uu[i][0] = here ? to_f32(u[(size_t)t * part]) : 0.0f;
-                yy[i][0] = here ? to_f32(y[(size_t)t * m.ld]) : 0.0f;
             }
         }
         float A[VEC], H[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) { A[e] = 1.0f; H[e] = 0.0f; }
 #pragma unroll
-        for (uint32_t i = 0; i < RG_SEG; ++i)
+        for (uint32_t i = 0; i < RG_SEG; ++i) {
+            const float2 uv = rg_values(uu[i]);
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
-                if (first + i < place.chunk) rg_token<T>(ch[e], a[i][e], b[i][e], uu[i][e], a[i][e], b[i][e]);
+                if (first + i < place.chunk) rg_token<T>(ch[e], a[i][e], b[i][e], e ? uv.y : uv.x, a[i][e], b[i][e]);
                 else { a[i][e] = 1.0f; b[i][e] = 0.0f; }
                 A[e] *= a[i][e];
                 H[e] = fmaf(a[i][e], H[e], b[i][e]);
             }
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) { seg_a[buf][warp][lane * VEC + e] = A[e]; seg_h[buf][warp][lane * VEC + e] = H[e]; }
+        }
+        seg[buf][warp][lane] = make_float4(A[0], A[VEC - 1], H[0], H[VEC - 1]);
         __syncthreads();       // the other buffer is rewritten only after the next barrier
         float S[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            float x = carry[e];
-            S[e] = x;
+        for (uint32_t w = 0; w < RG_WARPS; ++w) {
+            const float4 q = seg[buf][w][lane];
 #pragma unroll
-            for (uint32_t w = 0; w < RG_WARPS; ++w) {
-                if (w == warp) S[e] = x;
-                x = fmaf(seg_a[buf][w][lane * VEC + e], x, seg_h[buf][w][lane * VEC + e]);
+            for (int e = 0; e < VEC; ++e) {
+                if (w == warp) S[e] = carry[e];
+                carry[e] = e ? fmaf(q.y, carry[e], q.w) : fmaf(q.x, carry[e], q.z);
             }
-            carry[e] = x;
         }
 #pragma unroll
         for (uint32_t i = 0; i < RG_SEG; ++i) {
             const uint32_t t = first + i;
+            const float2 yv = rg_values(yy[i]);
             float o[VEC];
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) { S[e] = fmaf(a[i][e], S[e], b[i][e]); o[e] = S[e] * yy[i][e]; }
+            for (int e = 0; e < VEC; ++e) { S[e] = fmaf(a[i][e], S[e], b[i][e]); o[e] = S[e] * (e ? yv.y : yv.x); }
             if (!live || t >= place.chunk) continue;
             if (VEC == 2) store_pair<T>(out + (size_t)t * m.out_ld, make_float2(o[0], o[VEC - 1]), true, true);
             else out[(size_t)t * m.out_ld] = from_f32<T>(o[0]);
