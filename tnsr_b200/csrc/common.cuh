@@ -144,7 +144,8 @@ enum GemmMode : int {
     GEMM_QKV = 1,     // n = 3*d: columns [0,d) -> q (bf16), [d,2d) -> K cache rows, [2d,3d) -> V cache rows
     GEMM_SWIGLU = 2,  // n = 2*f packed in blocks of 16: out[m, f] bf16 = silu(gate) * up
     GEMM_ARGMAX = 3,  // no matrix leaves the kernel: per (row, column tile) the greedy candidate (key, index)
-    GEMM_SEGMENTS = 4 // column ranges with destinations of their own (GemmSegments): one product for all projections of a layer
+    GEMM_SEGMENTS = 4, // column ranges with destinations of their own (GemmSegments): one product for all projections of a layer
+    GEMM_SCALED = 5   // GEMM_PLAIN with GemmEpilogue::scale, f32 out: a kernel of its own, so that the plain epilogue stays as lean as it is
 };
 // Destinations of the column ranges of one product: range i covers accumulator columns [col0, col0 of i + 1) and lands in
 // `out` (row pitch ld, local column = column - col0), bf16 or f32, with an activation of its own.  Range boundaries and n
@@ -379,7 +380,6 @@ __device__ __forceinline__ float apply_activation(float x, int act) {
     if (act == ACT_RELU) return fmaxf(x, 0.0f);
     if (act == ACT_GELU) return fast_gelu(x);
     if (act == ACT_GELU_TANH) return fast_gelu_tanh(x);
-    if (act == ACT_RELU_SQUARED) { const float y = fmaxf(x, 0.0f); return y * y; }
     return x;
 }
 

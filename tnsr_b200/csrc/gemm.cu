@@ -186,6 +186,7 @@ static int launch_simple(const bf16* a, uint32_t lda, const bf16* bt, const EpiP
         return TNSR_B200_ERR_UNSUPPORTED;
     }
     switch (mode) {
+        case GEMM_SCALED:     // the scalar epilogue looks at the pointer
         case GEMM_PLAIN: launch_kernel(gemm_simple_kernel<GEMM_PLAIN>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
         case GEMM_QKV: launch_kernel(gemm_simple_kernel<GEMM_QKV>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
         case GEMM_SWIGLU: launch_kernel(gemm_simple_kernel<GEMM_SWIGLU>, grid, dim3(256), 0, stream, a, lda, bt, P, k); break;
@@ -282,7 +283,7 @@ __device__ __forceinline__ float4 act4(float4 v, int act) {
 // pointers and leading dimensions).
 __device__ __forceinline__ bool f32_vector_path(const EpiParams& P, uint32_t col0) {
     const float* res = P.ep.residual;
-    return col0 + 32 <= P.n && ((reinterpret_cast<uintptr_t>(P.ep.bias) | reinterpret_cast<uintptr_t>(P.ep.scale)) & 15) == 0 && P.ldc % 4 == 0 &&
+    return col0 + 32 <= P.n && (reinterpret_cast<uintptr_t>(P.ep.bias) & 15) == 0 && P.ldc % 4 == 0 &&
            (reinterpret_cast<uintptr_t>(P.out) & 15) == 0 &&
            (!res || (P.ep.ldr % 4 == 0 && (reinterpret_cast<uintptr_t>(res) & 15) == 0));
 }
@@ -305,6 +306,7 @@ __device__ __forceinline__ void load_residual_block(const EpiParams& P, uint32_t
 // box into the residual stream in global memory.  The warp neither reads the residual nor issues stores; rows and
 // columns outside the matrix are clipped by the tensor map.  One add per element, so the result is the same
 // residual + value an explicit read-add-store gives.
+template <bool SCALED>
 __device__ __forceinline__ void epilogue_block_reduce(const EpiParams& P, const CUtensorMap* map_out, float* stage,
                                                       uint32_t row0, uint32_t col0, const float* acc, uint32_t lane,
                                                       bool store = false, bool with_bias = true, uint32_t row_out = 0) {
@@ -313,7 +315,7 @@ __device__ __forceinline__ void epilogue_block_reduce(const EpiParams& P, const 
     __syncwarp();
     float4* row = reinterpret_cast<float4*>(stage) + lane * 8;
     const bool bias_vec = with_bias && P.ep.bias && (reinterpret_cast<uintptr_t>(P.ep.bias) & 15) == 0 && col0 + 32 <= P.n;
-    const bool scale_vec = (reinterpret_cast<uintptr_t>(P.ep.scale) & 15) == 0 && col0 + 32 <= P.n;
+    const bool scale_vec = SCALED && (reinterpret_cast<uintptr_t>(P.ep.scale) & 15) == 0 && col0 + 32 <= P.n;
 #pragma unroll
     for (int g = 0; g < 8; ++g) {
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -325,7 +327,7 @@ __device__ __forceinline__ void epilogue_block_reduce(const EpiParams& P, const 
                             c + 2 < P.n ? P.ep.bias[c + 2] : 0.f, c + 3 < P.n ? P.ep.bias[c + 3] : 0.f);
         }
         float4 v = act4(make_float4(acc[4 * g] + b.x, acc[4 * g + 1] + b.y, acc[4 * g + 2] + b.z, acc[4 * g + 3] + b.w), P.ep.activation);
-        if (P.ep.scale) {
+        if (SCALED) {
             const uint32_t c = col0 + 4 * g;
             if (scale_vec) {
                 const float4 f = __ldg(reinterpret_cast<const float4*>(P.ep.scale + c));
@@ -559,7 +561,10 @@ __device__ __forceinline__ void epilogue_block(const EpiParams& P, float* stage,
             float4 bv = make_float4(0.f, 0.f, 0.f, 0.f);
             if (P.ep.bias) bv = __ldg(reinterpret_cast<const float4*>(P.ep.bias + col0 + c4));
             float4 sv = make_float4(1.f, 1.f, 1.f, 1.f);
-            if (P.ep.scale) sv = __ldg(reinterpret_cast<const float4*>(P.ep.scale + col0 + c4));
+            if (MODE == GEMM_SCALED) {
+                const float* f = P.ep.scale + col0 + c4;       // any alignment
+                sv = make_float4(__ldg(f), __ldg(f + 1), __ldg(f + 2), __ldg(f + 3));
+            }
 #pragma unroll
             for (uint32_t it = 0; it < 8; ++it) {
                 const uint32_t rr = it * 4 + rsub;
@@ -578,7 +583,7 @@ __device__ __forceinline__ void epilogue_block(const EpiParams& P, float* stage,
             for (int rr = 0; rr < 32; ++rr)
                 rv[rr] = (res && col_ok && (uint32_t)rr < rows) ? res[(size_t)(row0 + rr) * P.ep.ldr + col] : 0.0f;
             const float bv = (P.ep.bias && col_ok) ? __ldg(P.ep.bias + col) : 0.0f;
-            const float sv = (P.ep.scale && col_ok) ? __ldg(P.ep.scale + col) : 1.0f;
+            const float sv = (MODE == GEMM_SCALED && col_ok) ? __ldg(P.ep.scale + col) : 1.0f;
 #pragma unroll
             for (int rr = 0; rr < 32; ++rr)
                 if (col_ok && (uint32_t)rr < rows)
@@ -594,6 +599,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                const __grid_constant__ CUtensorMap map_out, const __grid_constant__ CUtensorMap map_k,
                const __grid_constant__ CUtensorMap map_v, TcParams prm) {
     using S = TcShape<BN, EPI>;
+    constexpr bool PLAIN = MODE == GEMM_PLAIN || MODE == GEMM_SCALED;
     constexpr int PER_QUARTER = EPI / 4;             // epilogue warps per TMEM lane quarter
     constexpr uint32_t CHUNK_STRIDE = 32 * PER_QUARTER;
     extern __shared__ uint8_t smem_raw[];
@@ -609,7 +615,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t split = (MODE == GEMM_PLAIN && prm.tma_reduce == 2) ? prm.split_k : 1u;
+    const uint32_t split = (PLAIN && prm.tma_reduce == 2) ? prm.split_k : 1u;
     const uint32_t num_tiles = prm.tiles_m * prm.tiles_n * split;
     const uint32_t num_kb = (prm.k + BK - 1) / BK;
     const uint32_t kb_per = (num_kb + split - 1) / split;    // the host picks split so that no range is empty
@@ -703,8 +709,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             // being accumulated (the rows are final: only this warp rewrites them, after this read)
             float4 res_pre[8];
             bool have_pre = false;
-            const bool reduce = MODE == GEMM_PLAIN && prm.tma_reduce;
-            if (!reduce && MODE == GEMM_PLAIN && prm.epi.ep.out_dtype == TNSR_B200_F32 && prm.epi.ep.residual && half * 32 < (uint32_t)BN) {
+            const bool reduce = PLAIN && prm.tma_reduce;
+            if (!reduce && PLAIN && prm.epi.ep.out_dtype == TNSR_B200_F32 && prm.epi.ep.residual && half * 32 < (uint32_t)BN) {
                 const uint32_t col0 = tn * BN + half * 32;
                 if (row0 < prm.epi.m && col0 < prm.epi.n && f32_vector_path(prm.epi, col0)) {
                     load_residual_block(prm.epi, row0, col0, lane, res_pre);
@@ -754,7 +760,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     const uint32_t col0 = tn * BN + c;
                     if (reduce) {
                         if (row0 < prm.epi.m && col0 < prm.epi.n)
-                            epilogue_block_reduce(prm.epi, &map_out, stage, row0, col0, acc, lane, prm.tma_reduce == 2, ks == 0,
+                            epilogue_block_reduce<MODE == GEMM_SCALED>(prm.epi, &map_out, stage, row0, col0, acc, lane, prm.tma_reduce == 2, ks == 0,
                                                   ks * prm.split_rows + row0);
                     } else if (prm.tma_store) {
                         if (row0 < prm.epi.m && col0 < prm.epi.n)
@@ -769,7 +775,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             if (lane == 0) mbar_arrive(acc_empty + ab);
         }
         // bulk reduce operations of this warp must be complete before the CTA gives up its shared memory
-        if (((MODE == GEMM_PLAIN && prm.tma_reduce) || prm.tma_store) && lane == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+        if (((PLAIN && prm.tma_reduce) || prm.tma_store) && lane == 0) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
     }
 
     // ---------------- teardown ----------------
@@ -849,6 +855,7 @@ template <int BN>
 static int launch_tc_mode(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap* mo, const TcParams& prm, GemmMode mode, cudaStream_t stream) {
     switch (mode) {
         case GEMM_PLAIN: return launch_tc_t<BN, GEMM_PLAIN>(ma, mb, mo, prm, stream);
+        case GEMM_SCALED: return launch_tc_t<BN, GEMM_SCALED>(ma, mb, mo, prm, stream);
         case GEMM_QKV: return launch_tc_t<BN, GEMM_QKV>(ma, mb, mo, prm, stream);
         case GEMM_SWIGLU: return launch_tc_t<BN, GEMM_SWIGLU>(ma, mb, mo, prm, stream);
         case GEMM_ARGMAX: return launch_tc_t<BN, GEMM_ARGMAX>(ma, mb, mo, prm, stream);
@@ -874,7 +881,7 @@ static int launch_gemm_impl(const bf16* a, const bf16* bt, void* out, uint32_t l
         set_thread_error("gemm: packed SwiGLU width must be a multiple of 32");
         return TNSR_B200_ERR_UNSUPPORTED;
     }
-    if (ep.residual && ep.out_dtype != TNSR_B200_F32) return TNSR_B200_ERR_INVALID_ARGUMENT;
+    if ((ep.residual || ep.scale) && ep.out_dtype != TNSR_B200_F32) return TNSR_B200_ERR_INVALID_ARGUMENT;
     EpiParams P;
     if (mode == GEMM_SEGMENTS) {
         bool fits = segments && segments->count >= 1 && segments->count <= 3 && segments->s[0].col0 == 0 && n % 32 == 0;
@@ -1040,6 +1047,7 @@ static int launch_gemm_impl(const bf16* a, const bf16* bt, void* out, uint32_t l
         else mo[0] = mo[1] = mo[2] = ma;
     }
     prm.epi = P;
+    if (mode == GEMM_PLAIN && ep.scale) mode = GEMM_SCALED;
     switch (bn) {
         case 256: return launch_tc_mode<256>(ma, mb, mo, prm, mode, stream);
         case 128: return launch_tc_mode<128>(ma, mb, mo, prm, mode, stream);

@@ -46,6 +46,11 @@ struct GgParams {
     uint64_t wait_limit_ns;
 };
 
+__device__ __forceinline__ float gg_activation(float x, int act) {
+    if (act == ACT_RELU_SQUARED) { const float y = fmaxf(x, 0.0f); return y * y; }
+    return apply_activation(x, act);
+}
+
 // Walks the tile list: tiles of a group are consecutive, weight tiles fastest.
 struct GgWalk {
     uint32_t g = 0, row0 = 0, end = 0, n0 = 0;      // group, first token row, end of the group's rows, first weight row
@@ -180,7 +185,7 @@ gemm_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
                 const uint32_t n_rows = min(32u, live - j0);
                 const size_t base = (size_t)(at.row0 + j0) * prm.n;
 #pragma unroll
-                for (int j = 0; j < 32; ++j) acc[j] = apply_activation(acc[j], prm.activation);
+                for (int j = 0; j < 32; ++j) acc[j] = gg_activation(acc[j], prm.activation);
                 if (prm.out_dtype == TNSR_B200_F32) {
                     float* out = reinterpret_cast<float*>(prm.out) + base + col;
                     if (col < prm.n) {
@@ -269,7 +274,7 @@ gemm_grouped_simple_kernel(const T* __restrict__ a, const T* __restrict__ w, GgP
             for (int j = 0; j < 2; ++j) {
                 const uint32_t row = row0 + ty + 16 * i, col = n0 + tx + 16 * j;
                 if (row >= end || col >= P.n) continue;
-                const float v = apply_activation(acc[i][j], P.activation);
+                const float v = gg_activation(acc[i][j], P.activation);
                 if (P.out_dtype == TNSR_B200_BF16) reinterpret_cast<bf16*>(P.out)[(size_t)row * P.n + col] = __float2bfloat16_rn(v);
                 else reinterpret_cast<float*>(P.out)[(size_t)row * P.n + col] = v;
             }

@@ -90,7 +90,8 @@ struct PtParams {
 
 enum : int { PT_SOFTMAX = 0, PT_CAPPED = 1, PT_SIGMOID = 2 };
 
-template <int KIND>
+// WINDOW: prm.window is set (compiled apart: the masks of the unwindowed kernels stay one comparison per key).
+template <int KIND, bool WINDOW>
 __global__ void __launch_bounds__(PT_THREADS, 2)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, PtParams prm) {
@@ -129,7 +130,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t last_q = min(q0 + PT_BQ, prm.chunk) - 1;
         const uint32_t total = prm.position + last_q + 1;          // keys visible to the tile's last query
         const uint32_t first = prm.position + q0 + 1;              // keys up to the tile's first query
-        block0 = prm.window && first > prm.window ? (first - prm.window) / PT_BK : 0u;
+        block0 = WINDOW && first > prm.window ? (first - prm.window) / PT_BK : 0u;
         n_blocks = (total + PT_BK - 1) / PT_BK - block0;
     };
 
@@ -253,7 +254,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             item_coords(item, q0, h, s, block0, n_blocks);
             const uint32_t q_idx = min(q0 + row, prm.chunk - 1);
             const uint32_t limit = prm.position + q_idx;             // last visible key of this row
-            const uint32_t low = prm.window && limit >= prm.window ? limit + 1 - prm.window : 0u;   // first one
+            const uint32_t low = WINDOW && limit >= prm.window ? limit + 1 - prm.window : 0u;   // first one
             const float bias2 = SIGMOID && prm.head_bias ? -1.4426950408889634f * prm.head_bias[h] : 0.0f;
             float acc[32];                                           // output columns [32 half, 32 half + 32)
 #pragma unroll
@@ -277,8 +278,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tc_fence_after();
                 const uint32_t taddr = lane_taddr + half * 64;
                 const uint32_t kbase = (block0 + j) * PT_BK + half * 64;           // first key of this thread's columns
-                const bool need_mask = kbase + 63 > limit || kbase < low;
-                auto hidden = [&](uint32_t key) { return key > limit || key < low; };
+                const bool need_mask = kbase + 63 > limit || (WINDOW && kbase < low);
+                auto hidden = [&](uint32_t key) { return key > limit || (WINDOW && key < low); };
                 float corr = 0.0f, neg = 0.0f;
                 if (SIGMOID) {
                     // the previous P V must have read the upper P tile; its result stays in TMEM
@@ -431,8 +432,8 @@ bool prefill_attention_tc_eligible(uint32_t sessions, uint32_t chunk, uint32_t p
     return encode_fn() != nullptr;
 }
 
-template <int KIND>
-static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, uint32_t kv_heads, uint32_t capacity, PtParams& prm, cudaStream_t stream) {
+template <int KIND, bool WINDOW>
+static int launch_pt_kind(const bf16* q, const bf16* k_cache, const bf16* v_cache, uint32_t kv_heads, uint32_t capacity, PtParams& prm, cudaStream_t stream) {
     const uint64_t width = (uint64_t)prm.heads * PT_HD, kv_width = (uint64_t)kv_heads * PT_HD;
     CUtensorMap mq, mk, mv;
     if (!make_map3(&mq, q, width, prm.chunk, prm.sessions, prm.chunk) ||
@@ -445,8 +446,8 @@ static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, ui
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-        if (cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
-            cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND>, cudaFuncAttributePreferredSharedMemoryCarveout,
+        if (cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND, WINDOW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PT_SMEM_BYTES) != cudaSuccess ||
+            cudaFuncSetAttribute(prefill_attention_tc_kernel<KIND, WINDOW>, cudaFuncAttributePreferredSharedMemoryCarveout,
                                  (int)cudaSharedmemCarveoutMaxShared) != cudaSuccess)
             return check_launch("prefill_attention_tc attribute");
         if (dev >= 0 && dev < 64) configured[dev] = true;
@@ -460,9 +461,15 @@ static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, ui
     if (dev_sms <= 0) dev_sms = 148;
     const uint64_t items = (uint64_t)prm.q_tiles * prm.heads * prm.sessions;
     dim3 grid((unsigned)std::min<uint64_t>(items, 2ull * dev_sms));
-    launch_kernel(prefill_attention_tc_kernel<KIND>, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
+    launch_kernel(prefill_attention_tc_kernel<KIND, WINDOW>, grid, dim3(PT_THREADS), (size_t)PT_SMEM_BYTES, stream, mq, mk, mv, prm);
     count_launch();
     return check_launch("prefill_attention_tc");
+}
+
+template <int KIND>
+static int launch_pt(const bf16* q, const bf16* k_cache, const bf16* v_cache, uint32_t kv_heads, uint32_t capacity, PtParams& prm, cudaStream_t stream) {
+    return prm.window ? launch_pt_kind<KIND, true>(q, k_cache, v_cache, kv_heads, capacity, prm, stream)
+                      : launch_pt_kind<KIND, false>(q, k_cache, v_cache, kv_heads, capacity, prm, stream);
 }
 
 int launch_prefill_attention_tc(const bf16* q, const bf16* k_cache, const bf16* v_cache, bf16* out, uint32_t sessions,
