@@ -171,9 +171,9 @@ typedef struct tnsr_b200_decoder tnsr_b200_decoder;
  * parts.
  * MIXER_ATTENTION_HGRN2: two mixers side by side, their results added with the
  * gains attention_gain and recurrent_gain.  Attention as above without biases,
- * convolutions, norms and gate; with window > 0 a position sees itself and the
- * window - 1 before it; with score_kind SCORE_SIGMOID a visible key counts with
- * sigmoid(score + bias of the head), not normalised over keys.  HGRN2: per head a
+ * convolutions, norms and gate; with window > 0 position i sees
+ * j with i - window < j <= i; with score_kind SCORE_SIGMOID a visible key counts with
+ * sigmoid(score + bias of the head) and no sum divides.  HGRN2: per head a
  * [rec_dim, rec_vdim] f32 state, f = l + (1 - l) sigmoid(W_f h + b),
  * S <- diag(f) S + (1 - f) v^T, o = S^T silu(W_q h), then an RMS norm per head.
  * MIXER_RGLRU: y = gelu_tanh(W_y h + b) beside u = convolution of W_x h + b over
@@ -612,7 +612,7 @@ typedef struct tnsr_b200_grouped_attention_args {
     float scale, softcap;
     int32_t dtype, engine;
     const float* head_bias; /* [heads], sigmoid scores */
-    uint32_t window;        /* > 0: a query sees itself and the window - 1 keys before it */
+    uint32_t window;        /* > 0: a query at i sees keys i - window + 1 .. i */
     uint32_t score_kind;    /* tnsr_b200_score_kind; SIGMOID: out = gain * sum_j sigmoid(q . k_j * scale + head_bias) v_j */
     float gain;             /* factor of the result; 0 counts as 1 */
     uint32_t pad0;

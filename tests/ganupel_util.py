@@ -36,7 +36,7 @@ CONFIGS = {
                               parallel((6, 3, 16, 24, 16, 50, 0.2), (2, 36, 12), dense(80), (1.1, 0.4)), rglru(48, 2, 4, moe(24, 4, 1, 2, 0.8)),
                               rglru(40, 4, 2), parallel((2, 1, 32, 16, 8, 33, 0.25), (4, 16, 24))]),
     # heads of 64, states of 128 x 64, widths of whole 16-byte groups: the tensor-core kernels
-    "even": config(128, 320, [parallel((8, 2, 64, 64, 64, 48, 0.125), (2, 128, 64), dense(192)), rglru(128, 2, 4, moe(64, 8, 1, 2)),
+    "even": config(128, 320, [parallel((8, 2, 64, 64, 64, 48, 0.13), (2, 128, 64), dense(192)), rglru(192, 3, 4, moe(96, 7, 1, 2)),
                               parallel((4, 4, 64, 64, 32, 131, 0.1), (3, 64, 128), moe(128, 6, 3, 4, 2.5))]),
     # nothing divides anything: odd widths, one expert chosen, no identity expert
     "odd": config(70, 97, [parallel((3, 3, 10, 7, 6, 5, 0.4), (5, 5, 7), dense(37)), rglru(45, 5, 5, moe(13, 3, 0, 1)),

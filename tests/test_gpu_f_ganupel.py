@@ -372,7 +372,7 @@ def run_rglru(shape, x, t, portions, dtype, positions=None, state=None):
     return np.concatenate(outs, axis=1), (ring, carried)
 
 
-@pytest.mark.parametrize("shape", [(128, 2, 4), (72, 3, 3), (45, 5, 5), (160, 1, 1), (96, 12, 16), (30, 2, 2), (33, 33, 4), (320, 4, 4)])
+@pytest.mark.parametrize("shape", [(128, 4, 4), (72, 3, 3), (45, 5, 5), (160, 1, 1), (96, 12, 16), (30, 2, 2), (33, 33, 4), (320, 4, 4)])
 def test_rglru_portions_and_tokens(shape):
     n = 300
     x, t = rglru_case(shape, 2, n)
@@ -387,7 +387,7 @@ def test_rglru_portions_and_tokens(shape):
 
 
 # ---- feed-forwards ----------------------------------------------------------------------------------------
-@pytest.mark.parametrize("width", [8, 64, 37, 384, 1000, 2048, 8200, 9000, 7])
+@pytest.mark.parametrize("width", [8, 64, 37, 392, 1000, 2048, 8200, 9000, 7])
 def test_polynorm(width):
     rng = np.random.default_rng(width)
     z, act = bf16_exact((rng.normal(size=(5, width)) * [[0.03], [1], [4], [20], [0]]).astype(np.float32)), np.float32([0.7, -0.4, 0.9, 0.2])
@@ -578,7 +578,7 @@ def test_each_constant_matters(dtype):
 
 
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
-@pytest.mark.parametrize("window", [16, 40, 129])
+@pytest.mark.parametrize("window", [16, 45, 129])
 def test_planted_token_at_the_window_edge_decides(dtype, window):
     """q and k of the only layer depend on the token alone, and the last token's query matches one earlier token's key only:
     the logits must follow its value up to the window's last place, and not beyond."""
@@ -811,3 +811,101 @@ def test_command_line_generation(tmp_path):
                           "--prompt", " ".join(map(str, prompt))], capture_output=True, text=True, timeout=300, cwd=ROOT)
     assert run.returncode == 0, run.stderr[-2000:]
     assert [int(x) for x in run.stdout.split()] == greedy(cfg, tensors, prompt, 8)[6:]
+
+
+# ---- mechanisms in other company -------------------------------------------------------------------------------
+class OtherDesign:
+    """The block forms, mixers and feed-forwards of the library in combinations that no model here has."""
+    vocab_size, embed_dim, num_layers, layer_norm_epsilon, max_sequence_length = 83, 64, 4, 1e-4, 1 << 20
+    layers = (0, 1, 2, 3)
+
+    def __init__(self, weight_dtype):
+        self.weight_dtype = weight_dtype
+
+    def stack(self):
+        a = (_native.LayerDesc * 4)()
+        for x in a:
+            x.weights_of, x.feed_forward = -1, 40
+        a[0].mixer, a[0].block_form, a[0].heads, a[0].vdim, a[0].state, a[0].groups, a[0].norm_groups, a[0].conv_taps = 1, 1, 4, 16, 24, 2, 2, 3
+        b = a[1]       # a parallel block of softmax attention in a window beside HGRN2
+        b.mixer, b.heads, b.kv_heads, b.dim, b.vdim, b.window, b.score_kind, b.score_scale = 2, 4, 2, 24, 16, 9, 0, 0.4
+        b.rotary_dims, b.rotary_layout, b.rotary_base, b.rec_heads, b.rec_dim, b.rec_vdim, b.attention_gain, b.recurrent_gain = 8, 0, 50.0, 2, 12, 20, 1.3, 0.6
+        a[2].mixer, a[2].width, a[2].blocks, a[2].conv_taps = 3, 96, 3, 4
+        c = a[3]
+        c.mixer, c.block_form, c.heads, c.kv_heads, c.dim, c.vdim, c.conv_taps, c.score_scale = 0, 1, 4, 1, 16, 24, 2, 0.5
+        c.rotary_dims, c.rotary_base, c.feed_forward_kind, c.experts, c.identity_experts, c.top, c.router_scale = 16, 50.0, 2, 3, 2, 2, 1.2
+        return _native.StackDesc(1.5, 1.0, a, 4)
+
+    def tensor_shapes(self):
+        d = 64
+        s = {"embed": (83, d), "head": (83, d), "final.norm": (d,)}
+        s.update({"0.norm1": (d,), "0.in": (64 + 160 + 4, d), "0.conv": (160, 3), "0.conv.b": (160,), "0.dt_bias": (4,), "0.A_log": (4,), "0.D": (4,),
+                  "0.norm": (64,), "0.o": (d, 64), "0.ls1": (d,), "0.norm2": (d,), "0.up": (40, d), "0.down": (d, 40), "0.ls2": (d,)})
+        s.update({"1.norm1": (d,), "1.left.q": (96, d), "1.left.k": (48, d), "1.left.v": (32, d), "1.left.o": (d, 64), "1.right.q": (24, d), "1.right.f": (24, d),
+                  "1.right.f.b": (24,), "1.right.lower": (24,), "1.right.v": (40, d), "1.right.norm": (20,), "1.right.o": (d, 40), "1.up": (40, d),
+                  "1.down": (d, 40)})
+        s.update({"2.norm1": (d,), "2.y": (96, d), "2.y.b": (96,), "2.x": (96, d), "2.x.b": (96,), "2.conv": (96, 4), "2.conv.b": (96,), "2.ra": (3, 32, 32),
+                  "2.ra.b": (3, 32), "2.ri": (3, 32, 32), "2.ri.b": (3, 32), "2.lam": (96,), "2.o": (d, 96), "2.up": (40, d), "2.down": (d, 40)})
+        s.update({"3.norm1": (d,), "3.q": (64, d), "3.q.b": (64,), "3.k": (16, d), "3.k.b": (16,), "3.v": (24, d), "3.v.b": (24,), "3.q.norm": (16,), "3.k.norm": (16,),
+                  "3.q.conv": (64, 2), "3.k.conv": (16, 2), "3.v.conv": (24, 2), "3.g": (4, d), "3.o": (d, 96), "3.ls1": (d,), "3.norm2": (d,)})
+        for e in range(3):
+            s[f"3.e{e}.up"], s[f"3.e{e}.down"] = (40, d), (d, 40)
+        s.update({"3.router": (5, d), "3.correction": (5,), "3.ls2": (d,)})
+        return s
+
+    def forward(self, tensors, tokens):
+        get, eps = {k: v.astype(np.float64) for k, v in tensors.items()}, self.layer_norm_epsilon
+
+        def of(i):
+            return plain.under(get, f"{i}.")
+
+        def gelu(h, t):
+            return plain.gelu_tanh(h @ t["up"].T) @ t["down"].T
+
+        x = get["embed"][np.asarray(tokens)] * 1.5
+        t = of(0)
+        x = x + interleaved.mamba2_mixer(plain.norm_around_zero(x, t["norm1"], eps), dict(heads=4, vdim=16, state=24, groups=2, norm_groups=2), t, eps) * t["ls1"]
+        x = x + gelu(plain.norm_around_zero(x, t["norm2"], eps), t) * t["ls2"]
+        t = of(1)
+        h, n = plain.norm_around_zero(x, t["norm1"], eps), len(tokens)
+        rot = {"base": 50.0, "dims": 8, "scaling": None}
+        q, k = (interleaved.rotate_interleaved((h @ t["left." + name].T).reshape(n, -1, 24), rot) for name in "qk")
+        v = (h @ t["left.v"].T).reshape(n, 2, 16)
+        o = expected_attention(q[None], k[None], v[None], None, (0,), 0.4, 9, "softmax")[0]
+        right = plain.hgrn2(h, dict(heads=2, dim=12, vdim=20), plain.under(t, "right."), eps)
+        x = x + 1.3 * o.reshape(n, -1) @ t["left.o"].T + 0.6 * right + gelu(h, t)
+        t = of(2)
+        h = plain.norm_around_zero(x, t["norm1"], eps)
+        x = x + plain.rglru_mixer(h, None, t, eps) + gelu(h, t)
+        t = of(3)
+        m = dict(heads=4, kv_heads=1, dim=16, vdim=24, scale=0.5, rot={"base": 50.0, "dims": 16, "scaling": None})
+        x = x + interleaved.attention_mixer(plain.norm_around_zero(x, t["norm1"], eps), m, t, eps) * t["ls1"]
+        router = {"experts": 3, "identity": 2, "top": 2, "scale": 1.2}
+        x = x + plain.mixture(plain.norm_around_zero(x, t["norm2"], eps), {"router": router}, t, eps) * t["ls2"]
+        return plain.norm_around_zero(x, get["final.norm"], eps) @ get["head"].T
+
+
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_mechanisms_combine_freely(dtype):
+    from tnsr_b200.described import DescribedModel
+    design, rng = OtherDesign(dtype), np.random.default_rng(8)
+    tensors = {}
+    for name, shape in design.tensor_shapes().items():
+        leaf = name.split(".")[-1]
+        scale = {"conv": 0.4, "b": 0.3, "norm1": 0.3, "norm2": 0.3, "A_log": 0.5, "dt_bias": 1.0}.get(leaf, shape[-1] ** -0.5)
+        v = rng.normal(0, 1.0 if name == "embed" else scale, shape)
+        if leaf in ("ls1", "ls2", "norm", "D") and name != "final.norm":
+            v = rng.uniform(0.5, 1.3, shape)
+        elif leaf == "lower":
+            v = rng.uniform(0, 0.9, shape)
+        elif leaf == "lam":
+            v = rng.uniform(-5, 0, shape)
+        elif leaf == "correction":
+            v = np.array([4.0, 0.0, 2.0, 8.0, 0.0])
+        tensors[name] = bf16_exact(v.astype(np.float32))
+    model = DescribedModel(design, tensors)
+    ids = [int(x) for x in rng.integers(0, 83, 90)]
+    want = design.forward(tensors, ids)
+    decoder = model.decoder_with_capacity(Backend.Cuda, 1, 90)
+    for portions in ([90], [40] + [1] * 50, [2, 17, 33, 38]):
+        assert close(row_errors(logits_of(decoder, ids, portions), want), dtype), portions

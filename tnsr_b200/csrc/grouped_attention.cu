@@ -1,5 +1,5 @@
-// Grouped-query attention with capped scores and a sigmoid gate per head, or with sigmoid weights that are not normalised
-// over keys, over all earlier keys or a window of them; bf16 caches, any widths up to 256.
+// Grouped-query attention with capped scores and a sigmoid gate per head, or with sigmoid weights (no sum to divide by),
+// over all earlier keys or a window of them; bf16 caches, any widths up to 256.
 //
 // The query heads that share a key/value head are rows of one matrix product: row r of a (session, key/value head) is
 // query token r / per and head r % per of the group (per = heads / kv_heads), so a K/V tile is loaded once for the whole

@@ -1,4 +1,4 @@
-// HGRN2: linear attention whose forget gate also decides what is written.  Per head an f32 state S [dim, vdim]:
+// HGRN2: linear attention in which every channel writes the share that it forgets.  Per head an f32 state S [dim, vdim]:
 //     f = l + (1 - l) sigmoid(f_raw + b),   S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,   o_t = S_t^T silu(q_t)
 // then an RMS norm of o per head.  1 - f is formed as (1 - l) sigmoid(-(f_raw + b)), so that a gate close to one writes
 // what it should.

@@ -54,8 +54,8 @@ int launch_attention_prep(const AttentionPrep& a, const StepPlace& place, int dt
 
 // Grouped-query causal attention with capped scores and a sigmoid gate per head:
 // out[row, h * vdim ..] = gain * sigmoid(gate[row, h]) * softmax(cap(q . k * scale)) . v ; columns [heads * vdim, out_cols)
-// are zeroed.  window > 0: a query sees itself and the window - 1 keys before it.  score_kind SIGMOID: the weight of a
-// visible key is sigmoid(q . k * scale + head_bias[h]), not normalised over keys (softcap does not apply).
+// are zeroed.  window > 0: a query at i sees keys i - window + 1 .. i.  score_kind SIGMOID: the weight of a
+// visible key is sigmoid(q . k * scale + head_bias[h]), and no sum divides the result (softcap does not apply).
 struct GroupedAttention {
     const void* q = nullptr;
     const void* k_cache = nullptr;

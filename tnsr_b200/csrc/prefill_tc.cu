@@ -80,7 +80,7 @@ struct PtParams {
     uint32_t out_ld, out_cols; // output rows: pitch, columns (those past the heads are zeroed)
     const float* gate;         // [rows, gate_ld] or nullptr
     uint32_t gate_ld;
-    uint32_t window;           // 0: all earlier keys; else a query sees itself and the window - 1 keys before it
+    uint32_t window;           // 0: all earlier keys; else a query at i sees keys i - window + 1 .. i
     float gain;                // factor of the output
     const float* head_bias;    // sigmoid scores: added to q . k * scale, may be null
     float cap_pre, cap_post;   // capped scores in log2 units: cap_post - 2 cap_post / (1 + exp2(s cap_pre))
